@@ -114,7 +114,8 @@ typedef enum nnq_path {
     NNQ_PATH_AUTO = 0,
     NNQ_PATH_GENERIC = 1, /* portable dequant-fused row kernel on the raw block layout */
     NNQ_PATH_SKINNY = 2,  /* M <= 16: tiled layout, mma-based streaming kernel           */
-    NNQ_PATH_TENSOR = 3   /* M >= 128: TMA + tcgen05/TMEM tile pipeline                  */
+    NNQ_PATH_TENSOR = 3,  /* M >= 128: TMA + tcgen05/TMEM tile pipeline                  */
+    NNQ_PATH_F32 = 4      /* f32 activations: f32 products and sums, no operand rounded to bf16 */
 } nnq_path;
 
 /* ---- library / context ---------------------------------------------------------- */
@@ -608,6 +609,78 @@ NNQ_API nnq_status nnq_decoder_state(nnq_decoder *d, int *token, int *pos, int *
  * generated tokens [max_seq] (token produced at position p is stored at index p) */
 NNQ_API nnq_status nnq_decoder_buffers(nnq_decoder *d, float **k_cache, float **v_cache, float **logits, int **tokens);
 NNQ_API void nnq_decoder_destroy(nnq_decoder *d);
+
+/* ---- decoders whose layers each name their own mixer -------------------------------------
+ * A block is x <- x + mixer(h) + ff(h) with h = RMSNorm(x) * w: one norm, both parts read it. The
+ * decoder object, its step / prompt pass / state / token loop are the ones above; nnq_decoder_create_blocks
+ * takes the place of nnq_decoder_create, and nnq_decoder_set_block that of nnq_decoder_set_layer. Of the
+ * nnq_decoder_config only hidden, n_layers, vocab, max_seq, rms_eps and act_dtype are read (the other
+ * fields are ignored; tensor parallelism is not available: tp_world must be 0 or 1). With act_dtype
+ * NNQ_F32 every product runs in f32 (NNQ_PATH_F32); with NNQ_BF16 the inputs of the products are bf16 and
+ * everything else -- residual, norms, rotation, scores, softmax, decays, recurrent state -- is f32. */
+typedef enum nnq_mixer {
+    NNQ_MIXER_ATTENTION = 0,  /* softmax attention over a sliding window, query heads grouped over kv_heads */
+    NNQ_MIXER_RECURRENT = 1   /* S_t = diag(decay) S_{t-1} + k v^T, o = S^T q per head; o / rms(o) (* head_norm) * silu(g) */
+} nnq_mixer;
+typedef struct nnq_block_config {
+    int32_t mixer;           /* nnq_mixer */
+    int32_t heads, kv_heads; /* kv_heads: attention only */
+    int32_t dim, vdim;       /* query / key size and value size of a head (at most 256 each where a limit applies) */
+    int32_t ffn;             /* width of the silu-gated feed-forward, 0 = none */
+    int32_t rot_dims;        /* first dimensions of q and k that are rotated (half-split pairs), 0 = none */
+    double rot_base;         /* angle of pair i at position p: p * rot_base^(-2 i / rot_dims) */
+    /* attention */
+    float scale;             /* score = scale * q . k */
+    int32_t window;          /* position i sees j with 0 <= i - j < window; 0 = every earlier position */
+    int32_t conv_taps;       /* short causal convolution on q, k and v after the projection; 0 = none */
+    int32_t value_mix;       /* 1: v <- (1 - lambda) v + lambda v_first, v_first the values of the first such block */
+    int32_t out_gate;        /* 1: output times sigmoid(g) before the output projection */
+    /* recurrent */
+    float q_scale, k_scale;  /* factors on q and k (after the rotation) */
+    int32_t decay_rank;      /* > 0: decay per key channel sigmoid(W_2 W_1 h + b)^(1 / decay_tau) with a W_1 of this
+                              * many rows; 0: a fixed decay per head */
+    float decay_tau;
+} nnq_block_config;
+/* Where the parts of a block sit in its two products (filled by nnq_decoder_block_layout). Input product:
+ * weight [in_cols, in_k], rows of q, k, v, g (gate), a1 (W_1 of the decay), gate, up from these row numbers on
+ * (-1: absent), zero rows between and zero columns beyond hidden. Output product: weight [hidden, out_k],
+ * columns of the mixer's output projection from column 0 (heads * vdim of them), of the feed-forward's down
+ * projection from column ffn_col, zeros elsewhere. */
+typedef struct nnq_block_layout {
+    int32_t in_cols, in_k, out_k, ffn_col;
+    int32_t q, k, v, g, a1, gate, up;
+} nnq_block_layout;
+/* Weights of a block. The f32 arrays are host or device memory and are copied; in / out stay owned by the
+ * caller. Arrays a block does not use may be NULL. */
+typedef struct nnq_block_weights {
+    const nnq_weight *in, *out;
+    const float *norm;        /* [hidden] */
+    const float *bias_in;     /* [in_cols] or NULL */
+    const float *bias_out;    /* [hidden] or NULL */
+    const float *conv;        /* [heads*dim + kv_heads*(dim + vdim), conv_taps], channels q | k | v */
+    const float *head_norm;   /* [vdim] or NULL */
+    const float *decay_w;     /* [heads*dim, decay_rank] (W_2) */
+    const float *decay_b;     /* [heads*dim] */
+    const float *decay;       /* [heads] */
+    float lambda;             /* value_mix */
+} nnq_block_weights;
+/* `blocks` holds cfg->n_layers entries. block_rows: prompt rows that go through the blocks together (0 =
+ * 1024). An attention block keeps a ring of min(max_seq, window - 1 + block_rows) keys and values. */
+NNQ_API nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg, const nnq_block_config *blocks,
+                                             int block_rows, nnq_decoder **out);
+NNQ_API nnq_status nnq_decoder_block_layout(const nnq_decoder *d, int layer, nnq_block_layout *out);
+NNQ_API nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_block_weights *w);
+/* As nnq_decoder_set_head with the embedding held as an unquantized bf16 weight [vocab, in_k] (zero columns
+ * beyond hidden); lm_head [vocab, in_k]. The two may be the same weight. */
+NNQ_API nnq_status nnq_decoder_set_head_weights(nnq_decoder *d, const nnq_weight *embed, const float *final_norm,
+                                                const nnq_weight *lm_head);
+/* Continues the sequence with `count` given tokens (host array) at positions start_pos .., and writes the
+ * logits after the `n_want` tokens want[] (indexes into tokens, ascending) to logits_host [n_want, vocab].
+ * One token runs the decode step, several the prompt pass. start_pos 0 starts a new sequence; otherwise it
+ * must be the decoder's position where blocks with recurrent state or convolutions continue. With n_want = 0
+ * no logits are formed. Synchronises the stream. */
+NNQ_API nnq_status nnq_decoder_extend(nnq_decoder *d, const int32_t *tokens_host, int count, int start_pos, const int32_t *want,
+                                      int n_want, float *logits_host, void *stream);
 
 /* Number of kernels this library has launched on this context since creation. */
 NNQ_API int64_t nnq_launch_count(const nnq_ctx *ctx);

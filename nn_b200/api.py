@@ -92,7 +92,7 @@ _STATUS_ERRORS = {
 _BACKEND_KINDS = {20: "OutOfMemory", 21: "DispatchFailed", 22: "Timeout", 23: "NoDevice", 24: "Other"}
 
 F32, BF16 = 0, 1
-PATH_AUTO, PATH_GENERIC, PATH_SKINNY, PATH_TENSOR = 0, 1, 2, 3
+PATH_AUTO, PATH_GENERIC, PATH_SKINNY, PATH_TENSOR, PATH_F32 = 0, 1, 2, 3, 4
 
 
 def _torch():

@@ -49,12 +49,16 @@ def build(force: bool = False, verbose: bool = False) -> str:
         cmd += ["-ccbin", host_cxx]
     if verbose:
         cmd += ["-Xptxas", "-v"]
-    cmd += ["-o", LIB] + sources()
+    part = f"{LIB}.{os.getpid()}.part"   # renamed when whole: a concurrent or interrupted build leaves no broken library
+    cmd += ["-o", part] + sources()
     res = subprocess.run(cmd, capture_output=True, text=True)
     if verbose:
         sys.stderr.write(res.stderr)
     if res.returncode != 0:
+        if os.path.exists(part):
+            os.unlink(part)
         raise RuntimeError("nvcc failed:\n" + res.stdout + res.stderr)
+    os.replace(part, LIB)
     return LIB
 
 

@@ -6,6 +6,7 @@
 #include <new>
 
 #include "nnq_internal.h"
+#include "blocks.h"
 #include "gemm_tc.h"
 #include "skinny.h"
 
@@ -73,9 +74,10 @@ static nnq_status wait_host_stream(nnq_ctx *ctx) {
 
 static nnq_status finish_weight(nnq_ctx *ctx, nnq_weight *w) {
     // Build the tiled copy when a skinny kernel exists for this format and shape, and make the
-    // bf16 scratch of the large-prefill GEMM large enough for this weight.
+    // bf16 scratch of the large-prefill GEMM large enough for this weight (a bf16 weight is its own
+    // decoded form).
     nnq_status s = build_tiled(ctx, w);
-    if (s == NNQ_OK && w->d_raw) s = dense_scratch_reserve(ctx, w->n, w->k);
+    if (s == NNQ_OK && w->d_raw && w->fmt != NNQ_BF16_DENSE) s = dense_scratch_reserve(ctx, w->n, w->k);
     return s;
 }
 
@@ -182,7 +184,7 @@ const char *nnq_last_error(const nnq_ctx *ctx) { return ctx ? ctx->last_error : 
 
 nnq_status nnq_set_path(nnq_ctx *ctx, nnq_path path) {
     if (!ctx) return NNQ_ERR_INVALID_ARG;
-    if ((int)path < NNQ_PATH_AUTO || path > NNQ_PATH_TENSOR) return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown path %d", (int)path);
+    if ((int)path < NNQ_PATH_AUTO || path > NNQ_PATH_F32) return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown path %d", (int)path);
     ctx->path = path;
     return NNQ_OK;
 }
@@ -400,6 +402,10 @@ static nnq_status linear_dispatch(nnq_ctx *ctx, const nnq_weight *w, const void 
                                   cudaStream_t stream) {
     if (m == 0 || w->n == 0) return NNQ_OK;
     int path = ctx->path;
+    if (path == NNQ_PATH_F32) {
+        LinearArgs a = {w->d_raw, w->d_scales, x_dev, bias_dev, y_dev, m, w->n, w->k, w->fmt, x_dt, y_dt};
+        return launch_linear_f32(ctx, a, stream);
+    }
     bool skinny_ok = skinny_supported(w, m, x_dt);
     if (path == NNQ_PATH_SKINNY && !skinny_ok)
         return fail(ctx, NNQ_ERR_UNSUPPORTED, "skinny path does not cover format %d, N=%lld, K=%lld, M=%lld",
@@ -454,7 +460,7 @@ nnq_status nnq_linear_batch(nnq_ctx *ctx, int count, const nnq_weight *const *w,
     if (!ctx) return NNQ_ERR_INVALID_ARG;
     if (count < 0 || (count && (!w || !x_dev || !y_dev))) return fail(ctx, NNQ_ERR_INVALID_ARG, "bad batch arguments");
     nnq_status s;
-    bool all_skinny = count > 0 && ctx->path != NNQ_PATH_GENERIC && ctx->path != NNQ_PATH_TENSOR;
+    bool all_skinny = count > 0 && ctx->path != NNQ_PATH_GENERIC && ctx->path != NNQ_PATH_TENSOR && ctx->path != NNQ_PATH_F32;
     for (int i = 0; i < count; i++) {
         s = linear_checked(ctx, w[i], x_dev[i], x_dt, m, bias_dev ? bias_dev[i] : nullptr, y_dev[i], y_dt);
         if (s != NNQ_OK) return s;

@@ -10,15 +10,20 @@
 // The quantized products are the library's own (nnq_linear / nnq_linear_batch); this file adds the
 // small kernels between them. Token and position live in device memory and are advanced by the
 // last kernel of a step, so the launches of one step can be captured once and replayed per token.
+//
+// A decoder is built either from Qwen3 layers (nnq_decoder_create) or from blocks that each name their own
+// mixer (nnq_decoder_create_blocks): norm -> one product for everything that reads the normed row -> mixer
+// and feed-forward activation (attn_window.cu, recurrent.cu) -> one product back to the model width. Token
+// loop, prompt pass, position keeping, head and greedy commit are the same for both.
 #include <cuda_bf16.h>
 #include <math.h>
 #include <string.h>
 
 #include <new>
 
+#include "blocks.h"
 #include "comm.cuh"
-#include "nnq_internal.h"
-#include "pdl.cuh"
+#include "decoder_common.cuh"
 
 namespace nnq {
 nnq_status comm_view(nnq_comm *c, CommView *out);   // comm.cu
@@ -53,6 +58,25 @@ struct nnq_decoder {
     float *pf_h, *pf_delta, *pf_q, *pf_k, *pf_v, *pf_qrot, *pf_g, *pf_u;
     void *pf_xn, *pf_attn, *pf_mid;
     int *pf_tokens;
+    int *pf_want;               // rows of a block whose logits are asked for, [kPrefillRows]
+    float *d_want_logits;       // [kWantRows, vocab], allocated by the first nnq_decoder_extend that asks for any
+    int embed_ld, xn_ld;        // row strides of the embedding table and of the normed rows
+    // block decoder: the row buffers above are allocated at creation (pf_rows rows; a step uses row 0)
+    struct Block {
+        nnq_block_config cfg;
+        nnq_block_layout lay;
+        const nnq_weight *in, *out;
+        float *norm, *bias_in, *bias_out, *conv, *head_norm, *a2t, *a2b, *decay;
+        float lambda;
+        float *cosv, *sinv;     // rotation tables, owned by the first block with the same base and width
+        bool owns_tables;
+        int dim_ld, vdim_ld;
+        int cap, ranges;        // attention: ring capacity, key ranges of the decode kernel
+        float *kcache, *vcache, *conv_ring, *rec_state;
+        int mix_mode;
+    } *blocks;
+    float *b_proj, *b_q, *b_k, *b_a, *b_o, *b_vfirst;   // rows of proj; prepared q / k / decay, mixer output, first values
+    void *b_act;
 };
 
 namespace nnq {
@@ -64,30 +88,14 @@ constexpr int kAttnWarps = 4;
 // the Qwen3-8B shape).
 constexpr int kPrefillRows = 1024;
 constexpr int kArgmaxBlocks = 128;
-
-__device__ __forceinline__ float block_sum(float v, float *red) {
-#pragma unroll
-    for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, off);
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
-    __syncthreads();
-    if (lane == 0) red[warp] = v;
-    __syncthreads();
-    float t = 0.0f;
-    for (int w = 0; w < nw; w++) t += red[w];
-    return t;
-}
-
-__device__ __forceinline__ void store_act(void *dst, int dt, int i, float v) {
-    if (dt == NNQ_F32) reinterpret_cast<float *>(dst)[i] = v;
-    else reinterpret_cast<__nv_bfloat16 *>(dst)[i] = __float2bfloat16_rn(v);
-}
+constexpr int kWantRows = 64;     // rows of logits formed together
 
 // h = embedding row of the current token (first layer), or h += delta; xn = RMSNorm(h) * w.
 // One CTA; every thread keeps its (up to 8) elements in registers between the two phases.
 __global__ void __launch_bounds__(1024)
 dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
                 const int *__restrict__ state, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                int hidden) {
+                int hidden, int embed_ld, int xn_ld) {
     pdl_prologue();
     __shared__ float red[32];
     const int tok = embed ? state[0] : 0;
@@ -99,14 +107,14 @@ dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __
         v[r] = 0.0f;
         wv[r] = 0.0f;
         if (i < hidden) {
-            v[r] = embed ? __bfloat162float(embed[(size_t)tok * hidden + i]) : h[i] + delta[i];
+            v[r] = embed ? __bfloat162float(embed[(size_t)tok * embed_ld + i]) : h[i] + delta[i];
             wv[r] = w[i];
             h[i] = v[r];
             ss = fmaf(v[r], v[r], ss);
         }
     }
     for (int i = threadIdx.x + 8 * 1024; i < hidden; i += 1024) {   // wider models: the tail goes through memory
-        const float t = embed ? __bfloat162float(embed[(size_t)tok * hidden + i]) : h[i] + delta[i];
+        const float t = embed ? __bfloat162float(embed[(size_t)tok * embed_ld + i]) : h[i] + delta[i];
         h[i] = t;
         ss = fmaf(t, t, ss);
     }
@@ -118,6 +126,7 @@ dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __
         if (i < hidden) store_act(xn, act_dt, i, (v[r] / rms) * wv[r]);
     }
     for (int i = threadIdx.x + 8 * 1024; i < hidden; i += 1024) store_act(xn, act_dt, i, (h[i] / rms) * w[i]);
+    for (int i = hidden + threadIdx.x; i < xn_ld; i += 1024) store_act(xn, act_dt, i, 0.0f);
 }
 
 // One CTA per head (query heads, then key heads, then value heads), one thread per dimension:
@@ -446,25 +455,27 @@ __global__ void dec_argmax_exchange_kernel(const float *__restrict__ bv_in, cons
 
 // ---- prompt pass: the same operations over a block of rows (one row per prompt token) ----
 
-// row r: h = embedding of tokens[r] (first layer) or h += delta; xn = RMSNorm(h) * w. One CTA per row.
+// row r: h = embedding of tokens[r] (first layer) or h += delta; xn = RMSNorm(h) * w, zeros from hidden to
+// xn_ld. One CTA per row. With `rows` given CTA i norms row rows[i] into row i of xn and leaves h as it is.
 __global__ void __launch_bounds__(256)
 dec_norm_rows_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
                      const int *__restrict__ tokens, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                     int hidden) {
+                     int hidden, int embed_ld, int xn_ld, const int *__restrict__ rows) {
     __shared__ float red[32];
-    const size_t r = blockIdx.x;
+    const size_t r = rows ? rows[blockIdx.x] : blockIdx.x;
     float *hr = h + r * hidden;
     const float *dr = delta ? delta + r * hidden : nullptr;
-    const __nv_bfloat16 *er = embed ? embed + (size_t)tokens[r] * hidden : nullptr;
+    const __nv_bfloat16 *er = embed ? embed + (size_t)tokens[r] * embed_ld : nullptr;
     float ss = 0.0f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         const float v = er ? __bfloat162float(er[i]) : hr[i] + dr[i];
-        hr[i] = v;
+        if (!rows) hr[i] = v;
         ss = fmaf(v, v, ss);
     }
     const float rms = sqrtf(block_sum(ss, red) / (float)hidden + eps);
-    char *xr = reinterpret_cast<char *>(xn) + r * hidden * (act_dt == NNQ_F32 ? 4 : 2);
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) store_act(xr, act_dt, i, (hr[i] / rms) * w[i]);
+    char *xr = reinterpret_cast<char *>(xn) + (size_t)blockIdx.x * xn_ld * (act_dt == NNQ_F32 ? 4 : 2);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) store_act(xr, act_dt, i, ((rows ? hr[i] + dr[i] : hr[i]) / rms) * w[i]);
+    for (int i = hidden + threadIdx.x; i < xn_ld; i += blockDim.x) store_act(xr, act_dt, i, 0.0f);
 }
 
 // grid (heads, rows): per-head RMSNorm + half-split rotation at position pos0 + row, append of k / v
@@ -629,6 +640,7 @@ nnq_status nnq_decoder_create(nnq_ctx *ctx, const nnq_decoder_config *cfg, nnq_d
     d->ctx = ctx;
     d->cfg = c;
     d->act_dt = c.act_dtype;
+    d->embed_ld = d->xn_ld = c.hidden;
     d->lh = c.n_heads / c.tp_world;
     d->lkv = c.n_kv_heads / c.tp_world;
     d->head_rows = c.vocab;
@@ -706,6 +718,7 @@ nnq_status nnq_decoder_set_layer(nnq_decoder *d, int layer, const nnq_weight *q,
     if (!d) return NNQ_ERR_INVALID_ARG;
     nnq_ctx *ctx = d->ctx;
     const nnq_decoder_config &c = d->cfg;
+    if (!d->layers) return fail(ctx, NNQ_ERR_INVALID_ARG, "this decoder is made of blocks: use nnq_decoder_set_block");
     if (layer < 0 || layer >= c.n_layers) return fail(ctx, NNQ_ERR_INVALID_ARG, "layer %d out of range", layer);
     if (!in_norm || !post_norm || !q_norm || !k_norm) return fail(ctx, NNQ_ERR_INVALID_ARG, "NULL norm weight");
     // with tensor parallelism: this rank's column shards of q / k / v / gate / up and row shards of o / down
@@ -728,6 +741,7 @@ nnq_status nnq_decoder_set_layer(nnq_decoder *d, int layer, const nnq_weight *q,
 nnq_status nnq_decoder_set_head(nnq_decoder *d, const void *embed_bf16_dev, const float *final_norm, const nnq_weight *lm_head) {
     if (!d) return NNQ_ERR_INVALID_ARG;
     nnq_ctx *ctx = d->ctx;
+    if (!d->layers) return fail(ctx, NNQ_ERR_INVALID_ARG, "this decoder is made of blocks: use nnq_decoder_set_head_weights");
     if (!embed_bf16_dev || !final_norm) return fail(ctx, NNQ_ERR_INVALID_ARG, "NULL tensor");
     // tensor parallel: either the whole [vocab, hidden] projection on every rank, or this rank's
     // rows [rank * vocab / world, (rank + 1) * vocab / world) of it (vocabulary parallel: the ranks
@@ -750,6 +764,260 @@ nnq_status nnq_decoder_set_head(nnq_decoder *d, const void *embed_bf16_dev, cons
     return check_cuda(ctx, cudaMemcpy(d->d_final_norm, final_norm, (size_t)d->cfg.hidden * 4, cudaMemcpyDefault), "final norm");
 }
 
+// ---- block decoders ----
+
+static nnq_status check_block(nnq_ctx *ctx, int l, const nnq_block_config &b) {
+    if (b.mixer != NNQ_MIXER_ATTENTION && b.mixer != NNQ_MIXER_RECURRENT) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: unknown mixer %d", l, b.mixer);
+    if (b.heads < 1 || b.dim < 1 || b.vdim < 1 || b.ffn < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad sizes", l);
+    if (b.rot_dims < 0 || b.rot_dims % 2 || b.rot_dims > b.dim || (b.rot_dims && !(b.rot_base > 0.0)))
+        return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad rotation (%d of %d dimensions)", l, b.rot_dims, b.dim);
+    if (b.mixer == NNQ_MIXER_ATTENTION) {
+        if (b.kv_heads < 1 || b.heads % b.kv_heads) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: %d query heads over %d key/value heads", l, b.heads, b.kv_heads);
+        if (b.window < 0 || b.conv_taps < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad window or convolution", l);
+        if (b.dim > 1024 || b.vdim > kAttnMaxValueDim)
+            return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: attention heads of %d / %d are above 1024 / %d", l, b.dim, b.vdim, kAttnMaxValueDim);
+    } else {
+        if (b.decay_rank < 0 || (b.decay_rank > 0 && !(b.decay_tau > 0.0f))) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad decay", l);
+        if (b.dim > kRecMaxKeyDim || b.vdim > 2048)
+            return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: recurrent heads of %d / %d are above %d / 2048", l, b.dim, b.vdim, kRecMaxKeyDim);
+    }
+    return NNQ_OK;
+}
+
+static nnq_block_layout layout_of(const nnq_block_config &b, int hidden) {
+    nnq_block_layout y = {};
+    const bool attn = b.mixer == NNQ_MIXER_ATTENTION;
+    const int kvh = attn ? b.kv_heads : b.heads;
+    int at = 0;
+    auto take = [&](int width) {
+        if (width == 0) return -1;
+        const int c = at;
+        at += round_up(width, 8);
+        return c;
+    };
+    y.q = take(b.heads * b.dim);
+    y.k = take(kvh * b.dim);
+    y.v = take(kvh * b.vdim);
+    y.g = take(!attn || b.out_gate ? b.heads * b.vdim : 0);
+    y.a1 = take(attn ? 0 : b.decay_rank);
+    y.gate = take(b.ffn);
+    y.up = take(b.ffn);
+    y.in_cols = at;
+    y.in_k = round_up(hidden, 64);   // one k step of the tensor-core products
+    y.ffn_col = round_up(b.heads * b.vdim, 8);
+    y.out_k = round_up(y.ffn_col + b.ffn, 64);
+    return y;
+}
+
+nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg, const nnq_block_config *blocks, int block_rows, nnq_decoder **out) {
+    if (!ctx || !cfg || !blocks || !out) return NNQ_ERR_INVALID_ARG;
+    *out = nullptr;
+    nnq_decoder_config c = *cfg;
+    if (c.tp_world == 0) c.tp_world = 1;
+    if (c.tp_world != 1) return fail(ctx, NNQ_ERR_UNSUPPORTED, "block decoders run on one device");
+    if (c.hidden < 1 || c.n_layers < 1 || c.vocab < 1 || c.max_seq < 1 || block_rows < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "bad decoder dimensions");
+    if (c.act_dtype != NNQ_F32 && c.act_dtype != NNQ_BF16) return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown activation dtype");
+    nnq_status s = NNQ_OK;
+    int first_mix = -1;
+    for (int l = 0; l < c.n_layers; l++) {
+        if ((s = check_block(ctx, l, blocks[l])) != NNQ_OK) return s;
+        if (blocks[l].mixer != NNQ_MIXER_ATTENTION || !blocks[l].value_mix) continue;
+        if (first_mix < 0) first_mix = l;
+        else if (blocks[l].kv_heads * blocks[l].vdim != blocks[first_mix].kv_heads * blocks[first_mix].vdim)
+            return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d mixes values of another width than block %d", l, first_mix);
+    }
+    if ((s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice")) != NNQ_OK) return s;
+    nnq_decoder *d = new (std::nothrow) nnq_decoder();
+    if (!d) return fail(ctx, NNQ_ERR_OUT_OF_MEMORY, "host allocation failed");
+    memset(d, 0, sizeof(*d));
+    d->ctx = ctx;
+    d->cfg = c;
+    d->act_dt = c.act_dtype;
+    d->head_rows = c.vocab;
+    d->host_pos = -1;
+    d->xn_ld = d->embed_ld = round_up(c.hidden, 64);
+    d->blocks = new (std::nothrow) nnq_decoder::Block[c.n_layers]();
+    if (!d->blocks) {
+        delete d;
+        return fail(ctx, NNQ_ERR_OUT_OF_MEMORY, "host allocation failed");
+    }
+    const int want_rows = block_rows ? block_rows : kPrefillRows;
+    const int rows = d->pf_rows = want_rows < c.max_seq ? want_rows : c.max_seq;
+    const size_t R = rows, es = c.act_dtype == NNQ_F32 ? 4 : 2;
+    size_t proj = 0, act = 0, q = 0, k = 0, o = 0, vf = 0, part = 0, counters = 1;
+    auto alloc = [&](void *pp, size_t bytes, const char *what) {
+        if (s == NNQ_OK) s = dev_alloc(ctx, (void **)pp, bytes, what);
+    };
+    auto most = [](size_t &m, size_t v) { if (v > m) m = v; };
+    for (int l = 0; l < c.n_layers && s == NNQ_OK; l++) {
+        nnq_decoder::Block &B = d->blocks[l];
+        B.cfg = blocks[l];
+        B.lay = layout_of(B.cfg, c.hidden);
+        const nnq_block_config &b = B.cfg;
+        most(proj, B.lay.in_cols);
+        most(act, B.lay.out_k);
+        alloc(&B.norm, (size_t)c.hidden * 4, "norm weight");
+        if (b.mixer == NNQ_MIXER_ATTENTION) {
+            B.dim_ld = round_up(b.dim, 4);
+            B.vdim_ld = round_up(b.vdim, 4);
+            // a block of rows writes its keys before it reads: window - 1 older positions stay beside them
+            B.cap = b.window > 0 && (long long)b.window - 1 + rows < c.max_seq ? b.window - 1 + rows : c.max_seq;
+            B.ranges = attn_decode_ranges(b.window > 0 ? b.window : c.max_seq, c.max_seq);
+            B.mix_mode = !b.value_mix ? 0 : (l == first_mix ? 1 : 2);
+            const int channels = b.heads * b.dim + b.kv_heads * (b.dim + b.vdim);
+            alloc(&B.kcache, (size_t)b.kv_heads * B.cap * B.dim_ld * 4, "key cache");
+            alloc(&B.vcache, (size_t)b.kv_heads * B.cap * B.vdim_ld * 4, "value cache");
+            if (b.conv_taps > 0) {
+                alloc(&B.conv, (size_t)channels * b.conv_taps * 4, "convolution taps");
+                alloc(&B.conv_ring, (size_t)channels * b.conv_taps * 4, "convolution state");
+            }
+            most(q, (size_t)b.heads * B.dim_ld);
+            if (b.value_mix) most(vf, (size_t)b.kv_heads * b.vdim);
+            most(part, attn_decode_part_floats(b.heads, b.kv_heads, B.vdim_ld, B.ranges));
+            most(counters, attn_decode_counters(b.heads, b.kv_heads));
+        } else {
+            B.dim_ld = round_up(b.dim, 32);
+            alloc(&B.rec_state, (size_t)b.heads * b.dim * b.vdim * 4, "recurrent state");
+            if (b.decay_rank > 0) {
+                alloc(&B.a2t, (size_t)b.heads * b.dim * b.decay_rank * 4, "decay weight");
+                alloc(&B.a2b, (size_t)b.heads * b.dim * 4, "decay bias");
+            } else {
+                alloc(&B.decay, (size_t)b.heads * 4, "decay");
+            }
+            most(q, (size_t)b.heads * B.dim_ld);
+            most(k, (size_t)b.heads * B.dim_ld);
+            most(o, (size_t)b.heads * b.vdim);
+        }
+        if (b.rot_dims > 0) {
+            for (int j = 0; j < l && !B.cosv; j++)
+                if (d->blocks[j].cfg.rot_dims == b.rot_dims && d->blocks[j].cfg.rot_base == b.rot_base) {
+                    B.cosv = d->blocks[j].cosv;
+                    B.sinv = d->blocks[j].sinv;
+                }
+            if (!B.cosv) {
+                const int half = b.rot_dims / 2;
+                const size_t n = (size_t)c.max_seq * half;
+                B.owns_tables = true;
+                alloc(&B.cosv, n * 4, "rotation table");
+                alloc(&B.sinv, n * 4, "rotation table");
+                float *hc = new (std::nothrow) float[n], *hs = new (std::nothrow) float[n];
+                if (!hc || !hs) s = fail(ctx, NNQ_ERR_OUT_OF_MEMORY, "host allocation failed");
+                if (s == NNQ_OK) {
+                    // angles in f64: the tables are the correctly rounded sine and cosine at any position
+                    for (int i = 0; i < half; i++) {
+                        const double f = pow(b.rot_base, -2.0 * i / b.rot_dims);
+                        for (int p = 0; p < c.max_seq; p++) {
+                            hc[(size_t)p * half + i] = (float)cos(p * f);
+                            hs[(size_t)p * half + i] = (float)sin(p * f);
+                        }
+                    }
+                    s = check_cuda(ctx, cudaMemcpy(B.cosv, hc, n * 4, cudaMemcpyHostToDevice), "rotation table");
+                    if (s == NNQ_OK) s = check_cuda(ctx, cudaMemcpy(B.sinv, hs, n * 4, cudaMemcpyHostToDevice), "rotation table");
+                }
+                delete[] hc;
+                delete[] hs;
+            }
+        }
+    }
+    alloc(&d->d_h, (size_t)c.hidden * 4, "decoder buffer");
+    alloc(&d->d_delta, (size_t)c.hidden * 4, "decoder buffer");
+    alloc(&d->d_xn, (size_t)d->xn_ld * es, "decoder buffer");
+    alloc(&d->d_logits, (size_t)c.vocab * 4, "decoder buffer");
+    alloc(&d->d_final_norm, (size_t)c.hidden * 4, "final norm");
+    alloc(&d->d_state, (4 + 2 * kArgmaxBlocks) * 4, "decoder state");
+    alloc(&d->d_tokens, (size_t)c.max_seq * 4, "token log");
+    alloc(&d->d_part, part * 4, "attention partials");
+    alloc(&d->d_arrived, counters * 4, "attention arrival counters");
+    alloc(&d->pf_h, R * c.hidden * 4, "row buffer");
+    alloc(&d->pf_delta, R * c.hidden * 4, "row buffer");
+    alloc(&d->pf_xn, R * d->xn_ld * es, "row buffer");
+    alloc(&d->pf_tokens, R * 4, "row buffer");
+    alloc(&d->pf_want, R * 4, "row buffer");
+    alloc(&d->b_proj, R * proj * 4, "row buffer");
+    alloc(&d->b_act, R * act * es, "row buffer");
+    alloc(&d->b_q, R * q * 4, "row buffer");
+    alloc(&d->b_k, R * k * 4, "row buffer");
+    alloc(&d->b_a, R * k * 4, "row buffer");
+    alloc(&d->b_o, R * o * 4, "row buffer");
+    alloc(&d->b_vfirst, R * vf * 4, "row buffer");
+    if (s != NNQ_OK) {
+        nnq_decoder_destroy(d);
+        return s;
+    }
+    *out = d;
+    return NNQ_OK;
+}
+
+nnq_status nnq_decoder_block_layout(const nnq_decoder *d, int layer, nnq_block_layout *out) {
+    if (!d || !out) return NNQ_ERR_INVALID_ARG;
+    if (!d->blocks || layer < 0 || layer >= d->cfg.n_layers) return fail(d->ctx, NNQ_ERR_INVALID_ARG, "no block %d", layer);
+    *out = d->blocks[layer].lay;
+    return NNQ_OK;
+}
+
+nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_block_weights *w) {
+    if (!d || !w) return NNQ_ERR_INVALID_ARG;
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    if (!d->blocks || layer < 0 || layer >= c.n_layers) return fail(ctx, NNQ_ERR_INVALID_ARG, "no block %d", layer);
+    nnq_decoder::Block &B = d->blocks[layer];
+    const nnq_block_config &b = B.cfg;
+    if (!shape_is(w->in, B.lay.in_cols, B.lay.in_k) || !shape_is(w->out, c.hidden, B.lay.out_k))
+        return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "products of block %d must be [%d, %d] and [%d, %d]", layer, B.lay.in_cols, B.lay.in_k, c.hidden, B.lay.out_k);
+    if (!w->norm || (B.conv && !w->conv) || (B.a2t && (!w->decay_w || !w->decay_b)) || (B.decay && !w->decay))
+        return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d lacks a tensor", layer);
+    nnq_status s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
+    auto copy = [&](float *dst, const float *src, size_t n, const char *what) {
+        if (s == NNQ_OK) s = check_cuda(ctx, cudaMemcpy(dst, src, n * 4, cudaMemcpyDefault), what);
+    };
+    auto optional = [&](float **dst, const float *src, size_t n, const char *what) {
+        if (!src || s != NNQ_OK) return;
+        if (!*dst) s = dev_alloc(ctx, (void **)dst, n * 4, what);
+        copy(*dst, src, n, what);
+    };
+    copy(B.norm, w->norm, c.hidden, "norm weight");
+    optional(&B.bias_in, w->bias_in, B.lay.in_cols, "bias");
+    optional(&B.bias_out, w->bias_out, c.hidden, "bias");
+    optional(&B.head_norm, b.mixer == NNQ_MIXER_RECURRENT ? w->head_norm : nullptr, b.vdim, "head norm weight");
+    if (B.conv) copy(B.conv, w->conv, (size_t)(b.heads * b.dim + b.kv_heads * (b.dim + b.vdim)) * b.conv_taps, "convolution taps");
+    if (B.decay) copy(B.decay, w->decay, b.heads, "decay");
+    if (B.a2t && s == NNQ_OK) {
+        // [channels, rank] -> [rank, channels]: neighbouring channels are neighbouring lanes
+        const size_t n = (size_t)b.heads * b.dim, r = b.decay_rank;
+        float *src = new (std::nothrow) float[2 * n * r];
+        if (!src) return fail(ctx, NNQ_ERR_OUT_OF_MEMORY, "host allocation failed");
+        float *t = src + n * r;
+        s = check_cuda(ctx, cudaMemcpy(src, w->decay_w, n * r * 4, cudaMemcpyDefault), "decay weight");
+        for (size_t i = 0; i < n; i++)
+            for (size_t j = 0; j < r; j++) t[j * n + i] = src[i * r + j];
+        copy(B.a2t, t, n * r, "decay weight");
+        delete[] src;
+        copy(B.a2b, w->decay_b, n, "decay bias");
+    }
+    B.lambda = w->lambda;
+    if (s == NNQ_OK) {
+        B.in = w->in;
+        B.out = w->out;
+    }
+    return s;
+}
+
+nnq_status nnq_decoder_set_head_weights(nnq_decoder *d, const nnq_weight *embed, const float *final_norm, const nnq_weight *lm_head) {
+    if (!d) return NNQ_ERR_INVALID_ARG;
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    if (!d->blocks) return fail(ctx, NNQ_ERR_INVALID_ARG, "not a block decoder: use nnq_decoder_set_head");
+    if (!final_norm || !shape_is(embed, c.vocab, d->embed_ld) || embed->fmt != NNQ_BF16_DENSE || !shape_is(lm_head, c.vocab, d->xn_ld))
+        return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "embedding (bf16) and vocabulary projection must be [%d, %d]", c.vocab, d->xn_ld);
+    nnq_status s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
+    if (s == NNQ_OK) s = check_cuda(ctx, cudaMemcpy(d->d_final_norm, final_norm, (size_t)c.hidden * 4, cudaMemcpyDefault), "final norm");
+    if (s != NNQ_OK) return s;
+    d->d_embed = embed->d_raw;
+    d->lm_head = lm_head;
+    d->ready = 1;
+    return NNQ_OK;
+}
+
 nnq_status nnq_decoder_set_comm(nnq_decoder *d, nnq_comm *comm) {
     if (!d) return NNQ_ERR_INVALID_ARG;
     if (d->cfg.tp_world > 1 && !comm) return fail(d->ctx, NNQ_ERR_INVALID_ARG, "a tensor-parallel decoder needs a communicator");
@@ -762,8 +1030,15 @@ nnq_status nnq_decoder_reset(nnq_decoder *d, int token, int pos, void *stream) {
     if (token < 0 || token >= d->cfg.vocab || pos < 0 || pos >= d->cfg.max_seq) return fail(d->ctx, NNQ_ERR_INVALID_ARG, "token or position out of range");
     cudaSetDevice(d->ctx->device);
     const int st[4] = {token, pos, 0, 0};
+    nnq_status s = NNQ_OK;
+    if (d->blocks && pos != 0) {
+        // recurrent state and convolution inputs exist for one position only
+        int at = 0;
+        if ((s = nnq_decoder_state(d, nullptr, &at, nullptr, stream)) != NNQ_OK) return s;
+        if (at != pos) return fail(d->ctx, NNQ_ERR_INVALID_ARG, "the decoder's state is at position %d: it can continue there or restart at 0, not at %d", at, pos);
+    }
     d->host_pos = pos;
-    nnq_status s = check_cuda(d->ctx, cudaMemcpyAsync(d->d_state, st, sizeof(st), cudaMemcpyHostToDevice, (cudaStream_t)stream), "decoder state");
+    s = check_cuda(d->ctx, cudaMemcpyAsync(d->d_state, st, sizeof(st), cudaMemcpyHostToDevice, (cudaStream_t)stream), "decoder state");
     if (s == NNQ_OK) s = check_cuda(d->ctx, cudaStreamSynchronize((cudaStream_t)stream), "decoder state");   // st is on the stack
     return s;
 }
@@ -777,6 +1052,13 @@ nnq_status nnq_decoder_buffers(nnq_decoder *d, float **k_cache, float **v_cache,
     return NNQ_OK;
 }
 
+// A product of the decoder: blocks with f32 activations keep f32 operands throughout.
+static nnq_status product(nnq_decoder *d, const nnq_weight *w, const void *x, int64_t m, const float *bias, float *y, cudaStream_t st) {
+    if (!d->blocks || d->act_dt != NNQ_F32) return nnq_linear(d->ctx, w, x, (nnq_dtype)d->act_dt, m, bias, y, NNQ_F32, st);
+    LinearArgs a = {w->d_raw, w->d_scales, x, bias, y, m, w->n, w->k, w->fmt, NNQ_F32, NNQ_F32};
+    return launch_linear_f32(d->ctx, a, st);
+}
+
 // Vocabulary projection of the normed state in d_xn, greedy argmax (exchanged between the ranks
 // when the projection is split by rows), commit of the token and advance of the position.
 static nnq_status launch_head(nnq_decoder *d, bool vocab_parallel, const CommView &cv, cudaStream_t st) {
@@ -785,7 +1067,7 @@ static nnq_status launch_head(nnq_decoder *d, bool vocab_parallel, const CommVie
     nnq_status s;
     // the logits of this rank's rows land at their global offsets in the [vocab] buffer
     float *logits = d->d_logits + d->head_row0;
-    if ((s = nnq_linear(ctx, d->lm_head, d->d_xn, (nnq_dtype)d->act_dt, 1, nullptr, logits, NNQ_F32, st)) != NNQ_OK) return s;
+    if ((s = product(d, d->lm_head, d->d_xn, 1, nullptr, logits, st)) != NNQ_OK) return s;
     float *bv = reinterpret_cast<float *>(d->d_state + 4);
     int *bi = d->d_state + 4 + kArgmaxBlocks;
     launch_pdl(dec_argmax_stage1_kernel, dim3(kArgmaxBlocks), dim3(256), st, logits, d->head_rows, bv, bi);
@@ -824,27 +1106,90 @@ static int dec_skip() {
 #define DEC_RUN(bit, ...) do { __VA_ARGS__; } while (0)
 #endif
 
-nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
-    if (!d) return NNQ_ERR_INVALID_ARG;
+static nnq_status ready_to_run(const nnq_decoder *d) {
     nnq_ctx *ctx = d->ctx;
-    if (!d->ready) return fail(ctx, NNQ_ERR_INVALID_ARG, "decoder head has not been set");
     const nnq_decoder_config &c = d->cfg;
+    if (!d->ready) return fail(ctx, NNQ_ERR_INVALID_ARG, "decoder head has not been set");
     if (c.tp_world > 1 && !d->comm) return fail(ctx, NNQ_ERR_INVALID_ARG, "communicator has not been set");
     for (int l = 0; l < c.n_layers; l++)
-        if (!d->layers[l].q) return fail(ctx, NNQ_ERR_INVALID_ARG, "layer %d has not been set", l);
-    // The caches hold max_seq positions and never grow (the reference's KvCacheLayer::append doubles
-    // its buffer instead): a step past the last position is refused here, and -- for captured graphs
-    // that the host does not see being replayed -- by the device-side flag behind nnq_device_status.
-    if (d->host_pos >= c.max_seq)
-        return fail(ctx, NNQ_ERR_UNSUPPORTED, "the decoder's context is full (max_seq = %d positions): reset it", c.max_seq);
-    if (d->host_pos >= 0) d->host_pos++;
-    bool vocab_parallel = false;
-    CommView cv = {};
-    nnq_status s = head_mode(d, &vocab_parallel, &cv);
-    if (s != NNQ_OK) return s;
-    s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
-    if (s != NNQ_OK) return s;
-    cudaStream_t st = (cudaStream_t)stream;
+        if (d->blocks ? !d->blocks[l].in : !d->layers[l].q) return fail(ctx, NNQ_ERR_INVALID_ARG, "layer %d has not been set", l);
+    return NNQ_OK;
+}
+
+// Everything between the norm and the residual of block l for n rows: xn -> delta. `state` given: a decode
+// step (n = 1, position in state[1]), else rows from position pos0.
+static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *state, const void *xn, float *delta, cudaStream_t st) {
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder::Block &B = d->blocks[l];
+    const nnq_block_config &k = B.cfg;
+    nnq_status s;
+    if ((s = product(d, B.in, xn, n, B.bias_in, d->b_proj, st)) != NNQ_OK) return s;
+    const RowSpan span = {n, pos0, state};
+    const FfnPart ffn = {d->b_proj, B.lay.in_cols, B.lay.gate, B.lay.up, k.ffn, d->b_act, d->act_dt, B.lay.out_k, k.heads * k.vdim, B.lay.ffn_col};
+    if (k.mixer == NNQ_MIXER_ATTENTION) {
+        WindowAttn a = {};
+        a.span = span;
+        a.ffn = ffn;
+        a.heads = k.heads; a.kv_heads = k.kv_heads; a.dim = k.dim; a.vdim = k.vdim; a.dim_ld = B.dim_ld; a.vdim_ld = B.vdim_ld;
+        a.c_q = B.lay.q; a.c_k = B.lay.k; a.c_v = B.lay.v; a.c_g = B.lay.g;
+        a.gated = k.out_gate;
+        a.taps = k.conv_taps; a.conv = B.conv; a.conv_ring = B.conv_ring;
+        a.rot_dims = k.rot_dims; a.cosv = B.cosv; a.sinv = B.sinv;
+        a.mix_mode = B.mix_mode; a.lambda = B.lambda; a.vfirst = d->b_vfirst;
+        a.scale = k.scale; a.window = k.window > 0 ? k.window : (1 << 30);
+        a.qrot = d->b_q; a.kcache = B.kcache; a.vcache = B.vcache; a.cap = B.cap;
+        a.ranges = B.ranges; a.part = d->d_part; a.arrived = d->d_arrived;
+        if ((s = launch_attn_prep(ctx, a, st)) != NNQ_OK) return s;
+        if (state) {
+            if ((s = launch_attn_decode(ctx, a, st)) != NNQ_OK) return s;
+        } else {
+            if ((s = launch_attn_conv_tail(ctx, a, st)) != NNQ_OK) return s;
+            if ((s = launch_attn_rows(ctx, a, st)) != NNQ_OK) return s;
+        }
+    } else {
+        Recurrence r = {};
+        r.span = span;
+        r.ffn = ffn;
+        r.heads = k.heads; r.dim = k.dim; r.vdim = k.vdim; r.dim_ld = B.dim_ld;
+        r.c_q = B.lay.q; r.c_k = B.lay.k; r.c_v = B.lay.v; r.c_g = B.lay.g; r.c_a1 = B.lay.a1;
+        r.q_scale = k.q_scale; r.k_scale = k.k_scale;
+        r.rot_dims = k.rot_dims; r.cosv = B.cosv; r.sinv = B.sinv;
+        r.rank = k.decay_rank; r.a2t = B.a2t; r.a2b = B.a2b; r.inv_tau = k.decay_rank > 0 ? 1.0f / k.decay_tau : 0.0f; r.decay = B.decay;
+        r.head_norm = B.head_norm; r.eps = d->cfg.rms_eps;
+        r.state = B.rec_state; r.q = d->b_q; r.k = d->b_k; r.a = d->b_a; r.o = d->b_o;
+        if ((s = state ? launch_rec_step(ctx, r, st) : launch_rec_rows(ctx, r, st)) != NNQ_OK) return s;
+    }
+    return product(d, B.out, d->b_act, n, B.bias_out, delta, st);
+}
+
+static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
+    const nnq_decoder_config &c = d->cfg;
+    for (int l = 0; l < c.n_layers; l++) {
+        launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->d_state,
+                   d->blocks[l].norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld);
+        d->ctx->launches++;
+        nnq_status s = run_block(d, l, 1, 0, d->d_state, d->d_xn, d->d_delta, st);
+        if (s != NNQ_OK) return s;
+    }
+    return NNQ_OK;
+}
+
+static nnq_status rows_blocks(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
+    const nnq_decoder_config &c = d->cfg;
+    for (int l = 0; l < c.n_layers; l++) {
+        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->pf_tokens,
+                                                d->blocks[l].norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
+        d->ctx->launches++;
+        nnq_status s = run_block(d, l, n, pos0, nullptr, d->pf_xn, d->pf_delta, st);
+        if (s != NNQ_OK) return s;
+    }
+    return NNQ_OK;
+}
+
+static nnq_status step_qwen3(nnq_decoder *d, cudaStream_t st) {
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    nnq_status s = NNQ_OK;
     const int hd = c.head_dim, group = c.n_heads / c.n_kv_heads, lh = d->lh, lkv = d->lkv, lffn = c.ffn / c.tp_world;
     const nnq_dtype adt = (nnq_dtype)d->act_dt;
     const size_t layer_cache = (size_t)lkv * c.max_seq * hd;
@@ -852,7 +1197,7 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
     const __nv_bfloat16 *embed = (const __nv_bfloat16 *)d->d_embed;
     for (int l = 0; l < c.n_layers; l++) {
         const nnq_decoder::Layer &L = d->layers[l];
-        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? embed : nullptr, d->d_state, L.in_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden));
+        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? embed : nullptr, d->d_state, L.in_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld));
         const nnq_weight *w3[3] = {L.q, L.k, L.v};
         const void *x3[3] = {d->d_xn, d->d_xn, d->d_xn};
         void *y3[3] = {d->d_q, d->d_k, d->d_v};
@@ -874,7 +1219,7 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
         DEC_RUN(32, s = d->comm ? nnq_comm_linear(d->comm, L.o, d->d_attn, adt, 1, nullptr, d->d_delta, NNQ_F32, st)
                                 : nnq_linear(ctx, L.o, d->d_attn, adt, 1, nullptr, d->d_delta, NNQ_F32, st));
         if (s != NNQ_OK) return s;
-        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, L.post_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden));
+        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, L.post_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld));
         const nnq_weight *w2[2] = {L.gate, L.up};
         const void *x2[2] = {d->d_xn, d->d_xn};
         void *y2[2] = {d->d_g, d->d_u};
@@ -885,43 +1230,111 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
         if (s != NNQ_OK) return s;
         ctx->launches += 5;
     }
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden);
+    return NNQ_OK;
+}
+
+static nnq_status rows_qwen3(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    nnq_status s = NNQ_OK;
+    const int hd = c.head_dim, group = c.n_heads / c.n_kv_heads, lh = d->lh, lkv = d->lkv, lffn = c.ffn / c.tp_world;
+    const nnq_dtype adt = (nnq_dtype)d->act_dt;
+    const size_t layer_cache = (size_t)lkv * c.max_seq * hd;
+    const float scale = (float)(1.0 / sqrt((double)hd));
+    const __nv_bfloat16 *embed = (const __nv_bfloat16 *)d->d_embed;
+    for (int l = 0; l < c.n_layers; l++) {
+        const nnq_decoder::Layer &L = d->layers[l];
+        float *kc = d->d_kcache + l * layer_cache, *vc = d->d_vcache + l * layer_cache;
+        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? embed : nullptr, d->pf_tokens, L.in_norm,
+                                                c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
+        const nnq_weight *w3[3] = {L.q, L.k, L.v};
+        const void *x3[3] = {d->pf_xn, d->pf_xn, d->pf_xn};
+        void *y3[3] = {d->pf_q, d->pf_k, d->pf_v};
+        if ((s = nnq_linear_batch(ctx, 3, w3, x3, adt, n, nullptr, y3, NNQ_F32, st)) != NNQ_OK) return s;
+        dec_qk_rope_rows_kernel<<<dim3(lh + 2 * lkv, n), hd, 0, st>>>(d->pf_q, d->pf_k, d->pf_v, L.q_norm, L.k_norm, d->d_cos, d->d_sin, pos0,
+                                                                     c.rms_eps, d->pf_qrot, kc, vc, lh, lkv, hd, c.max_seq);
+        // 16 query vectors per warp: R = 16 / G rows share each key / value row
+        switch (group) {
+            case 1: dec_attn_rows_kernel<1, 16><<<dim3(lkv, (n + 15) / 16), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
+            case 2: dec_attn_rows_kernel<2, 8><<<dim3(lkv, (n + 7) / 8), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
+            case 4: dec_attn_rows_kernel<4, 4><<<dim3(lkv, (n + 3) / 4), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
+            case 8: dec_attn_rows_kernel<8, 2><<<dim3(lkv, (n + 1) / 2), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
+            default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "query heads per key/value head must be 1, 2, 4 or 8");
+        }
+        s = d->comm ? nnq_comm_linear(d->comm, L.o, d->pf_attn, adt, n, nullptr, d->pf_delta, NNQ_F32, st)
+                    : nnq_linear(ctx, L.o, d->pf_attn, adt, n, nullptr, d->pf_delta, NNQ_F32, st);
+        if (s != NNQ_OK) return s;
+        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, d->pf_delta, nullptr, d->pf_tokens, L.post_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
+        const nnq_weight *w2[2] = {L.gate, L.up};
+        const void *x2[2] = {d->pf_xn, d->pf_xn};
+        void *y2[2] = {d->pf_g, d->pf_u};
+        if ((s = nnq_linear_batch(ctx, 2, w2, x2, adt, n, nullptr, y2, NNQ_F32, st)) != NNQ_OK) return s;
+        const int total = n * lffn;
+        dec_silu_mul_kernel<<<(total + 255) / 256, 256, 0, st>>>(d->pf_g, d->pf_u, d->pf_mid, d->act_dt, total);
+        s = d->comm ? nnq_comm_linear(d->comm, L.down, d->pf_mid, adt, n, nullptr, d->pf_delta, NNQ_F32, st)
+                    : nnq_linear(ctx, L.down, d->pf_mid, adt, n, nullptr, d->pf_delta, NNQ_F32, st);
+        if (s != NNQ_OK) return s;
+        ctx->launches += 5;
+    }
+    return NNQ_OK;
+}
+
+nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
+    if (!d) return NNQ_ERR_INVALID_ARG;
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    nnq_status s = ready_to_run(d);
+    if (s != NNQ_OK) return s;
+    // The caches hold max_seq positions and never grow (the reference's KvCacheLayer::append doubles
+    // its buffer instead): a step past the last position is refused here, and -- for captured graphs
+    // that the host does not see being replayed -- by the device-side flag behind nnq_device_status.
+    if (d->host_pos >= c.max_seq)
+        return fail(ctx, NNQ_ERR_UNSUPPORTED, "the decoder's context is full (max_seq = %d positions): reset it", c.max_seq);
+    if (d->host_pos >= 0) d->host_pos++;
+    bool vocab_parallel = false;
+    CommView cv = {};
+    if ((s = head_mode(d, &vocab_parallel, &cv)) != NNQ_OK) return s;
+    s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
+    if (s != NNQ_OK) return s;
+    cudaStream_t st = (cudaStream_t)stream;
+    if ((s = d->blocks ? step_blocks(d, st) : step_qwen3(d, st)) != NNQ_OK) return s;
+    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld);
     ctx->launches++;
     return launch_head(d, vocab_parallel, cv, st);
 }
 
-nnq_status nnq_decoder_prefill(nnq_decoder *d, const int32_t *tokens_host, int count, int start_pos, void *stream) {
-    if (!d) return NNQ_ERR_INVALID_ARG;
+// Checks of a call that feeds `count` given tokens from position start_pos on.
+static nnq_status check_tokens(nnq_decoder *d, const int32_t *tokens_host, int count, int start_pos) {
     nnq_ctx *ctx = d->ctx;
     const nnq_decoder_config &c = d->cfg;
-    if (!d->ready) return fail(ctx, NNQ_ERR_INVALID_ARG, "decoder head has not been set");
-    if (c.tp_world > 1 && !d->comm) return fail(ctx, NNQ_ERR_INVALID_ARG, "communicator has not been set");
-    for (int l = 0; l < c.n_layers; l++)
-        if (!d->layers[l].q) return fail(ctx, NNQ_ERR_INVALID_ARG, "layer %d has not been set", l);
+    nnq_status s = ready_to_run(d);
+    if (s != NNQ_OK) return s;
     if (!tokens_host || count < 1 || start_pos < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "bad prompt arguments");
     if ((long long)start_pos + count > c.max_seq)
         return fail(ctx, NNQ_ERR_UNSUPPORTED, "a prompt of %d tokens at position %d does not fit max_seq = %d", count, start_pos, c.max_seq);
     for (int i = 0; i < count; i++)
         if (tokens_host[i] < 0 || tokens_host[i] >= c.vocab) return fail(ctx, NNQ_ERR_INVALID_ARG, "prompt token %d out of range", i);
-    bool vocab_parallel = false;
-    CommView cv = {};
-    nnq_status s = head_mode(d, &vocab_parallel, &cv);
-    if (s != NNQ_OK) return s;
-    if ((s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice")) != NNQ_OK) return s;
-    cudaStream_t st = (cudaStream_t)stream;
-    const int hd = c.head_dim, group = c.n_heads / c.n_kv_heads, lh = d->lh, lkv = d->lkv, lffn = c.ffn / c.tp_world;
-    const int qdim = lh * hd, kvdim = lkv * hd;
-    const nnq_dtype adt = (nnq_dtype)d->act_dt;
-    const size_t es = adt == NNQ_F32 ? 4 : 2;
-    // rows per pass: bounded by the scratch below and, with tensor parallelism, by what one exchange carries
-    int rows_max = kPrefillRows;
+    if (d->blocks && start_pos != 0 && start_pos != d->host_pos)
+        return fail(ctx, NNQ_ERR_INVALID_ARG, "the decoder's state is at position %lld: it can continue there or restart at 0, not at %d", d->host_pos, start_pos);
+    return NNQ_OK;
+}
+
+// Rows that go through the layers together: bounded by the row buffers (allocated here for Qwen3 layers)
+// and, with tensor parallelism, by what one exchange carries.
+static nnq_status row_buffers(nnq_decoder *d, int *rows_max) {
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    nnq_status s = NNQ_OK;
+    *rows_max = d->blocks ? d->pf_rows : kPrefillRows;
     if (d->comm) {
         CommView v;
         if ((s = comm_view(d->comm, &v)) != NNQ_OK) return s;
         const size_t fit = v.slot_bytes / ((size_t)c.hidden * 4);
         if (fit < 1) return fail(ctx, NNQ_ERR_UNSUPPORTED, "communicator slots are smaller than one row of the hidden state");
-        if ((size_t)rows_max > fit) rows_max = (int)fit;
+        if ((size_t)*rows_max > fit) *rows_max = (int)fit;
     }
+    const int qdim = d->lh * c.head_dim, kvdim = d->lkv * c.head_dim, lffn = d->blocks ? 0 : c.ffn / c.tp_world;
+    const size_t es = d->act_dt == NNQ_F32 ? 4 : 2;
     if (!d->pf_h) {
         d->pf_rows = kPrefillRows;
         const size_t R = kPrefillRows;
@@ -937,60 +1350,102 @@ nnq_status nnq_decoder_prefill(nnq_decoder *d, const int32_t *tokens_host, int c
         if (s == NNQ_OK) s = dev_alloc(ctx, &d->pf_attn, R * qdim * es, "prompt buffer");
         if (s == NNQ_OK) s = dev_alloc(ctx, &d->pf_mid, R * lffn * es, "prompt buffer");
         if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->pf_tokens, R * 4, "prompt buffer");
+        if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->pf_want, R * 4, "prompt buffer");
         if (s != NNQ_OK) return s;
     }
-    const size_t layer_cache = (size_t)lkv * c.max_seq * hd;
-    const float scale = (float)(1.0 / sqrt((double)hd));
-    const __nv_bfloat16 *embed = (const __nv_bfloat16 *)d->d_embed;
+    return NNQ_OK;
+}
+
+// n <= rows_max tokens through the layers: afterwards pf_h + pf_delta are the rows' final residuals.
+static nnq_status run_rows(nnq_decoder *d, const int32_t *tokens_host, int n, int pos0, cudaStream_t st) {
+    nnq_status s = check_cuda(d->ctx, cudaMemcpyAsync(d->pf_tokens, tokens_host, (size_t)n * 4, cudaMemcpyHostToDevice, st), "prompt tokens");
+    if (s != NNQ_OK) return s;
+    return d->blocks ? rows_blocks(d, n, pos0, st) : rows_qwen3(d, n, pos0, st);
+}
+
+nnq_status nnq_decoder_prefill(nnq_decoder *d, const int32_t *tokens_host, int count, int start_pos, void *stream) {
+    if (!d) return NNQ_ERR_INVALID_ARG;
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    nnq_status s = check_tokens(d, tokens_host, count, start_pos);
+    if (s != NNQ_OK) return s;
+    bool vocab_parallel = false;
+    CommView cv = {};
+    if ((s = head_mode(d, &vocab_parallel, &cv)) != NNQ_OK) return s;
+    if ((s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice")) != NNQ_OK) return s;
+    cudaStream_t st = (cudaStream_t)stream;
+    int rows_max = 0;
+    if ((s = row_buffers(d, &rows_max)) != NNQ_OK) return s;
+    d->host_pos = -1;   // until the call has gone through
     int n = 0;
     for (int c0 = 0; c0 < count; c0 += n) {
         n = count - c0 < rows_max ? count - c0 : rows_max;
-        const int pos0 = start_pos + c0;
-        if ((s = check_cuda(ctx, cudaMemcpyAsync(d->pf_tokens, tokens_host + c0, (size_t)n * 4, cudaMemcpyHostToDevice, st), "prompt tokens")) != NNQ_OK) return s;
-        for (int l = 0; l < c.n_layers; l++) {
-            const nnq_decoder::Layer &L = d->layers[l];
-            float *kc = d->d_kcache + l * layer_cache, *vc = d->d_vcache + l * layer_cache;
-            dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? embed : nullptr, d->pf_tokens, L.in_norm,
-                                                    c.rms_eps, d->pf_xn, d->act_dt, c.hidden);
-            const nnq_weight *w3[3] = {L.q, L.k, L.v};
-            const void *x3[3] = {d->pf_xn, d->pf_xn, d->pf_xn};
-            void *y3[3] = {d->pf_q, d->pf_k, d->pf_v};
-            if ((s = nnq_linear_batch(ctx, 3, w3, x3, adt, n, nullptr, y3, NNQ_F32, st)) != NNQ_OK) return s;
-            dec_qk_rope_rows_kernel<<<dim3(lh + 2 * lkv, n), hd, 0, st>>>(d->pf_q, d->pf_k, d->pf_v, L.q_norm, L.k_norm, d->d_cos, d->d_sin, pos0,
-                                                                         c.rms_eps, d->pf_qrot, kc, vc, lh, lkv, hd, c.max_seq);
-            // 16 query vectors per warp: R = 16 / G rows share each key / value row
-            switch (group) {
-                case 1: dec_attn_rows_kernel<1, 16><<<dim3(lkv, (n + 15) / 16), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
-                case 2: dec_attn_rows_kernel<2, 8><<<dim3(lkv, (n + 7) / 8), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
-                case 4: dec_attn_rows_kernel<4, 4><<<dim3(lkv, (n + 3) / 4), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
-                case 8: dec_attn_rows_kernel<8, 2><<<dim3(lkv, (n + 1) / 2), 32, 0, st>>>(d->pf_qrot, kc, vc, pos0, n, scale, d->pf_attn, d->act_dt, lh, hd, c.max_seq); break;
-                default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "query heads per key/value head must be 1, 2, 4 or 8");
-            }
-            s = d->comm ? nnq_comm_linear(d->comm, L.o, d->pf_attn, adt, n, nullptr, d->pf_delta, NNQ_F32, st)
-                        : nnq_linear(ctx, L.o, d->pf_attn, adt, n, nullptr, d->pf_delta, NNQ_F32, st);
-            if (s != NNQ_OK) return s;
-            dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, d->pf_delta, nullptr, d->pf_tokens, L.post_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden);
-            const nnq_weight *w2[2] = {L.gate, L.up};
-            const void *x2[2] = {d->pf_xn, d->pf_xn};
-            void *y2[2] = {d->pf_g, d->pf_u};
-            if ((s = nnq_linear_batch(ctx, 2, w2, x2, adt, n, nullptr, y2, NNQ_F32, st)) != NNQ_OK) return s;
-            const int total = n * lffn;
-            dec_silu_mul_kernel<<<(total + 255) / 256, 256, 0, st>>>(d->pf_g, d->pf_u, d->pf_mid, d->act_dt, total);
-            s = d->comm ? nnq_comm_linear(d->comm, L.down, d->pf_mid, adt, n, nullptr, d->pf_delta, NNQ_F32, st)
-                        : nnq_linear(ctx, L.down, d->pf_mid, adt, n, nullptr, d->pf_delta, NNQ_F32, st);
-            if (s != NNQ_OK) return s;
-            ctx->launches += 5;
-        }
+        if ((s = run_rows(d, tokens_host + c0, n, start_pos + c0, st)) != NNQ_OK) return s;
     }
     // the last prompt token's state: final norm, vocabulary projection, greedy successor
     const size_t last = (size_t)(n - 1) * c.hidden;
     const int st4[4] = {tokens_host[count - 1], start_pos + count - 1, 0, 0};
     if ((s = check_cuda(ctx, cudaMemcpyAsync(d->d_state, st4, sizeof(st4), cudaMemcpyHostToDevice, st), "decoder state")) != NNQ_OK) return s;
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->pf_h + last, d->pf_delta + last, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden);
+    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->pf_h + last, d->pf_delta + last, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld);
     ctx->launches++;
     if ((s = launch_head(d, vocab_parallel, cv, st)) != NNQ_OK) return s;
-    d->host_pos = (long long)start_pos + count;
-    return check_cuda(ctx, cudaStreamSynchronize(st), "prompt pass");   // tokens_host and st4 are the caller's / the stack's
+    s = check_cuda(ctx, cudaStreamSynchronize(st), "prompt pass");   // tokens_host and st4 are the caller's / the stack's
+    if (s == NNQ_OK) d->host_pos = (long long)start_pos + count;
+    return s;
+}
+
+nnq_status nnq_decoder_extend(nnq_decoder *d, const int32_t *tokens_host, int count, int start_pos, const int32_t *want, int n_want,
+                              float *logits_host, void *stream) {
+    if (!d) return NNQ_ERR_INVALID_ARG;
+    nnq_ctx *ctx = d->ctx;
+    const nnq_decoder_config &c = d->cfg;
+    nnq_status s = check_tokens(d, tokens_host, count, start_pos);
+    if (s != NNQ_OK) return s;
+    if (n_want < 0 || (n_want && (!want || !logits_host))) return fail(ctx, NNQ_ERR_INVALID_ARG, "bad list of wanted positions");
+    for (int i = 0; i < n_want; i++)
+        if (want[i] < 0 || want[i] >= count || (i && want[i] <= want[i - 1])) return fail(ctx, NNQ_ERR_INVALID_ARG, "wanted positions must be ascending and inside the tokens");
+    if (d->head_rows != c.vocab) return fail(ctx, NNQ_ERR_UNSUPPORTED, "wanted logits need the whole vocabulary projection on this rank");
+    if ((s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice")) != NNQ_OK) return s;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (count == 1) {
+        if ((s = nnq_decoder_reset(d, tokens_host[0], start_pos, stream)) != NNQ_OK) return s;
+        if ((s = nnq_decoder_step(d, stream)) != NNQ_OK) return s;
+        if (n_want) s = check_cuda(ctx, cudaMemcpyAsync(logits_host, d->d_logits, (size_t)c.vocab * 4, cudaMemcpyDeviceToHost, st), "logits");
+        if (s == NNQ_OK) s = check_cuda(ctx, cudaStreamSynchronize(st), "decoder step");
+        return s;
+    }
+    int rows_max = 0;
+    if ((s = row_buffers(d, &rows_max)) != NNQ_OK) return s;
+    if (n_want && !d->d_want_logits && (s = dev_alloc(ctx, (void **)&d->d_want_logits, (size_t)kWantRows * c.vocab * 4, "logits of wanted rows")) != NNQ_OK) return s;
+    d->host_pos = -1;   // until the call has gone through
+    int n = 0, w0 = 0;
+    for (int c0 = 0; c0 < count; c0 += n) {
+        n = count - c0 < rows_max ? count - c0 : rows_max;
+        if ((s = run_rows(d, tokens_host + c0, n, start_pos + c0, st)) != NNQ_OK) return s;
+        while (w0 < n_want && want[w0] < c0 + n) {
+            int32_t rows[kWantRows];
+            int m = 0;
+            while (m < kWantRows && w0 + m < n_want && want[w0 + m] < c0 + n) {
+                rows[m] = want[w0 + m] - c0;
+                m++;
+            }
+            if ((s = check_cuda(ctx, cudaMemcpyAsync(d->pf_want, rows, (size_t)m * 4, cudaMemcpyHostToDevice, st), "wanted rows")) != NNQ_OK) return s;
+            dec_norm_rows_kernel<<<m, 256, 0, st>>>(d->pf_h, d->pf_delta, nullptr, d->pf_tokens, d->d_final_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden,
+                                                    d->embed_ld, d->xn_ld, d->pf_want);
+            ctx->launches++;
+            if ((s = product(d, d->lm_head, d->pf_xn, m, nullptr, d->d_want_logits, st)) != NNQ_OK) return s;
+            s = check_cuda(ctx, cudaMemcpyAsync(logits_host + (size_t)w0 * c.vocab, d->d_want_logits, (size_t)m * c.vocab * 4, cudaMemcpyDeviceToHost, st), "logits");
+            if (s == NNQ_OK) s = check_cuda(ctx, cudaStreamSynchronize(st), "logits");   // rows[] is on the stack
+            if (s != NNQ_OK) return s;
+            w0 += m;
+        }
+    }
+    const bool full = start_pos + count >= c.max_seq;
+    const int st4[4] = {tokens_host[count - 1], full ? c.max_seq - 1 : start_pos + count, 0, full ? 1 : 0};
+    s = check_cuda(ctx, cudaMemcpyAsync(d->d_state, st4, sizeof(st4), cudaMemcpyHostToDevice, st), "decoder state");
+    if (s == NNQ_OK) s = check_cuda(ctx, cudaStreamSynchronize(st), "prompt pass");
+    if (s == NNQ_OK) d->host_pos = (long long)start_pos + count;
+    return s;
 }
 
 nnq_status nnq_decoder_state(nnq_decoder *d, int *token, int *pos, int *steps, void *stream) {
@@ -999,6 +1454,7 @@ nnq_status nnq_decoder_state(nnq_decoder *d, int *token, int *pos, int *steps, v
     int st[4] = {0, 0, 0, 0};
     nnq_status s = check_cuda(d->ctx, cudaMemcpyAsync(st, d->d_state, sizeof(st), cudaMemcpyDeviceToHost, (cudaStream_t)stream), "decoder state");
     if (s == NNQ_OK) s = check_cuda(d->ctx, cudaStreamSynchronize((cudaStream_t)stream), "decoder state");
+    if (s == NNQ_OK && (d->host_pos >= 0 || st[2] > 0)) d->host_pos = st[3] ? d->cfg.max_seq : st[1];   // replayed graphs advance it unseen
     if (token) *token = st[0];
     if (pos) *pos = st[1];
     if (steps) *steps = st[2];
@@ -1016,6 +1472,20 @@ void nnq_decoder_destroy(nnq_decoder *d) {
         }
         delete[] d->layers;
     }
+    if (d->blocks) {
+        for (int l = 0; l < d->cfg.n_layers; l++) {
+            nnq_decoder::Block &B = d->blocks[l];
+            cudaFree(B.norm); cudaFree(B.bias_in); cudaFree(B.bias_out); cudaFree(B.conv); cudaFree(B.head_norm);
+            cudaFree(B.a2t); cudaFree(B.a2b); cudaFree(B.decay); cudaFree(B.kcache); cudaFree(B.vcache);
+            cudaFree(B.conv_ring); cudaFree(B.rec_state);
+            if (B.owns_tables) {
+                cudaFree(B.cosv); cudaFree(B.sinv);
+            }
+        }
+        delete[] d->blocks;
+    }
+    cudaFree(d->b_proj); cudaFree(d->b_q); cudaFree(d->b_k); cudaFree(d->b_a); cudaFree(d->b_o); cudaFree(d->b_vfirst); cudaFree(d->b_act);
+    cudaFree(d->pf_want); cudaFree(d->d_want_logits);
     cudaFree(d->d_final_norm); cudaFree(d->d_cos); cudaFree(d->d_sin); cudaFree(d->d_kcache); cudaFree(d->d_vcache);
     cudaFree(d->d_h); cudaFree(d->d_delta); cudaFree(d->d_q); cudaFree(d->d_k); cudaFree(d->d_v); cudaFree(d->d_qrot);
     cudaFree(d->d_g); cudaFree(d->d_u); cudaFree(d->d_logits); cudaFree(d->d_part); cudaFree(d->d_arrived); cudaFree(d->d_xn); cudaFree(d->d_attn);

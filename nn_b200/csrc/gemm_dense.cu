@@ -530,8 +530,7 @@ static bool make_map(const void *base, int64_t rows, int64_t k, int box_rows, CU
 bool gemm_dense_shape_ok(const nnq_ctx *ctx, int64_t m, int64_t n, int64_t k, int x_dt) {
     static const char *env_min = diag_env("NNQ_DENSE_MIN_M");   // tuning aid
     const int64_t min_m = env_min ? atoll(env_min) : 256;
-    return ctx->d_dense && x_dt == NNQ_BF16 && m >= min_m && k >= kDgBK && k % kDgBK == 0 && n >= 1 &&
-           (size_t)n * (size_t)k * 2 <= ctx->dense_bytes && m < (1ll << 31) && n < (1ll << 31) && encode_fn() != nullptr;
+    return x_dt == NNQ_BF16 && m >= min_m && k >= kDgBK && k % kDgBK == 0 && n >= 1 && m < (1ll << 31) && n < (1ll << 31) && encode_fn() != nullptr;
 }
 bool gemm_dense_supported(const nnq_ctx *ctx, const nnq_weight *w, int64_t m, int x_dt) {
     // Formats whose fused decode reads its raw blocks through the TMA ring keep it for longer. Measured on
@@ -544,7 +543,9 @@ bool gemm_dense_supported(const nnq_ctx *ctx, const nnq_weight *w, int64_t m, in
         const bool q8 = w->fmt == NNQ_Q8_0 && w->k % 256 == 0;
         if ((q4k && m <= 512) || (q8 && m < 384)) return false;
     }
-    return w && w->d_raw && gemm_dense_shape_ok(ctx, m, w->n, w->k, x_dt);
+    if (!w || !w->d_raw || !gemm_dense_shape_ok(ctx, m, w->n, w->k, x_dt)) return false;
+    // a bf16 weight is multiplied in place, the others are decoded into the scratch
+    return (w->fmt == NNQ_BF16_DENSE && !((uintptr_t)w->d_raw & 15u)) || (ctx->d_dense && (size_t)w->n * (size_t)w->k * 2 <= ctx->dense_bytes);
 }
 
 nnq_status dense_scratch_reserve(nnq_ctx *ctx, int64_t n, int64_t k) {

@@ -633,7 +633,7 @@ nnq_status nnq_gq_linear(nnq_gq_weight *w, const void *x_dev, nnq_dtype x_dt, in
     cudaStream_t st = (cudaStream_t)stream;
     const int64_t n = w->n, k = w->k;
     // from 17 tokens on: one decode to bf16 in the context's scratch, then the tensor-core product
-    if (m > 16 && k >= 64 && k % 64 == 0 && ctx->d_dense && (size_t)n * (size_t)k * 2 <= ctx->dense_bytes && ctx->path != NNQ_PATH_GENERIC) {
+    if (m > 16 && k >= 64 && k % 64 == 0 && ctx->d_dense && (size_t)n * (size_t)k * 2 <= ctx->dense_bytes && ctx->path != NNQ_PATH_GENERIC && ctx->path != NNQ_PATH_F32) {
         s = check_cuda(ctx, launch_decode<__nv_bfloat16, float>(ctx, w->codes, w->scale, w->zpf, n, k, w->groups, w->group_size, w->bits, w->is_signed,
                                                                 reinterpret_cast<__nv_bfloat16 *>(ctx->d_dense), st), "bf16 decode launch");
         if (s != NNQ_OK) return s;

@@ -6,13 +6,20 @@ quantized products: Qwen3DecoderLayer / Qwen3Attention / Qwen3MLP forward
 ``Decoder`` binds nnq_decoder_* of the C ABI. Weights stay owned by the caller
 (``api.DeviceWeight`` / ``api.QuantizedTensor``); token and position live on the device, so
 ``step`` can be captured in a CUDA graph once and replayed per token (``generate`` does that).
+
+``BlockDecoder`` is the same decoder object made of blocks that each name their own mixer (sliding-window
+attention, linear-attention recurrences) and read one normed row per block.
 """
 from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
+from typing import List, Optional
+
+import numpy as np
 
 from . import api
+from .formats import QuantFormat
 
 
 class _Config(ctypes.Structure):
@@ -50,12 +57,18 @@ class _DevArray:
 class Decoder:
     def __init__(self, backend: api.Backend, cfg: DecoderConfig):
         self.backend, self.cfg = backend, cfg
-        c = _Config(cfg.hidden, cfg.n_heads, cfg.n_kv_heads, cfg.head_dim, cfg.ffn, cfg.n_layers, cfg.vocab,
-                    cfg.max_seq, cfg.rms_eps, cfg.rope_theta, cfg.act_dtype, cfg.tp_rank, cfg.tp_world)
         h = ctypes.c_void_p()
-        backend.check(backend._lib.nnq_decoder_create(backend._ctx, ctypes.byref(c), ctypes.byref(h)))
+        backend.check(self._create(self._c_config(), ctypes.byref(h)))
         self._handle = h
         self._keep = []   # tensors the library holds pointers to
+
+    def _c_config(self):
+        cfg = self.cfg
+        return _Config(cfg.hidden, cfg.n_heads, cfg.n_kv_heads, cfg.head_dim, cfg.ffn, cfg.n_layers, cfg.vocab,
+                       cfg.max_seq, cfg.rms_eps, cfg.rope_theta, cfg.act_dtype, cfg.tp_rank, cfg.tp_world)
+
+    def _create(self, c_config, out):
+        return self.backend._lib.nnq_decoder_create(self.backend._ctx, ctypes.byref(c_config), out)
 
     def set_layer(self, layer: int, q, k, v, o, gate, up, down, in_norm, post_norm, q_norm, k_norm):
         """Projections: quantized weights; norms: contiguous f32 torch tensors (any device) or numpy arrays."""
@@ -86,10 +99,21 @@ class Decoder:
     def prefill(self, tokens, start_pos: int = 0, stream=None):
         """Prompt pass over `tokens` (a sequence of ids) at positions start_pos ..: fills the caches,
         leaves the last prompt token's logits and its greedy successor as the next input."""
-        import numpy as np
         arr = np.ascontiguousarray(tokens, dtype=np.int32)
         self.backend.check(self.backend._lib.nnq_decoder_prefill(self._handle, arr.ctypes.data, int(arr.size), int(start_pos),
                                                                  api._stream_ptr(stream)))
+
+    def extend(self, tokens, start_pos: int, want=(), stream=None):
+        """Continue the sequence with given tokens at positions start_pos ..; returns the logits (numpy f32
+        [len(want), vocab]) after the tokens whose indexes `want` lists in ascending order. One token runs the
+        decode step, several run the prompt pass; start_pos 0 starts a new sequence."""
+        arr = np.ascontiguousarray(tokens, dtype=np.int32)
+        idx = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((idx.size, self.cfg.vocab), np.float32)
+        self.backend.check(self.backend._lib.nnq_decoder_extend(self._handle, arr.ctypes.data, int(arr.size), int(start_pos),
+                                                                idx.ctypes.data, int(idx.size), out.ctypes.data,
+                                                                api._stream_ptr(stream)))
+        return out
 
     def step(self, stream=None):
         self.backend.check(self.backend._lib.nnq_decoder_step(self._handle, api._stream_ptr(stream)))
@@ -119,31 +143,209 @@ class Decoder:
 
     def generate(self, first_token: int, pos: int, n_tokens: int, use_graph: bool = True):
         """Greedy decode of n_tokens starting with `first_token` at position `pos`; returns the
-        generated token ids (a list) — one captured graph replayed per token."""
+        generated token ids (a list) — one captured graph replayed per token after the first."""
         import torch
         dev = torch.device("cuda", self.backend.device)
         stream = torch.cuda.Stream(device=dev)
         self.reset(first_token, pos, stream)
         with torch.cuda.stream(stream):
+            self.step(stream)   # outside a capture: lazy module loading, attribute set-up
             if use_graph and n_tokens > 1:
-                self.step(stream)   # warm-up outside capture (lazy module loading, attribute set-up)
                 stream.synchronize()
-                self.reset(first_token, pos, stream)
                 g = torch.cuda.CUDAGraph()
                 with torch.cuda.graph(g, stream=stream):
                     self.step(torch.cuda.current_stream())
-                for _ in range(n_tokens):
+                for _ in range(n_tokens - 1):
                     g.replay()
             else:
-                for _ in range(n_tokens):
+                for _ in range(n_tokens - 1):
                     self.step(stream)
             stream.synchronize()
         self.backend.device_status(stream)
+        self.state(stream)   # the library's host side learns the position the replays reached
         toks = self.buffers()[3]
         return toks[pos:pos + n_tokens].cpu().tolist()
+
+    def complete(self, prompt, n_tokens: int, use_graph: bool = True):
+        """Greedy continuation of a prompt (token ids) by n_tokens: prompt pass, then the decode loop."""
+        prompt = list(prompt)
+        self.prefill(prompt, 0)
+        first = self.state()[0]
+        return [first] + (self.generate(first, len(prompt), n_tokens - 1, use_graph) if n_tokens > 1 else [])
 
     def release(self):
         if self._handle is not None:
             self.backend._lib.nnq_decoder_destroy(self._handle)
             self._handle = None
             self._keep = []
+
+
+# --------------------------------------------------------------------------- #
+# decoders made of blocks
+# --------------------------------------------------------------------------- #
+
+MIXER_ATTENTION, MIXER_RECURRENT = 0, 1
+
+
+class _BlockConfig(ctypes.Structure):
+    _fields_ = [("mixer", ctypes.c_int32), ("heads", ctypes.c_int32), ("kv_heads", ctypes.c_int32), ("dim", ctypes.c_int32),
+                ("vdim", ctypes.c_int32), ("ffn", ctypes.c_int32), ("rot_dims", ctypes.c_int32), ("rot_base", ctypes.c_double),
+                ("scale", ctypes.c_float), ("window", ctypes.c_int32), ("conv_taps", ctypes.c_int32), ("value_mix", ctypes.c_int32),
+                ("out_gate", ctypes.c_int32), ("q_scale", ctypes.c_float), ("k_scale", ctypes.c_float),
+                ("decay_rank", ctypes.c_int32), ("decay_tau", ctypes.c_float)]
+
+
+class _BlockLayout(ctypes.Structure):
+    _fields_ = [(n, ctypes.c_int32) for n in ("in_cols", "in_k", "out_k", "ffn_col", "q", "k", "v", "g", "a1", "gate", "up")]
+
+
+class _BlockWeights(ctypes.Structure):
+    _fields_ = [("w_in", ctypes.c_void_p), ("w_out", ctypes.c_void_p)] + \
+        [(n, ctypes.c_void_p) for n in ("norm", "bias_in", "bias_out", "conv", "head_norm", "decay_w", "decay_b", "decay")] + \
+        [("value_lambda", ctypes.c_float)]
+
+
+@dataclass
+class BlockConfig:
+    """nnq_block_config of the C ABI; window 0 = every earlier position, decay_rank 0 = a fixed decay per head."""
+    mixer: int = MIXER_ATTENTION
+    heads: int = 1
+    kv_heads: int = 1
+    dim: int = 64
+    vdim: int = 64
+    ffn: int = 0
+    rot_dims: int = 0
+    rot_base: float = 1e4
+    scale: float = 1.0
+    window: int = 0
+    conv_taps: int = 0
+    value_mix: bool = False
+    out_gate: bool = False
+    q_scale: float = 1.0
+    k_scale: float = 1.0
+    decay_rank: int = 0
+    decay_tau: float = 1.0
+
+    def _c(self) -> _BlockConfig:
+        return _BlockConfig(self.mixer, self.heads, self.kv_heads, self.dim, self.vdim, self.ffn, self.rot_dims, self.rot_base,
+                            self.scale, self.window, self.conv_taps, int(self.value_mix), int(self.out_gate), self.q_scale,
+                            self.k_scale, self.decay_rank, self.decay_tau)
+
+
+@dataclass
+class BlockTensors:
+    """Tensors of one block: matrices [out, in] as bf16 bit patterns (uint16), everything else f32."""
+    norm: np.ndarray
+    q: np.ndarray
+    k: np.ndarray
+    v: np.ndarray
+    o: np.ndarray
+    g: Optional[np.ndarray] = None
+    q_bias: Optional[np.ndarray] = None
+    k_bias: Optional[np.ndarray] = None
+    v_bias: Optional[np.ndarray] = None
+    o_bias: Optional[np.ndarray] = None
+    conv: Optional[np.ndarray] = None        # [channels of q | k | v, taps]
+    value_lambda: float = 0.0
+    a1: Optional[np.ndarray] = None
+    decay_w: Optional[np.ndarray] = None
+    decay_b: Optional[np.ndarray] = None
+    decay: Optional[np.ndarray] = None       # [heads]
+    head_norm: Optional[np.ndarray] = None
+    gate: Optional[np.ndarray] = None
+    up: Optional[np.ndarray] = None
+    down: Optional[np.ndarray] = None
+
+
+class BlockDecoder(Decoder):
+    """Decoder whose layers are blocks x <- x + mixer(h) + ff(h), h = RMSNorm(x) * w."""
+
+    def __init__(self, backend: api.Backend, *, hidden: int, vocab: int, blocks: List[BlockConfig], max_seq: int,
+                 rms_eps: float = 1e-6, act_dtype: int = api.BF16, block_rows: int = 0):
+        self.blocks, self._block_rows = list(blocks), int(block_rows)
+        super().__init__(backend, DecoderConfig(hidden=hidden, n_heads=0, n_kv_heads=0, head_dim=0, ffn=0, n_layers=len(blocks),
+                                                vocab=vocab, max_seq=max_seq, rms_eps=rms_eps, rope_theta=0.0, act_dtype=act_dtype))
+
+    def _create(self, c_config, out):
+        arr = (_BlockConfig * len(self.blocks))(*[b._c() for b in self.blocks])
+        return self.backend._lib.nnq_decoder_create_blocks(self.backend._ctx, ctypes.byref(c_config), arr, self._block_rows, out)
+
+    def layout(self, layer: int) -> _BlockLayout:
+        y = _BlockLayout()
+        self.backend.check(self.backend._lib.nnq_decoder_block_layout(self._handle, layer, ctypes.byref(y)))
+        return y
+
+    def _weight(self, rows: int, cols: int, parts) -> api.DeviceWeight:
+        """A bf16 weight [rows, cols] of zeros with the given (row, column, matrix) parts, on the device."""
+        w = np.zeros((rows, cols), np.uint16)
+        for r, c, m in parts:
+            if m is not None:
+                if r < 0 or r + m.shape[0] > rows or c + m.shape[1] > cols:
+                    raise api.ShapeMismatch(f"a matrix of shape {m.shape} does not fit its block")
+                w[r:r + m.shape[0], c:c + m.shape[1]] = m
+        b, h = self.backend, ctypes.c_void_p()
+        b.check(b._lib.nnq_weight_create(b._ctx, int(QuantFormat.BF16_DENSE), w.ctypes.data, w.nbytes, None, 0, rows, cols, ctypes.byref(h)))
+        t = api.DeviceWeight(b, h)
+        self._keep.append(t)
+        return t
+
+    def set_block(self, layer: int, t: BlockTensors):
+        y, b, hidden = self.layout(layer), self.blocks[layer], self.cfg.hidden
+        kvh = b.kv_heads if b.mixer == MIXER_ATTENTION else b.heads
+        qn, kn, vn, mix = b.heads * b.dim, kvh * b.dim, kvh * b.vdim, b.heads * b.vdim
+        want = {"q": (qn, hidden), "k": (kn, hidden), "v": (vn, hidden), "o": (hidden, mix), "norm": (hidden,)}
+        if y.g >= 0:
+            want["g"] = (mix, hidden)
+        if b.ffn:
+            want.update(gate=(b.ffn, hidden), up=(b.ffn, hidden), down=(hidden, b.ffn))
+        if b.mixer == MIXER_ATTENTION and b.conv_taps:
+            want["conv"] = (qn + kn + vn, b.conv_taps)
+        if b.mixer == MIXER_RECURRENT:
+            if b.decay_rank:
+                want.update(a1=(b.decay_rank, hidden), decay_w=(qn, b.decay_rank), decay_b=(qn,))
+            else:
+                want["decay"] = (b.heads,)
+        optional = {"q_bias": (qn,), "k_bias": (kn,), "v_bias": (vn,), "o_bias": (hidden,), "head_norm": (b.vdim,)}
+        for name, shape in list(want.items()) + list(optional.items()):
+            a = getattr(t, name)
+            if a is None and name in optional:
+                continue
+            if a is None or tuple(a.shape) != shape:
+                raise api.ShapeMismatch(f"block {layer}: {name} must be {shape}, got {None if a is None else tuple(a.shape)}")
+        w_in = self._weight(y.in_cols, y.in_k, [(y.q, 0, t.q), (y.k, 0, t.k), (y.v, 0, t.v), (y.g, 0, t.g), (y.a1, 0, t.a1),
+                                                (y.gate, 0, t.gate), (y.up, 0, t.up)])
+        w_out = self._weight(hidden, y.out_k, [(0, 0, t.o), (0, y.ffn_col, t.down)])
+        bias = None
+        if any(x is not None for x in (t.q_bias, t.k_bias, t.v_bias)):
+            bias = np.zeros(y.in_cols, np.float32)
+            for c, x in ((y.q, t.q_bias), (y.k, t.k_bias), (y.v, t.v_bias)):
+                if x is not None:
+                    bias[c:c + x.size] = x
+        f32 = [None if a is None else np.ascontiguousarray(a, np.float32)
+               for a in (t.norm, bias, t.o_bias, t.conv, t.head_norm, t.decay_w, t.decay_b, t.decay)]
+        w = _BlockWeights(w_in.handle(), w_out.handle(), *[None if a is None else a.ctypes.data for a in f32], float(t.value_lambda))
+        self.backend.check(self.backend._lib.nnq_decoder_set_block(self._handle, layer, ctypes.byref(w)))
+
+    def set_head(self, embed, final_norm, lm_head):
+        """embed, lm_head: [vocab, hidden] as bf16 bit patterns (uint16); final_norm f32 [hidden]."""
+        c = self.cfg
+        ld = self.layout(0).in_k
+        for a in (embed, lm_head):
+            if tuple(a.shape) != (c.vocab, c.hidden):
+                raise api.ShapeMismatch(f"embedding and vocabulary projection must be {(c.vocab, c.hidden)}, got {tuple(a.shape)}")
+        e = self._weight(c.vocab, ld, [(0, 0, embed)])
+        h = e if lm_head is embed else self._weight(c.vocab, ld, [(0, 0, lm_head)])
+        fn = np.ascontiguousarray(final_norm, np.float32)
+        self.backend.check(self.backend._lib.nnq_decoder_set_head_weights(self._handle, e.handle(), fn.ctypes.data, h.handle()))
+
+    def set_layer(self, *a, **k):
+        raise api.Unsupported("a block decoder takes set_block")
+
+    def buffers(self):
+        """(None, None, logits, tokens): the blocks keep their own caches and states."""
+        import torch
+        lg, tk = ctypes.c_void_p(), ctypes.c_void_p()
+        self.backend.check(self.backend._lib.nnq_decoder_buffers(self._handle, None, None, ctypes.byref(lg), ctypes.byref(tk)))
+        dev = torch.device("cuda", self.backend.device)
+        return (None, None, torch.as_tensor(_DevArray(lg.value, (self.cfg.vocab,), "<f4"), device=dev),
+                torch.as_tensor(_DevArray(tk.value, (self.cfg.max_seq,), "<i4"), device=dev))
