@@ -423,6 +423,10 @@ static nnq_status linear_dispatch(nnq_ctx *ctx, const nnq_weight *w, const void 
         nnq_status s = launch_skinny(ctx, &lo, 1, x_dt, cols, y_dt, stream);
         return s != NNQ_OK ? s : launch_skinny(ctx, &hi, 1, x_dt, m - cols, y_dt, stream);
     }
+    if (path == NNQ_PATH_AUTO && dense_gemv_supported(w, m, x_dt)) {
+        TcArgs a = {w->d_raw, w->d_scales, x_dev, bias_dev, y_dev, m, w->n, w->k, w->fmt, x_dt, y_dt};
+        return launch_dense_gemv(ctx, a, stream);
+    }
     const bool tc_ok = gemm_tc_supported(w, m);
     if (path == NNQ_PATH_TENSOR && !tc_ok)
         return fail(ctx, NNQ_ERR_UNSUPPORTED, "tensor path needs K to be a multiple of 64 (K=%lld)", (long long)w->k);

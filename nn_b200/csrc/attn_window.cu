@@ -8,69 +8,94 @@
 
 namespace nnq {
 
-constexpr int kPrepWarps = 4;
+constexpr int kPrepWarps = 4, kPrepRows = 8;
 
-// Projected value of channel c (column col of proj) after the convolution, for row r at position pos.
-// Rows of this launch come from proj, earlier ones from the ring, positions before 0 are zero.
-__device__ __forceinline__ float conv_value(const WindowAttn &a, int r, int pos, int c, int col) {
-    const float cur = a.ffn.proj[(size_t)r * a.ffn.in_cols + col];
-    if (a.taps == 0) return cur;
-    const int channels = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
-    const float *w = a.conv + (size_t)c * a.taps;
-    float y = 0.0f;
-    for (int j = 0; j < a.taps - 1; j++) {
-        const int s = a.taps - 1 - j;   // rows back
-        float u = 0.0f;
-        if (r - s >= 0) u = a.ffn.proj[(size_t)(r - s) * a.ffn.in_cols + col];
-        else if (pos - s >= 0) u = a.conv_ring[(size_t)((pos - s) % a.taps) * channels + c];
-        y = fmaf(w[j], u, y);
-    }
-    return fmaf(w[a.taps - 1], cur, y);
+// Projected value (before the convolution) of channel c, column col of proj, `back` rows before row r at
+// position pos: rows of this launch come from proj, earlier ones from the ring, positions before 0 are zero.
+__device__ __forceinline__ float conv_input(const WindowAttn &a, int channels, int r, int pos, int back, int c, int col) {
+    if (r >= back) return a.ffn.proj[(size_t)(r - back) * a.ffn.in_cols + col];
+    return pos >= back ? a.conv_ring[(size_t)((pos - back) % a.taps) * channels + c] : 0.0f;
 }
 
-// One warp per (row, head), heads numbered q | k | v. CTAs from prep_ctas on do the feed-forward part.
+// One warp per (head, kPrepRows consecutive rows), heads numbered q | k | v; a lane slides over the rows of its
+// channels, so that a projected value is read once. TAPS 0: no convolution; -1: any other number of taps.
+// CTAs from prep_ctas on do the feed-forward part.
+template <int TAPS>
 __global__ void __launch_bounds__(kPrepWarps * 32) attn_prep_kernel(const WindowAttn a, int prep_ctas) {
     pdl_prologue();
+    pdl_release();
     extern __shared__ float prep_smem[];
     if ((int)blockIdx.x >= prep_ctas) {
         ffn_part(a.ffn, a.span.n, prep_ctas);
         return;
     }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int nh = a.heads + 2 * a.kv_heads;
-    const long long item = (long long)blockIdx.x * kPrepWarps + warp;
-    if (item >= (long long)a.span.n * nh) return;
-    const int row = (int)(item / nh), head = (int)(item - (long long)row * nh);
-    const int pos = span_pos(a.span) + row;
+    const int nh = a.heads + 2 * a.kv_heads, n = a.span.n;
+    const int item = blockIdx.x * kPrepWarps + warp;
+    const int tile = item / nh, head = item - tile * nh, row0 = tile * kPrepRows;
+    if (row0 >= n) return;
+    const int rows = min(kPrepRows, n - row0), pos0 = span_pos(a.span) + row0;
     const bool is_q = head < a.heads, is_v = head >= a.heads + a.kv_heads;
     const int h = is_q ? head : (is_v ? head - a.heads - a.kv_heads : head - a.heads);
-    const int width = is_v ? a.vdim : a.dim;
+    const int width = is_v ? a.vdim : a.dim, wmax = max(a.dim, a.vdim);
+    const int channels = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
     const int c0 = is_q ? h * a.dim : (is_v ? (a.heads + a.kv_heads) * a.dim + h * a.vdim : (a.heads + h) * a.dim);
     const int col0 = (is_q ? a.c_q : (is_v ? a.c_v : a.c_k)) + h * width;
-    float *xs = prep_smem + warp * (a.dim > a.vdim ? a.dim : a.vdim);
+    float *xs = prep_smem + warp * kPrepRows * wmax;   // [rows, wmax]
     for (int d = lane; d < width; d += 32) {
-        xs[d] = conv_value(a, row, pos, c0 + d, col0 + d);
+        float cur[kPrepRows];
+#pragma unroll
+        for (int r = 0; r < kPrepRows; r++) cur[r] = r < rows ? a.ffn.proj[(size_t)(row0 + r) * a.ffn.in_cols + col0 + d] : 0.0f;
         // one row: this position's slot is read by nobody in this launch (readers look 1 .. taps - 1 back)
-        if (a.taps > 1 && a.span.n == 1) {
-            const int channels = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
-            a.conv_ring[(size_t)(pos % a.taps) * channels + c0 + d] = a.ffn.proj[col0 + d];
+        if (TAPS != 0 && n == 1 && a.taps > 1) a.conv_ring[(size_t)(pos0 % a.taps) * channels + c0 + d] = cur[0];
+        if constexpr (TAPS > 0) {
+            float w[TAPS], u[TAPS];   // u[b]: value b rows back
+#pragma unroll
+            for (int t = 0; t < TAPS; t++) w[t] = a.conv[(size_t)(c0 + d) * TAPS + t];
+#pragma unroll
+            for (int b = 1; b < TAPS; b++) u[b] = conv_input(a, channels, row0, pos0, b, c0 + d, col0 + d);
+#pragma unroll
+            for (int r = 0; r < kPrepRows; r++) {
+                u[0] = cur[r];
+                float y = 0.0f;
+#pragma unroll
+                for (int t = 0; t < TAPS; t++) y = fmaf(w[t], u[TAPS - 1 - t], y);
+                if (r < rows) xs[r * wmax + d] = y;
+#pragma unroll
+                for (int b = TAPS - 1; b > 0; b--) u[b] = u[b - 1];
+            }
+        } else if constexpr (TAPS == 0) {
+#pragma unroll
+            for (int r = 0; r < kPrepRows; r++)
+                if (r < rows) xs[r * wmax + d] = cur[r];
+        } else {
+            for (int r = 0; r < rows; r++) {
+                float y = 0.0f;
+                for (int t = 0; t < a.taps; t++)
+                    y = fmaf(a.conv[(size_t)(c0 + d) * a.taps + t], conv_input(a, channels, row0 + r, pos0 + r, a.taps - 1 - t, c0 + d, col0 + d), y);
+                xs[r * wmax + d] = y;
+            }
         }
     }
     __syncwarp();
     const int half = a.rot_dims >> 1;
-    const float *cs = a.cosv + (size_t)pos * half, *sn = a.sinv + (size_t)pos * half;
-    if (is_v) {
-        const size_t vf = ((size_t)row * a.kv_heads + h) * a.vdim;
-        float *dst = a.vcache + ((size_t)h * a.cap + pos % a.cap) * a.vdim_ld;
-        for (int d = lane; d < width; d += 32) {
-            float v = xs[d];
-            if (a.mix_mode == 1) a.vfirst[vf + d] = v;
-            else if (a.mix_mode == 2) v = (1.0f - a.lambda) * v + a.lambda * a.vfirst[vf + d];
-            dst[d] = v;
+    for (int r = 0; r < rows; r++) {
+        const int pos = pos0 + r, row = row0 + r;
+        const float *x = xs + r * wmax;
+        if (is_v) {
+            const size_t vf = ((size_t)row * a.kv_heads + h) * a.vdim;
+            float *dst = a.vcache + ((size_t)h * a.cap + pos % a.cap) * a.vdim_ld;
+            for (int d = lane; d < width; d += 32) {
+                float v = x[d];
+                if (a.mix_mode == 1) a.vfirst[vf + d] = v;
+                else if (a.mix_mode == 2) v = (1.0f - a.lambda) * v + a.lambda * a.vfirst[vf + d];
+                dst[d] = v;
+            }
+        } else {
+            const float *cs = a.cosv + (size_t)pos * half, *sn = a.sinv + (size_t)pos * half;
+            float *dst = is_q ? a.qrot + ((size_t)row * a.heads + h) * a.dim_ld : a.kcache + ((size_t)h * a.cap + pos % a.cap) * a.dim_ld;
+            for (int d = lane; d < a.dim_ld; d += 32) dst[d] = d < width ? rotated(x, d, a.rot_dims, cs, sn) : 0.0f;
         }
-    } else {
-        float *dst = is_q ? a.qrot + ((size_t)row * a.heads + h) * a.dim_ld : a.kcache + ((size_t)h * a.cap + pos % a.cap) * a.dim_ld;
-        for (int d = lane; d < a.dim_ld; d += 32) dst[d] = d < width ? rotated(xs, d, a.rot_dims, cs, sn) : 0.0f;
     }
 }
 
@@ -233,6 +258,7 @@ constexpr int kDecMaxRanges = 32;
 template <int P, int VC>
 __global__ void __launch_bounds__(kDecWarps * 32) attn_decode_kernel(const WindowAttn a) {
     pdl_prologue();
+    pdl_release();
     extern __shared__ __align__(16) float dec_smem[];
     __shared__ float wm[kDecWarps][P], wl[kDecWarps][P];
     __shared__ int s_last;
@@ -349,16 +375,27 @@ static nnq_status allow_smem(nnq_ctx *ctx, K kernel, size_t bytes) {
     return check_cuda(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes), "attention shared memory");
 }
 
-nnq_status launch_attn_prep(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
-    const long long items = (long long)a.span.n * (a.heads + 2 * a.kv_heads);
-    const int prep = (int)((items + kPrepWarps - 1) / kPrepWarps);
+template <int TAPS>
+static nnq_status go_prep(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
+    const int items = (a.span.n + kPrepRows - 1) / kPrepRows * (a.heads + 2 * a.kv_heads);
+    const int prep = (items + kPrepWarps - 1) / kPrepWarps;
     const int ffn = ffn_ctas(a.ffn, a.span.n, kPrepWarps * 32, ctx->sm_count);
-    const size_t smem = (size_t)kPrepWarps * (a.dim > a.vdim ? a.dim : a.vdim) * sizeof(float);
-    nnq_status s = allow_smem(ctx, attn_prep_kernel, smem);
+    const size_t smem = (size_t)kPrepWarps * kPrepRows * (a.dim > a.vdim ? a.dim : a.vdim) * sizeof(float);
+    nnq_status s = allow_smem(ctx, attn_prep_kernel<TAPS>, smem);
     if (s != NNQ_OK) return s;
-    launch_pdl_smem(attn_prep_kernel, dim3(prep + ffn), dim3(kPrepWarps * 32), smem, st, a, prep);
+    launch_pdl_smem(attn_prep_kernel<TAPS>, dim3(prep + ffn), dim3(kPrepWarps * 32), smem, st, a, prep);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "attention prologue launch");
+}
+
+nnq_status launch_attn_prep(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
+    switch (a.taps) {
+        case 0: return go_prep<0>(ctx, a, st);
+        case 2: return go_prep<2>(ctx, a, st);
+        case 3: return go_prep<3>(ctx, a, st);
+        case 4: return go_prep<4>(ctx, a, st);
+        default: return go_prep<-1>(ctx, a, st);
+    }
 }
 
 nnq_status launch_attn_conv_tail(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {

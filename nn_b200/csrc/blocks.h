@@ -72,7 +72,7 @@ int attn_decode_counters(int heads, int kv_heads);
 struct Recurrence {
     RowSpan span;
     FfnPart ffn;
-    int heads, dim, vdim, dim_ld;   // dim_ld: rounded up to 32
+    int heads, dim, vdim, dim_ld;   // dim_ld: rounded up to 64
     int c_q, c_k, c_v, c_g, c_a1;
     float q_scale, k_scale;         // applied after the rotation
     int rot_dims;

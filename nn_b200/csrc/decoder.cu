@@ -95,8 +95,9 @@ constexpr int kWantRows = 64;     // rows of logits formed together
 __global__ void __launch_bounds__(1024)
 dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
                 const int *__restrict__ state, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                int hidden, int embed_ld, int xn_ld) {
+                int hidden, int embed_ld, int xn_ld, int release) {
     pdl_prologue();
+    if (release) pdl_release();
     __shared__ float red[32];
     const int tok = embed ? state[0] : 0;
     float v[8], wv[8];
@@ -467,6 +468,37 @@ dec_norm_rows_kernel(float *__restrict__ h, const float *__restrict__ delta, con
     const float *dr = delta ? delta + r * hidden : nullptr;
     const __nv_bfloat16 *er = embed ? embed + (size_t)tokens[r] * embed_ld : nullptr;
     float ss = 0.0f;
+    if (!er && hidden % 4 == 0 && hidden <= 256 * 4 * 8) {
+        float4 v[8];
+#pragma unroll
+        for (int k = 0; k < 8; k++) {
+            const int i = 4 * (threadIdx.x + 256 * k);
+            v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (i < hidden) {
+                const float4 a = *reinterpret_cast<const float4 *>(hr + i), b = *reinterpret_cast<const float4 *>(dr + i);
+                v[k] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+                if (!rows) *reinterpret_cast<float4 *>(hr + i) = v[k];
+            }
+            ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+        }
+        const float rms = sqrtf(block_sum(ss, red) / (float)hidden + eps);
+        char *xr = reinterpret_cast<char *>(xn) + (size_t)blockIdx.x * xn_ld * (act_dt == NNQ_F32 ? 4 : 2);
+#pragma unroll
+        for (int k = 0; k < 8; k++) {
+            const int i = 4 * (threadIdx.x + 256 * k);
+            if (i >= hidden) continue;
+            const float4 g = *reinterpret_cast<const float4 *>(w + i);
+            const float y0 = v[k].x / rms * g.x, y1 = v[k].y / rms * g.y, y2 = v[k].z / rms * g.z, y3 = v[k].w / rms * g.w;
+            if (act_dt == NNQ_F32) {
+                reinterpret_cast<float4 *>(xr)[i >> 2] = make_float4(y0, y1, y2, y3);
+            } else {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(y0, y1), b = __floats2bfloat162_rn(y2, y3);
+                reinterpret_cast<uint2 *>(xr)[i >> 2] = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+            }
+        }
+        for (int i = hidden + threadIdx.x; i < xn_ld; i += blockDim.x) store_act(xr, act_dt, i, 0.0f);
+        return;
+    }
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         const float v = er ? __bfloat162float(er[i]) : hr[i] + dr[i];
         if (!rows) hr[i] = v;
@@ -805,7 +837,8 @@ static nnq_block_layout layout_of(const nnq_block_config &b, int hidden) {
     y.in_cols = at;
     y.in_k = round_up(hidden, 64);   // one k step of the tensor-core products
     y.ffn_col = round_up(b.heads * b.vdim, 8);
-    y.out_k = round_up(y.ffn_col + b.ffn, 64);
+    // (a gap in front of the feed-forward's columns is cleared together with them: there are some then)
+    y.out_k = round_up(y.ffn_col + (b.ffn > 0 || y.ffn_col == b.heads * b.vdim ? b.ffn : 8), 64);
     return y;
 }
 
@@ -876,7 +909,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
             most(part, attn_decode_part_floats(b.heads, b.kv_heads, B.vdim_ld, B.ranges));
             most(counters, attn_decode_counters(b.heads, b.kv_heads));
         } else {
-            B.dim_ld = round_up(b.dim, 32);
+            B.dim_ld = round_up(b.dim, 64);
             alloc(&B.rec_state, (size_t)b.heads * b.dim * b.vdim * 4, "recurrent state");
             if (b.decay_rank > 0) {
                 alloc(&B.a2t, (size_t)b.heads * b.dim * b.decay_rank * 4, "decay weight");
@@ -1166,7 +1199,7 @@ static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
     const nnq_decoder_config &c = d->cfg;
     for (int l = 0; l < c.n_layers; l++) {
         launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->d_state,
-                   d->blocks[l].norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld);
+                   d->blocks[l].norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
         d->ctx->launches++;
         nnq_status s = run_block(d, l, 1, 0, d->d_state, d->d_xn, d->d_delta, st);
         if (s != NNQ_OK) return s;
@@ -1197,7 +1230,7 @@ static nnq_status step_qwen3(nnq_decoder *d, cudaStream_t st) {
     const __nv_bfloat16 *embed = (const __nv_bfloat16 *)d->d_embed;
     for (int l = 0; l < c.n_layers; l++) {
         const nnq_decoder::Layer &L = d->layers[l];
-        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? embed : nullptr, d->d_state, L.in_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld));
+        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? embed : nullptr, d->d_state, L.in_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0));
         const nnq_weight *w3[3] = {L.q, L.k, L.v};
         const void *x3[3] = {d->d_xn, d->d_xn, d->d_xn};
         void *y3[3] = {d->d_q, d->d_k, d->d_v};
@@ -1219,7 +1252,7 @@ static nnq_status step_qwen3(nnq_decoder *d, cudaStream_t st) {
         DEC_RUN(32, s = d->comm ? nnq_comm_linear(d->comm, L.o, d->d_attn, adt, 1, nullptr, d->d_delta, NNQ_F32, st)
                                 : nnq_linear(ctx, L.o, d->d_attn, adt, 1, nullptr, d->d_delta, NNQ_F32, st));
         if (s != NNQ_OK) return s;
-        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, L.post_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld));
+        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, L.post_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0));
         const nnq_weight *w2[2] = {L.gate, L.up};
         const void *x2[2] = {d->d_xn, d->d_xn};
         void *y2[2] = {d->d_g, d->d_u};
@@ -1298,7 +1331,7 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
     if (s != NNQ_OK) return s;
     cudaStream_t st = (cudaStream_t)stream;
     if ((s = d->blocks ? step_blocks(d, st) : step_qwen3(d, st)) != NNQ_OK) return s;
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld);
+    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
     ctx->launches++;
     return launch_head(d, vocab_parallel, cv, st);
 }
@@ -1386,7 +1419,7 @@ nnq_status nnq_decoder_prefill(nnq_decoder *d, const int32_t *tokens_host, int c
     const size_t last = (size_t)(n - 1) * c.hidden;
     const int st4[4] = {tokens_host[count - 1], start_pos + count - 1, 0, 0};
     if ((s = check_cuda(ctx, cudaMemcpyAsync(d->d_state, st4, sizeof(st4), cudaMemcpyHostToDevice, st), "decoder state")) != NNQ_OK) return s;
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->pf_h + last, d->pf_delta + last, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld);
+    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->pf_h + last, d->pf_delta + last, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
     ctx->launches++;
     if ((s = launch_head(d, vocab_parallel, cv, st)) != NNQ_OK) return s;
     s = check_cuda(ctx, cudaStreamSynchronize(st), "prompt pass");   // tokens_host and st4 are the caller's / the stack's

@@ -1,0 +1,173 @@
+// y[M, N] = x[M, K] W^T (+ bias) for an unquantized bf16 weight and one to four bf16 rows (a decode step).
+//
+// The work is one pass over the weight, so the kernel is built around keeping enough of it in flight: one CTA
+// per SM, sixteen warps (eight for three and four rows), each with a private ring of bulk copies (cp.async.bulk on mbarriers, up to 160 KB in
+// flight per SM). A warp owns one chunk of at most 1024 columns for all of its rows: its x values stay in
+// registers (a lane's 32 of them as bf16 pairs) and a tile is one row's chunk, 2 KB. KS warps share a row; their
+// partial sums meet in shared memory once, at the end. The ring is filled before the kernel waits for its
+// predecessor (programmatic dependent launch): the small kernels in front of a product release it early, so the
+// weights stream while they run. Products bf16 x bf16 in f32, f32 sums. Every wait is bounded.
+#include <cuda_bf16.h>
+
+#include "gemm_tc.h"
+#include "pdl.cuh"
+#include "sync.cuh"
+
+namespace nnq {
+
+constexpr int kGvChunk = 1024, kGvTileBytes = kGvChunk * 2, kGvTiles = 80, kGvRing = kGvTiles * kGvTileBytes;
+// warps of a CTA: three and four rows need the registers of half as many
+__host__ __device__ constexpr int gv_warps(int m) { return m <= 2 ? 16 : 8; }
+
+__device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xFFFF0000u); }
+
+// grid: rows dealt to CTAs in contiguous runs. ks: warps per row (power of two), passes: chunks of a warp.
+template <int M>
+__global__ void __launch_bounds__(gv_warps(M) * 32, 1)
+dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__restrict__ x, const float *__restrict__ bias, void *__restrict__ y,
+                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status) {
+    constexpr int kGvWarps = gv_warps(M), kGvStages = kGvTiles / kGvWarps;
+    extern __shared__ __align__(128) uint8_t gv_smem[];
+    __shared__ __align__(8) uint64_t bars[kGvWarps * kGvStages];
+    float *part = reinterpret_cast<float *>(gv_smem + kGvRing);   // [rows of this CTA][ks][M]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r0 = (int)((long long)N * blockIdx.x / gridDim.x), r1 = (int)((long long)N * (blockIdx.x + 1) / gridDim.x);
+    const int groups = kGvWarps / ks, group = warp / ks, kw = warp % ks;
+    const int rows = r1 - r0 > group ? (r1 - r0 - group + groups - 1) / groups : 0;   // rows r0 + group, + groups, ...
+    const uint32_t bar0 = smem_u32(bars + warp * kGvStages);
+    const uint32_t ring = smem_u32(gv_smem) + warp * kGvStages * kGvTileBytes;
+    const uint8_t *ring_p = gv_smem + warp * kGvStages * kGvTileBytes;
+    if (lane == 0) {
+        for (int s = 0; s < kGvStages; s++) mbar_init(bar0 + 8 * s, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncwarp();
+    // tile i of this warp: pass i / rows, row r0 + group + groups * (i % rows); a chunk past the end has no tiles
+    const int my_passes = max(0, min(passes, ((K + chunk - 1) / chunk - kw + ks - 1) / ks));
+    const int tiles = rows * my_passes;
+    auto issue = [&](int i) {   // lane 0
+        const int pass = i / rows, row = r0 + group + groups * (i - pass * rows);
+        const int k0 = (pass * ks + kw) * chunk, kc = min(chunk, K - k0);
+        const uint32_t bar = bar0 + 8 * (i % kGvStages);
+        mbar_expect_tx(bar, kc * 2);
+        bulk_g2s(ring + (i % kGvStages) * kGvTileBytes, w + (size_t)row * K + k0, kc * 2, bar);
+    };
+    if (lane == 0)
+        for (int i = 0; i < kGvStages && i < tiles; i++) issue(i);
+    pdl_prologue();
+    bool ok = true;
+    int stage = 0, issued = min(tiles, kGvStages);
+    uint32_t phase = 0;
+    for (int pass = 0, i = 0; pass < my_passes && ok; pass++) {
+        const int k0 = (pass * ks + kw) * chunk, kc = min(chunk, K - k0);
+        uint4 xv[M][4];
+#pragma unroll
+        for (int m = 0; m < M; m++)
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+                xv[m][j] = 8 * (lane + 32 * j) < kc ? *reinterpret_cast<const uint4 *>(x + (size_t)m * K + k0 + 8 * (lane + 32 * j)) : make_uint4(0, 0, 0, 0);
+        for (int r = 0; r < rows; r++, i++) {
+            if (!mbar_wait_fast(bar0 + 8 * stage, phase)) {
+                ok = false;
+                break;
+            }
+            const uint4 *tile = reinterpret_cast<const uint4 *>(ring_p + stage * kGvTileBytes);
+            float acc[M][2];
+#pragma unroll
+            for (int m = 0; m < M; m++) acc[m][0] = acc[m][1] = 0.0f;
+            uint4 wv[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) wv[j] = 8 * (lane + 32 * j) < kc ? tile[lane + 32 * j] : make_uint4(0, 0, 0, 0);
+            __syncwarp();
+            if (lane == 0 && issued < tiles) issue(issued);   // the tile's values are in registers
+            issued++;
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const uint32_t wq[4] = {wv[j].x, wv[j].y, wv[j].z, wv[j].w};
+#pragma unroll
+                for (int q = 0; q < 4; q++) {
+                    const float wl = bf_lo(wq[q]), wh = bf_hi(wq[q]);
+#pragma unroll
+                    for (int m = 0; m < M; m++) {
+                        const uint32_t xq = q == 0 ? xv[m][j].x : (q == 1 ? xv[m][j].y : (q == 2 ? xv[m][j].z : xv[m][j].w));
+                        acc[m][0] = fmaf(wl, bf_lo(xq), acc[m][0]);
+                        acc[m][1] = fmaf(wh, bf_hi(xq), acc[m][1]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < M; m++) {
+                float v = acc[m][0] + acc[m][1];
+#pragma unroll
+                for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, off);
+                if (lane == 0) {
+                    float *p = part + ((size_t)(group + groups * r) * ks + kw) * M + m;
+                    *p = pass == 0 ? v : *p + v;
+                }
+            }
+            if (++stage == kGvStages) {
+                stage = 0;
+                phase ^= 1u;
+            }
+        }
+    }
+    if (my_passes == 0)   // fewer chunks than warps per row
+        for (int r = lane; r < rows; r += 32)
+#pragma unroll
+            for (int m = 0; m < M; m++) part[((size_t)(group + groups * r) * ks + kw) * M + m] = 0.0f;
+    if (!ok) {
+        // give the copies in flight a bounded chance to land before the shared memory goes
+        for (int s = 0; s < kGvStages; s++) mbar_wait(bar0 + 8 * s, phase);
+        if (lane == 0) atomicExch(status, 1);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < (r1 - r0) * M; i += kGvWarps * 32) {
+        const int m = i / (r1 - r0), r = i - m * (r1 - r0);
+        float v = 0.0f;
+        for (int q = 0; q < ks; q++) v += part[((size_t)r * ks + q) * M + m];
+        if (bias) v += __ldg(bias + r0 + r);
+        if (y_dt == NNQ_F32) reinterpret_cast<float *>(y)[(size_t)m * N + r0 + r] = v;
+        else reinterpret_cast<__nv_bfloat16 *>(y)[(size_t)m * N + r0 + r] = __float2bfloat16_rn(v);
+    }
+}
+
+bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt) {
+    return w && w->fmt == NNQ_BF16_DENSE && w->d_raw && x_dt == NNQ_BF16 && m >= 1 && m <= 4 && w->k >= 64 && w->k % 8 == 0 && w->n >= 1 &&
+           w->n < (1ll << 31) && w->k < (1ll << 31) && !((uintptr_t)w->d_raw & 15u);
+}
+
+template <int M>
+static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, cudaStream_t st) {
+    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+    launch_pdl_smem(dense_gemv_kernel<M>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
+                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status);
+    return cudaGetLastError();
+}
+
+nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) {
+    // as few warps per row as keep a warp's columns within one chunk
+    int ks = 1;
+    while (ks < gv_warps((int)a.m) && a.k > (int64_t)ks * kGvChunk) ks *= 2;
+    int chunk = (int)(((a.k + ks - 1) / ks + 7) / 8 * 8);
+    if (chunk > kGvChunk) chunk = kGvChunk;
+    const int chunks = (int)((a.k + chunk - 1) / chunk), passes = (chunks + ks - 1) / ks;
+    // partial sums of a CTA's rows within 32 KB: more CTAs than SMs for very tall weights
+    const int64_t max_rows = (32 << 10) / (4 * ks * a.m);
+    int64_t grid = a.n < ctx->sm_count ? a.n : ctx->sm_count;
+    while ((a.n + grid - 1) / grid > max_rows) grid += ctx->sm_count;
+    const size_t smem = kGvRing + (size_t)((a.n + grid - 1) / grid) * ks * a.m * 4;
+    cudaError_t e;
+    switch (a.m) {
+        case 1: e = gv_go<1>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
+        case 2: e = gv_go<2>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
+        case 3: e = gv_go<3>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
+        case 4: e = gv_go<4>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
+        default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "1 to 4 rows");
+    }
+    ctx->launches++;
+    return check_cuda(ctx, e, "bf16 row product launch");
+}
+
+}  // namespace nnq

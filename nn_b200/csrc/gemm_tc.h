@@ -55,6 +55,9 @@ nnq_status dense_scratch_reserve(nnq_ctx *ctx, int64_t n, int64_t k);
 nnq_status launch_gemm_dense(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream);
 // the GEMM alone over an already decoded bf16 [n, k] weight (a.w / a.fmt are not read)
 nnq_status launch_gemm_dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs &a, cudaStream_t stream);
+// dense_gemv.cu: one to four bf16 rows against an unquantized bf16 weight
+bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt);
+nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream);
 bool gemm_dense_shape_ok(const nnq_ctx *ctx, int64_t m, int64_t n, int64_t k, int x_dt);
 // the expert products of a prefill-sized MoE call: all local experts decoded at once
 bool gemm_dense_grouped_supported(const nnq_ctx *ctx, const TcGroupArgs &g);

@@ -12,6 +12,13 @@ __device__ __forceinline__ void pdl_prologue() {
     asm volatile("griddepcontrol.wait;" ::: "memory");
 }
 
+// Lets the successor become resident once every CTA of this kernel has come here. For the small kernels of
+// a block decoder: the successor of the last of them is the bf16 row product (dense_gemv.cu), which keeps few
+// registers, fills its ring of weight copies and then sleeps until this kernel has ended.
+__device__ __forceinline__ void pdl_release() {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+}
+
 template <typename... KArgs, typename... Args>
 static void launch_pdl_smem(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args... args) {
     cudaLaunchConfig_t cfg = {};

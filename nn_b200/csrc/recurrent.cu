@@ -3,9 +3,9 @@
 // from a low-rank gate (gated linear attention); optional half-split rotation of q and k; RMS norm of
 // each head's o, silu output gate. Everything in f32.
 //
-// The state of a block of rows is advanced token by token (each CTA keeps a [dim, 16] tile of it in
-// registers and streams the prepared q / k / decay rows through shared memory), so the result does not
-// depend on how a sequence was cut into blocks: a cut only stores and reloads the same f32 state.
+// The state of a block of rows is advanced token by token (a warp keeps a [dim, 8] tile of it in registers,
+// the prepared q / k / decay rows stream through shared memory), so the result does not depend on how a
+// sequence was cut into blocks: a cut only stores and reloads the same f32 state.
 #include <math.h>
 
 #include "blocks.cuh"
@@ -68,136 +68,211 @@ __global__ void __launch_bounds__(kRecPrepWarps * 32) rec_prep_kernel(const Recu
     }
 }
 
-constexpr int kScanCols = 16, kScanThreads = 128;   // 8 threads per column, each every eighth group of four key rows
+// ---- the scan over a block of rows ----
+//
+// A warp owns eight columns of the state over all key rows: lane = 16 row groups x 2 column groups, a lane
+// holds rows 64 j + 4 (lane % 16) .. + 3 and four columns as packed f32 pairs (two rows of a column), so that
+// q, k and the decay come as pairs out of one 16-byte shared-memory read and the three operations of a state
+// element -- k v, s a + (k v), o + s q -- are packed f32x2 instructions. After eight tokens the lanes' partial
+// o are reduced across the row groups by halving exchanges: every lane ends with one token and two columns.
+// Tokens stream through a three-stage ring of cp.async copies, one barrier per stage.
 
-__device__ __forceinline__ void cp_async16(void *dst, const void *src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+constexpr int kScanTokens = 8, kScanStages = 3;
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+// four bytes, or four zero bytes
+__device__ __forceinline__ void cp_async4(uint32_t dst, const void *src, bool real) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(real ? 4 : 0) : "memory");
+}
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float &lo, float &hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
 }
 
-// grid (heads, ceil(vdim / 16)); NI = dim_ld / 32, TC tokens per stage of the double buffer
-template <int NI, int TC, bool FIXED>
-__global__ void __launch_bounds__(kScanThreads) rec_scan_kernel(const Recurrence r) {
+// grid (heads, ceil(vdim / (8 WARPS))); NJ = dim_ld / 64
+template <int NJ, int WARPS, bool FIXED>
+__global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r) {
     constexpr int NS = FIXED ? 2 : 3;   // streams: q, k (, decay)
-    constexpr int LD = NI * 32;
-    extern __shared__ __align__(16) float scan_smem[];   // [2][NS][TC][LD], then v [2][TC][16]
-    float *vbuf = scan_smem + 2 * NS * TC * LD;
-    const int tid = threadIdx.x, rg = tid & 7, col = tid >> 3;
-    const int head = blockIdx.x, v0 = blockIdx.y * kScanCols;
-    const int n = r.span.n;
-    const bool live = v0 + col < r.vdim;
-    float S[NI * 4];
-    float *state = r.state + (size_t)head * r.dim * r.vdim + v0 + col;
+    constexpr int LD = NJ * 64, COLS = WARPS * 8, T = kScanTokens, THREADS = WARPS * 32;
+    constexpr int STAGE = T * (NS * LD + COLS);   // floats
+    extern __shared__ __align__(16) float scan_smem[];
+    const int tid = threadIdx.x, lane = tid & 31, rl = lane & 15;
+    const int wcol = (tid >> 5) * 8 + (lane >> 4) * 4;
+    const int head = blockIdx.x, v0 = blockIdx.y * COLS, n = r.span.n;
+    float *state = r.state + (size_t)head * r.dim * r.vdim;
+    uint64_t S[NJ][2][4];
 #pragma unroll
-    for (int i = 0; i < NI; i++)
+    for (int j = 0; j < NJ; j++)
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const int row = 32 * i + 4 * rg + j;
-            S[4 * i + j] = live && r.span.pos0 > 0 && row < r.dim ? state[(size_t)row * r.vdim] : 0.0f;
-        }
+        for (int h = 0; h < 2; h++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                float s[2];
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int row = 64 * j + 4 * rl + 2 * h + e, col = v0 + wcol + c;
+                    s[e] = r.span.pos0 > 0 && row < r.dim && col < r.vdim ? state[(size_t)row * r.vdim + col] : 0.0f;
+                }
+                S[j][h][c] = pack2(s[0], s[1]);
+            }
     const float fixed = FIXED ? r.decay[head] : 0.0f;
+    const uint64_t fixed2 = pack2(fixed, fixed);
     const size_t row_ld = (size_t)r.heads * LD;
     const float *src[3] = {r.q + (size_t)head * LD, r.k + (size_t)head * LD, r.a + (size_t)head * LD};
-    const int chunks = (n + TC - 1) / TC;
+    const float *vsrc = r.ffn.proj + r.c_v + head * r.vdim;
+    const int chunks = (n + T - 1) / T;
+    const uint32_t smem0 = (uint32_t)__cvta_generic_to_shared(scan_smem);
     auto load = [&](int ch) {
-        float *dst = scan_smem + (ch & 1) * NS * TC * LD;
-        const int t0 = ch * TC;
+        if (ch < chunks) {
+            const uint32_t dst = smem0 + 4u * STAGE * (ch % kScanStages);
+            const int t0 = ch * T;
 #pragma unroll
-        for (int s = 0; s < NS; s++)
-            for (int i = tid; i < TC * (LD / 4); i += kScanThreads) {
-                const int t = i / (LD / 4), c = i % (LD / 4);
-                if (t0 + t < n) cp_async16(dst + (s * TC + t) * LD + 4 * c, src[s] + (size_t)(t0 + t) * row_ld + 4 * c);
+            for (int s = 0; s < NS; s++)
+#pragma unroll
+                for (int i = tid; i < T * (LD / 4); i += THREADS) {
+                    const int t = i / (LD / 4), c = i % (LD / 4);
+                    if (t0 + t < n) cp_async16(dst + 4u * ((s * T + t) * LD + 4 * c), src[s] + (size_t)(t0 + t) * row_ld + 4 * c);
+                }
+#pragma unroll
+            for (int i = tid; i < T * COLS; i += THREADS) {
+                const int t = i / COLS, c = i % COLS;
+                const bool real = t0 + t < n && v0 + c < r.vdim;
+                cp_async4(dst + 4u * (NS * T * LD + i), real ? vsrc + (size_t)(t0 + t) * r.ffn.in_cols + v0 + c : vsrc, real);
             }
-        for (int i = tid; i < TC * kScanCols; i += kScanThreads) {
-            const int t = i / kScanCols, c = i % kScanCols;
-            vbuf[(ch & 1) * TC * kScanCols + i] =
-                t0 + t < n && v0 + c < r.vdim ? r.ffn.proj[(size_t)(t0 + t) * r.ffn.in_cols + r.c_v + head * r.vdim + v0 + c] : 0.0f;
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.commit_group;" ::: "memory");   // (empty past the end: the group count stays in step)
     };
     load(0);
+    load(1);
     for (int ch = 0; ch < chunks; ch++) {
-        if (ch + 1 < chunks) {
-            load(ch + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const float4 *b4 = reinterpret_cast<const float4 *>(scan_smem + (ch & 1) * NS * TC * LD);
-        const float *vb = vbuf + (ch & 1) * TC * kScanCols + col;
-        const int nt = min(TC, n - ch * TC);
-        float po[TC];
+        asm volatile("cp.async.wait_group 1;" ::: "memory");   // chunk ch has landed
+        __syncthreads();                                       // for everybody, and everybody is done with chunk ch - 1
+        load(ch + 2);
+        const float *b = scan_smem + STAGE * (ch % kScanStages);
+        const int nt = min(T, n - ch * T);
+        float po[T * 4];
 #pragma unroll
-        for (int t = 0; t < TC; t++) {
-            po[t] = 0.0f;
+        for (int t = 0; t < T; t++) {
+            uint64_t o[4] = {0, 0, 0, 0};
             if (t < nt) {
-                const float v = vb[t * kScanCols];
-                float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
+                const float4 v = *reinterpret_cast<const float4 *>(b + NS * T * LD + t * COLS + wcol);
+                const uint64_t vd[4] = {pack2(v.x, v.x), pack2(v.y, v.y), pack2(v.z, v.z), pack2(v.w, v.w)};
 #pragma unroll
-                for (int i = 0; i < NI; i++) {
-                    const float4 q = b4[t * (LD / 4) + rg + 8 * i], k = b4[(TC + t) * (LD / 4) + rg + 8 * i];
-                    const float4 a = FIXED ? make_float4(fixed, fixed, fixed, fixed) : b4[((NS - 1) * TC + t) * (LD / 4) + rg + 8 * i];
-                    float *s = S + 4 * i;
-                    s[0] = fmaf(s[0], a.x, k.x * v);
-                    s[1] = fmaf(s[1], a.y, k.y * v);
-                    s[2] = fmaf(s[2], a.z, k.z * v);
-                    s[3] = fmaf(s[3], a.w, k.w * v);
-                    o0 = fmaf(s[0], q.x, o0);
-                    o1 = fmaf(s[1], q.y, o1);
-                    o2 = fmaf(s[2], q.z, o2);
-                    o3 = fmaf(s[3], q.w, o3);
+                for (int j = 0; j < NJ; j++) {
+                    const int at = 64 * j + 4 * rl;
+                    const ulonglong2 q = *reinterpret_cast<const ulonglong2 *>(b + t * LD + at);
+                    const ulonglong2 k = *reinterpret_cast<const ulonglong2 *>(b + (T + t) * LD + at);
+                    const ulonglong2 al = FIXED ? make_ulonglong2(fixed2, fixed2) : *reinterpret_cast<const ulonglong2 *>(b + ((NS - 1) * T + t) * LD + at);
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        S[j][0][c] = fma2(S[j][0][c], al.x, mul2(k.x, vd[c]));
+                        o[c] = fma2(S[j][0][c], q.x, o[c]);
+                    }
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        S[j][1][c] = fma2(S[j][1][c], al.y, mul2(k.y, vd[c]));
+                        o[c] = fma2(S[j][1][c], q.y, o[c]);
+                    }
                 }
-                po[t] = (o0 + o1) + (o2 + o3);
+            }
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                float lo, hi;
+                unpack2(o[c], lo, hi);
+                po[t * 4 + c] = lo + hi;
             }
         }
-        // sum over the eight threads of a column; thread rg ends up with token rg of the stage
-        if (TC == 8) {
+        // 32 sums over 16 lanes; bit 3 of the lane picks tokens 4 .. 7, bit 2 and 1 within them, bit 0 columns 2, 3
 #pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const float send = (rg & 4) ? po[i] : po[(i + 4) % TC], keep = (rg & 4) ? po[(i + 4) % TC] : po[i];
-                po[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 4);
+        for (int step = 0; step < 4; step++) {
+            const int half = 16 >> step, bit = 8 >> step;
+#pragma unroll
+            for (int i = 0; i < half; i++) {
+                const float send = (rl & bit) ? po[i] : po[i + half], keep = (rl & bit) ? po[i + half] : po[i];
+                po[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, bit);
             }
-        } else {
-#pragma unroll
-            for (int i = 0; i < 4; i++) po[i] += __shfl_xor_sync(0xFFFFFFFFu, po[i], 4);
         }
-#pragma unroll
-        for (int i = 0; i < 2; i++) {
-            const float send = (rg & 2) ? po[i] : po[i + 2], keep = (rg & 2) ? po[i + 2] : po[i];
-            po[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 2);
+        const int t = ch * T + (rl >> 1), col = v0 + wcol + 2 * (rl & 1);
+        if (t < n) {
+            float *o = r.o + ((size_t)t * r.heads + head) * r.vdim + col;
+            if (col < r.vdim) o[0] = po[0];
+            if (col + 1 < r.vdim) o[1] = po[1];
         }
-        {
-            const float send = (rg & 1) ? po[0] : po[1], keep = (rg & 1) ? po[1] : po[0];
-            po[0] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 1);
-        }
-        const int t = ch * TC + (rg & (TC - 1));
-        if (live && rg < TC && t < n) r.o[(size_t)t * r.heads * r.vdim + head * r.vdim + v0 + col] = po[0];
-        __syncthreads();   // this stage's buffer is free for chunk ch + 2
     }
 #pragma unroll
-    for (int i = 0; i < NI; i++)
+    for (int j = 0; j < NJ; j++)
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const int row = 32 * i + 4 * rg + j;
-            if (live && row < r.dim) state[(size_t)row * r.vdim] = S[4 * i + j];
-        }
+        for (int h = 0; h < 2; h++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                float s[2];
+                unpack2(S[j][h][c], s[0], s[1]);
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int row = 64 * j + 4 * rl + 2 * h + e, col = v0 + wcol + c;
+                    if (row < r.dim && col < r.vdim) state[(size_t)row * r.vdim + col] = s[e];
+                }
+            }
 }
 
 // act[row, head] = o / rms(o) (* weight) * silu(g): one warp per (row, head)
+template <bool VEC>
 __global__ void __launch_bounds__(128) rec_finish_kernel(const Recurrence r) {
     const int lane = threadIdx.x & 31;
-    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (item >= (long long)r.span.n * r.heads) return;
-    const int row = (int)(item / r.heads), head = (int)(item - (long long)row * r.heads);
-    const float *o = r.o + item * r.vdim;
-    float ss = 0.0f;
-    for (int d = lane; d < r.vdim; d += 32) ss = fmaf(o[d], o[d], ss);
-    const float rms = sqrtf(warp_sum(ss) / (float)r.vdim + r.eps);
+    const int item = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (item >= r.span.n * r.heads) return;
+    const int row = item / r.heads, head = item - row * r.heads;
+    const float *o = r.o + (size_t)item * r.vdim;
     const float *g = r.ffn.proj + (size_t)row * r.ffn.in_cols + r.c_g + head * r.vdim;
-    for (int d = lane; d < r.vdim; d += 32) {
-        float v = o[d] / rms;
-        if (r.head_norm) v *= r.head_norm[d];
-        store_act(r.ffn.act, r.ffn.act_dt, (size_t)row * r.ffn.out_k + head * r.vdim + d, v * silu_f32(g[d]));
+    const size_t at = (size_t)row * r.ffn.out_k + head * r.vdim;
+    float ss = 0.0f;
+    if constexpr (VEC) {   // vdim a multiple of 4, at most 512
+        float4 ov[4], gv[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int d = 4 * lane + 128 * i;
+            ov[i] = d < r.vdim ? *reinterpret_cast<const float4 *>(o + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            gv[i] = d < r.vdim ? *reinterpret_cast<const float4 *>(g + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            ss = fmaf(ov[i].x, ov[i].x, fmaf(ov[i].y, ov[i].y, fmaf(ov[i].z, ov[i].z, fmaf(ov[i].w, ov[i].w, ss))));
+        }
+        const float rms = sqrtf(warp_sum(ss) / (float)r.vdim + r.eps);
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int d = 4 * lane + 128 * i;
+            if (d >= r.vdim) continue;
+            const float4 w = r.head_norm ? *reinterpret_cast<const float4 *>(r.head_norm + d) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+            const float y0 = ov[i].x / rms * w.x * silu_f32(gv[i].x), y1 = ov[i].y / rms * w.y * silu_f32(gv[i].y);
+            const float y2 = ov[i].z / rms * w.z * silu_f32(gv[i].z), y3 = ov[i].w / rms * w.w * silu_f32(gv[i].w);
+            if (r.ffn.act_dt == NNQ_F32) {
+                *reinterpret_cast<float4 *>(reinterpret_cast<float *>(r.ffn.act) + at + d) = make_float4(y0, y1, y2, y3);
+            } else {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(y0, y1), b = __floats2bfloat162_rn(y2, y3);
+                *reinterpret_cast<uint2 *>(reinterpret_cast<__nv_bfloat16 *>(r.ffn.act) + at + d) =
+                    make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+            }
+        }
+    } else {
+        for (int d = lane; d < r.vdim; d += 32) ss = fmaf(o[d], o[d], ss);
+        const float rms = sqrtf(warp_sum(ss) / (float)r.vdim + r.eps);
+        for (int d = lane; d < r.vdim; d += 32) {
+            float v = o[d] / rms;
+            if (r.head_norm) v *= r.head_norm[d];
+            store_act(r.ffn.act, r.ffn.act_dt, at + d, v * silu_f32(g[d]));
+        }
     }
 }
 
@@ -207,6 +282,7 @@ constexpr int kStepWarps = 16, kStepBatch = 8;
 // the head's state (read and written once), norms and gates the output; the other CTAs do the feed-forward part.
 __global__ void __launch_bounds__(kStepWarps * 32) rec_step_kernel(const Recurrence r) {
     pdl_prologue();
+    pdl_release();
     extern __shared__ float step_smem[];   // q, k, decay [dim], v [vdim], partial o [warps, vdim]
     __shared__ float red[32];
     if ((int)blockIdx.x >= r.heads) {
@@ -276,22 +352,28 @@ __global__ void __launch_bounds__(kStepWarps * 32) rec_step_kernel(const Recurre
 
 // ---- host side ----
 
-template <int NI>
+template <int NJ, int WARPS, bool FIXED>
 static nnq_status go_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
-    constexpr int TC = NI <= 4 ? 8 : 4;
-    const bool fixed = r.rank == 0;
-    const size_t smem = (size_t)(2 * (fixed ? 2 : 3) * TC * NI * 32 + 2 * TC * kScanCols) * sizeof(float);
-    const dim3 grid(r.heads, (r.vdim + kScanCols - 1) / kScanCols);
+    constexpr size_t smem = (size_t)kScanStages * kScanTokens * ((FIXED ? 2 : 3) * NJ * 64 + WARPS * 8) * sizeof(float);
+    auto kernel = rec_scan_kernel<NJ, WARPS, FIXED>;
     if (smem > 48 * 1024) {
-        nnq_status s = check_cuda(ctx, fixed ? cudaFuncSetAttribute(rec_scan_kernel<NI, TC, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
-                                             : cudaFuncSetAttribute(rec_scan_kernel<NI, TC, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem),
-                                  "recurrence shared memory");
+        nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "recurrence shared memory");
         if (s != NNQ_OK) return s;
     }
-    if (fixed) rec_scan_kernel<NI, TC, true><<<grid, kScanThreads, smem, st>>>(r);
-    else rec_scan_kernel<NI, TC, false><<<grid, kScanThreads, smem, st>>>(r);
+    kernel<<<dim3(r.heads, (r.vdim + WARPS * 8 - 1) / (WARPS * 8)), WARPS * 32, smem, st>>>(r);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "recurrence launch");
+}
+
+// Four warps share a head's q / k / decay rows where that leaves enough CTAs, else fewer do.
+template <int NJ>
+static nnq_status pick_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
+    auto ctas = [&](int cols) { return r.heads * ((r.vdim + cols - 1) / cols); };
+    const int enough = ctx->sm_count * 3 / 4;
+    const bool fixed = r.rank == 0;
+    if (ctas(32) >= enough) return fixed ? go_scan<NJ, 4, true>(ctx, r, st) : go_scan<NJ, 4, false>(ctx, r, st);
+    if (ctas(16) >= enough) return fixed ? go_scan<NJ, 2, true>(ctx, r, st) : go_scan<NJ, 2, false>(ctx, r, st);
+    return fixed ? go_scan<NJ, 1, true>(ctx, r, st) : go_scan<NJ, 1, false>(ctx, r, st);
 }
 
 nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
@@ -302,20 +384,17 @@ nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
     ctx->launches++;
     nnq_status s = check_cuda(ctx, cudaGetLastError(), "recurrence prologue launch");
     if (s != NNQ_OK) return s;
-    switch (r.dim_ld / 32) {
-        case 1: s = go_scan<1>(ctx, r, st); break;
-        case 2: s = go_scan<2>(ctx, r, st); break;
-        case 3: s = go_scan<3>(ctx, r, st); break;
-        case 4: s = go_scan<4>(ctx, r, st); break;
-        case 5: s = go_scan<5>(ctx, r, st); break;
-        case 6: s = go_scan<6>(ctx, r, st); break;
-        case 7: s = go_scan<7>(ctx, r, st); break;
-        case 8: s = go_scan<8>(ctx, r, st); break;
+    switch (r.dim_ld / 64) {
+        case 1: s = pick_scan<1>(ctx, r, st); break;
+        case 2: s = pick_scan<2>(ctx, r, st); break;
+        case 3: s = pick_scan<3>(ctx, r, st); break;
+        case 4: s = pick_scan<4>(ctx, r, st); break;
         default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "key dimension %d of a recurrence is above %d", r.dim, kRecMaxKeyDim);
     }
     if (s != NNQ_OK) return s;
-    const long long items = (long long)r.span.n * r.heads;
-    rec_finish_kernel<<<(unsigned)((items + 3) / 4), 128, 0, st>>>(r);
+    const int ctas = (r.span.n * r.heads + 3) / 4;
+    if (r.vdim % 4 == 0 && r.vdim <= 512) rec_finish_kernel<true><<<ctas, 128, 0, st>>>(r);
+    else rec_finish_kernel<false><<<ctas, 128, 0, st>>>(r);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "recurrence epilogue launch");
 }
