@@ -419,6 +419,7 @@ static nnq_status go_rows(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
 }
 
 nnq_status launch_attn_rows(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
+    if (attn_tc_supported(a)) return launch_attn_tc(ctx, a, st);
     return a.vdim_ld <= 128 ? go_rows<8, 1>(ctx, a, st) : go_rows<8, 2>(ctx, a, st);
 }
 

@@ -62,6 +62,8 @@ struct WindowAttn {
 nnq_status launch_attn_prep(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);       // convolution, rotation, mixing, cache append, ffn part
 nnq_status launch_attn_conv_tail(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);  // n > 1: the last taps - 1 rows enter the ring
 nnq_status launch_attn_rows(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);       // block of rows
+bool attn_tc_supported(const WindowAttn &a);                                           // attn_tc.cu: block of rows on the tensor cores
+nnq_status launch_attn_tc(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);
 nnq_status launch_attn_decode(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);     // one row
 int attn_decode_ranges(int window, int max_seq);                                       // key ranges of the decode kernel
 size_t attn_decode_part_floats(int heads, int kv_heads, int vdim_ld, int ranges);

@@ -25,6 +25,7 @@
 #include "decode.cuh"
 #include "gemm_tc.h"
 #include "sync.cuh"
+#include "tcgen05.cuh"
 
 namespace nnq {
 
@@ -204,43 +205,10 @@ constexpr int kDgABytes = kDgBM * 128;
 constexpr int kDgThreads = 192;
 __host__ __device__ constexpr int dg_stage_bytes(int bn) { return kDgABytes + bn * 128; }
 
-__device__ __forceinline__ void dg_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void dg_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-
-// K-major tile, 128-byte swizzle: rows of 128 bytes, 8-row groups 1024 bytes apart
-__device__ __forceinline__ uint64_t dg_smem_desc(uint32_t addr) {
-    const uint32_t lo = ((addr >> 4) & 0x3FFFu) | (1u << 16);
-    const uint32_t hi = (1024u >> 4) | (1u << 14) | (2u << 29);
-    return ((uint64_t)hi << 32) | lo;
-}
-
-__device__ __forceinline__ void dg_mma(uint32_t tmem_d, uint64_t da, uint64_t db, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
-        " tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}"
-        ::"r"(tmem_d), "l"(da), "l"(db), "r"(idesc), "r"(accumulate) : "memory");
-}
-
-__device__ __forceinline__ void dg_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-
 __device__ __forceinline__ void dg_tma_2d(uint32_t dst, const CUtensorMap *map, int x, int y, uint32_t bar) {
     asm volatile(
         "cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
         ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(bar) : "memory");
-}
-
-__device__ __forceinline__ void dg_tmem_ld32(uint32_t addr, uint32_t (&v)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
-          "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
-          "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-        : "r"(addr));
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
 
 // Grouped mode (expert products): the rows of x are sorted by expert (offsets[e] .. offsets[e+1]
@@ -313,9 +281,9 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_s)), "r"(512u) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    dg_fence_before();
+    tc_fence_before();
     __syncthreads();
-    dg_fence_after();
+    tc_fence_after();
     const uint32_t tmem_base = tmem_base_s;
     bool ok = true;
 
@@ -361,25 +329,25 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
                     ok = false;
                     break;
                 }
-                dg_fence_after();
+                tc_fence_after();
                 const uint32_t acc = tmem_base + (uint32_t)(a * kDgBN);
                 for (int kb = 0; kb < nkb; kb++) {
                     if (!mbar_wait_fast(full_s + 8 * slot, phase)) {
                         ok = false;
                         break;
                     }
-                    dg_fence_after();
+                    tc_fence_after();
                     const uint32_t a_s = smem_u32(smem + (size_t)slot * kDgStageBytes);
-                    const uint64_t da = dg_smem_desc(a_s), db = dg_smem_desc(a_s + kDgABytes);
+                    const uint64_t da = smem_desc(a_s), db = smem_desc(a_s + kDgABytes);
 #pragma unroll
-                    for (int k = 0; k < 4; k++) dg_mma(acc, da + 2 * k, db + 2 * k, idesc, (kb | k) != 0);
-                    dg_commit(empty_s + 8 * slot);
+                    for (int k = 0; k < 4; k++) umma_bf16(acc, da + 2 * k, db + 2 * k, idesc, (kb | k) != 0);
+                    umma_commit(empty_s + 8 * slot);
                     if (++slot == kDgStages) {
                         slot = 0;
                         phase ^= 1u;
                     }
                 }
-                if (ok) dg_commit(accf_s + 8 * a);
+                if (ok) umma_commit(accf_s + 8 * a);
             }
         }
     } else {
@@ -395,12 +363,12 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
                 ok = false;
                 break;
             }
-            dg_fence_after();
+            tc_fence_after();
             const int row = m0 + q * 32 + lane;
 #pragma unroll 1
             for (int cc = 0; cc < kDgBN / 32; cc++) {
                 uint32_t v[32];
-                dg_tmem_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * kDgBN + cc * 32), v);
+                tmem_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * kDgBN + cc * 32), v);
                 const int col0 = n0 + cc * 32;
                 if (h_out) {
                     // interleaved gate / up columns (2j, 2j + 1): h[row, j] = clamp(silu(g), +-limit) * u in bf16,
@@ -472,7 +440,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
                     }
                 }
             }
-            dg_fence_before();
+            tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(acce_s + 8 * a);
         }
@@ -488,7 +456,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
             mbar_wait(accf_s, 0);
             mbar_wait(accf_s + 8, 0);
         }
-        dg_fence_after();
+        tc_fence_after();
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(512u) : "memory");
     }
 }

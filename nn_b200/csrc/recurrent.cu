@@ -70,11 +70,11 @@ __global__ void __launch_bounds__(kRecPrepWarps * 32) rec_prep_kernel(const Recu
 
 // ---- the scan over a block of rows ----
 //
-// A warp owns eight columns of the state over all key rows: lane = 16 row groups x 2 column groups, a lane
-// holds rows 64 j + 4 (lane % 16) .. + 3 and four columns as packed f32 pairs (two rows of a column), so that
+// A warp owns 2 C columns of the state over all key rows: lane = 16 row groups x 2 column groups, a lane
+// holds rows 64 j + 4 (lane % 16) .. + 3 and C columns as packed f32 pairs (two rows of a column), so that
 // q, k and the decay come as pairs out of one 16-byte shared-memory read and the three operations of a state
 // element -- k v, s a + (k v), o + s q -- are packed f32x2 instructions. After eight tokens the lanes' partial
-// o are reduced across the row groups by halving exchanges: every lane ends with one token and two columns.
+// o are reduced across the row groups by halving exchanges: a lane ends with one token of one or two columns.
 // Tokens stream through a three-stage ring of cp.async copies, one barrier per stage.
 
 constexpr int kScanTokens = 8, kScanStages = 3;
@@ -103,24 +103,24 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
     return r;
 }
 
-// grid (heads, ceil(vdim / (8 WARPS))); NJ = dim_ld / 64
-template <int NJ, int WARPS, bool FIXED>
+// grid (heads, ceil(vdim / (2 C WARPS))); NJ = dim_ld / 64
+template <int NJ, int C, int WARPS, bool FIXED>
 __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r) {
     constexpr int NS = FIXED ? 2 : 3;   // streams: q, k (, decay)
-    constexpr int LD = NJ * 64, COLS = WARPS * 8, T = kScanTokens, THREADS = WARPS * 32;
+    constexpr int LD = NJ * 64, COLS = WARPS * 2 * C, T = kScanTokens, THREADS = WARPS * 32;
     constexpr int STAGE = T * (NS * LD + COLS);   // floats
     extern __shared__ __align__(16) float scan_smem[];
     const int tid = threadIdx.x, lane = tid & 31, rl = lane & 15;
-    const int wcol = (tid >> 5) * 8 + (lane >> 4) * 4;
+    const int wcol = ((tid >> 5) * 2 + (lane >> 4)) * C;
     const int head = blockIdx.x, v0 = blockIdx.y * COLS, n = r.span.n;
     float *state = r.state + (size_t)head * r.dim * r.vdim;
-    uint64_t S[NJ][2][4];
+    uint64_t S[NJ][2][C];
 #pragma unroll
     for (int j = 0; j < NJ; j++)
 #pragma unroll
         for (int h = 0; h < 2; h++)
 #pragma unroll
-            for (int c = 0; c < 4; c++) {
+            for (int c = 0; c < C; c++) {
                 float s[2];
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
@@ -164,13 +164,17 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
         load(ch + 2);
         const float *b = scan_smem + STAGE * (ch % kScanStages);
         const int nt = min(T, n - ch * T);
-        float po[T * 4];
+        float po[T * C];
 #pragma unroll
         for (int t = 0; t < T; t++) {
-            uint64_t o[4] = {0, 0, 0, 0};
+            uint64_t o[C];
+#pragma unroll
+            for (int c = 0; c < C; c++) o[c] = 0;
             if (t < nt) {
-                const float4 v = *reinterpret_cast<const float4 *>(b + NS * T * LD + t * COLS + wcol);
-                const uint64_t vd[4] = {pack2(v.x, v.x), pack2(v.y, v.y), pack2(v.z, v.z), pack2(v.w, v.w)};
+                const float *v = b + NS * T * LD + t * COLS + wcol;
+                uint64_t vd[C];
+#pragma unroll
+                for (int c = 0; c < C; c++) vd[c] = pack2(v[c], v[c]);
 #pragma unroll
                 for (int j = 0; j < NJ; j++) {
                     const int at = 64 * j + 4 * rl;
@@ -178,39 +182,45 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
                     const ulonglong2 k = *reinterpret_cast<const ulonglong2 *>(b + (T + t) * LD + at);
                     const ulonglong2 al = FIXED ? make_ulonglong2(fixed2, fixed2) : *reinterpret_cast<const ulonglong2 *>(b + ((NS - 1) * T + t) * LD + at);
 #pragma unroll
-                    for (int c = 0; c < 4; c++) {
+                    for (int c = 0; c < C; c++) {
                         S[j][0][c] = fma2(S[j][0][c], al.x, mul2(k.x, vd[c]));
                         o[c] = fma2(S[j][0][c], q.x, o[c]);
                     }
 #pragma unroll
-                    for (int c = 0; c < 4; c++) {
+                    for (int c = 0; c < C; c++) {
                         S[j][1][c] = fma2(S[j][1][c], al.y, mul2(k.y, vd[c]));
                         o[c] = fma2(S[j][1][c], q.y, o[c]);
                     }
                 }
             }
 #pragma unroll
-            for (int c = 0; c < 4; c++) {
+            for (int c = 0; c < C; c++) {
                 float lo, hi;
                 unpack2(o[c], lo, hi);
-                po[t * 4 + c] = lo + hi;
+                po[t * C + c] = lo + hi;
             }
         }
-        // 32 sums over 16 lanes; bit 3 of the lane picks tokens 4 .. 7, bit 2 and 1 within them, bit 0 columns 2, 3
+        // 8 C sums over 16 lanes: bits 3, 2, 1 of the lane pick a token, bit 0 the upper half of the columns
 #pragma unroll
         for (int step = 0; step < 4; step++) {
-            const int half = 16 >> step, bit = 8 >> step;
+            const int half = (T * C / 2) >> step, bit = 8 >> step;
+            if (half == 0) {
+                po[0] += __shfl_xor_sync(0xFFFFFFFFu, po[0], bit);
+            } else {
 #pragma unroll
-            for (int i = 0; i < half; i++) {
-                const float send = (rl & bit) ? po[i] : po[i + half], keep = (rl & bit) ? po[i + half] : po[i];
-                po[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, bit);
+                for (int i = 0; i < half; i++) {
+                    const float send = (rl & bit) ? po[i] : po[i + half], keep = (rl & bit) ? po[i + half] : po[i];
+                    po[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, bit);
+                }
             }
         }
-        const int t = ch * T + (rl >> 1), col = v0 + wcol + 2 * (rl & 1);
-        if (t < n) {
+        constexpr int LEFT = C >= 2 ? C / 2 : 1;
+        const int t = ch * T + (rl >> 1), col = v0 + wcol + (C >= 2 ? LEFT * (rl & 1) : 0);
+        if (t < n && (C >= 2 || (rl & 1) == 0)) {
             float *o = r.o + ((size_t)t * r.heads + head) * r.vdim + col;
-            if (col < r.vdim) o[0] = po[0];
-            if (col + 1 < r.vdim) o[1] = po[1];
+#pragma unroll
+            for (int i = 0; i < LEFT; i++)
+                if (col + i < r.vdim) o[i] = po[i];
         }
     }
 #pragma unroll
@@ -218,7 +228,7 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
 #pragma unroll
         for (int h = 0; h < 2; h++)
 #pragma unroll
-            for (int c = 0; c < 4; c++) {
+            for (int c = 0; c < C; c++) {
                 float s[2];
                 unpack2(S[j][h][c], s[0], s[1]);
 #pragma unroll
@@ -352,28 +362,31 @@ __global__ void __launch_bounds__(kStepWarps * 32) rec_step_kernel(const Recurre
 
 // ---- host side ----
 
-template <int NJ, int WARPS, bool FIXED>
+template <int NJ, int C, int WARPS, bool FIXED>
 static nnq_status go_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
-    constexpr size_t smem = (size_t)kScanStages * kScanTokens * ((FIXED ? 2 : 3) * NJ * 64 + WARPS * 8) * sizeof(float);
-    auto kernel = rec_scan_kernel<NJ, WARPS, FIXED>;
+    constexpr int cols = WARPS * 2 * C;
+    constexpr size_t smem = (size_t)kScanStages * kScanTokens * ((FIXED ? 2 : 3) * NJ * 64 + cols) * sizeof(float);
+    auto kernel = rec_scan_kernel<NJ, C, WARPS, FIXED>;
     if (smem > 48 * 1024) {
         nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "recurrence shared memory");
         if (s != NNQ_OK) return s;
     }
-    kernel<<<dim3(r.heads, (r.vdim + WARPS * 8 - 1) / (WARPS * 8)), WARPS * 32, smem, st>>>(r);
+    kernel<<<dim3(r.heads, (r.vdim + cols - 1) / cols), WARPS * 32, smem, st>>>(r);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "recurrence launch");
 }
 
-// Four warps share a head's q / k / decay rows where that leaves enough CTAs, else fewer do.
+// Wide tiles amortise the shared-memory reads of q / k / decay over more columns, narrow ones give more warps.
+// Measured on 128 x 256 heads (us per 1024 rows, all kernels of the mixer): 16 heads 259 / 279 / 377 with C = 4 / 2 / 1,
+// 8 heads 229 / 191 / 234; 8 heads of 64 x 64: 148 / 138 / 117.
 template <int NJ>
 static nnq_status pick_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
-    auto ctas = [&](int cols) { return r.heads * ((r.vdim + cols - 1) / cols); };
-    const int enough = ctx->sm_count * 3 / 4;
     const bool fixed = r.rank == 0;
-    if (ctas(32) >= enough) return fixed ? go_scan<NJ, 4, true>(ctx, r, st) : go_scan<NJ, 4, false>(ctx, r, st);
-    if (ctas(16) >= enough) return fixed ? go_scan<NJ, 2, true>(ctx, r, st) : go_scan<NJ, 2, false>(ctx, r, st);
-    return fixed ? go_scan<NJ, 1, true>(ctx, r, st) : go_scan<NJ, 1, false>(ctx, r, st);
+    auto warps = [&](int c) { return r.heads * ((r.vdim + 2 * c - 1) / (2 * c)); };
+    const int enough = ctx->sm_count * 5 / 2;
+    if (warps(4) >= enough) return fixed ? go_scan<NJ, 4, 4, true>(ctx, r, st) : go_scan<NJ, 4, 4, false>(ctx, r, st);
+    if (warps(2) >= enough) return fixed ? go_scan<NJ, 2, 4, true>(ctx, r, st) : go_scan<NJ, 2, 4, false>(ctx, r, st);
+    return fixed ? go_scan<NJ, 1, 4, true>(ctx, r, st) : go_scan<NJ, 1, 4, false>(ctx, r, st);
 }
 
 nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {

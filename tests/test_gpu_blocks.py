@@ -369,3 +369,24 @@ def test_f32_products_round_nothing(m, n, k, fmt):
     want = x.astype(np.float64) @ w.astype(np.float64).T
     assert np.abs(y - want).max() <= 2e-6 * np.sqrt(k) * np.abs(want).max()
     t.release()
+
+
+# ---- attention of a block of rows on the tensor cores (bf16 decoders) ----
+
+@pytest.mark.parametrize("heads,kv,dim,vdim,window", [(4, 2, 24, 20, 9), (8, 1, 96, 48, 96), (6, 3, 128, 128, 70), (4, 4, 64, 40, 300), (12, 2, 72, 100, 33),
+                                                       (5, 5, 8, 8, 1), (16, 2, 128, 96, 2000)])
+def test_tensor_core_attention_is_as_exact_as_the_decode_kernel(tmp_path, heads, kv, dim, vdim, window):
+    """A bf16 decoder's prompt pass (operands split into two bf16 terms) against its own decode steps (f32 on the
+    CUDA cores): everything before and after the attention rounds alike, so the two agree far more closely than
+    either agrees with the unrounded model."""
+    cfg = M.config([M.attention(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, window=window, rot=(1e4, dim // 4 * 2), scale=3.0 * dim ** -0.5)], width=64, vocab=96)
+    t = M.tensors(cfg, seed=heads)
+    ids = tokens(330, 96, 2)
+    dec = load(tmp_path, cfg, t, api.BF16, max_seq=400, block_rows=150)
+    want = run(dec, ids, [1] * 330).astype(np.float64)
+    for cuts in ([], [40, 111, 33], [200]):
+        d = run(dec, ids, cuts) - want
+        assert np.sqrt((d * d).mean() / (want * want).mean()) <= 2e-3, cuts
+    assert err(want, ref.forward(cfg, t, ids, np.float32)) <= BF16_TOL
+    dec.backend.device_status()
+    dec.release()
