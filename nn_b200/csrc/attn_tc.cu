@@ -42,8 +42,8 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t 
 // byte offset of element e (0 .. 63) of row r inside a swizzled tile of 128-byte rows
 __device__ __forceinline__ uint32_t swz_at(int r, int e) { return swz(r, e >> 3) + 2 * (e & 7); }
 
-template <int NV>
-__global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn a, int atoms, int *status) {
+template <int ATOMS, int NV>
+__global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn a, int *status) {
     extern __shared__ __align__(1024) uint8_t at_smem_raw[];
     uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(at_smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ __align__(8) uint64_t bars[6];   // kv_full[2], kv_empty[2], s_full, p_full
@@ -55,8 +55,8 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
     const int pos0 = a.span.pos0;
     const int first = max(0, pos0 + t0 / group - a.window + 1), last = pos0 + last_pair / group;   // keys some row sees
     const int tiles = (last - first) / kAtKeys + 1;
-    uint8_t *q_s = smem, *kv_s = q_s + at_q_bytes(atoms), *p_s = kv_s + 2 * (at_k_bytes(atoms) + at_v_bytes(NV));
-    const int kv_stage = at_k_bytes(atoms) + at_v_bytes(NV);
+    uint8_t *q_s = smem, *kv_s = q_s + at_q_bytes(ATOMS), *p_s = kv_s + 2 * (at_k_bytes(ATOMS) + at_v_bytes(NV));
+    const int kv_stage = at_k_bytes(ATOMS) + at_v_bytes(NV);
 
     if (tid == 0) {
         for (int i = 0; i < 2; i++) {
@@ -76,14 +76,14 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
         for (int r = warp; r < kAtRows; r += 4) {
             const int t = t0 + r;
             const float *src = a.qrot + ((size_t)(t / group) * a.heads + kvh * group + t % group) * a.dim_ld;
-            for (int d = 4 * lane; d < 64 * atoms; d += 128) {
+            for (int d = 4 * lane; d < 64 * ATOMS; d += 128) {
                 const float4 v = t <= last_pair && d < a.dim_ld ? *reinterpret_cast<const float4 *>(src + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 uint2 hi, lo;
                 split2(v.x, v.y, hi.x, lo.x);
                 split2(v.z, v.w, hi.y, lo.y);
                 uint8_t *dst = q_s + (d >> 6) * kAtQAtom + swz_at(r, d & 63);
                 *reinterpret_cast<uint2 *>(dst) = hi;
-                *reinterpret_cast<uint2 *>(dst + atoms * kAtQAtom) = lo;
+                *reinterpret_cast<uint2 *>(dst + ATOMS * kAtQAtom) = lo;
             }
         }
         fence_async_smem();
@@ -184,43 +184,57 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
         }
     } else if (warp < 4 + kAtLoaders) {
         // ---------------- loaders ----------------
-        const int w = warp - 4;
+        // The cache is read from L2 in batches held in registers, always one batch ahead of the conversion (the
+        // next tile's keys are under way before this tile is handed over).
+        constexpr int LT = kAtLoaders * 32;
+        constexpr int KU = kAtKeys * 16 * ATOMS, KB = (KU + 2 * LT - 1) / (2 * LT);                // units of four dimensions of a key, two batches
+        constexpr int VB = (NV * 8 + 2 * kAtLoaders - 1) / (2 * kAtLoaders);                       // groups of four value dimensions, two batches
+        const int w = warp - 4, lt = tid - 128;
         const float *kb = a.kcache + (size_t)kvh * a.cap * a.dim_ld, *vb = a.vcache + (size_t)kvh * a.cap * a.vdim_ld;
-        for (int t = 0; t < tiles; t++) {
-            const int st = t & 1;
-            if (t >= 2 && !mbar_wait_fast(kve + 8 * st, ((t >> 1) - 1) & 1)) {
-                ok = false;
-                break;
-            }
-            uint8_t *k_s = kv_s + st * kv_stage, *v_s = k_s + at_k_bytes(atoms);
-            const int k0 = first + t * kAtKeys, have = min(kAtKeys, last - k0 + 1), s0 = k0 % a.cap;
-            // keys: a warp per key, lanes over the dimensions
-#pragma unroll 4
-            for (int j = w; j < kAtKeys; j += kAtLoaders) {
-                int slot = s0 + j;
+        const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const int j = 2 * lane;   // values: lane = pair of keys, a warp every third group of dimensions
+        auto load_k = [&](int t, int b, float4 (&v)[KB]) {   // neighbouring lanes take neighbouring dimensions
+            const int k0 = first + t * kAtKeys, have = t < tiles ? min(kAtKeys, last - k0 + 1) : 0, s0 = k0 % a.cap;
+#pragma unroll
+            for (int i = 0; i < KB; i++) {
+                const int u = lt + LT * (b * KB + i), key = u / (16 * ATOMS), d = 4 * (u % (16 * ATOMS));
+                int slot = s0 + key;
                 if (slot >= a.cap) slot -= a.cap;
-                const float *src = kb + (size_t)slot * a.dim_ld;
-                for (int d = 4 * lane; d < 64 * atoms; d += 128) {
-                    const float4 v = j < have && d < a.dim_ld ? *reinterpret_cast<const float4 *>(src + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                    uint2 hi, lo;
-                    split2(v.x, v.y, hi.x, lo.x);
-                    split2(v.z, v.w, hi.y, lo.y);
-                    uint8_t *dst = k_s + (d >> 6) * kAtKAtom + swz_at(j, d & 63);
-                    *reinterpret_cast<uint2 *>(dst) = hi;
-                    *reinterpret_cast<uint2 *>(dst + atoms * kAtKAtom) = lo;
-                }
+                v[i] = key < have && d < a.dim_ld ? *reinterpret_cast<const float4 *>(kb + (size_t)slot * a.dim_ld + d) : zero;
             }
-            // values, transposed: lane = pair of keys, a warp every third group of four dimensions
-            const int j = 2 * lane;
+        };
+        auto store_k = [&](uint8_t *k_s, int b, const float4 (&v)[KB]) {
+#pragma unroll
+            for (int i = 0; i < KB; i++) {
+                const int u = lt + LT * (b * KB + i), key = u / (16 * ATOMS), d = 4 * (u % (16 * ATOMS));
+                if (u >= KU) continue;
+                uint2 hi, lo;
+                split2(v[i].x, v[i].y, hi.x, lo.x);
+                split2(v[i].z, v[i].w, hi.y, lo.y);
+                uint8_t *dst = k_s + (d >> 6) * kAtKAtom + swz_at(key, d & 63);
+                *reinterpret_cast<uint2 *>(dst) = hi;
+                *reinterpret_cast<uint2 *>(dst + ATOMS * kAtKAtom) = lo;
+            }
+        };
+        auto load_v = [&](int t, int b, float4 (&x)[VB], float4 (&y)[VB]) {
+            const int k0 = first + t * kAtKeys, have = min(kAtKeys, last - k0 + 1), s0 = k0 % a.cap;
             int sa = s0 + j, sb = s0 + j + 1;
             if (sa >= a.cap) sa -= a.cap;
             if (sb >= a.cap) sb -= a.cap;
             const float *va = vb + (size_t)sa * a.vdim_ld, *vc = vb + (size_t)sb * a.vdim_ld;
-#pragma unroll 4
-            for (int d = 4 * w; d < NV * 32; d += 4 * kAtLoaders) {
-                const float4 x = j < have && d < a.vdim_ld ? *reinterpret_cast<const float4 *>(va + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                const float4 y = j + 1 < have && d < a.vdim_ld ? *reinterpret_cast<const float4 *>(vc + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+            for (int i = 0; i < VB; i++) {
+                const int d = 4 * (w + kAtLoaders * (b * VB + i));
+                x[i] = j < have && d < a.vdim_ld ? *reinterpret_cast<const float4 *>(va + d) : zero;
+                y[i] = j + 1 < have && d < a.vdim_ld ? *reinterpret_cast<const float4 *>(vc + d) : zero;
+            }
+        };
+        auto store_v = [&](uint8_t *v_s, int b, const float4 (&x)[VB], const float4 (&y)[VB]) {   // transposed
+#pragma unroll
+            for (int i = 0; i < VB; i++) {
+                const int d = 4 * (w + kAtLoaders * (b * VB + i));
+                if (d >= NV * 32) continue;
+                const float xv[4] = {x[i].x, x[i].y, x[i].z, x[i].w}, yv[4] = {y[i].x, y[i].y, y[i].z, y[i].w};
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     uint32_t hi, lo;
@@ -230,6 +244,25 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
                     *reinterpret_cast<uint32_t *>(dst + NV * 32 * 128) = lo;
                 }
             }
+        };
+        float4 ka[KB], kc[KB], vx[VB], vy[VB];
+        load_k(0, 0, ka);
+        load_k(0, 1, kc);
+        for (int t = 0; t < tiles; t++) {
+            const int st = t & 1;
+            uint8_t *k_s = kv_s + st * kv_stage, *v_s = k_s + at_k_bytes(ATOMS);
+            if (t >= 2 && !mbar_wait_fast(kve + 8 * st, ((t >> 1) - 1) & 1)) {
+                ok = false;
+                break;
+            }
+            load_v(t, 0, vx, vy);
+            store_k(k_s, 0, ka);
+            store_k(k_s, 1, kc);
+            load_k(t + 1, 0, ka);
+            store_v(v_s, 0, vx, vy);
+            load_v(t, 1, vx, vy);
+            load_k(t + 1, 1, kc);
+            store_v(v_s, 1, vx, vy);
             fence_async_smem();
             mbar_arrive(kvf + 8 * st);
         }
@@ -243,8 +276,8 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
             bool add = false;
 #pragma unroll 1
             for (int x = 0; x < 3; x++) {   // hi hi, hi lo, lo hi
-                const uint32_t qo = qa + (x == 2 ? atoms * kAtQAtom : 0), ko = ka + (x == 1 ? atoms * kAtKAtom : 0);
-                for (int at = 0; at < atoms; at++) {
+                const uint32_t qo = qa + (x == 2 ? ATOMS * kAtQAtom : 0), ko = ka + (x == 1 ? ATOMS * kAtKAtom : 0);
+                for (int at = 0; at < ATOMS; at++) {
                     const uint64_t dq = smem_desc(qo + at * kAtQAtom), dk = smem_desc(ko + at * kAtKAtom);
 #pragma unroll
                     for (int k = 0; k < 4; k++) {
@@ -264,7 +297,7 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
                 break;
             }
             tc_fence_after();
-            const uint32_t va = smem_u32(kv_s + (t & 1) * kv_stage) + at_k_bytes(atoms);
+            const uint32_t va = smem_u32(kv_s + (t & 1) * kv_stage) + at_k_bytes(ATOMS);
 #pragma unroll 1
             for (int x = 0; x < 3; x++) {
                 const uint64_t dp = smem_desc(pa + (x == 2 ? kAtQAtom : 0)), dv = smem_desc(va + (x == 1 ? NV * 32 * 128 : 0));
@@ -304,22 +337,23 @@ bool attn_tc_supported(const WindowAttn &a) {
     return a.ffn.act_dt == NNQ_BF16 && a.dim <= 128 && a.vdim <= 128 && a.span.n * (a.heads / a.kv_heads) >= 32;
 }
 
-template <int NV>
+template <int ATOMS, int NV>
 static nnq_status at_go(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
-    const int atoms = (a.dim + 63) / 64, smem = at_smem_bytes(atoms, NV), pairs = a.span.n * (a.heads / a.kv_heads);
-    nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(attn_tc_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "attention shared memory");
+    const int smem = at_smem_bytes(ATOMS, NV), pairs = a.span.n * (a.heads / a.kv_heads);
+    nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(attn_tc_kernel<ATOMS, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "attention shared memory");
     if (s != NNQ_OK) return s;
-    attn_tc_kernel<NV><<<dim3(a.kv_heads, (pairs + kAtRows - 1) / kAtRows), kAtThreads, smem, st>>>(a, atoms, ctx->d_status);
+    attn_tc_kernel<ATOMS, NV><<<dim3(a.kv_heads, (pairs + kAtRows - 1) / kAtRows), kAtThreads, smem, st>>>(a, ctx->d_status);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "tensor-core attention launch");
 }
 
 nnq_status launch_attn_tc(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
+    const bool two = a.dim > 64;
     switch ((a.vdim + 31) / 32) {
-        case 1: return at_go<1>(ctx, a, st);
-        case 2: return at_go<2>(ctx, a, st);
-        case 3: return at_go<3>(ctx, a, st);
-        default: return at_go<4>(ctx, a, st);
+        case 1: return two ? at_go<2, 1>(ctx, a, st) : at_go<1, 1>(ctx, a, st);
+        case 2: return two ? at_go<2, 2>(ctx, a, st) : at_go<1, 2>(ctx, a, st);
+        case 3: return two ? at_go<2, 3>(ctx, a, st) : at_go<1, 3>(ctx, a, st);
+        default: return two ? at_go<2, 4>(ctx, a, st) : at_go<1, 4>(ctx, a, st);
     }
 }
 

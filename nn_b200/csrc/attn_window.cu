@@ -248,125 +248,318 @@ __global__ void __launch_bounds__(32) attn_rows_kernel(const WindowAttn a) {
     }
 }
 
-constexpr int kDecWarps = 4;
-constexpr int kDecMaxRanges = 32;
+// ---- one token: everything of the layer between its two products in one launch ----
+//
+// CTA = (kv head, tile of P query heads of its group, range of keys); 256 threads. Before it waits for the product
+// in front of it, a CTA asks for the keys and values of its range (they do not depend on this token) and forms the
+// part of its convolutions that lies in the past. After the wait: convolution and rotation of its query heads (and
+// of the new key and value in the CTAs that hold the current position), scores with a warp per eighth of the
+// dimensions, softmax with a lane per two keys, values with a thread per dimension. Ranges are merged by the CTA of
+// a (kv head, tile) that finishes last. Further CTAs do the feed-forward part.
+constexpr int kStepThreads = 256, kStepKeys = 64, kStepMaxRanges = 64;
 
-// One token: grid (kv head, key range, tile of P query heads of the group). The window's batches of 32
-// keys are dealt to the ranges (contiguous) and to a CTA's warps; the warps merge through shared memory.
-// With several ranges a CTA publishes a record (m, l, acc) per head and the last CTA of its (kv head,
-// tile) to arrive merges the records; the counter is back at zero for the next launch.
-template <int P, int VC>
-__global__ void __launch_bounds__(kDecWarps * 32) attn_decode_kernel(const WindowAttn a) {
-    pdl_prologue();
-    pdl_release();
-    extern __shared__ __align__(16) float dec_smem[];
-    __shared__ float wm[kDecWarps][P], wl[kDecWarps][P];
+struct StepSmem {   // offsets in floats
+    int k, v, q, raw, dots, probs, total;
+    int k_ld;
+};
+__host__ __device__ inline StepSmem step_smem(int P, int dim, int dim_ld, int vdim_ld) {
+    StepSmem m;
+    m.k_ld = dim_ld + 4;   // rows four banks apart: eight lanes reading 16 bytes of eight rows meet no bank twice
+    int at = 0;
+    auto take = [&](int n) {
+        const int o = at;
+        at += (n + 3) / 4 * 4;
+        return o;
+    };
+    m.k = take(kStepKeys * m.k_ld);
+    m.v = take(kStepKeys * vdim_ld);
+    m.q = take(P * dim_ld);
+    m.raw = take(P * dim + dim + vdim_ld);        // convolved values before the rotation: query heads, key, value
+    m.dots = take(8 * P * kStepKeys);          // partial scores of the eight warps
+    m.probs = take(kStepKeys * P);
+    m.total = at;
+    return m;
+}
+
+__device__ __forceinline__ void cp_async16_attn(void *dst, const void *src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+template <int P>
+__global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const WindowAttn a, int attn_ctas, int per) {
+    extern __shared__ __align__(16) float st_smem[];
+    __shared__ float run_m[P], run_l[P], corr_s[P];
     __shared__ int s_last;
-    const int kvh = blockIdx.x, range = blockIdx.y, tile = blockIdx.z;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int group = a.heads / a.kv_heads, g0 = tile * P, ng = min(P, group - g0);
-    const int n4 = a.dim_ld >> 2, vld = a.vdim_ld;
-    float *qs = dec_smem;                    // [P, dim_ld]
-    float *wacc = dec_smem + P * a.dim_ld;   // [warps, P, vdim_ld]
+    if ((int)blockIdx.x >= attn_ctas) {
+        pdl_prologue();
+        pdl_release();
+        ffn_part(a.ffn, 1, attn_ctas);
+        return;
+    }
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int group = a.heads / a.kv_heads, tiles = (group + P - 1) / P;
+    const int range = blockIdx.x % a.ranges, kt = blockIdx.x / a.ranges, tile = kt % tiles, kvh = kt / tiles;
+    const int g0 = tile * P, ng = min(P, group - g0), h0 = kvh * group + g0;
+    const StepSmem m = step_smem(P, a.dim, a.dim_ld, a.vdim_ld);
+    const int n4 = a.dim_ld >> 2, v4 = a.vdim_ld >> 2;
     const int pos = a.span.state[1];
-    const int first = max(0, pos - a.window + 1);
-    const int nb = (pos - first + 32) >> 5;                     // batches of 32 keys
-    const int bper = (nb + gridDim.y - 1) / gridDim.y;
-    const int used = (nb + bper - 1) / bper;                    // ranges that hold keys
-    const int b_lo = range * bper, b_hi = min(nb, b_lo + bper);
-    const int slot0 = (kvh * gridDim.z + tile) * gridDim.y;     // this tile's records
-    const int rec = vld + 4;                                    // m, l, pad, pad, acc
-    if (b_lo < b_hi) {
-        for (int i = threadIdx.x; i < P * n4; i += kDecWarps * 32) {
-            const int p = i / n4, d4 = i - p * n4;
-            reinterpret_cast<float4 *>(qs)[i] =
-                reinterpret_cast<const float4 *>(a.qrot + (size_t)(kvh * group + g0 + min(p, ng - 1)) * a.dim_ld)[d4];
+    const int first = max(0, pos - a.window + 1), keys = pos - first + 1;
+    const int used = (keys + per - 1) / per;                        // ranges that hold keys
+    const int lo = first + range * per, hi = min(pos + 1, lo + per);  // this CTA's keys [lo, hi)
+    const bool active = lo < hi, owns_pos = active && hi == pos + 1;
+    const float *kb = a.kcache + (size_t)kvh * a.cap * a.dim_ld, *vb = a.vcache + (size_t)kvh * a.cap * a.vdim_ld;
+    // keys and values b0 .. b0 + 63 of the range, the current position's excepted
+    auto fetch = [&](int b0) {
+        const int n = min(kStepKeys, min(hi, pos) - b0), s0 = b0 % a.cap;
+        for (int i = tid; i < n * n4; i += kStepThreads) {
+            const int r = i / n4, c = i - r * n4;
+            int slot = s0 + r;
+            if (slot >= a.cap) slot -= a.cap;
+            cp_async16_attn(st_smem + m.k + r * m.k_ld + 4 * c, kb + (size_t)slot * a.dim_ld + 4 * c);
         }
-        __syncthreads();
-        const float *kb = a.kcache + (size_t)kvh * a.cap * a.dim_ld, *vb = a.vcache + (size_t)kvh * a.cap * vld;
-        WarpSoftmax<P, VC> ws;
-        ws.init();
-        for (int b = b_lo + warp; b < b_hi; b += kDecWarps)
-            ws.batch(a, qs, kb, vb, first + (b << 5), pos, [](int, int) { return true; });
-#pragma unroll
-        for (int p = 0; p < P; p++) {
-            if (lane == 0) {
-                wm[warp][p] = ws.m[p];
-                wl[warp][p] = ws.l[p];
-            }
-#pragma unroll
-            for (int c = 0; c < VC; c++)
-                if (4 * lane + 128 * c < vld) *reinterpret_cast<float4 *>(&wacc[(warp * P + p) * vld + 4 * lane + 128 * c]) = ws.acc[p][c];
+        for (int i = tid; i < n * v4; i += kStepThreads) {
+            const int r = i / v4, c = i - r * v4;
+            int slot = s0 + r;
+            if (slot >= a.cap) slot -= a.cap;
+            cp_async16_attn(st_smem + m.v + r * a.vdim_ld + 4 * c, vb + (size_t)slot * a.vdim_ld + 4 * c);
         }
-        __syncthreads();
-        for (int i = threadIdx.x; i < ng * vld; i += kDecWarps * 32) {
-            const int p = i / vld, d = i - p * vld;
-            float M = wm[0][p];   // warp 0 always holds a batch: finite
-#pragma unroll
-            for (int w = 1; w < kDecWarps; w++) M = fmaxf(M, wm[w][p]);
-            float L = 0.0f, s = 0.0f;
-#pragma unroll
-            for (int w = 0; w < kDecWarps; w++) {
-                const float e = wm[w][p] == -INFINITY ? 0.0f : expf(wm[w][p] - M);
-                L = fmaf(wl[w][p], e, L);
-                s = fmaf(wacc[(w * P + p) * vld + d], e, s);
-            }
-            if (used == 1) {
-                attn_store(a, 0, kvh * group + g0 + p, d, s / L);
-            } else {
-                float *o = a.part + ((size_t)(slot0 + range) * P + p) * rec;
-                if (d == 0) {
-                    o[0] = M;
-                    o[1] = L;
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    // the channels this CTA convolves: its query heads, then (with the current position) the key and the value
+    const int qn = ng * a.dim, total = qn + (owns_pos ? a.dim + a.vdim : 0);
+    const int channels = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
+    auto locate = [&](int i, int &c, int &col) {
+        if (i < qn) {
+            c = h0 * a.dim + i;
+            col = a.c_q + c;
+        } else if (i < qn + a.dim) {
+            c = (a.heads + kvh) * a.dim + i - qn;
+            col = a.c_k + kvh * a.dim + i - qn;
+        } else {
+            c = (a.heads + a.kv_heads) * a.dim + kvh * a.vdim + i - qn - a.dim;
+            col = a.c_v + kvh * a.vdim + i - qn - a.dim;
+        }
+    };
+    float *raw = st_smem + m.raw;
+    if (active) {
+        fetch(lo);
+        if (a.taps > 1) {
+            for (int i = tid; i < total; i += kStepThreads) {
+                int c, col;
+                locate(i, c, col);
+                float y = 0.0f;
+                for (int t = 0; t < a.taps - 1; t++) {
+                    const int back = a.taps - 1 - t;
+                    const float u = pos >= back ? a.conv_ring[(size_t)((pos - back) % a.taps) * channels + c] : 0.0f;
+                    y = fmaf(a.conv[(size_t)c * a.taps + t], u, y);
                 }
-                o[4 + d] = s;
+                raw[(i < qn ? 0 : P * a.dim - qn) + i] = y;   // key and value behind all P query heads' places
             }
         }
     }
-    if (used == 1) return;   // the same for every CTA of the launch: nobody counts
+    if (tid < P) {
+        run_m[tid] = -INFINITY;
+        run_l[tid] = 0.0f;
+    }
+    pdl_prologue();
+    pdl_release();
+    float acc[P];
+#pragma unroll
+    for (int p = 0; p < P; p++) acc[p] = 0.0f;
+    if (active) {
+        for (int i = tid; i < total; i += kStepThreads) {
+            int c, col;
+            locate(i, c, col);
+            const float u = a.ffn.proj[col];
+            float &y = raw[(i < qn ? 0 : P * a.dim - qn) + i];
+            if (a.taps > 1) {
+                y = fmaf(a.conv[(size_t)c * a.taps + a.taps - 1], u, y);
+                // this position's slot is read by nobody in this launch (readers look 1 .. taps - 1 back)
+                if (i < qn ? range == 0 : tile == 0) a.conv_ring[(size_t)(pos % a.taps) * channels + c] = u;
+            } else {
+                y = a.taps == 1 ? a.conv[c] * u : u;
+            }
+        }
+        __syncthreads();
+        const int half = a.rot_dims >> 1;
+        const float *cs = a.cosv + (size_t)pos * half, *sn = a.sinv + (size_t)pos * half;
+        for (int i = tid; i < P * a.dim_ld; i += kStepThreads) {
+            const int p = i / a.dim_ld, d = i - p * a.dim_ld;
+            st_smem[m.q + i] = p < ng && d < a.dim ? rotated(raw + p * a.dim, d, a.rot_dims, cs, sn) : 0.0f;
+        }
+        if (owns_pos) {
+            // the new key and value: into the cache, and into the shared tile that holds them (the last one)
+            const int slot = pos % a.cap, r = (pos - lo) % kStepKeys;
+            const bool now = pos - lo < kStepKeys;
+            const float *rk = raw + P * a.dim, *rv = rk + a.dim;
+            for (int d = tid; d < a.dim_ld; d += kStepThreads) {
+                const float k = d < a.dim ? rotated(rk, d, a.rot_dims, cs, sn) : 0.0f;
+                if (now) st_smem[m.k + r * m.k_ld + d] = k;
+                if (tile == 0) a.kcache[((size_t)kvh * a.cap + slot) * a.dim_ld + d] = k;
+            }
+            for (int d = tid; d < a.vdim_ld; d += kStepThreads) {
+                float v = d < a.vdim ? rv[d] : 0.0f;
+                if (d < a.vdim && a.mix_mode == 1 && tile == 0) a.vfirst[kvh * a.vdim + d] = v;
+                else if (d < a.vdim && a.mix_mode == 2) v = (1.0f - a.lambda) * v + a.lambda * a.vfirst[kvh * a.vdim + d];
+                if (now) st_smem[m.v + r * a.vdim_ld + d] = v;
+                if (tile == 0) a.vcache[((size_t)kvh * a.cap + slot) * a.vdim_ld + d] = v;
+                if (!now) raw[P * a.dim + a.dim + d] = v;   // (vdim_ld - vdim zeros fit: the area is rounded up)
+            }
+        }
+        for (int b0 = lo; b0 < hi; b0 += kStepKeys) {
+            if (b0 > lo) fetch(b0);
+            const int n = min(kStepKeys, hi - b0);
+            if (b0 > lo && owns_pos && b0 + n == hi) {   // a later tile holds the current position
+                const int r = n - 1;
+                const float *rk = raw + P * a.dim, *rv = rk + a.dim;
+                for (int d = tid; d < a.dim_ld; d += kStepThreads) st_smem[m.k + r * m.k_ld + d] = d < a.dim ? rotated(rk, d, a.rot_dims, cs, sn) : 0.0f;
+                for (int d = tid; d < a.vdim_ld; d += kStepThreads) st_smem[m.v + r * a.vdim_ld + d] = d < a.vdim ? rv[d] : 0.0f;
+            }
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            __syncthreads();
+            // scores: warp w takes every eighth group of four dimensions, a lane two keys
+            {
+                float dot[2][P];
+#pragma unroll
+                for (int p = 0; p < P; p++) dot[0][p] = dot[1][p] = 0.0f;
+                const float *k0 = st_smem + m.k + lane * m.k_ld, *k1 = k0 + 32 * m.k_ld;
+                for (int c = warp; c < n4; c += 8) {
+                    const float4 x = *reinterpret_cast<const float4 *>(k0 + 4 * c), y = *reinterpret_cast<const float4 *>(k1 + 4 * c);
+#pragma unroll
+                    for (int p = 0; p < P; p++) {
+                        const float4 q = *reinterpret_cast<const float4 *>(st_smem + m.q + p * a.dim_ld + 4 * c);
+                        dot[0][p] = fmaf(q.x, x.x, fmaf(q.y, x.y, fmaf(q.z, x.z, fmaf(q.w, x.w, dot[0][p]))));
+                        dot[1][p] = fmaf(q.x, y.x, fmaf(q.y, y.y, fmaf(q.z, y.z, fmaf(q.w, y.w, dot[1][p]))));
+                    }
+                }
+#pragma unroll
+                for (int p = 0; p < P; p++) {
+                    st_smem[m.dots + (warp * P + p) * kStepKeys + lane] = dot[0][p];
+                    st_smem[m.dots + (warp * P + p) * kStepKeys + 32 + lane] = dot[1][p];
+                }
+            }
+            __syncthreads();
+            if (warp < P) {   // softmax of head `warp` over the tile
+                float sc[2];
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    float d = 0.0f;
+#pragma unroll
+                    for (int w = 0; w < 8; w++) d += st_smem[m.dots + (w * P + warp) * kStepKeys + 32 * e + lane];
+                    sc[e] = 32 * e + lane < n ? d * a.scale : -INFINITY;
+                }
+                const float mo = run_m[warp], mn = fmaxf(mo, warp_max(fmaxf(sc[0], sc[1])));   // finite: the tile holds a key
+                const float p0 = expf(sc[0] - mn), p1 = expf(sc[1] - mn), corr = expf(mo - mn);
+                const float sum = warp_sum(p0 + p1);
+                st_smem[m.probs + lane * P + warp] = p0;
+                st_smem[m.probs + (32 + lane) * P + warp] = p1;
+                if (lane == 0) {
+                    run_m[warp] = mn;
+                    run_l[warp] = run_l[warp] * corr + sum;
+                    corr_s[warp] = corr;
+                }
+            }
+            __syncthreads();
+            // values: a thread per dimension; with at most 128 of them the two halves of the CTA take every other key
+            const bool split = a.vdim_ld <= 128;
+            const int d0 = split ? tid & 127 : tid, j0 = split ? tid >> 7 : 0, dj = split ? 2 : 1;
+#pragma unroll
+            for (int p = 0; p < P; p++) acc[p] *= corr_s[p];
+            if (d0 < a.vdim_ld) {
+#pragma unroll 4
+                for (int jj = j0; jj < n; jj += dj) {
+                    const float v = st_smem[m.v + jj * a.vdim_ld + d0];
+#pragma unroll
+                    for (int p = 0; p < P; p++) acc[p] = fmaf(st_smem[m.probs + jj * P + p], v, acc[p]);
+                }
+            }
+            __syncthreads();   // the tile may be overwritten
+        }
+        if (a.vdim_ld <= 128) {   // the halves meet (in the score area)
+            if (tid >= 128 && (tid & 127) < a.vdim_ld)
+#pragma unroll
+                for (int p = 0; p < P; p++) st_smem[m.dots + p * 128 + (tid & 127)] = acc[p];
+            __syncthreads();
+            if (tid < a.vdim_ld)
+#pragma unroll
+                for (int p = 0; p < P; p++) acc[p] += st_smem[m.dots + p * 128 + tid];
+        }
+        if (tid < a.vdim_ld) {
+#pragma unroll
+            for (int p = 0; p < P; p++) {
+                if (p >= ng) continue;
+                if (used == 1) {
+                    attn_store(a, 0, h0 + p, tid, acc[p] / run_l[p]);
+                } else {
+                    float *o = a.part + ((size_t)(kt * a.ranges + range) * P + p) * (a.vdim_ld + 4);   // record: m, l, pad, pad, acc
+                    if (tid == 0) {
+                        o[0] = run_m[p];
+                        o[1] = run_l[p];
+                    }
+                    o[4 + tid] = acc[p];
+                }
+            }
+        }
+    }
+    if (used == 1 || !active) return;   // ranges without keys are not counted
     __threadfence();
     __syncthreads();
-    unsigned int *cnt = a.arrived + kvh * gridDim.z + tile;
-    if (threadIdx.x == 0) s_last = atomicAdd(cnt, 1u) == gridDim.y - 1;
+    unsigned int *cnt = a.arrived + kt;
+    if (tid == 0) s_last = atomicAdd(cnt, 1u) == (unsigned)(used - 1);
     __syncthreads();
     if (!s_last) return;
     __threadfence();
-    for (int i = threadIdx.x; i < ng * vld; i += kDecWarps * 32) {
-        const int p = i / vld, d = i - p * vld;
-        const float *r0 = a.part + ((size_t)slot0 * P + p) * rec;
-        const size_t step = (size_t)P * rec;
-        float M = -INFINITY;
-        for (int s = 0; s < used; s++) M = fmaxf(M, __ldcg(r0 + s * step));
-        float L = 0.0f, v = 0.0f;
-#pragma unroll 4
-        for (int s = 0; s < used; s++) {
-            const float e = expf(__ldcg(r0 + s * step) - M);
-            L = fmaf(__ldcg(r0 + s * step + 1), e, L);
-            v = fmaf(__ldcg(r0 + s * step + 4 + d), e, v);
+    for (int i = tid; i < ng * a.vdim_ld; i += kStepThreads) {
+        const int p = i / a.vdim_ld, d = i - p * a.vdim_ld;
+        const size_t step = (size_t)P * (a.vdim_ld + 4);
+        const float *r0 = a.part + ((size_t)(kt * a.ranges) * P + p) * (a.vdim_ld + 4);
+        float M = -INFINITY, L = 0.0f, v = 0.0f;
+        for (int s0 = 0; s0 < used; s0 += 8) {
+            float2 ml[8];
+            float x[8];
+#pragma unroll
+            for (int s = 0; s < 8; s++) {   // all loads of a pass before the first is used
+                ml[s] = s0 + s < used ? __ldcg(reinterpret_cast<const float2 *>(r0 + (s0 + s) * step)) : make_float2(-INFINITY, 0.0f);
+                x[s] = s0 + s < used ? __ldcg(r0 + (s0 + s) * step + 4 + d) : 0.0f;
+            }
+            float mx = M;
+#pragma unroll
+            for (int s = 0; s < 8; s++) mx = fmaxf(mx, ml[s].x);
+            const float c = expf(M - mx);
+            L *= c;
+            v *= c;
+#pragma unroll
+            for (int s = 0; s < 8; s++) {
+                const float e = expf(ml[s].x - mx);
+                L = fmaf(ml[s].y, e, L);
+                v = fmaf(x[s], e, v);
+            }
+            M = mx;
         }
-        attn_store(a, 0, kvh * group + g0 + p, d, v / L);
+        attn_store(a, 0, h0 + p, d, v / L);
     }
-    if (threadIdx.x == 0) *cnt = 0;   // the next launch starts after this grid has ended
+    if (tid == 0) *cnt = 0;   // the next launch starts after this grid has ended
 }
 
 // ---- host side ----
 
 static int dec_tile(int group) { return group > 4 ? 8 : (group > 2 ? 4 : (group > 1 ? 2 : 1)); }
+static int dec_tiles(int heads, int kv_heads) { return kv_heads * ((heads / kv_heads + dec_tile(heads / kv_heads) - 1) / dec_tile(heads / kv_heads)); }
 
-int attn_decode_ranges(int window, int max_seq) {
+// Ranges of whole 64-key tiles, as many as leave at most one CTA per SM.
+static int step_per(int ranges, int keys) { return ((keys + ranges - 1) / ranges + kStepKeys - 1) / kStepKeys * kStepKeys; }
+
+int attn_step_ranges(int sm_count, int heads, int kv_heads, int window, int max_seq) {
     const int keys = window < max_seq ? window : max_seq;
-    const int per = 32 * kDecWarps;   // one batch per warp
-    const int r = (keys + per - 1) / per;
-    return r < 1 ? 1 : (r > kDecMaxRanges ? kDecMaxRanges : r);
+    int r = sm_count / dec_tiles(heads, kv_heads);
+    r = r < 1 ? 1 : (r > kStepMaxRanges ? kStepMaxRanges : r);
+    return (keys + step_per(r, keys) - 1) / step_per(r, keys);
 }
 
-int attn_decode_counters(int heads, int kv_heads) {
-    const int group = heads / kv_heads, P = dec_tile(group);
-    return kv_heads * ((group + P - 1) / P);
-}
+int attn_step_counters(int heads, int kv_heads) { return dec_tiles(heads, kv_heads); }
 
-size_t attn_decode_part_floats(int heads, int kv_heads, int vdim_ld, int ranges) {
-    return (size_t)attn_decode_counters(heads, kv_heads) * ranges * dec_tile(heads / kv_heads) * (vdim_ld + 4);
+size_t attn_step_part_floats(int heads, int kv_heads, int vdim_ld, int ranges) {
+    return (size_t)dec_tiles(heads, kv_heads) * ranges * dec_tile(heads / kv_heads) * (vdim_ld + 4);
 }
 
 template <typename K>
@@ -423,24 +616,24 @@ nnq_status launch_attn_rows(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) 
     return a.vdim_ld <= 128 ? go_rows<8, 1>(ctx, a, st) : go_rows<8, 2>(ctx, a, st);
 }
 
-template <int P, int VC>
-static nnq_status go_decode(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
-    const int group = a.heads / a.kv_heads;
-    const size_t smem = (size_t)P * (a.dim_ld + kDecWarps * a.vdim_ld) * sizeof(float);
-    nnq_status s = allow_smem(ctx, attn_decode_kernel<P, VC>, smem);
+template <int P>
+static nnq_status go_step(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
+    const int ctas = dec_tiles(a.heads, a.kv_heads) * a.ranges;
+    const size_t smem = (size_t)step_smem(P, a.dim, a.dim_ld, a.vdim_ld).total * sizeof(float);
+    nnq_status s = allow_smem(ctx, attn_step_kernel<P>, smem);
     if (s != NNQ_OK) return s;
-    launch_pdl_smem(attn_decode_kernel<P, VC>, dim3(a.kv_heads, a.ranges, (group + P - 1) / P), dim3(kDecWarps * 32), smem, st, a);
+    launch_pdl_smem(attn_step_kernel<P>, dim3(ctas + ffn_ctas(a.ffn, 1, kStepThreads, ctx->sm_count)), dim3(kStepThreads), smem, st, a, ctas,
+                    step_per(a.ranges, a.keys_max));
     ctx->launches++;
-    return check_cuda(ctx, cudaGetLastError(), "decode attention launch");
+    return check_cuda(ctx, cudaGetLastError(), "attention step launch");
 }
 
-nnq_status launch_attn_decode(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
-    const bool wide = a.vdim_ld > 128;
+nnq_status launch_attn_step(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st) {
     switch (dec_tile(a.heads / a.kv_heads)) {
-        case 1: return wide ? go_decode<1, 2>(ctx, a, st) : go_decode<1, 1>(ctx, a, st);
-        case 2: return wide ? go_decode<2, 2>(ctx, a, st) : go_decode<2, 1>(ctx, a, st);
-        case 4: return wide ? go_decode<4, 2>(ctx, a, st) : go_decode<4, 1>(ctx, a, st);
-        default: return wide ? go_decode<8, 2>(ctx, a, st) : go_decode<8, 1>(ctx, a, st);
+        case 1: return go_step<1>(ctx, a, st);
+        case 2: return go_step<2>(ctx, a, st);
+        case 4: return go_step<4>(ctx, a, st);
+        default: return go_step<8>(ctx, a, st);
     }
 }
 

@@ -11,7 +11,7 @@
 
 namespace nnq {
 
-constexpr int kAttnMaxValueDim = 256;   // a lane holds up to two groups of four value dimensions
+constexpr int kAttnMaxDim = 256;        // key and value dimensions of an attention head
 constexpr int kRecMaxKeyDim = 256;      // key rows of a state tile held in a thread's registers
 
 inline int round_up(int v, int m) { return (v + m - 1) / m * m; }
@@ -53,7 +53,9 @@ struct WindowAttn {
     float *qrot;                    // [rows, heads, dim_ld]
     float *kcache, *vcache;         // [kv_heads, cap, dim_ld / vdim_ld], position p at slot p % cap
     int cap;
-    // decode: key ranges per (kv head, head tile), records of the ranges and their arrival counters
+    // decode step: keys a window can hold, key ranges per (kv head, head tile), records of the ranges and their
+    // arrival counters
+    int keys_max;
     int ranges;
     float *part;
     unsigned int *arrived;
@@ -64,10 +66,10 @@ nnq_status launch_attn_conv_tail(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t
 nnq_status launch_attn_rows(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);       // block of rows
 bool attn_tc_supported(const WindowAttn &a);                                           // attn_tc.cu: block of rows on the tensor cores
 nnq_status launch_attn_tc(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);
-nnq_status launch_attn_decode(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);     // one row
-int attn_decode_ranges(int window, int max_seq);                                       // key ranges of the decode kernel
-size_t attn_decode_part_floats(int heads, int kv_heads, int vdim_ld, int ranges);
-int attn_decode_counters(int heads, int kv_heads);
+nnq_status launch_attn_step(nnq_ctx *ctx, const WindowAttn &a, cudaStream_t st);       // one row, prologue and feed-forward part included
+int attn_step_ranges(int sm_count, int heads, int kv_heads, int window, int max_seq);  // key ranges of the step kernel
+size_t attn_step_part_floats(int heads, int kv_heads, int vdim_ld, int ranges);
+int attn_step_counters(int heads, int kv_heads);
 
 // S_t = diag(decay_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t per head; then per-head RMS norm of o, times
 // silu(g). The decay is a constant per head, or sigmoid(W_2 a1 + b)^(1 / tau) per key channel and token.

@@ -24,6 +24,7 @@
 #include "blocks.h"
 #include "comm.cuh"
 #include "decoder_common.cuh"
+#include "gemm_tc.h"
 
 namespace nnq {
 nnq_status comm_view(nnq_comm *c, CommView *out);   // comm.cu
@@ -75,6 +76,7 @@ struct nnq_decoder {
         float *kcache, *vcache, *conv_ring, *rec_state;
         int mix_mode;
     } *blocks;
+    float *b_h2;                // the step's residual row alternates between d_h and this buffer
     float *b_proj, *b_q, *b_k, *b_a, *b_o, *b_vfirst;   // rows of proj; prepared q / k / decay, mixer output, first values
     void *b_act;
 };
@@ -397,15 +399,18 @@ __device__ __forceinline__ void dec_commit_token(int bi, int *state, int *tokens
 __global__ void dec_argmax_stage2_kernel(const float *__restrict__ bv_in, const int *__restrict__ bi_in, int blocks,
                                          int *__restrict__ state, int *__restrict__ tokens, int max_seq, int *status) {
     pdl_prologue();
-    if (threadIdx.x != 0 || blockIdx.x != 0) return;
-    if (state[3]) {
-        atomicExch(status, 2);
-        return;
-    }
-    float bv = -INFINITY;
+    float bv = -INFINITY;   // one warp
     int bi = -1;
-    for (int b = 0; b < blocks; b++) arg_better(bv, bi, bv_in[b], bi_in[b]);
-    dec_commit_token(bi, state, tokens, max_seq);
+    for (int b = threadIdx.x; b < blocks; b += 32) arg_better(bv, bi, bv_in[b], bi_in[b]);
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+        const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, off);
+        const int oi = __shfl_xor_sync(0xFFFFFFFFu, bi, off);
+        arg_better(bv, bi, ov, oi);
+    }
+    if (threadIdx.x != 0) return;
+    if (state[3]) atomicExch(status, 2);
+    else dec_commit_token(bi, state, tokens, max_seq);
 }
 
 // Vocabulary-parallel head: every rank holds the maximum of its slice of the logits; the ranks
@@ -806,8 +811,8 @@ static nnq_status check_block(nnq_ctx *ctx, int l, const nnq_block_config &b) {
     if (b.mixer == NNQ_MIXER_ATTENTION) {
         if (b.kv_heads < 1 || b.heads % b.kv_heads) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: %d query heads over %d key/value heads", l, b.heads, b.kv_heads);
         if (b.window < 0 || b.conv_taps < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad window or convolution", l);
-        if (b.dim > 1024 || b.vdim > kAttnMaxValueDim)
-            return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: attention heads of %d / %d are above 1024 / %d", l, b.dim, b.vdim, kAttnMaxValueDim);
+        if (b.dim > kAttnMaxDim || b.vdim > kAttnMaxDim)
+            return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: attention heads of %d / %d are above %d", l, b.dim, b.vdim, kAttnMaxDim);
     } else {
         if (b.decay_rank < 0 || (b.decay_rank > 0 && !(b.decay_tau > 0.0f))) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad decay", l);
         if (b.dim > kRecMaxKeyDim || b.vdim > 2048)
@@ -895,7 +900,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
             B.vdim_ld = round_up(b.vdim, 4);
             // a block of rows writes its keys before it reads: window - 1 older positions stay beside them
             B.cap = b.window > 0 && (long long)b.window - 1 + rows < c.max_seq ? b.window - 1 + rows : c.max_seq;
-            B.ranges = attn_decode_ranges(b.window > 0 ? b.window : c.max_seq, c.max_seq);
+            B.ranges = attn_step_ranges(ctx->sm_count, b.heads, b.kv_heads, b.window > 0 ? b.window : c.max_seq, c.max_seq);
             B.mix_mode = !b.value_mix ? 0 : (l == first_mix ? 1 : 2);
             const int channels = b.heads * b.dim + b.kv_heads * (b.dim + b.vdim);
             alloc(&B.kcache, (size_t)b.kv_heads * B.cap * B.dim_ld * 4, "key cache");
@@ -906,8 +911,8 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
             }
             most(q, (size_t)b.heads * B.dim_ld);
             if (b.value_mix) most(vf, (size_t)b.kv_heads * b.vdim);
-            most(part, attn_decode_part_floats(b.heads, b.kv_heads, B.vdim_ld, B.ranges));
-            most(counters, attn_decode_counters(b.heads, b.kv_heads));
+            most(part, attn_step_part_floats(b.heads, b.kv_heads, B.vdim_ld, B.ranges));
+            most(counters, attn_step_counters(b.heads, b.kv_heads));
         } else {
             B.dim_ld = round_up(b.dim, 64);
             alloc(&B.rec_state, (size_t)b.heads * b.dim * b.vdim * 4, "recurrent state");
@@ -953,6 +958,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
         }
     }
     alloc(&d->d_h, (size_t)c.hidden * 4, "decoder buffer");
+    alloc(&d->b_h2, (size_t)c.hidden * 4, "decoder buffer");
     alloc(&d->d_delta, (size_t)c.hidden * 4, "decoder buffer");
     alloc(&d->d_xn, (size_t)d->xn_ld * es, "decoder buffer");
     alloc(&d->d_logits, (size_t)c.vocab * 4, "decoder buffer");
@@ -1094,13 +1100,10 @@ static nnq_status product(nnq_decoder *d, const nnq_weight *w, const void *x, in
 
 // Vocabulary projection of the normed state in d_xn, greedy argmax (exchanged between the ranks
 // when the projection is split by rows), commit of the token and advance of the position.
-static nnq_status launch_head(nnq_decoder *d, bool vocab_parallel, const CommView &cv, cudaStream_t st) {
+static nnq_status launch_argmax(nnq_decoder *d, bool vocab_parallel, const CommView &cv, cudaStream_t st) {
     nnq_ctx *ctx = d->ctx;
     const nnq_decoder_config &c = d->cfg;
-    nnq_status s;
-    // the logits of this rank's rows land at their global offsets in the [vocab] buffer
-    float *logits = d->d_logits + d->head_row0;
-    if ((s = product(d, d->lm_head, d->d_xn, 1, nullptr, logits, st)) != NNQ_OK) return s;
+    const float *logits = d->d_logits + d->head_row0;
     float *bv = reinterpret_cast<float *>(d->d_state + 4);
     int *bi = d->d_state + 4 + kArgmaxBlocks;
     launch_pdl(dec_argmax_stage1_kernel, dim3(kArgmaxBlocks), dim3(256), st, logits, d->head_rows, bv, bi);
@@ -1111,6 +1114,12 @@ static nnq_status launch_head(nnq_decoder *d, bool vocab_parallel, const CommVie
         launch_pdl(dec_argmax_stage2_kernel, dim3(1), dim3(32), st, bv, bi, kArgmaxBlocks, d->d_state, d->d_tokens, c.max_seq, ctx->d_status);
     ctx->launches += 2;
     return check_cuda(ctx, cudaGetLastError(), "decoder head launch");
+}
+
+static nnq_status launch_head(nnq_decoder *d, bool vocab_parallel, const CommView &cv, cudaStream_t st) {
+    // the logits of this rank's rows land at their global offsets in the [vocab] buffer
+    nnq_status s = product(d, d->lm_head, d->d_xn, 1, nullptr, d->d_logits + d->head_row0, st);
+    return s != NNQ_OK ? s : launch_argmax(d, vocab_parallel, cv, st);
 }
 
 static nnq_status head_mode(nnq_decoder *d, bool *vocab_parallel, CommView *cv) {
@@ -1149,14 +1158,13 @@ static nnq_status ready_to_run(const nnq_decoder *d) {
     return NNQ_OK;
 }
 
-// Everything between the norm and the residual of block l for n rows: xn -> delta. `state` given: a decode
-// step (n = 1, position in state[1]), else rows from position pos0.
-static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *state, const void *xn, float *delta, cudaStream_t st) {
+// The mixer, the feed-forward activation and the output product of block l for n rows: b_proj -> delta. `state`
+// given: a decode step (n = 1, position in state[1]), else rows from position pos0.
+static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *state, float *delta, cudaStream_t st) {
     nnq_ctx *ctx = d->ctx;
     const nnq_decoder::Block &B = d->blocks[l];
     const nnq_block_config &k = B.cfg;
     nnq_status s;
-    if ((s = product(d, B.in, xn, n, B.bias_in, d->b_proj, st)) != NNQ_OK) return s;
     const RowSpan span = {n, pos0, state};
     const FfnPart ffn = {d->b_proj, B.lay.in_cols, B.lay.gate, B.lay.up, k.ffn, d->b_act, d->act_dt, B.lay.out_k, k.heads * k.vdim, B.lay.ffn_col};
     if (k.mixer == NNQ_MIXER_ATTENTION) {
@@ -1171,11 +1179,12 @@ static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *s
         a.mix_mode = B.mix_mode; a.lambda = B.lambda; a.vfirst = d->b_vfirst;
         a.scale = k.scale; a.window = k.window > 0 ? k.window : (1 << 30);
         a.qrot = d->b_q; a.kcache = B.kcache; a.vcache = B.vcache; a.cap = B.cap;
+        a.keys_max = k.window > 0 && k.window < d->cfg.max_seq ? k.window : d->cfg.max_seq;
         a.ranges = B.ranges; a.part = d->d_part; a.arrived = d->d_arrived;
-        if ((s = launch_attn_prep(ctx, a, st)) != NNQ_OK) return s;
         if (state) {
-            if ((s = launch_attn_decode(ctx, a, st)) != NNQ_OK) return s;
+            if ((s = launch_attn_step(ctx, a, st)) != NNQ_OK) return s;
         } else {
+            if ((s = launch_attn_prep(ctx, a, st)) != NNQ_OK) return s;
             if ((s = launch_attn_conv_tail(ctx, a, st)) != NNQ_OK) return s;
             if ((s = launch_attn_rows(ctx, a, st)) != NNQ_OK) return s;
         }
@@ -1195,14 +1204,31 @@ static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *s
     return product(d, B.out, d->b_act, n, B.bias_out, delta, st);
 }
 
-static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
+// y = RMSNorm(residual) * norm times w^T for the step's row. The residual row is h + delta (the first block: the
+// embedding row); where the norm is part of the product kernel the sum goes to the other of two buffers.
+static nnq_status step_norm_product(nnq_decoder *d, const float *norm, bool embed, const nnq_weight *w, const float *bias, float *y, cudaStream_t st) {
     const nnq_decoder_config &c = d->cfg;
-    for (int l = 0; l < c.n_layers; l++) {
-        launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->d_state,
-                   d->blocks[l].norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
-        d->ctx->launches++;
-        nnq_status s = run_block(d, l, 1, 0, d->d_state, d->d_xn, d->d_delta, st);
-        if (s != NNQ_OK) return s;
+    const __nv_bfloat16 *table = embed ? (const __nv_bfloat16 *)d->d_embed : nullptr;
+    if (d->act_dt == NNQ_BF16 && d->ctx->path == NNQ_PATH_AUTO && dense_gemv_norm_supported(w, c.hidden)) {
+        const TcArgs a = {w->d_raw, w->d_scales, nullptr, bias, y, 1, w->n, w->k, w->fmt, NNQ_BF16, NNQ_F32};
+        const GemvNorm g = {d->d_h, d->d_delta, d->b_h2, table, d->embed_ld, d->d_state, norm, c.rms_eps, c.hidden, 0};
+        nnq_status s = launch_dense_gemv_norm(d->ctx, a, g, st);
+        float *t = d->d_h;
+        d->d_h = d->b_h2;
+        d->b_h2 = t;
+        return s;
+    }
+    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, table, d->d_state, norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, 1);
+    d->ctx->launches++;
+    return product(d, w, d->d_xn, 1, bias, y, st);
+}
+
+static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
+    nnq_status s = NNQ_OK;
+    for (int l = 0; l < d->cfg.n_layers; l++) {
+        const nnq_decoder::Block &B = d->blocks[l];
+        if ((s = step_norm_product(d, B.norm, l == 0, B.in, B.bias_in, d->b_proj, st)) != NNQ_OK) return s;
+        if ((s = run_block(d, l, 1, 0, d->d_state, d->d_delta, st)) != NNQ_OK) return s;
     }
     return NNQ_OK;
 }
@@ -1213,7 +1239,8 @@ static nnq_status rows_blocks(nnq_decoder *d, int n, int pos0, cudaStream_t st) 
         dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->pf_tokens,
                                                 d->blocks[l].norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
         d->ctx->launches++;
-        nnq_status s = run_block(d, l, n, pos0, nullptr, d->pf_xn, d->pf_delta, st);
+        nnq_status s = product(d, d->blocks[l].in, d->pf_xn, n, d->blocks[l].bias_in, d->b_proj, st);
+        if (s == NNQ_OK) s = run_block(d, l, n, pos0, nullptr, d->pf_delta, st);
         if (s != NNQ_OK) return s;
     }
     return NNQ_OK;
@@ -1330,7 +1357,12 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
     s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
     if (s != NNQ_OK) return s;
     cudaStream_t st = (cudaStream_t)stream;
-    if ((s = d->blocks ? step_blocks(d, st) : step_qwen3(d, st)) != NNQ_OK) return s;
+    if (d->blocks) {
+        if ((s = step_blocks(d, st)) != NNQ_OK) return s;
+        if ((s = step_norm_product(d, d->d_final_norm, false, d->lm_head, nullptr, d->d_logits, st)) != NNQ_OK) return s;
+        return launch_argmax(d, vocab_parallel, cv, st);
+    }
+    if ((s = step_qwen3(d, st)) != NNQ_OK) return s;
     launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
     ctx->launches++;
     return launch_head(d, vocab_parallel, cv, st);
@@ -1517,7 +1549,7 @@ void nnq_decoder_destroy(nnq_decoder *d) {
         }
         delete[] d->blocks;
     }
-    cudaFree(d->b_proj); cudaFree(d->b_q); cudaFree(d->b_k); cudaFree(d->b_a); cudaFree(d->b_o); cudaFree(d->b_vfirst); cudaFree(d->b_act);
+    cudaFree(d->b_h2); cudaFree(d->b_proj); cudaFree(d->b_q); cudaFree(d->b_k); cudaFree(d->b_a); cudaFree(d->b_o); cudaFree(d->b_vfirst); cudaFree(d->b_act);
     cudaFree(d->pf_want); cudaFree(d->d_want_logits);
     cudaFree(d->d_final_norm); cudaFree(d->d_cos); cudaFree(d->d_sin); cudaFree(d->d_kcache); cudaFree(d->d_vcache);
     cudaFree(d->d_h); cudaFree(d->d_delta); cudaFree(d->d_q); cudaFree(d->d_k); cudaFree(d->d_v); cudaFree(d->d_qrot);

@@ -7,15 +7,19 @@
 // partial sums meet in shared memory once, at the end. The ring is filled before the kernel waits for its
 // predecessor (programmatic dependent launch): the small kernels in front of a product release it early, so the
 // weights stream while they run. Products bf16 x bf16 in f32, f32 sums. Every wait is bounded.
+//
+// With NORM the kernel also does what stands in front of a decoder's product: every CTA adds the last block's output
+// to the residual row (or reads the embedding row), takes its root mean square and keeps the normed row as bf16 in
+// shared memory; CTA 0 writes the new residual to another buffer (the others may still be reading the old one).
 #include <cuda_bf16.h>
 
+#include "decoder_common.cuh"
 #include "gemm_tc.h"
-#include "pdl.cuh"
 #include "sync.cuh"
 
 namespace nnq {
 
-constexpr int kGvChunk = 1024, kGvTileBytes = kGvChunk * 2, kGvTiles = 80, kGvRing = kGvTiles * kGvTileBytes;
+constexpr int kGvChunk = 1024, kGvTileBytes = kGvChunk * 2, kGvTiles = 64, kGvRing = kGvTiles * kGvTileBytes;
 // warps of a CTA: three and four rows need the registers of half as many
 __host__ __device__ constexpr int gv_warps(int m) { return m <= 2 ? 16 : 8; }
 
@@ -23,10 +27,12 @@ __device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u <<
 __device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xFFFF0000u); }
 
 // grid: rows dealt to CTAs in contiguous runs. ks: warps per row (power of two), passes: chunks of a warp.
-template <int M>
+constexpr int kGvNormMax = 8192;   // width of the normed row: 16 values per thread
+
+template <int M, bool NORM>
 __global__ void __launch_bounds__(gv_warps(M) * 32, 1)
 dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__restrict__ x, const float *__restrict__ bias, void *__restrict__ y,
-                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status) {
+                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm) {
     constexpr int kGvWarps = gv_warps(M), kGvStages = kGvTiles / kGvWarps;
     extern __shared__ __align__(128) uint8_t gv_smem[];
     __shared__ __align__(8) uint64_t bars[kGvWarps * kGvStages];
@@ -56,6 +62,42 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
     if (lane == 0)
         for (int i = 0; i < kGvStages && i < tiles; i++) issue(i);
     pdl_prologue();
+    pdl_release();   // (the whole grid is resident; the mixer behind it asks for its caches while this kernel streams)
+    const __nv_bfloat16 *xrow = x;
+    if constexpr (NORM) {
+        __shared__ float red[32];
+        __nv_bfloat16 *xn = reinterpret_cast<__nv_bfloat16 *>(gv_smem + kGvRing + nrm.xn_at);
+        const __nv_bfloat16 *er = nrm.embed ? nrm.embed + (size_t)nrm.state[0] * nrm.embed_ld : nullptr;
+        float4 h[4];
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int d = 4 * (threadIdx.x + kGvWarps * 32 * i);
+            h[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (d < nrm.hidden) {
+                if (er) {
+                    const uint2 u = *reinterpret_cast<const uint2 *>(er + d);
+                    h[i] = make_float4(bf_lo(u.x), bf_hi(u.x), bf_lo(u.y), bf_hi(u.y));
+                } else {
+                    const float4 a = *reinterpret_cast<const float4 *>(nrm.h_in + d), b = *reinterpret_cast<const float4 *>(nrm.delta + d);
+                    h[i] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+                }
+                if (blockIdx.x == 0 && nrm.h_out) *reinterpret_cast<float4 *>(nrm.h_out + d) = h[i];
+            }
+            ss = fmaf(h[i].x, h[i].x, fmaf(h[i].y, h[i].y, fmaf(h[i].z, h[i].z, fmaf(h[i].w, h[i].w, ss))));
+        }
+        const float rms = sqrtf(block_sum(ss, red) / (float)nrm.hidden + nrm.eps);
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int d = 4 * (threadIdx.x + kGvWarps * 32 * i);
+            if (d >= K) continue;   // columns from hidden on are zero
+            const float4 g = d < nrm.hidden ? *reinterpret_cast<const float4 *>(nrm.w + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            const __nv_bfloat162 a = __floats2bfloat162_rn(h[i].x / rms * g.x, h[i].y / rms * g.y), b = __floats2bfloat162_rn(h[i].z / rms * g.z, h[i].w / rms * g.w);
+            *reinterpret_cast<uint2 *>(xn + d) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+        }
+        __syncthreads();
+        xrow = xn;
+    }
     bool ok = true;
     int stage = 0, issued = min(tiles, kGvStages);
     uint32_t phase = 0;
@@ -66,7 +108,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
         for (int m = 0; m < M; m++)
 #pragma unroll
             for (int j = 0; j < 4; j++)
-                xv[m][j] = 8 * (lane + 32 * j) < kc ? *reinterpret_cast<const uint4 *>(x + (size_t)m * K + k0 + 8 * (lane + 32 * j)) : make_uint4(0, 0, 0, 0);
+                xv[m][j] = 8 * (lane + 32 * j) < kc ? *reinterpret_cast<const uint4 *>(xrow + (size_t)m * K + k0 + 8 * (lane + 32 * j)) : make_uint4(0, 0, 0, 0);
         for (int r = 0; r < rows; r++, i++) {
             if (!mbar_wait_fast(bar0 + 8 * stage, phase)) {
                 ok = false;
@@ -137,16 +179,20 @@ bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt) {
            w->n < (1ll << 31) && w->k < (1ll << 31) && !((uintptr_t)w->d_raw & 15u);
 }
 
-template <int M>
-static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, cudaStream_t st) {
-    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+template <int M, bool NORM>
+static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, const GemvNorm &nrm, cudaStream_t st) {
+    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M, NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
-    launch_pdl_smem(dense_gemv_kernel<M>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
-                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status);
+    launch_pdl_smem(dense_gemv_kernel<M, NORM>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
+                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm);
     return cudaGetLastError();
 }
 
-nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) {
+bool dense_gemv_norm_supported(const nnq_weight *w, int hidden) {
+    return dense_gemv_supported(w, 1, NNQ_BF16) && hidden % 4 == 0 && hidden <= w->k && w->k <= kGvNormMax;
+}
+
+static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, cudaStream_t stream) {
     // as few warps per row as keep a warp's columns within one chunk
     int ks = 1;
     while (ks < gv_warps((int)a.m) && a.k > (int64_t)ks * kGvChunk) ks *= 2;
@@ -157,17 +203,31 @@ nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream)
     const int64_t max_rows = (32 << 10) / (4 * ks * a.m);
     int64_t grid = a.n < ctx->sm_count ? a.n : ctx->sm_count;
     while ((a.n + grid - 1) / grid > max_rows) grid += ctx->sm_count;
-    const size_t smem = kGvRing + (size_t)((a.n + grid - 1) / grid) * ks * a.m * 4;
+    size_t smem = kGvRing + ((size_t)((a.n + grid - 1) / grid) * ks * a.m * 4 + 15) / 16 * 16;
     cudaError_t e;
-    switch (a.m) {
-        case 1: e = gv_go<1>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
-        case 2: e = gv_go<2>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
-        case 3: e = gv_go<3>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
-        case 4: e = gv_go<4>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, stream); break;
-        default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "1 to 4 rows");
+    const GemvNorm none = {};
+    if (nrm) {
+        nrm->xn_at = (int)(smem - kGvRing);
+        smem += (size_t)a.k * 2;
+        e = gv_go<1, true>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, stream);
+    } else {
+        switch (a.m) {
+            case 1: e = gv_go<1, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
+            case 2: e = gv_go<2, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
+            case 3: e = gv_go<3, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
+            case 4: e = gv_go<4, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
+            default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "1 to 4 rows");
+        }
     }
     ctx->launches++;
     return check_cuda(ctx, e, "bf16 row product launch");
+}
+
+nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) { return gemv(ctx, a, nullptr, stream); }
+
+nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, cudaStream_t stream) {
+    GemvNorm n = norm;
+    return gemv(ctx, a, &n, stream);
 }
 
 }  // namespace nnq

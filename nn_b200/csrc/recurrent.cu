@@ -286,78 +286,110 @@ __global__ void __launch_bounds__(128) rec_finish_kernel(const Recurrence r) {
     }
 }
 
-constexpr int kStepWarps = 16, kStepBatch = 8;
+// ---- one token ----
+//
+// Everything between the two products: a cluster of CTAs per head, each with a slice of the value columns (a
+// multiple of 32). Every CTA prepares q / k / decay of the head, advances its slice of the state (lanes over
+// columns, warps over key rows; the slice's first 32 columns are asked for before the kernel waits for the product
+// in front of it), sums o over the warps; the squares of o are summed over the cluster through its shared memory
+// for the norm, then the slice is gated and stored. Further CTAs do the feed-forward part.
+constexpr int kStepWarps = 8, kStepThreads = kStepWarps * 32, kStepRows = kRecMaxKeyDim / kStepWarps;
 
-// One token, everything between the two products: CTA h < heads prepares q / k / decay of its head, advances
-// the head's state (read and written once), norms and gates the output; the other CTAs do the feed-forward part.
-__global__ void __launch_bounds__(kStepWarps * 32) rec_step_kernel(const Recurrence r) {
-    pdl_prologue();
-    pdl_release();
-    extern __shared__ float step_smem[];   // q, k, decay [dim], v [vdim], partial o [warps, vdim]
+__global__ void __launch_bounds__(kStepThreads) rec_step_kernel(const Recurrence r, int cluster, int slice) {
+    extern __shared__ float step_smem[];   // q, k, decay [dim], v, o [slice], partial o [warps, 32]
     __shared__ float red[32];
-    if ((int)blockIdx.x >= r.heads) {
-        ffn_part(r.ffn, 1, r.heads);
+    __shared__ float squares;              // this CTA's sum of o^2
+    if ((int)blockIdx.x >= r.heads * cluster) {
+        pdl_prologue();
+        pdl_release();
+        ffn_part(r.ffn, 1, r.heads * cluster);
         return;
     }
-    const int head = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int head = blockIdx.x / cluster, c0 = (blockIdx.x - head * cluster) * slice, cn = min(slice, r.vdim - c0);   // (cn <= 0: nothing of its own)
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int pos = r.span.state[1];
-    float *q = step_smem, *k = q + r.dim, *al = k + r.dim, *v = al + r.dim, *po = v + r.vdim;
+    float *q = step_smem, *k = q + r.dim, *al = k + r.dim, *v = al + r.dim, *o = v + slice, *po = o + slice;
+    float *S = r.state + (size_t)head * r.dim * r.vdim + c0;
+    float s[kStepRows];
+    auto fetch = [&](int c) {
+#pragma unroll
+        for (int i = 0; i < kStepRows; i++) {
+            const int row = warp + i * kStepWarps;
+            s[i] = pos > 0 && row < r.dim && c < cn ? S[(size_t)row * r.vdim + c] : 0.0f;
+        }
+    };
+    fetch(lane);
+    pdl_prologue();
+    pdl_release();
     const float *p = r.ffn.proj;
     const int half = r.rot_dims >> 1;
     const float *cs = r.cosv + (size_t)pos * half, *sn = r.sinv + (size_t)pos * half;
-    for (int d = tid; d < r.dim; d += kStepWarps * 32) {
+    for (int d = tid; d < r.dim; d += kStepThreads) {
         q[d] = rotated(p + r.c_q + head * r.dim, d, r.rot_dims, cs, sn) * r.q_scale;
         k[d] = rotated(p + r.c_k + head * r.dim, d, r.rot_dims, cs, sn) * r.k_scale;
         if (r.rank > 0) {
             const int c = head * r.dim + d;
             float z = 0.0f;
-#pragma unroll 8
+#pragma unroll 16
             for (int j = 0; j < r.rank; j++) z = fmaf(p[r.c_a1 + j], r.a2t[(size_t)j * r.heads * r.dim + c], z);
             al[d] = gate_decay(z + r.a2b[c], r.inv_tau);
         } else {
             al[d] = r.decay[head];
         }
     }
-    for (int d = tid; d < r.vdim; d += kStepWarps * 32) v[d] = p[r.c_v + head * r.vdim + d];
-    __syncthreads();
-    float *S = r.state + (size_t)head * r.dim * r.vdim;
-    for (int c = lane; c < r.vdim; c += 32) {
-        const float vc = v[c];
-        float acc = 0.0f;
-        for (int r0 = warp; r0 < r.dim; r0 += kStepWarps * kStepBatch) {
-            float s[kStepBatch];
-#pragma unroll
-            for (int i = 0; i < kStepBatch; i++) {
-                const int row = r0 + i * kStepWarps;
-                s[i] = pos > 0 && row < r.dim ? S[(size_t)row * r.vdim + c] : 0.0f;
-            }
-#pragma unroll
-            for (int i = 0; i < kStepBatch; i++) {
-                const int row = r0 + i * kStepWarps;
-                if (row < r.dim) {
-                    s[i] = fmaf(s[i], al[row], k[row] * vc);
-                    acc = fmaf(s[i], q[row], acc);
-                    S[(size_t)row * r.vdim + c] = s[i];
-                }
-            }
-        }
-        po[warp * r.vdim + c] = acc;
-    }
+    for (int d = tid; d < cn; d += kStepThreads) v[d] = p[r.c_v + head * r.vdim + c0 + d];
     __syncthreads();
     float ss = 0.0f;
-    for (int d = tid; d < r.vdim; d += kStepWarps * 32) {
-        float o = 0.0f;
+    for (int b = 0; b < cn; b += 32) {
+        const int c = b + lane;
+        if (b > 0) fetch(c);
+        const float vc = c < cn ? v[c] : 0.0f;
+        float acc = 0.0f;
 #pragma unroll
-        for (int w = 0; w < kStepWarps; w++) o += po[w * r.vdim + d];
-        v[d] = o;   // the value vector has been used
-        ss = fmaf(o, o, ss);
+        for (int i = 0; i < kStepRows; i++) {
+            const int row = warp + i * kStepWarps;
+            if (row < r.dim) {
+                s[i] = fmaf(s[i], al[row], k[row] * vc);
+                acc = fmaf(s[i], q[row], acc);
+                if (c < cn) S[(size_t)row * r.vdim + c] = s[i];
+            }
+        }
+        po[warp * 32 + lane] = acc;
+        __syncthreads();
+        if (warp == 0) {
+            float t = 0.0f;
+#pragma unroll
+            for (int w = 0; w < kStepWarps; w++) t += po[w * 32 + lane];
+            if (c < cn) {
+                o[c] = t;
+                ss = fmaf(t, t, ss);
+            }
+        }
+        __syncthreads();
     }
-    const float rms = sqrtf(block_sum(ss, red) / (float)r.vdim + r.eps);
-    for (int d = tid; d < r.vdim; d += kStepWarps * 32) {
-        float o = v[d] / rms;
-        if (r.head_norm) o *= r.head_norm[d];
-        store_act(r.ffn.act, r.ffn.act_dt, (size_t)head * r.vdim + d, o * silu_f32(p[r.c_g + head * r.vdim + d]));
+    ss = block_sum(ss, red);
+    if (cluster > 1) {
+        if (tid == 0) squares = ss;
+        asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        ss = 0.0f;
+        const uint32_t mine = (uint32_t)__cvta_generic_to_shared(&squares);
+        for (int i = 0; i < cluster; i++) {   // the same order in every CTA
+            uint32_t at;
+            float x;
+            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"(mine), "r"(i));
+            asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(x) : "r"(at) : "memory");
+            ss += x;
+        }
     }
+    const float rms = sqrtf(ss / (float)r.vdim + r.eps);
+    for (int d = tid; d < cn; d += kStepThreads) {
+        float x = o[d] / rms;
+        if (r.head_norm) x *= r.head_norm[c0 + d];
+        const int c = head * r.vdim + c0 + d;
+        store_act(r.ffn.act, r.ffn.act_dt, c, x * silu_f32(p[r.c_g + c]));
+    }
+    // nobody leaves while its sum may still be read
+    if (cluster > 1) asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
 // ---- host side ----
@@ -413,14 +445,26 @@ nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
 }
 
 nnq_status launch_rec_step(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
-    const size_t smem = (size_t)(3 * r.dim + (1 + kStepWarps) * r.vdim) * sizeof(float);
-    if (smem > 48 * 1024) {
-        nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(rec_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "recurrence shared memory");
-        if (s != NNQ_OK) return s;
-    }
-    launch_pdl_smem(rec_step_kernel, dim3(r.heads + ffn_ctas(r.ffn, 1, kStepWarps * 32, ctx->sm_count)), dim3(kStepWarps * 32), smem, st, r);
+    // up to eight CTAs per head with at least 32 columns each
+    const int want = (r.vdim + 31) / 32 < 8 ? (r.vdim + 31) / 32 : 8;
+    const int slice = ((r.vdim + want - 1) / want + 31) / 32 * 32, cluster = (r.vdim + slice - 1) / slice;
+    const size_t smem = (size_t)(3 * r.dim + 2 * slice + kStepThreads) * sizeof(float);
+    const int ctas = r.heads * cluster + (ffn_ctas(r.ffn, 1, kStepThreads, ctx->sm_count) + cluster - 1) / cluster * cluster;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(ctas);
+    cfg.blockDim = dim3(kStepThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = cluster;
+    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
     ctx->launches++;
-    return check_cuda(ctx, cudaGetLastError(), "recurrence step launch");
+    return check_cuda(ctx, cudaLaunchKernelEx(&cfg, rec_step_kernel, r, cluster, slice), "recurrence step launch");
 }
 
 }  // namespace nnq
