@@ -134,11 +134,11 @@ def measure(backend, name, z, prompt, new_tokens, reps=5):
             "decode_launches": int(launches)}
 
 
-def run(prompt=4096, new_tokens=128):
+def run(prompt=4096, new_tokens=128, reps=5):
     backend = api.gpu_backend()
     out = {}
     for size, z in SIZES.items():
-        out[size] = {n: measure(backend, n, z, prompt, new_tokens) for n in ("sikivik", "qwen3")}
+        out[size] = {n: measure(backend, n, z, prompt, new_tokens, reps) for n in ("sikivik", "qwen3")}
         r = out[size]
         out[size]["sikivik_over_qwen3"] = {k: r["sikivik"][k] / r["qwen3"][k] for k in ("prefill_tokens_per_s", "decode_tokens_per_s")}
     return out

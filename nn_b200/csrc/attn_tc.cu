@@ -71,20 +71,26 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_s)), "r"(256u) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    if (warp < 4) {
-        // the 128 query vectors, a warp per vector in turn
-        for (int r = warp; r < kAtRows; r += 4) {
-            const int t = t0 + r;
-            const float *src = a.qrot + ((size_t)(t / group) * a.heads + kvh * group + t % group) * a.dim_ld;
-            for (int d = 4 * lane; d < 64 * ATOMS; d += 128) {
-                const float4 v = t <= last_pair && d < a.dim_ld ? *reinterpret_cast<const float4 *>(src + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                uint2 hi, lo;
-                split2(v.x, v.y, hi.x, lo.x);
-                split2(v.z, v.w, hi.y, lo.y);
-                uint8_t *dst = q_s + (d >> 6) * kAtQAtom + swz_at(r, d & 63);
-                *reinterpret_cast<uint2 *>(dst) = hi;
-                *reinterpret_cast<uint2 *>(dst + ATOMS * kAtQAtom) = lo;
-            }
+    {
+        // the 128 query vectors: neighbouring lanes take neighbouring dimensions, all loads before the first store
+        constexpr int QN = kAtRows * 16 * ATOMS / kAtThreads;
+        float4 v[QN];
+#pragma unroll
+        for (int i = 0; i < QN; i++) {
+            const int u = tid + kAtThreads * i, t = t0 + u / (16 * ATOMS), d = 4 * (u % (16 * ATOMS));
+            v[i] = t <= last_pair && d < a.dim_ld
+                       ? *reinterpret_cast<const float4 *>(a.qrot + ((size_t)(t / group) * a.heads + kvh * group + t % group) * a.dim_ld + d)
+                       : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+#pragma unroll
+        for (int i = 0; i < QN; i++) {
+            const int u = tid + kAtThreads * i, r = u / (16 * ATOMS), d = 4 * (u % (16 * ATOMS));
+            uint2 hi, lo;
+            split2(v[i].x, v[i].y, hi.x, lo.x);
+            split2(v[i].z, v[i].w, hi.y, lo.y);
+            uint8_t *dst = q_s + (d >> 6) * kAtQAtom + swz_at(r, d & 63);
+            *reinterpret_cast<uint2 *>(dst) = hi;
+            *reinterpret_cast<uint2 *>(dst + ATOMS * kAtQAtom) = lo;
         }
         fence_async_smem();
     }
@@ -163,18 +169,25 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_tc_kernel(const WindowAttn
             const size_t at = (size_t)row * a.ffn.out_k + head * a.vdim;
             if (a.ffn.act_dt == NNQ_BF16 && (a.vdim & 7) == 0) {
 #pragma unroll
-                for (int d = 0; d < NV * 32; d += 8) {
-                    if (d >= a.vdim) continue;
-                    float v[8];
+                for (int b = 0; b < NV * 32; b += 32) {
+                    float4 gv[8];
 #pragma unroll
-                    for (int i = 0; i < 8; i++) v[i] = acc[d + i] * inv;
-                    if (a.gated) {
-                        const float4 g0 = reinterpret_cast<const float4 *>(g + d)[0], g1 = reinterpret_cast<const float4 *>(g + d)[1];
-                        v[0] *= sigmoid_f32(g0.x); v[1] *= sigmoid_f32(g0.y); v[2] *= sigmoid_f32(g0.z); v[3] *= sigmoid_f32(g0.w);
-                        v[4] *= sigmoid_f32(g1.x); v[5] *= sigmoid_f32(g1.y); v[6] *= sigmoid_f32(g1.z); v[7] *= sigmoid_f32(g1.w);
+                    for (int i = 0; i < 8; i++)
+                        gv[i] = a.gated && b + 4 * i < a.vdim ? *reinterpret_cast<const float4 *>(g + b + 4 * i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+                    for (int d = 0; d < 32; d += 8) {
+                        if (b + d >= a.vdim) continue;
+                        float v[8];
+#pragma unroll
+                        for (int i = 0; i < 8; i++) v[i] = acc[b + d + i] * inv;
+                        if (a.gated) {
+                            const float4 g0 = gv[d / 4], g1 = gv[d / 4 + 1];
+                            v[0] *= sigmoid_f32(g0.x); v[1] *= sigmoid_f32(g0.y); v[2] *= sigmoid_f32(g0.z); v[3] *= sigmoid_f32(g0.w);
+                            v[4] *= sigmoid_f32(g1.x); v[5] *= sigmoid_f32(g1.y); v[6] *= sigmoid_f32(g1.z); v[7] *= sigmoid_f32(g1.w);
+                        }
+                        *reinterpret_cast<uint4 *>(reinterpret_cast<__nv_bfloat16 *>(a.ffn.act) + at + b + d) =
+                            make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
                     }
-                    *reinterpret_cast<uint4 *>(reinterpret_cast<__nv_bfloat16 *>(a.ffn.act) + at + d) =
-                        make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
                 }
             } else {
 #pragma unroll

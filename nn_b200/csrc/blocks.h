@@ -76,7 +76,7 @@ int attn_step_counters(int heads, int kv_heads);
 struct Recurrence {
     RowSpan span;
     FfnPart ffn;
-    int heads, dim, vdim, dim_ld;   // dim_ld: rounded up to 64
+    int heads, dim, vdim, dim_ld;   // dim_ld: 64, 128 or 256
     int c_q, c_k, c_v, c_g, c_a1;
     float q_scale, k_scale;         // applied after the rotation
     int rot_dims;

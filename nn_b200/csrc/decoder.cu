@@ -914,7 +914,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
             most(part, attn_step_part_floats(b.heads, b.kv_heads, B.vdim_ld, B.ranges));
             most(counters, attn_step_counters(b.heads, b.kv_heads));
         } else {
-            B.dim_ld = round_up(b.dim, 64);
+            B.dim_ld = b.dim <= 64 ? 64 : round_up(b.dim, 128);
             alloc(&B.rec_state, (size_t)b.heads * b.dim * b.vdim * 4, "recurrent state");
             if (b.decay_rank > 0) {
                 alloc(&B.a2t, (size_t)b.heads * b.dim * b.decay_rank * 4, "decay weight");

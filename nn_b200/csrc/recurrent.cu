@@ -70,12 +70,12 @@ __global__ void __launch_bounds__(kRecPrepWarps * 32) rec_prep_kernel(const Recu
 
 // ---- the scan over a block of rows ----
 //
-// A warp owns 2 C columns of the state over all key rows: lane = 16 row groups x 2 column groups, a lane
-// holds rows 64 j + 4 (lane % 16) .. + 3 and C columns as packed f32 pairs (two rows of a column), so that
-// q, k and the decay come as pairs out of one 16-byte shared-memory read and the three operations of a state
-// element -- k v, s a + (k v), o + s q -- are packed f32x2 instructions. After eight tokens the lanes' partial
-// o are reduced across the row groups by halving exchanges: a lane ends with one token of one or two columns.
-// Tokens stream through a three-stage ring of cp.async copies, one barrier per stage.
+// A warp owns a few columns of the state over all key rows: RL row lanes (32; 16 for heads of at most 64, then two
+// column groups) hold rows 4 RL j + 4 rl .. + 3 of C columns each, as packed f32 pairs (two rows of a column), so that
+// q, k and the decay come as pairs out of one 16-byte shared-memory read without two lanes reading the same, and the
+// three operations of a state element -- k v, s a + (k v), o + s q -- are packed f32x2 instructions. After eight
+// tokens the lanes' partial o are reduced across the row lanes by halving exchanges: a lane ends with one token of
+// one or two columns. Tokens stream through a three-stage ring of cp.async copies, one barrier per stage.
 
 constexpr int kScanTokens = 8, kScanStages = 3;
 
@@ -103,15 +103,15 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
     return r;
 }
 
-// grid (heads, ceil(vdim / (2 C WARPS))); NJ = dim_ld / 64
-template <int NJ, int C, int WARPS, bool FIXED>
+// grid (heads, ceil(vdim / columns of a CTA)); NJ = dim_ld / (4 RL)
+template <int RL, int NJ, int C, int WARPS, bool FIXED>
 __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r) {
     constexpr int NS = FIXED ? 2 : 3;   // streams: q, k (, decay)
-    constexpr int LD = NJ * 64, COLS = WARPS * 2 * C, T = kScanTokens, THREADS = WARPS * 32;
+    constexpr int RW = 4 * RL, LD = NJ * RW, COLS = WARPS * (32 / RL) * C, T = kScanTokens, THREADS = WARPS * 32;
     constexpr int STAGE = T * (NS * LD + COLS);   // floats
     extern __shared__ __align__(16) float scan_smem[];
-    const int tid = threadIdx.x, lane = tid & 31, rl = lane & 15;
-    const int wcol = ((tid >> 5) * 2 + (lane >> 4)) * C;
+    const int tid = threadIdx.x, rl = tid % RL;
+    const int wcol = tid / RL * C;
     const int head = blockIdx.x, v0 = blockIdx.y * COLS, n = r.span.n;
     float *state = r.state + (size_t)head * r.dim * r.vdim;
     uint64_t S[NJ][2][C];
@@ -124,7 +124,7 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
                 float s[2];
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
-                    const int row = 64 * j + 4 * rl + 2 * h + e, col = v0 + wcol + c;
+                    const int row = RW * j + 4 * rl + 2 * h + e, col = v0 + wcol + c;
                     s[e] = r.span.pos0 > 0 && row < r.dim && col < r.vdim ? state[(size_t)row * r.vdim + col] : 0.0f;
                 }
                 S[j][h][c] = pack2(s[0], s[1]);
@@ -177,7 +177,7 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
                 for (int c = 0; c < C; c++) vd[c] = pack2(v[c], v[c]);
 #pragma unroll
                 for (int j = 0; j < NJ; j++) {
-                    const int at = 64 * j + 4 * rl;
+                    const int at = RW * j + 4 * rl;
                     const ulonglong2 q = *reinterpret_cast<const ulonglong2 *>(b + t * LD + at);
                     const ulonglong2 k = *reinterpret_cast<const ulonglong2 *>(b + (T + t) * LD + at);
                     const ulonglong2 al = FIXED ? make_ulonglong2(fixed2, fixed2) : *reinterpret_cast<const ulonglong2 *>(b + ((NS - 1) * T + t) * LD + at);
@@ -200,12 +200,15 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
                 po[t * C + c] = lo + hi;
             }
         }
-        // 8 C sums over 16 lanes: bits 3, 2, 1 of the lane pick a token, bit 0 the upper half of the columns
+        // 8 C sums over RL lanes: the upper three bits of the row lane pick a token, the next ones a column (or a pair)
+        constexpr int LR = RL == 32 ? 5 : 4, LC = C == 4 ? 2 : (C == 2 ? 1 : 0);
+        constexpr int CB = LC < LR - 3 ? LC : LR - 3, LEFT = C >> CB, SPARE = LR - 3 - CB;
 #pragma unroll
-        for (int step = 0; step < 4; step++) {
-            const int half = (T * C / 2) >> step, bit = 8 >> step;
-            if (half == 0) {
-                po[0] += __shfl_xor_sync(0xFFFFFFFFu, po[0], bit);
+        for (int step = 0; step < LR; step++) {
+            const int half = (T * C / 2) >> step, bit = (RL / 2) >> step;
+            if (step >= 3 + CB) {
+#pragma unroll
+                for (int i = 0; i < LEFT; i++) po[i] += __shfl_xor_sync(0xFFFFFFFFu, po[i], bit);
             } else {
 #pragma unroll
                 for (int i = 0; i < half; i++) {
@@ -214,9 +217,8 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
                 }
             }
         }
-        constexpr int LEFT = C >= 2 ? C / 2 : 1;
-        const int t = ch * T + (rl >> 1), col = v0 + wcol + (C >= 2 ? LEFT * (rl & 1) : 0);
-        if (t < n && (C >= 2 || (rl & 1) == 0)) {
+        const int t = ch * T + (rl >> (LR - 3)), col = v0 + wcol + ((rl >> SPARE) & ((1 << CB) - 1)) * LEFT;
+        if (t < n && (rl & ((1 << SPARE) - 1)) == 0) {
             float *o = r.o + ((size_t)t * r.heads + head) * r.vdim + col;
 #pragma unroll
             for (int i = 0; i < LEFT; i++)
@@ -233,7 +235,7 @@ __global__ void __launch_bounds__(WARPS * 32) rec_scan_kernel(const Recurrence r
                 unpack2(S[j][h][c], s[0], s[1]);
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
-                    const int row = 64 * j + 4 * rl + 2 * h + e, col = v0 + wcol + c;
+                    const int row = RW * j + 4 * rl + 2 * h + e, col = v0 + wcol + c;
                     if (row < r.dim && col < r.vdim) state[(size_t)row * r.vdim + col] = s[e];
                 }
             }
@@ -394,11 +396,11 @@ __global__ void __launch_bounds__(kStepThreads) rec_step_kernel(const Recurrence
 
 // ---- host side ----
 
-template <int NJ, int C, int WARPS, bool FIXED>
+template <int RL, int NJ, int C, int WARPS, bool FIXED>
 static nnq_status go_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
-    constexpr int cols = WARPS * 2 * C;
-    constexpr size_t smem = (size_t)kScanStages * kScanTokens * ((FIXED ? 2 : 3) * NJ * 64 + cols) * sizeof(float);
-    auto kernel = rec_scan_kernel<NJ, C, WARPS, FIXED>;
+    constexpr int cols = WARPS * (32 / RL) * C;
+    constexpr size_t smem = (size_t)kScanStages * kScanTokens * ((FIXED ? 2 : 3) * NJ * 4 * RL + cols) * sizeof(float);
+    auto kernel = rec_scan_kernel<RL, NJ, C, WARPS, FIXED>;
     if (smem > 48 * 1024) {
         nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "recurrence shared memory");
         if (s != NNQ_OK) return s;
@@ -409,16 +411,18 @@ static nnq_status go_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
 }
 
 // Wide tiles amortise the shared-memory reads of q / k / decay over more columns, narrow ones give more warps.
-// Measured on 128 x 256 heads (us per 1024 rows, all kernels of the mixer): 16 heads 259 / 279 / 377 with C = 4 / 2 / 1,
-// 8 heads 229 / 191 / 234; 8 heads of 64 x 64: 148 / 138 / 117.
-template <int NJ>
+// Measured (us per 1024 rows, all kernels of the mixer, C = 4 / 2 / 1): 16 heads of 128 x 256 254 / 284 / 410,
+// 8 heads of 128 x 256 222 / 191 / 244, 8 heads of 64 x 64 141 / 130 / 116.
+template <int RL, int NJ>
 static nnq_status pick_scan(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
+    constexpr int W = RL == 32 ? 8 : 4;
     const bool fixed = r.rank == 0;
-    auto warps = [&](int c) { return r.heads * ((r.vdim + 2 * c - 1) / (2 * c)); };
-    const int enough = ctx->sm_count * 5 / 2;
-    if (warps(4) >= enough) return fixed ? go_scan<NJ, 4, 4, true>(ctx, r, st) : go_scan<NJ, 4, 4, false>(ctx, r, st);
-    if (warps(2) >= enough) return fixed ? go_scan<NJ, 2, 4, true>(ctx, r, st) : go_scan<NJ, 2, 4, false>(ctx, r, st);
-    return fixed ? go_scan<NJ, 1, 4, true>(ctx, r, st) : go_scan<NJ, 1, 4, false>(ctx, r, st);
+    auto warps = [&](int c) { return r.heads * ((r.vdim + (32 / RL) * c - 1) / ((32 / RL) * c)); };
+    const int enough = 5 * ctx->sm_count;
+    const int c = warps(4) >= enough ? 4 : (warps(2) >= enough ? 2 : 1);
+    if (c == 4) return fixed ? go_scan<RL, NJ, 4, W, true>(ctx, r, st) : go_scan<RL, NJ, 4, W, false>(ctx, r, st);
+    if (c == 2) return fixed ? go_scan<RL, NJ, 2, W, true>(ctx, r, st) : go_scan<RL, NJ, 2, W, false>(ctx, r, st);
+    return fixed ? go_scan<RL, NJ, 1, W, true>(ctx, r, st) : go_scan<RL, NJ, 1, W, false>(ctx, r, st);
 }
 
 nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
@@ -429,11 +433,10 @@ nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st) {
     ctx->launches++;
     nnq_status s = check_cuda(ctx, cudaGetLastError(), "recurrence prologue launch");
     if (s != NNQ_OK) return s;
-    switch (r.dim_ld / 64) {
-        case 1: s = pick_scan<1>(ctx, r, st); break;
-        case 2: s = pick_scan<2>(ctx, r, st); break;
-        case 3: s = pick_scan<3>(ctx, r, st); break;
-        case 4: s = pick_scan<4>(ctx, r, st); break;
+    switch (r.dim_ld) {
+        case 64: s = pick_scan<16, 1>(ctx, r, st); break;
+        case 128: s = pick_scan<32, 1>(ctx, r, st); break;
+        case 256: s = pick_scan<32, 2>(ctx, r, st); break;
         default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "key dimension %d of a recurrence is above %d", r.dim, kRecMaxKeyDim);
     }
     if (s != NNQ_OK) return s;

@@ -371,6 +371,26 @@ def test_f32_products_round_nothing(m, n, k, fmt):
     t.release()
 
 
+@pytest.mark.parametrize("n,k", [(1, 64), (7, 128), (300, 256), (1000, 1536), (333, 5056), (4096, 4096), (50, 40000), (70000, 512)])
+@pytest.mark.parametrize("m", [1, 2, 3, 4])
+def test_row_product_of_bf16_weights(n, k, m):
+    """One to four rows: the streaming kernel multiplies bf16 by bf16 exactly and sums in f32."""
+    from nn_b200.formats import QuantFormat as Q
+    b = api.gpu_backend()
+    gen = torch.Generator(device="cuda:0")
+    gen.manual_seed(n + k)
+    w = torch.randn(n, k, device="cuda:0", generator=gen).to(torch.bfloat16)
+    x = torch.randn(m, k, device="cuda:0", generator=gen).to(torch.bfloat16)
+    bias = torch.randn(n, device="cuda:0", generator=gen)
+    t = api.DeviceWeight.from_device(b, Q.BF16_DENSE, w.view(torch.uint8).reshape(-1), n, k)
+    y = torch.full((m, n), float("nan"), device="cuda:0")
+    b.check(b._lib.nnq_linear(b._ctx, t.handle(), x.data_ptr(), api.BF16, m, bias.data_ptr(), y.data_ptr(), api.F32, api._stream_ptr(None)))
+    want = x.double() @ w.double().T + bias.double()
+    assert float((y.double() - want).abs().max() / want.abs().max()) <= 1e-5
+    b.device_status()
+    t.release()
+
+
 # ---- attention of a block of rows on the tensor cores (bf16 decoders) ----
 
 @pytest.mark.parametrize("heads,kv,dim,vdim,window", [(4, 2, 24, 20, 9), (8, 1, 96, 48, 96), (6, 3, 128, 128, 70), (4, 4, 64, 40, 300), (12, 2, 72, 100, 33),
