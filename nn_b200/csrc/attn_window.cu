@@ -259,7 +259,7 @@ __global__ void __launch_bounds__(32) attn_rows_kernel(const WindowAttn a) {
 constexpr int kStepThreads = 256, kStepKeys = 64, kStepMaxRanges = 64;
 
 struct StepSmem {   // offsets in floats
-    int k, v, q, raw, dots, probs, total;
+    int k, v, q, raw, trig, dots, probs, total;
     int k_ld;
 };
 __host__ __device__ inline StepSmem step_smem(int P, int dim, int dim_ld, int vdim_ld) {
@@ -275,6 +275,7 @@ __host__ __device__ inline StepSmem step_smem(int P, int dim, int dim_ld, int vd
     m.v = take(kStepKeys * vdim_ld);
     m.q = take(P * dim_ld);
     m.raw = take(P * dim + dim + vdim_ld);        // convolved values before the rotation: query heads, key, value
+    m.trig = take(dim);                        // cosines and sines of the current position
     m.dots = take(8 * P * kStepKeys);          // partial scores of the eight warps
     m.probs = take(kStepKeys * P);
     m.total = at;
@@ -341,8 +342,14 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const WindowAtt
         }
     };
     float *raw = st_smem + m.raw;
+    const int half = a.rot_dims >> 1;
+    const float *cs = st_smem + m.trig, *sn = cs + half;
     if (active) {
         fetch(lo);
+        for (int i = tid; i < half; i += kStepThreads) {
+            st_smem[m.trig + i] = a.cosv[(size_t)pos * half + i];
+            st_smem[m.trig + half + i] = a.sinv[(size_t)pos * half + i];
+        }
         if (a.taps > 1) {
             for (int i = tid; i < total; i += kStepThreads) {
                 int c, col;
@@ -381,8 +388,6 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const WindowAtt
             }
         }
         __syncthreads();
-        const int half = a.rot_dims >> 1;
-        const float *cs = a.cosv + (size_t)pos * half, *sn = a.sinv + (size_t)pos * half;
         for (int i = tid; i < P * a.dim_ld; i += kStepThreads) {
             const int p = i / a.dim_ld, d = i - p * a.dim_ld;
             st_smem[m.q + i] = p < ng && d < a.dim ? rotated(raw + p * a.dim, d, a.rot_dims, cs, sn) : 0.0f;
