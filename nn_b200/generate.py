@@ -1,6 +1,6 @@
 """Greedy generation from the command line:
 
-    python -m nn_b200.generate --model PATH --prompt 5,17,3 --new 32 [--dtype bfloat16|float32] [--max-seq N]
+    python -m nn_b200.generate --model PATH --prompt 11,4,90 --new 32 [--dtype bfloat16|float32] [--max-seq N]
 
 PATH is a model folder (config.json + model.safetensors) or a GGUF file; prompt and output are token ids.
 """

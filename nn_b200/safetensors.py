@@ -1,5 +1,5 @@
-"""Reader of safetensors files: an 8-byte little-endian length, that many bytes of JSON mapping a tensor's
-name to its dtype, shape and byte range, then the data. The file is mapped; a tensor is a view of it."""
+"""safetensors files: a u64 header size, a JSON header (per tensor: dtype, shape, byte range in the data section),
+the data section. The file is mapped; a tensor is a view of it."""
 from __future__ import annotations
 
 import json

@@ -4,7 +4,7 @@ A model is a folder with config.json and model.safetensors. config.json lists th
 ('attention': sliding-window softmax attention with short convolutions on q / k / v, value mixing and a
 sigmoid output gate; 'gla': gated linear attention; 'retention') beside a silu-gated feed-forward that reads
 the same normed row. Layer i's tensors are 'l<i>.norm1', 'l<i>.mix.*' and 'l<i>.mlp.*'; 'embed', 'final.norm'
-and 'head' complete the model. Every size and constant comes from config.json or a tensor's shape.
+and 'head' complete the model. Nothing here is tied to particular sizes: they are read.
 """
 from __future__ import annotations
 

@@ -2,12 +2,11 @@
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N
 
-Steps come from standard input, one JSON object a line:
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["a"]}
-An entry carries a request's next tokens and the places among them whose logits are wanted; 'end' lists the
-requests that are finished after the step. A step that wants something writes OUT/<step>.f32, the logits
-[wanted, vocab] as little-endian f32; after every step a line 'done <step>' is printed. The decoder holds one
-sequence: a request starts at position 0 when no other is live, and a step has one entry.
+Every input line is one step as JSON:
+    {"step": 7, "entries": [{"id": "x", "tokens": [11, 4, 90, 2], "want": [1, 3]}], "end": ["x"]}
+`tokens` continue sequence x, `want` indexes into them: after which of them logits are to be stored. `end` closes
+sequences behind the step. The wanted logits go to OUT/<step>.f32 (f32, [wanted, vocab]); 'done <step>' on
+standard output acknowledges the step. The decoder holds one sequence, so one is open at a time.
 """
 from __future__ import annotations
 
@@ -57,7 +56,7 @@ def main(argv=None) -> int:
     ap.add_argument("--model", required=True, help="a model folder or file (see nn_b200.models)")
     ap.add_argument("--dtype", default="bfloat16", choices=sorted(DTYPES))
     ap.add_argument("--out", required=True)
-    ap.add_argument("--max-tokens", type=int, default=4096, help="the most tokens a live request holds")
+    ap.add_argument("--max-tokens", type=int, default=4096, help="positions to make room for")
     a = ap.parse_args(argv)
     # stream 0 (the default stream) keeps the runner free of torch
     replay = Replay(models.load_model(a.model, max_seq=max(a.max_tokens, 16), act_dtype=DTYPES[a.dtype]), stream=0)

@@ -393,7 +393,7 @@ def test_row_product_of_bf16_weights(n, k, m):
 
 # ---- attention of a block of rows on the tensor cores (bf16 decoders) ----
 
-@pytest.mark.parametrize("heads,kv,dim,vdim,window", [(4, 2, 24, 20, 9), (8, 1, 96, 48, 96), (6, 3, 128, 128, 70), (4, 4, 64, 40, 300), (12, 2, 72, 100, 33),
+@pytest.mark.parametrize("heads,kv,dim,vdim,window", [(4, 2, 24, 20, 9), (8, 1, 88, 56, 100), (6, 3, 128, 128, 70), (4, 4, 64, 40, 300), (12, 2, 72, 100, 33),
                                                        (5, 5, 8, 8, 1), (16, 2, 128, 96, 2000)])
 def test_tensor_core_attention_is_as_exact_as_the_decode_kernel(tmp_path, heads, kv, dim, vdim, window):
     """A bf16 decoder's prompt pass (operands split into two bf16 terms) against its own decode steps (f32 on the
