@@ -270,6 +270,24 @@ def test_prompt_pass_matches_token_by_token(act_dtype, count):
     dec.release()
 
 
+def test_extend_gives_the_logits_of_chosen_tokens():
+    """Given tokens in portions (one token: the decode step, several: the prompt pass), logits after some of them."""
+    cfg, dec, _, keep = _build(api.F32)
+    ids = np.random.default_rng(3).integers(0, cfg.vocab, 24).tolist()
+    logits_dev = dec.buffers()[2]
+    want = []
+    for pos, t in enumerate(ids):
+        dec.reset(t, pos)
+        dec.step()
+        want.append(logits_dev.cpu().numpy().copy())
+    got = np.concatenate([dec.extend(ids[:9], 0, [2, 8]), dec.extend(ids[9:10], 9, [0]), dec.extend(ids[10:], 10, [0, 13])])
+    for row, pos in zip(got, (2, 8, 9, 10, 23)):
+        assert np.max(np.abs(row - want[pos])) / np.max(np.abs(want[pos])) <= 2e-3, pos
+    with pytest.raises(api.TensorError):
+        dec.extend(ids[:3], 0, [1, 1])
+    dec.backend.device_status()
+
+
 def test_generate_graph_replay_equals_stepwise():
     cfg, dec, model, keep = _build(api.BF16, seed=23)
     a = dec.generate(5, 0, 12, use_graph=False)
