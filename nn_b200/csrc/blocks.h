@@ -7,6 +7,8 @@
 // Every launcher serves both a block of prompt rows (n rows from position pos0) and a decode step
 // (n = 1, the position is read from state[1] so that the launch can be replayed from a graph).
 #pragma once
+#include <cuda_bf16.h>
+
 #include "nnq_internal.h"
 
 namespace nnq {
@@ -22,6 +24,20 @@ struct RowSpan {
     int pos0;           // position of the first row (state == NULL)
     const int *state;   // decode step: state[1] is the position (n = 1)
 };
+
+// block_norm.cu: h <- h + delta (or the embedding rows), xn <- RMSNorm(h) * w
+struct NormRows {
+    float *h;
+    const float *delta;
+    const __nv_bfloat16 *embed;   // NULL: h + delta
+    const float *w;
+    float eps;
+    void *xn;
+    int act_dt, hidden, embed_ld, xn_ld;
+};
+nnq_status launch_norm_step(nnq_ctx *ctx, const NormRows &a, const int *state, cudaStream_t st);   // one row, token in state[0]
+// n rows of tokens[]; with `rows` given, n rows picked by index (h is left as it is)
+nnq_status launch_norm_rows(nnq_ctx *ctx, const NormRows &a, int n, const int *tokens, const int *rows, cudaStream_t st);
 
 // silu(gate) * up of the feed-forward, and zeros in the columns of act that belong to neither part
 struct FfnPart {

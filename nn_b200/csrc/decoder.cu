@@ -97,9 +97,8 @@ constexpr int kWantRows = 64;     // rows of logits formed together
 __global__ void __launch_bounds__(1024)
 dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
                 const int *__restrict__ state, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                int hidden, int embed_ld, int xn_ld, int release) {
+                int hidden) {
     pdl_prologue();
-    if (release) pdl_release();
     __shared__ float red[32];
     const int tok = embed ? state[0] : 0;
     float v[8], wv[8];
@@ -110,14 +109,14 @@ dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __
         v[r] = 0.0f;
         wv[r] = 0.0f;
         if (i < hidden) {
-            v[r] = embed ? __bfloat162float(embed[(size_t)tok * embed_ld + i]) : h[i] + delta[i];
+            v[r] = embed ? __bfloat162float(embed[(size_t)tok * hidden + i]) : h[i] + delta[i];
             wv[r] = w[i];
             h[i] = v[r];
             ss = fmaf(v[r], v[r], ss);
         }
     }
     for (int i = threadIdx.x + 8 * 1024; i < hidden; i += 1024) {   // wider models: the tail goes through memory
-        const float t = embed ? __bfloat162float(embed[(size_t)tok * embed_ld + i]) : h[i] + delta[i];
+        const float t = embed ? __bfloat162float(embed[(size_t)tok * hidden + i]) : h[i] + delta[i];
         h[i] = t;
         ss = fmaf(t, t, ss);
     }
@@ -129,7 +128,6 @@ dec_norm_kernel(float *__restrict__ h, const float *__restrict__ delta, const __
         if (i < hidden) store_act(xn, act_dt, i, (v[r] / rms) * wv[r]);
     }
     for (int i = threadIdx.x + 8 * 1024; i < hidden; i += 1024) store_act(xn, act_dt, i, (h[i] / rms) * w[i]);
-    for (int i = hidden + threadIdx.x; i < xn_ld; i += 1024) store_act(xn, act_dt, i, 0.0f);
 }
 
 // One CTA per head (query heads, then key heads, then value heads), one thread per dimension:
@@ -461,58 +459,25 @@ __global__ void dec_argmax_exchange_kernel(const float *__restrict__ bv_in, cons
 
 // ---- prompt pass: the same operations over a block of rows (one row per prompt token) ----
 
-// row r: h = embedding of tokens[r] (first layer) or h += delta; xn = RMSNorm(h) * w, zeros from hidden to
-// xn_ld. One CTA per row. With `rows` given CTA i norms row rows[i] into row i of xn and leaves h as it is.
+// row r: h = embedding of tokens[r] (first layer) or h += delta; xn = RMSNorm(h) * w. One CTA per row.
 __global__ void __launch_bounds__(256)
 dec_norm_rows_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
                      const int *__restrict__ tokens, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                     int hidden, int embed_ld, int xn_ld, const int *__restrict__ rows) {
+                     int hidden) {
     __shared__ float red[32];
-    const size_t r = rows ? rows[blockIdx.x] : blockIdx.x;
+    const size_t r = blockIdx.x;
     float *hr = h + r * hidden;
     const float *dr = delta ? delta + r * hidden : nullptr;
-    const __nv_bfloat16 *er = embed ? embed + (size_t)tokens[r] * embed_ld : nullptr;
+    const __nv_bfloat16 *er = embed ? embed + (size_t)tokens[r] * hidden : nullptr;
     float ss = 0.0f;
-    if (!er && hidden % 4 == 0 && hidden <= 256 * 4 * 8) {
-        float4 v[8];
-#pragma unroll
-        for (int k = 0; k < 8; k++) {
-            const int i = 4 * (threadIdx.x + 256 * k);
-            v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (i < hidden) {
-                const float4 a = *reinterpret_cast<const float4 *>(hr + i), b = *reinterpret_cast<const float4 *>(dr + i);
-                v[k] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
-                if (!rows) *reinterpret_cast<float4 *>(hr + i) = v[k];
-            }
-            ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
-        }
-        const float rms = sqrtf(block_sum(ss, red) / (float)hidden + eps);
-        char *xr = reinterpret_cast<char *>(xn) + (size_t)blockIdx.x * xn_ld * (act_dt == NNQ_F32 ? 4 : 2);
-#pragma unroll
-        for (int k = 0; k < 8; k++) {
-            const int i = 4 * (threadIdx.x + 256 * k);
-            if (i >= hidden) continue;
-            const float4 g = *reinterpret_cast<const float4 *>(w + i);
-            const float y0 = v[k].x / rms * g.x, y1 = v[k].y / rms * g.y, y2 = v[k].z / rms * g.z, y3 = v[k].w / rms * g.w;
-            if (act_dt == NNQ_F32) {
-                reinterpret_cast<float4 *>(xr)[i >> 2] = make_float4(y0, y1, y2, y3);
-            } else {
-                const __nv_bfloat162 a = __floats2bfloat162_rn(y0, y1), b = __floats2bfloat162_rn(y2, y3);
-                reinterpret_cast<uint2 *>(xr)[i >> 2] = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
-            }
-        }
-        for (int i = hidden + threadIdx.x; i < xn_ld; i += blockDim.x) store_act(xr, act_dt, i, 0.0f);
-        return;
-    }
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         const float v = er ? __bfloat162float(er[i]) : hr[i] + dr[i];
-        if (!rows) hr[i] = v;
+        hr[i] = v;
         ss = fmaf(v, v, ss);
     }
     const float rms = sqrtf(block_sum(ss, red) / (float)hidden + eps);
-    char *xr = reinterpret_cast<char *>(xn) + (size_t)blockIdx.x * xn_ld * (act_dt == NNQ_F32 ? 4 : 2);
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) store_act(xr, act_dt, i, ((rows ? hr[i] + dr[i] : hr[i]) / rms) * w[i]);
-    for (int i = hidden + threadIdx.x; i < xn_ld; i += blockDim.x) store_act(xr, act_dt, i, 0.0f);
+    char *xr = reinterpret_cast<char *>(xn) + r * hidden * (act_dt == NNQ_F32 ? 4 : 2);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) store_act(xr, act_dt, i, (hr[i] / rms) * w[i]);
 }
 
 // grid (heads, rows): per-head RMSNorm + half-split rotation at position pos0 + row, append of k / v
@@ -1218,9 +1183,8 @@ static nnq_status step_norm_product(nnq_decoder *d, const float *norm, bool embe
         d->b_h2 = t;
         return s;
     }
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, table, d->d_state, norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, 1);
-    d->ctx->launches++;
-    return product(d, w, d->d_xn, 1, bias, y, st);
+    const nnq_status s = launch_norm_step(d->ctx, {d->d_h, d->d_delta, table, norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld}, d->d_state, st);
+    return s == NNQ_OK ? product(d, w, d->d_xn, 1, bias, y, st) : s;
 }
 
 static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
@@ -1236,10 +1200,9 @@ static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
 static nnq_status rows_blocks(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
     const nnq_decoder_config &c = d->cfg;
     for (int l = 0; l < c.n_layers; l++) {
-        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->pf_tokens,
-                                                d->blocks[l].norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
-        d->ctx->launches++;
-        nnq_status s = product(d, d->blocks[l].in, d->pf_xn, n, d->blocks[l].bias_in, d->b_proj, st);
+        nnq_status s = launch_norm_rows(d->ctx, {d->pf_h, d->pf_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->blocks[l].norm, c.rms_eps,
+                                                 d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld}, n, d->pf_tokens, nullptr, st);
+        if (s == NNQ_OK) s = product(d, d->blocks[l].in, d->pf_xn, n, d->blocks[l].bias_in, d->b_proj, st);
         if (s == NNQ_OK) s = run_block(d, l, n, pos0, nullptr, d->pf_delta, st);
         if (s != NNQ_OK) return s;
     }
@@ -1257,7 +1220,7 @@ static nnq_status step_qwen3(nnq_decoder *d, cudaStream_t st) {
     const __nv_bfloat16 *embed = (const __nv_bfloat16 *)d->d_embed;
     for (int l = 0; l < c.n_layers; l++) {
         const nnq_decoder::Layer &L = d->layers[l];
-        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? embed : nullptr, d->d_state, L.in_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0));
+        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, l == 0 ? embed : nullptr, d->d_state, L.in_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden));
         const nnq_weight *w3[3] = {L.q, L.k, L.v};
         const void *x3[3] = {d->d_xn, d->d_xn, d->d_xn};
         void *y3[3] = {d->d_q, d->d_k, d->d_v};
@@ -1279,7 +1242,7 @@ static nnq_status step_qwen3(nnq_decoder *d, cudaStream_t st) {
         DEC_RUN(32, s = d->comm ? nnq_comm_linear(d->comm, L.o, d->d_attn, adt, 1, nullptr, d->d_delta, NNQ_F32, st)
                                 : nnq_linear(ctx, L.o, d->d_attn, adt, 1, nullptr, d->d_delta, NNQ_F32, st));
         if (s != NNQ_OK) return s;
-        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, L.post_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0));
+        DEC_RUN(1, launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, L.post_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden));
         const nnq_weight *w2[2] = {L.gate, L.up};
         const void *x2[2] = {d->d_xn, d->d_xn};
         void *y2[2] = {d->d_g, d->d_u};
@@ -1305,8 +1268,7 @@ static nnq_status rows_qwen3(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
     for (int l = 0; l < c.n_layers; l++) {
         const nnq_decoder::Layer &L = d->layers[l];
         float *kc = d->d_kcache + l * layer_cache, *vc = d->d_vcache + l * layer_cache;
-        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? embed : nullptr, d->pf_tokens, L.in_norm,
-                                                c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
+        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? embed : nullptr, d->pf_tokens, L.in_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden);
         const nnq_weight *w3[3] = {L.q, L.k, L.v};
         const void *x3[3] = {d->pf_xn, d->pf_xn, d->pf_xn};
         void *y3[3] = {d->pf_q, d->pf_k, d->pf_v};
@@ -1324,7 +1286,7 @@ static nnq_status rows_qwen3(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
         s = d->comm ? nnq_comm_linear(d->comm, L.o, d->pf_attn, adt, n, nullptr, d->pf_delta, NNQ_F32, st)
                     : nnq_linear(ctx, L.o, d->pf_attn, adt, n, nullptr, d->pf_delta, NNQ_F32, st);
         if (s != NNQ_OK) return s;
-        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, d->pf_delta, nullptr, d->pf_tokens, L.post_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, nullptr);
+        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, d->pf_delta, nullptr, d->pf_tokens, L.post_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden);
         const nnq_weight *w2[2] = {L.gate, L.up};
         const void *x2[2] = {d->pf_xn, d->pf_xn};
         void *y2[2] = {d->pf_g, d->pf_u};
@@ -1363,7 +1325,7 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
         return launch_argmax(d, vocab_parallel, cv, st);
     }
     if ((s = step_qwen3(d, st)) != NNQ_OK) return s;
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
+    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->d_h, d->d_delta, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden);
     ctx->launches++;
     return launch_head(d, vocab_parallel, cv, st);
 }
@@ -1451,9 +1413,9 @@ nnq_status nnq_decoder_prefill(nnq_decoder *d, const int32_t *tokens_host, int c
     const size_t last = (size_t)(n - 1) * c.hidden;
     const int st4[4] = {tokens_host[count - 1], start_pos + count - 1, 0, 0};
     if ((s = check_cuda(ctx, cudaMemcpyAsync(d->d_state, st4, sizeof(st4), cudaMemcpyHostToDevice, st), "decoder state")) != NNQ_OK) return s;
-    launch_pdl(dec_norm_kernel, dim3(1), dim3(1024), st, d->pf_h + last, d->pf_delta + last, nullptr, d->d_state, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld, d->blocks ? 1 : 0);
-    ctx->launches++;
-    if ((s = launch_head(d, vocab_parallel, cv, st)) != NNQ_OK) return s;
+    s = launch_norm_step(ctx, {d->pf_h + last, d->pf_delta + last, nullptr, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld},
+                         d->d_state, st);
+    if (s != NNQ_OK || (s = launch_head(d, vocab_parallel, cv, st)) != NNQ_OK) return s;
     s = check_cuda(ctx, cudaStreamSynchronize(st), "prompt pass");   // tokens_host and st4 are the caller's / the stack's
     if (s == NNQ_OK) d->host_pos = (long long)start_pos + count;
     return s;
@@ -1495,10 +1457,9 @@ nnq_status nnq_decoder_extend(nnq_decoder *d, const int32_t *tokens_host, int co
                 m++;
             }
             if ((s = check_cuda(ctx, cudaMemcpyAsync(d->pf_want, rows, (size_t)m * 4, cudaMemcpyHostToDevice, st), "wanted rows")) != NNQ_OK) return s;
-            dec_norm_rows_kernel<<<m, 256, 0, st>>>(d->pf_h, d->pf_delta, nullptr, d->pf_tokens, d->d_final_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden,
-                                                    d->embed_ld, d->xn_ld, d->pf_want);
-            ctx->launches++;
-            if ((s = product(d, d->lm_head, d->pf_xn, m, nullptr, d->d_want_logits, st)) != NNQ_OK) return s;
+            s = launch_norm_rows(ctx, {d->pf_h, d->pf_delta, nullptr, d->d_final_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld}, m,
+                                 d->pf_tokens, d->pf_want, st);
+            if (s == NNQ_OK && (s = product(d, d->lm_head, d->pf_xn, m, nullptr, d->d_want_logits, st)) != NNQ_OK) return s;
             s = check_cuda(ctx, cudaMemcpyAsync(logits_host + (size_t)w0 * c.vocab, d->d_want_logits, (size_t)m * c.vocab * 4, cudaMemcpyDeviceToHost, st), "logits");
             if (s == NNQ_OK) s = check_cuda(ctx, cudaStreamSynchronize(st), "logits");   // rows[] is on the stack
             if (s != NNQ_OK) return s;
