@@ -611,8 +611,9 @@ NNQ_API nnq_status nnq_decoder_buffers(nnq_decoder *d, float **k_cache, float **
 NNQ_API void nnq_decoder_destroy(nnq_decoder *d);
 
 /* ---- decoders whose layers each name their own mixer -------------------------------------
- * A block is x <- x + mixer(h) + ff(h) with h = RMSNorm(x) * w: one norm, both parts read it. The
- * decoder object, its step / prompt pass / state / token loop are the ones above; nnq_decoder_create_blocks
+ * A block is one residual sum: x <- x + mixer(h) + ff(h) with h = RMSNorm(x) * w (one norm, both parts read it), or with
+ * post_norm x <- LN(alpha x + mixer(x) + ff(x)), LN the layer norm with weight and bias. Mixer or feed-forward may be
+ * absent, so a layer of two sequential sublayers is two blocks. The decoder object, its step / prompt pass / state / token loop are the ones above; nnq_decoder_create_blocks
  * takes the place of nnq_decoder_create, and nnq_decoder_set_block that of nnq_decoder_set_layer. Of the
  * nnq_decoder_config only hidden, n_layers, vocab, max_seq, rms_eps and act_dtype are read (the other
  * fields are ignored; tensor parallelism is not available: tp_world must be 0 or 1). With act_dtype
@@ -620,13 +621,20 @@ NNQ_API void nnq_decoder_destroy(nnq_decoder *d);
  * everything else -- residual, norms, rotation, scores, softmax, decays, recurrent state -- is f32. */
 typedef enum nnq_mixer {
     NNQ_MIXER_ATTENTION = 0,  /* softmax attention over a sliding window, query heads grouped over kv_heads */
-    NNQ_MIXER_RECURRENT = 1   /* S_t = diag(decay) S_{t-1} + k v^T, o = S^T q per head; o / rms(o) (* head_norm) * silu(g) */
+    NNQ_MIXER_RECURRENT = 1,  /* S_t = diag(decay) S_{t-1} + k v^T, o = S^T q per head; o / rms(o) (* head_norm) * silu(g) */
+    NNQ_MIXER_LATENT = 2,     /* softmax attention over a sliding window whose keys and values are linear images of one
+                               * normed latent per token, c = RMSNorm((W_dkv h)[0, kv_rank)) * kv_norm, and of one rotated
+                               * key part r = R (W_dkv h)[kv_rank, ..) that all heads share; queries
+                               * W_uq (RMSNorm(W_dq h) * q_norm), per head dim unrotated and rot_dims rotated dimensions;
+                               * score = scale (q_u . W_uk c + q_r . r), value W_uv c. post_norm blocks only. */
+    NNQ_MIXER_NONE = 3        /* feed-forward alone. post_norm blocks only. */
 } nnq_mixer;
+typedef enum nnq_gate_act { NNQ_ACT_SILU = 0, NNQ_ACT_GELU_TANH = 1 } nnq_gate_act;
 typedef struct nnq_block_config {
     int32_t mixer;           /* nnq_mixer */
     int32_t heads, kv_heads; /* kv_heads: attention only */
     int32_t dim, vdim;       /* query / key size and value size of a head (at most 256 each where a limit applies) */
-    int32_t ffn;             /* width of the silu-gated feed-forward, 0 = none */
+    int32_t ffn;             /* width of the gated feed-forward, 0 = none */
     int32_t rot_dims;        /* first dimensions of q and k that are rotated (half-split pairs), 0 = none */
     double rot_base;         /* angle of pair i at position p: p * rot_base^(-2 i / rot_dims) */
     /* attention */
@@ -640,21 +648,33 @@ typedef struct nnq_block_config {
     int32_t decay_rank;      /* > 0: decay per key channel sigmoid(W_2 W_1 h + b)^(1 / decay_tau) with a W_1 of this
                               * many rows; 0: a fixed decay per head */
     float decay_tau;
+    int32_t post_norm;       /* 1: layer norm behind the sum, the parts read x itself */
+    float alpha;             /* factor on x in the sum of a post_norm block */
+    int32_t ffn_act;         /* nnq_gate_act of the feed-forward (NNQ_MIXER_NONE blocks; silu elsewhere) */
+    int32_t experts;         /* NNQ_MIXER_NONE: > 0: a mixture of that many experts (nnq_block_weights.moe) in place of it */
+    /* latent */
+    int32_t q_rank, kv_rank; /* widths of the query latent and of the key / value latent */
+    int32_t kv_from;         /* block whose latents and rotated key parts this one reads; < 0: its own */
 } nnq_block_config;
 /* Where the parts of a block sit in its two products (filled by nnq_decoder_block_layout). Input product:
  * weight [in_cols, in_k], rows of q, k, v, g (gate), a1 (W_1 of the decay), gate, up from these row numbers on
  * (-1: absent), zero rows between and zero columns beyond hidden. Output product: weight [hidden, out_k],
  * columns of the mixer's output projection from column 0 (heads * vdim of them), of the feed-forward's down
- * projection from column ffn_col, zeros elsewhere. */
+ * projection from column ffn_col, zeros elsewhere. Latent blocks: input rows of W_dq from q on and of W_dkv from k on (-1:
+ * read from another block), second product uq [heads * (dim + rot_dims), q_ld], third ukv
+ * [heads * (dim_ld + vdim_ld), kv_ld]: row h * dim_ld + d is row h * dim + d of W_uk, row heads * dim_ld + h * vdim_ld + d
+ * row h * vdim + d of W_uv. NNQ_MIXER_NONE: gate row j at input row gate + 2 j, up row j at up + 2 j (ffn_step 2; 1
+ * elsewhere); a mixture of experts has no products of its own (in_cols 0). */
 typedef struct nnq_block_layout {
     int32_t in_cols, in_k, out_k, ffn_col;
     int32_t q, k, v, g, a1, gate, up;
+    int32_t ffn_step, q_ld, kv_ld, dim_ld, vdim_ld;
 } nnq_block_layout;
 /* Weights of a block. The f32 arrays are host or device memory and are copied; in / out stay owned by the
  * caller. Arrays a block does not use may be NULL. */
 typedef struct nnq_block_weights {
     const nnq_weight *in, *out;
-    const float *norm;        /* [hidden] */
+    const float *norm;        /* [hidden]: of h, or of the sum in a post_norm block */
     const float *bias_in;     /* [in_cols] or NULL */
     const float *bias_out;    /* [hidden] or NULL */
     const float *conv;        /* [heads*dim + kv_heads*(dim + vdim), conv_taps], channels q | k | v */
@@ -663,6 +683,11 @@ typedef struct nnq_block_weights {
     const float *decay_b;     /* [heads*dim] */
     const float *decay;       /* [heads] */
     float lambda;             /* value_mix */
+    const float *norm_bias;   /* [hidden], post_norm */
+    const nnq_weight *uq, *ukv;   /* latent; stay owned by the caller */
+    const float *q_norm;      /* [q_rank] */
+    const float *kv_norm;     /* [kv_rank], NULL with kv_from */
+    const nnq_moe *moe;       /* mixture of experts: hidden = in_k, [E, N, K] bf16 experts; stays owned by the caller */
 } nnq_block_weights;
 /* `blocks` holds cfg->n_layers entries. block_rows: prompt rows that go through the blocks together (0 =
  * 1024). An attention block keeps a ring of min(max_seq, window - 1 + block_rows) keys and values. */
@@ -674,6 +699,16 @@ NNQ_API nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_bl
  * beyond hidden); lm_head [vocab, in_k]. The two may be the same weight. */
 NNQ_API nnq_status nnq_decoder_set_head_weights(nnq_decoder *d, const nnq_weight *embed, const float *final_norm,
                                                 const nnq_weight *lm_head);
+/* Optional parts of a block decoder outside its blocks. */
+typedef struct nnq_head_options {
+    const float *final_norm_bias;   /* [hidden]: the final norm is a layer norm with this bias; NULL: RMS norm */
+    float logit_cap;                /* > 0: logits <- cap * tanh(logits / cap) */
+    const nnq_weight *pair_table;   /* bf16 [pair_buckets + 1, in_k], added to the embedding: row (previous token * pair_mul_prev
+                                     * + token * pair_mul_cur) mod pair_buckets, row pair_buckets for a sequence's first token;
+                                     * NULL: none */
+    int64_t pair_mul_prev, pair_mul_cur, pair_buckets;
+} nnq_head_options;
+NNQ_API nnq_status nnq_decoder_set_head_options(nnq_decoder *d, const nnq_head_options *o);
 /* Continues the sequence with `count` given tokens (host array) at positions start_pos .., and writes the
  * logits after the `n_want` tokens want[] (indexes into tokens, ascending) to logits_host [n_want, vocab].
  * One token runs the decode step, several the prompt pass. start_pos 0 starts a new sequence; otherwise it

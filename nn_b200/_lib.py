@@ -88,6 +88,7 @@ SIGNATURES = {
     "nnq_decoder_block_layout": (c_int, [c_void_p, c_int, c_void_p]),
     "nnq_decoder_set_block": (c_int, [c_void_p, c_int, c_void_p]),
     "nnq_decoder_set_head_weights": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p]),
+    "nnq_decoder_set_head_options": (c_int, [c_void_p, c_void_p]),
     "nnq_decoder_extend": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p]),
     "nnq_plan_create": (c_int, [c_void_p, c_int, c_int, c_int, ctypes.POINTER(c_void_p)]),
     "nnq_plan_add": (c_int, [c_void_p, c_int, ctypes.POINTER(c_void_p), c_void_p, ctypes.POINTER(c_void_p),

@@ -1,114 +1,118 @@
-// Residual add + RMSNorm of a block decoder, for the row of a decode step and for a block of rows. The normed
-// rows may be wider than the model (zero columns up to the products' k step).
-#include "blocks.h"
-#include "decoder_common.cuh"
+// Residual update + norm of a block decoder, for the row of a decode step and for a block of rows, and the small
+// row kernels around the products (gated activation of an interleaved product, logit cap). The normed rows may be
+// wider than the model (zero columns up to the products' k step).
+#include "block_norm.cuh"
+#include "blocks.cuh"
 
 namespace nnq {
 
-// h = embedding row of the current token, or h += delta; xn = RMSNorm(h) * w, zeros from hidden to xn_ld.
-// One CTA; every thread keeps its (up to 8) elements in registers between the two phases.
-__global__ void __launch_bounds__(1024)
-norm_step_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
-                 const int *__restrict__ state, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                 int hidden, int embed_ld, int xn_ld) {
+__device__ __forceinline__ void store_units(const NormRow &r, void *xn, int act_dt, int xn_ld, float *red) {
+    float4 v[8];
+    norm_units(r, v, red);
+#pragma unroll
+    for (int k = 0; k < 8; k++) {
+        const int u = threadIdx.x + blockDim.x * k;
+        if (4 * u >= r.hidden) continue;
+        if (act_dt == NNQ_F32) {
+            reinterpret_cast<float4 *>(xn)[u] = v[k];
+        } else {
+            const __nv_bfloat162 a = __floats2bfloat162_rn(v[k].x, v[k].y), b = __floats2bfloat162_rn(v[k].z, v[k].w);
+            reinterpret_cast<uint2 *>(xn)[u] = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+        }
+    }
+}
+
+// One CTA of 256 per row (the row of a step: `state` given, token state[0], position state[1], the token before it
+// state[4]). With `rows` given CTA i norms row rows[i] into row i of xn and leaves h as it is.
+__global__ void __launch_bounds__(256) norm_rows_kernel(const NormRows a, const int *__restrict__ tokens, int pos0, const int *__restrict__ rows,
+                                                        const int *__restrict__ state) {
     pdl_prologue();
     pdl_release();
     __shared__ float red[32];
-    const int tok = embed ? state[0] : 0;
-    float v[8], wv[8];
-    float ss = 0.0f;
-#pragma unroll
-    for (int r = 0; r < 8; r++) {
-        const int i = threadIdx.x + r * 1024;
-        v[r] = 0.0f;
-        wv[r] = 0.0f;
-        if (i < hidden) {
-            v[r] = embed ? __bfloat162float(embed[(size_t)tok * embed_ld + i]) : h[i] + delta[i];
-            wv[r] = w[i];
-            h[i] = v[r];
-            ss = fmaf(v[r], v[r], ss);
-        }
-    }
-    for (int i = threadIdx.x + 8 * 1024; i < hidden; i += 1024) {   // wider models: the tail goes through memory
-        const float t = embed ? __bfloat162float(embed[(size_t)tok * embed_ld + i]) : h[i] + delta[i];
-        h[i] = t;
-        ss = fmaf(t, t, ss);
-    }
-    const float mean = block_sum(ss, red) / (float)hidden;
-    const float rms = sqrtf(mean + eps);
-#pragma unroll
-    for (int r = 0; r < 8; r++) {
-        const int i = threadIdx.x + r * 1024;
-        if (i < hidden) store_act(xn, act_dt, i, (v[r] / rms) * wv[r]);
-    }
-    for (int i = threadIdx.x + 8 * 1024; i < hidden; i += 1024) store_act(xn, act_dt, i, (h[i] / rms) * w[i]);
-    for (int i = hidden + threadIdx.x; i < xn_ld; i += 1024) store_act(xn, act_dt, i, 0.0f);
-}
-
-// row r: h = embedding of tokens[r] or h += delta; xn = RMSNorm(h) * w, zeros from hidden to
-// xn_ld. One CTA per row. With `rows` given CTA i norms row rows[i] into row i of xn and leaves h as it is.
-__global__ void __launch_bounds__(256)
-norm_rows_kernel(float *__restrict__ h, const float *__restrict__ delta, const __nv_bfloat16 *__restrict__ embed,
-                 const int *__restrict__ tokens, const float *__restrict__ w, float eps, void *__restrict__ xn, int act_dt,
-                 int hidden, int embed_ld, int xn_ld, const int *__restrict__ rows) {
-    __shared__ float red[32];
     const size_t r = rows ? rows[blockIdx.x] : blockIdx.x;
-    float *hr = h + r * hidden;
-    const float *dr = delta ? delta + r * hidden : nullptr;
-    const __nv_bfloat16 *er = embed ? embed + (size_t)tokens[r] * embed_ld : nullptr;
-    float ss = 0.0f;
-    if (!er && hidden % 4 == 0 && hidden <= 256 * 4 * 8) {
-        float4 v[8];
-#pragma unroll
-        for (int k = 0; k < 8; k++) {
-            const int i = 4 * (threadIdx.x + 256 * k);
-            v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (i < hidden) {
-                const float4 a = *reinterpret_cast<const float4 *>(hr + i), b = *reinterpret_cast<const float4 *>(dr + i);
-                v[k] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
-                if (!rows) *reinterpret_cast<float4 *>(hr + i) = v[k];
-            }
-            ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+    NormRow n;
+    n.h_in = a.h + r * a.hidden;
+    n.h_out = rows ? nullptr : a.h + r * a.hidden;
+    n.delta = a.delta ? a.delta + r * a.delta_ld : nullptr;
+    n.e0 = n.e1 = nullptr;
+    if (a.embed) {
+        const int tok = state ? state[0] : tokens[(int)r], pos = state ? state[1] : pos0 + (int)r;
+        n.e0 = a.embed + (size_t)tok * a.embed_ld;
+        if (a.pairs.table) {
+            const int prev = pos == 0 ? 0 : (state ? state[4] : tokens[(int)r - 1]);   // (tokens[-1]: the one in front of this block)
+            n.e1 = a.pairs.table + pair_row(a.pairs, prev, tok, pos) * a.embed_ld;
         }
-        const float rms = sqrtf(block_sum(ss, red) / (float)hidden + eps);
-        char *xr = reinterpret_cast<char *>(xn) + (size_t)blockIdx.x * xn_ld * (act_dt == NNQ_F32 ? 4 : 2);
-#pragma unroll
-        for (int k = 0; k < 8; k++) {
-            const int i = 4 * (threadIdx.x + 256 * k);
-            if (i >= hidden) continue;
-            const float4 g = *reinterpret_cast<const float4 *>(w + i);
-            const float y0 = v[k].x / rms * g.x, y1 = v[k].y / rms * g.y, y2 = v[k].z / rms * g.z, y3 = v[k].w / rms * g.w;
-            if (act_dt == NNQ_F32) {
-                reinterpret_cast<float4 *>(xr)[i >> 2] = make_float4(y0, y1, y2, y3);
-            } else {
-                const __nv_bfloat162 a = __floats2bfloat162_rn(y0, y1), b = __floats2bfloat162_rn(y2, y3);
-                reinterpret_cast<uint2 *>(xr)[i >> 2] = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
-            }
-        }
-        for (int i = hidden + threadIdx.x; i < xn_ld; i += blockDim.x) store_act(xr, act_dt, i, 0.0f);
-        return;
     }
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-        const float v = er ? __bfloat162float(er[i]) : hr[i] + dr[i];
-        if (!rows) hr[i] = v;
-        ss = fmaf(v, v, ss);
-    }
-    const float rms = sqrtf(block_sum(ss, red) / (float)hidden + eps);
-    char *xr = reinterpret_cast<char *>(xn) + (size_t)blockIdx.x * xn_ld * (act_dt == NNQ_F32 ? 4 : 2);
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) store_act(xr, act_dt, i, ((rows ? hr[i] + dr[i] : hr[i]) / rms) * w[i]);
-    for (int i = hidden + threadIdx.x; i < xn_ld; i += blockDim.x) store_act(xr, act_dt, i, 0.0f);
+    n.alpha = a.alpha;
+    n.post_w = a.post_w;
+    n.post_b = a.post_b;
+    n.in = a.in;
+    n.eps = a.eps;
+    n.hidden = a.hidden;
+    char *xr = reinterpret_cast<char *>(a.xn) + (size_t)blockIdx.x * a.xn_ld * (a.act_dt == NNQ_F32 ? 4 : 2);
+    if (a.hidden % 4 == 0 && a.hidden <= 256 * 4 * 8) store_units(n, xr, a.act_dt, a.xn_ld, red);
+    else norm_elements(n, red, [&](int i, float v) { store_act(xr, a.act_dt, i, v); });
+    for (int i = a.hidden + threadIdx.x; i < a.xn_ld; i += blockDim.x) store_act(xr, a.act_dt, i, 0.0f);
 }
 
 nnq_status launch_norm_step(nnq_ctx *ctx, const NormRows &a, const int *state, cudaStream_t st) {
-    launch_pdl(norm_step_kernel, dim3(1), dim3(1024), st, a.h, a.delta, a.embed, state, a.w, a.eps, a.xn, a.act_dt, a.hidden, a.embed_ld, a.xn_ld);
+    launch_pdl(norm_rows_kernel, dim3(1), dim3(256), st, a, nullptr, 0, nullptr, state);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "norm launch");
 }
 
-nnq_status launch_norm_rows(nnq_ctx *ctx, const NormRows &a, int n, const int *tokens, const int *rows, cudaStream_t st) {
-    norm_rows_kernel<<<n, 256, 0, st>>>(a.h, a.delta, a.embed, tokens, a.w, a.eps, a.xn, a.act_dt, a.hidden, a.embed_ld, a.xn_ld, rows);
+nnq_status launch_norm_rows(nnq_ctx *ctx, const NormRows &a, int n, const int *tokens, int pos0, const int *rows, cudaStream_t st) {
+    launch_pdl(norm_rows_kernel, dim3(n), dim3(256), st, a, tokens, pos0, rows, nullptr);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "norm launch");
+}
+
+// act[row, j] = f(proj[row, 2 j]) * proj[row, 2 j + 1], zeros from ffn to act_ld; four columns per thread
+__global__ void __launch_bounds__(256) pair_act_kernel(const float *__restrict__ proj, int proj_ld, int ffn, int kind, void *__restrict__ act, int act_dt,
+                                                       int act_ld, long long total) {
+    pdl_prologue();
+    pdl_release();
+    const int units = act_ld >> 2;
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < total; i += (long long)gridDim.x * 256) {
+        const int row = (int)(i / units), j = (int)(i - (long long)row * units) * 4;
+        const float4 *p = reinterpret_cast<const float4 *>(proj + (size_t)row * proj_ld + 2 * j);
+        float v[4];
+        if (j + 4 <= ffn) {
+            const float4 a = p[0], b = p[1];
+            v[0] = gate_act(kind, a.x) * a.y; v[1] = gate_act(kind, a.z) * a.w; v[2] = gate_act(kind, b.x) * b.y; v[3] = gate_act(kind, b.z) * b.w;
+        } else {
+            const float *q = reinterpret_cast<const float *>(p);
+#pragma unroll
+            for (int e = 0; e < 4; e++) v[e] = j + e < ffn ? gate_act(kind, q[2 * e]) * q[2 * e + 1] : 0.0f;
+        }
+        const size_t at = (size_t)row * act_ld + j;
+        if (act_dt == NNQ_F32) {
+            *reinterpret_cast<float4 *>(reinterpret_cast<float *>(act) + at) = make_float4(v[0], v[1], v[2], v[3]);
+        } else {
+            const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+            *reinterpret_cast<uint2 *>(reinterpret_cast<__nv_bfloat16 *>(act) + at) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+        }
+    }
+}
+
+nnq_status launch_pair_act(nnq_ctx *ctx, const float *proj, int proj_ld, int n, int ffn, int kind, void *act, int act_dt, int act_ld, cudaStream_t st) {
+    const long long total = (long long)n * (act_ld >> 2), want = (total + 255) / 256, most = 16LL * ctx->sm_count;
+    launch_pdl(pair_act_kernel, dim3((unsigned)(want < most ? want : most)), dim3(256), st, proj, proj_ld, ffn, kind, act, act_dt, act_ld, total);
+    ctx->launches++;
+    return check_cuda(ctx, cudaGetLastError(), "activation launch");
+}
+
+__global__ void __launch_bounds__(256) logit_cap_kernel(float *__restrict__ z, float cap, long long n) {
+    pdl_prologue();
+    pdl_release();
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) z[i] = cap * tanhf(z[i] / cap);
+}
+
+nnq_status launch_logit_cap(nnq_ctx *ctx, float *z, float cap, long long n, cudaStream_t st) {
+    const long long want = (n + 255) / 256, most = 8LL * ctx->sm_count;
+    launch_pdl(logit_cap_kernel, dim3((unsigned)(want < most ? want : most)), dim3(256), st, z, cap, n);
+    ctx->launches++;
+    return check_cuda(ctx, cudaGetLastError(), "logit cap launch");
 }
 
 }  // namespace nnq

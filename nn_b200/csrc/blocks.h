@@ -25,19 +25,41 @@ struct RowSpan {
     const int *state;   // decode step: state[1] is the position (n = 1)
 };
 
-// block_norm.cu: h <- h + delta (or the embedding rows), xn <- RMSNorm(h) * w
+// hashed table of token pairs added to the embedding: row (previous * mul_prev + token * mul_cur) mod buckets, row
+// `buckets` for the first token of a sequence; rows as wide as the embedding's
+struct PairTable {
+    const __nv_bfloat16 *table;   // NULL: none
+    long long mul_prev, mul_cur, buckets;
+};
+
+// what a product reads: x itself, RMSNorm(x) * w or the layer norm (x - mean) / sd * w + b
+enum NormKind { kNormNone = 0, kNormRms = 1, kNormLayer = 2 };
+struct InNorm {
+    int kind;
+    const float *w, *b;
+};
+
+// block_norm.cu: h <- alpha h + delta, or the embedding rows; with post_w given h <- layer norm of that; xn <- in(h)
 struct NormRows {
     float *h;
     const float *delta;
-    const __nv_bfloat16 *embed;   // NULL: h + delta
-    const float *w;
+    int delta_ld;
+    float alpha;
+    const float *post_w, *post_b;
+    const __nv_bfloat16 *embed;   // NULL: alpha h + delta
+    PairTable pairs;
+    InNorm in;
     float eps;
     void *xn;
     int act_dt, hidden, embed_ld, xn_ld;
 };
 nnq_status launch_norm_step(nnq_ctx *ctx, const NormRows &a, const int *state, cudaStream_t st);   // one row, token in state[0]
-// n rows of tokens[]; with `rows` given, n rows picked by index (h is left as it is)
-nnq_status launch_norm_rows(nnq_ctx *ctx, const NormRows &a, int n, const int *tokens, const int *rows, cudaStream_t st);
+// n rows of tokens[] at positions pos0 .. (tokens[-1]: the token in front of them); with `rows` given, n rows picked by
+// index (h is left as it is)
+nnq_status launch_norm_rows(nnq_ctx *ctx, const NormRows &a, int n, const int *tokens, int pos0, const int *rows, cudaStream_t st);
+// act[row, j] = f(proj[row, 2 j]) * proj[row, 2 j + 1] for j < ffn, zeros up to act_ld (a multiple of 4); kind: nnq_gate_act
+nnq_status launch_pair_act(nnq_ctx *ctx, const float *proj, int proj_ld, int n, int ffn, int kind, void *act, int act_dt, int act_ld, cudaStream_t st);
+nnq_status launch_logit_cap(nnq_ctx *ctx, float *z, float cap, long long n, cudaStream_t st);   // z <- cap tanh(z / cap)
 
 // silu(gate) * up of the feed-forward, and zeros in the columns of act that belong to neither part
 struct FfnPart {
@@ -111,6 +133,51 @@ struct Recurrence {
 
 nnq_status launch_rec_rows(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st);
 nnq_status launch_rec_step(nnq_ctx *ctx, const Recurrence &r, cudaStream_t st);
+
+// Attention through a latent: per token one normed vector c (kv_rank) and one rotated key part r (rot), kept in a ring;
+// a head's key is [W_uk,h c | r], its value W_uv,h c. ukv holds the heads' W_uk rows (dim_ld apart), then their W_uv rows
+// (vdim_ld apart), zero rows between. A block of rows expands the keys and values its window reaches (kv = latents ukv^T);
+// a decode step moves W_uk to the query and W_uv behind the weighted sum, and reads the latents themselves.
+struct LatentAttn {
+    RowSpan span;
+    int heads, dim, rot, vdim, dim_ld, vdim_ld;   // dim: unrotated part; _ld: rounded up to 64
+    int q_rank, q_ld, kv_rank, kv_ld, rot_ld;     // _ld: rounded up to 64
+    const float *proj;              // rows of the input product
+    int in_cols, c_q, c_kv;         // its columns; c_kv < 0: the ring belongs to an earlier block
+    float eps;
+    const float *q_norm, *kv_norm;
+    const float *cosv, *sinv;       // [max_seq, rot / 2]
+    int act_dt;                     // of cq, the rings, kv and out
+    void *cq;                       // [rows, q_ld]
+    void *ring_c, *ring_r;          // [cap, kv_ld], [cap, rot_ld], position p at slot p % cap
+    int cap;
+    const float *q;                 // [rows, heads * (dim + rot)] as projected
+    float scale;
+    int window;
+    void *out;                      // [rows, out_ld], heads * vdim columns and zeros
+    int out_ld;
+    // block of rows: keys first .. pos0 + n - 1 in a row
+    int first, keys;
+    void *lin_c, *lin_r;            // [keys, kv_ld], [keys, rot_ld] (the ring itself where nothing wraps: linear = 0)
+    int linear;                     // copy the ring's older positions
+    const void *kv;                 // [keys, heads * (dim_ld + vdim_ld)]
+    float *qrot, *kfull, *vfull;    // rows on the general attention kernels: f32 copies with the shared part per head
+    // decode step
+    const __nv_bfloat16 *ukv;
+    float *qlat;                    // [heads, kv_ld + rot_ld]
+    int ranges, keys_max;
+    float *part;                    // [ranges, heads, kv_ld + 4]: maximum, sum, -, -, weighted latents
+};
+
+enum { kLatentQueries = 1, kLatentKeys = 2 };
+// the normed query latent (cq), the new latents into the ring (and lin), the older ones into lin; n rows
+nnq_status launch_latent_prep(nnq_ctx *ctx, const LatentAttn &a, int parts, cudaStream_t st);
+nnq_status launch_latent_rows(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st);   // attention of a block of rows (n > 1 or not)
+bool latent_tc_supported(int act_dt, int dim, int rot, int vdim);                    // attn_latent_tc.cu: on the tensor cores
+nnq_status launch_latent_tc(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st);
+nnq_status launch_latent_step(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st);   // one row, appends its latent
+bool latent_step_supported(int act_dt, int kv_ld, int rot_ld);
+int latent_step_ranges(int sm_count, int heads, int window, int max_seq, int act_dt);
 
 // linear_f32.cu: y = x W^T (+ bias) with f32 products and sums for unquantized weights, any row count
 nnq_status launch_linear_f32(nnq_ctx *ctx, const LinearArgs &a, cudaStream_t stream);

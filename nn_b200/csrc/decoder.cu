@@ -25,6 +25,7 @@
 #include "comm.cuh"
 #include "decoder_common.cuh"
 #include "gemm_tc.h"
+#include "moe.h"
 
 namespace nnq {
 nnq_status comm_view(nnq_comm *c, CommView *out);   // comm.cu
@@ -45,7 +46,7 @@ struct nnq_decoder {
     float *d_h, *d_delta, *d_q, *d_k, *d_v, *d_qrot, *d_g, *d_u, *d_logits, *d_part;
     unsigned int *d_arrived;   // per kv head: attention CTAs that have published their record
     void *d_xn, *d_attn, *d_mid;   // activations fed to the products (f32 or bf16)
-    int *d_state;               // [0] token, [1] position, [2] steps taken; then the argmax scratch
+    int *d_state;               // [0] token, [1] position, [2] steps taken, [3] context full, [4] token before [0]; then the argmax scratch
     int *d_tokens;              // generated tokens, [max_seq]
     int act_dt;
     int ready;                  // bit set of what has been supplied
@@ -75,10 +76,20 @@ struct nnq_decoder {
         int cap, ranges;        // attention: ring capacity, key ranges of the decode kernel
         float *kcache, *vcache, *conv_ring, *rec_state;
         int mix_mode;
+        float *norm_bias;       // post_norm
+        const nnq_weight *uq, *ukv;
+        const nnq_moe *moe;
+        float *q_norm, *kv_norm;
+        void *ring_c, *ring_r;  // latents and rotated key parts, owned by the block that forms them
     } *blocks;
     float *b_h2;                // the step's residual row alternates between d_h and this buffer
     float *b_proj, *b_q, *b_k, *b_a, *b_o, *b_vfirst;   // rows of proj; prepared q / k / decay, mixer output, first values
     void *b_act;
+    void *b_cq, *b_lin_c, *b_lin_r, *b_kv;              // latent attention: query latents, the window's latents in a row, expanded keys and values
+    float *b_q2, *b_qrot, *b_kfull, *b_vfull, *b_qlat;  // its queries; f32 copies for the general kernels; queries in the latent space
+    float *final_bias;          // layer norm in front of the head
+    float logit_cap;            // 0: none
+    nnq::PairTable pairs;
 };
 
 namespace nnq {
@@ -90,6 +101,7 @@ constexpr int kAttnWarps = 4;
 // the Qwen3-8B shape).
 constexpr int kPrefillRows = 1024;
 constexpr int kArgmaxBlocks = 128;
+constexpr int kStateWords = 8;    // token, position, steps, context full, previous token
 constexpr int kWantRows = 64;     // rows of logits formed together
 
 // h = embedding row of the current token (first layer), or h += delta; xn = RMSNorm(h) * w.
@@ -355,13 +367,17 @@ __device__ __forceinline__ void arg_better(float &bv, int &bi, float v, int i) {
 }
 
 __global__ void __launch_bounds__(256)
-dec_argmax_stage1_kernel(const float *__restrict__ logits, int n, float *__restrict__ bv_out, int *__restrict__ bi_out) {
+dec_argmax_stage1_kernel(float *__restrict__ logits, int n, float cap, float *__restrict__ bv_out, int *__restrict__ bi_out) {
     pdl_prologue();
     __shared__ float sv[8];
     __shared__ int si[8];
     float bv = -INFINITY;
     int bi = -1;
-    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) arg_better(bv, bi, logits[i], i);
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
+        float z = logits[i];
+        if (cap > 0.0f) logits[i] = z = cap * tanhf(z / cap);
+        arg_better(bv, bi, z, i);
+    }
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) {
         const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, off);
@@ -387,6 +403,7 @@ __device__ __forceinline__ void dec_commit_token(int bi, int *state, int *tokens
     if (bi < 0) bi = 0;   // all NaN: the reference returns index 0
     const int pos = state[1];
     tokens[pos] = bi;
+    state[4] = state[0];   // the token in front of the next one
     state[0] = bi;
     if (pos + 1 < max_seq) state[1] = pos + 1;
     else state[3] = 1;
@@ -675,7 +692,7 @@ nnq_status nnq_decoder_create(nnq_ctx *ctx, const nnq_decoder_config *cfg, nnq_d
     if (s == NNQ_OK) s = dev_alloc(ctx, &d->d_xn, (size_t)c.hidden * es, "decoder buffer");
     if (s == NNQ_OK) s = dev_alloc(ctx, &d->d_attn, (size_t)qdim * es, "decoder buffer");
     if (s == NNQ_OK) s = dev_alloc(ctx, &d->d_mid, (size_t)lffn * es, "decoder buffer");
-    if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->d_state, (4 + 2 * kArgmaxBlocks) * 4, "decoder state");
+    if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->d_state, (kStateWords + 2 * kArgmaxBlocks) * 4, "decoder state");
     if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->d_tokens, (size_t)c.max_seq * 4, "token log");
     if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->d_final_norm, (size_t)c.hidden * 4, "final norm");
     for (int l = 0; l < c.n_layers && s == NNQ_OK; l++) {
@@ -769,7 +786,20 @@ nnq_status nnq_decoder_set_head(nnq_decoder *d, const void *embed_bf16_dev, cons
 // ---- block decoders ----
 
 static nnq_status check_block(nnq_ctx *ctx, int l, const nnq_block_config &b) {
-    if (b.mixer != NNQ_MIXER_ATTENTION && b.mixer != NNQ_MIXER_RECURRENT) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: unknown mixer %d", l, b.mixer);
+    if (b.mixer < NNQ_MIXER_ATTENTION || b.mixer > NNQ_MIXER_NONE) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: unknown mixer %d", l, b.mixer);
+    if ((b.mixer == NNQ_MIXER_LATENT || b.mixer == NNQ_MIXER_NONE) && !b.post_norm) return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: this mixer takes post_norm", l);
+    if (b.ffn_act != NNQ_ACT_SILU && b.ffn_act != NNQ_ACT_GELU_TANH) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: unknown activation %d", l, b.ffn_act);
+    if (b.mixer == NNQ_MIXER_NONE) {
+        if (b.experts < 0 || b.ffn < 0 || (b.experts > 0) == (b.ffn > 0)) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: a feed-forward or a mixture of experts", l);
+        return NNQ_OK;
+    }
+    if (b.experts || b.ffn_act != NNQ_ACT_SILU) return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: experts and other activations than silu stand in blocks without a mixer", l);
+    if (b.mixer == NNQ_MIXER_LATENT) {
+        if (b.heads < 1 || b.dim < 1 || b.vdim < 1 || b.ffn || b.q_rank < 1 || b.kv_rank < 1 || b.window < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad sizes", l);
+        if (b.rot_dims < 0 || b.rot_dims % 2 || (b.rot_dims && !(b.rot_base > 0.0))) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad rotation", l);
+        if (b.vdim > kAttnMaxDim || b.dim + b.rot_dims > 2 * kAttnMaxDim) return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: attention heads of %d + %d / %d are above %d / %d", l, b.dim, b.rot_dims, b.vdim, 2 * kAttnMaxDim, kAttnMaxDim);
+        return NNQ_OK;
+    }
     if (b.heads < 1 || b.dim < 1 || b.vdim < 1 || b.ffn < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad sizes", l);
     if (b.rot_dims < 0 || b.rot_dims % 2 || b.rot_dims > b.dim || (b.rot_dims && !(b.rot_base > 0.0)))
         return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad rotation (%d of %d dimensions)", l, b.rot_dims, b.dim);
@@ -788,6 +818,29 @@ static nnq_status check_block(nnq_ctx *ctx, int l, const nnq_block_config &b) {
 
 static nnq_block_layout layout_of(const nnq_block_config &b, int hidden) {
     nnq_block_layout y = {};
+    y.in_k = round_up(hidden, 64);   // one k step of the tensor-core products
+    y.ffn_step = 1;
+    if (b.mixer == NNQ_MIXER_LATENT) {
+        y.q = 0;
+        y.k = b.kv_from < 0 ? round_up(b.q_rank, 8) : -1;
+        y.v = y.g = y.a1 = y.gate = y.up = -1;
+        y.in_cols = round_up(b.q_rank, 8) + (b.kv_from < 0 ? round_up(b.kv_rank + b.rot_dims, 8) : 0);
+        y.q_ld = round_up(b.q_rank, 64);
+        y.kv_ld = round_up(b.kv_rank, 64);
+        y.dim_ld = round_up(b.dim, 64);
+        y.vdim_ld = round_up(b.vdim, 64);
+        y.ffn_col = y.out_k = round_up(b.heads * b.vdim, 64);
+        return y;
+    }
+    if (b.mixer == NNQ_MIXER_NONE) {
+        y.q = y.k = y.v = y.g = y.a1 = -1;
+        y.gate = 0;
+        y.up = 1;
+        y.ffn_step = 2;
+        y.in_cols = round_up(2 * b.ffn, 8);
+        y.out_k = round_up(b.ffn, 64);
+        return y;
+    }
     const bool attn = b.mixer == NNQ_MIXER_ATTENTION;
     const int kvh = attn ? b.kv_heads : b.heads;
     int at = 0;
@@ -805,7 +858,6 @@ static nnq_block_layout layout_of(const nnq_block_config &b, int hidden) {
     y.gate = take(b.ffn);
     y.up = take(b.ffn);
     y.in_cols = at;
-    y.in_k = round_up(hidden, 64);   // one k step of the tensor-core products
     y.ffn_col = round_up(b.heads * b.vdim, 8);
     // (a gap in front of the feed-forward's columns is cleared together with them: there are some then)
     y.out_k = round_up(y.ffn_col + (b.ffn > 0 || y.ffn_col == b.heads * b.vdim ? b.ffn : 8), 64);
@@ -824,6 +876,11 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
     int first_mix = -1;
     for (int l = 0; l < c.n_layers; l++) {
         if ((s = check_block(ctx, l, blocks[l])) != NNQ_OK) return s;
+        if (blocks[l].mixer == NNQ_MIXER_LATENT && blocks[l].kv_from >= 0) {
+            const nnq_block_config &b = blocks[l], *o = b.kv_from < l ? &blocks[b.kv_from] : nullptr;
+            if (!o || o->mixer != NNQ_MIXER_LATENT || o->kv_from >= 0 || o->kv_rank != b.kv_rank || o->rot_dims != b.rot_dims || (b.rot_dims && o->rot_base != b.rot_base))
+                return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d cannot read the latents of block %d", l, b.kv_from);
+        }
         if (blocks[l].mixer != NNQ_MIXER_ATTENTION || !blocks[l].value_mix) continue;
         if (first_mix < 0) first_mix = l;
         else if (blocks[l].kv_heads * blocks[l].vdim != blocks[first_mix].kv_heads * blocks[first_mix].vdim)
@@ -848,6 +905,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
     const int rows = d->pf_rows = want_rows < c.max_seq ? want_rows : c.max_seq;
     const size_t R = rows, es = c.act_dtype == NNQ_F32 ? 4 : 2;
     size_t proj = 0, act = 0, q = 0, k = 0, o = 0, vf = 0, part = 0, counters = 1;
+    size_t cq = 0, lin_c = 0, lin_r = 0, kv = 0, q2 = 0, qrot = 0, kfull = 0, vfull = 0, qlat = 0;
     auto alloc = [&](void *pp, size_t bytes, const char *what) {
         if (s == NNQ_OK) s = dev_alloc(ctx, (void **)pp, bytes, what);
     };
@@ -860,6 +918,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
         most(proj, B.lay.in_cols);
         most(act, B.lay.out_k);
         alloc(&B.norm, (size_t)c.hidden * 4, "norm weight");
+        if (b.post_norm) alloc(&B.norm_bias, (size_t)c.hidden * 4, "norm bias");
         if (b.mixer == NNQ_MIXER_ATTENTION) {
             B.dim_ld = round_up(b.dim, 4);
             B.vdim_ld = round_up(b.vdim, 4);
@@ -878,7 +937,43 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
             if (b.value_mix) most(vf, (size_t)b.kv_heads * b.vdim);
             most(part, attn_step_part_floats(b.heads, b.kv_heads, B.vdim_ld, B.ranges));
             most(counters, attn_step_counters(b.heads, b.kv_heads));
-        } else {
+        } else if (b.mixer == NNQ_MIXER_LATENT) {
+            const nnq_block_layout &y = B.lay;
+            const int rot_ld = round_up(b.rot_dims, 64), window = b.window > 0 ? b.window : c.max_seq;
+            if (!latent_step_supported(c.act_dtype, y.kv_ld, rot_ld)) s = fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: a latent of %d + %d is too wide", l, b.kv_rank, b.rot_dims);
+            alloc(&B.q_norm, (size_t)b.q_rank * 4, "norm weight");
+            if (b.kv_from < 0) {
+                alloc(&B.kv_norm, (size_t)b.kv_rank * 4, "norm weight");
+                long long widest = window;   // the ring serves every block that reads it
+                for (int j = l + 1; j < c.n_layers; j++)
+                    if (blocks[j].mixer == NNQ_MIXER_LATENT && blocks[j].kv_from == l && (blocks[j].window > 0 ? blocks[j].window : c.max_seq) > widest)
+                        widest = blocks[j].window > 0 ? blocks[j].window : c.max_seq;
+                B.cap = widest - 1 + rows < c.max_seq ? (int)widest - 1 + rows : c.max_seq;
+                alloc(&B.ring_c, (size_t)B.cap * y.kv_ld * es, "latents");
+                alloc(&B.ring_r, (size_t)B.cap * rot_ld * es, "rotated key parts");
+            } else {
+                B.cap = d->blocks[b.kv_from].cap;
+                B.ring_c = d->blocks[b.kv_from].ring_c;
+                B.ring_r = d->blocks[b.kv_from].ring_r;
+            }
+            B.ranges = latent_step_ranges(ctx->sm_count, b.heads, window, c.max_seq, c.act_dtype);
+            const size_t keys = (long long)window - 1 + rows < c.max_seq ? window - 1 + rows : c.max_seq;
+            most(cq, y.q_ld);
+            if (B.cap < c.max_seq) {
+                most(lin_c, keys * y.kv_ld);
+                most(lin_r, keys * rot_ld);
+            }
+            most(kv, keys * b.heads * (y.dim_ld + y.vdim_ld));
+            most(q2, (size_t)b.heads * (b.dim + b.rot_dims));
+            if (!latent_tc_supported(c.act_dtype, b.dim, b.rot_dims, b.vdim)) {
+                const size_t dl = round_up(b.dim + b.rot_dims, 4), vl = round_up(b.vdim, 4);
+                most(qrot, b.heads * dl);
+                most(kfull, keys * b.heads * dl);
+                most(vfull, keys * b.heads * vl);
+            }
+            most(qlat, (size_t)b.heads * (y.kv_ld + rot_ld));
+            most(part, (size_t)B.ranges * b.heads * (y.kv_ld + 4));
+        } else if (b.mixer == NNQ_MIXER_RECURRENT) {
             B.dim_ld = b.dim <= 64 ? 64 : round_up(b.dim, 128);
             alloc(&B.rec_state, (size_t)b.heads * b.dim * b.vdim * 4, "recurrent state");
             if (b.decay_rank > 0) {
@@ -922,20 +1017,31 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
             }
         }
     }
+    if (s == NNQ_OK) {
+        alloc(&d->b_cq, R * cq * es, "row buffer");
+        alloc(&d->b_lin_c, lin_c * es, "row buffer");
+        alloc(&d->b_lin_r, lin_r * es, "row buffer");
+        alloc(&d->b_kv, kv * es, "expanded keys and values");
+        alloc(&d->b_q2, R * q2 * 4, "row buffer");
+        alloc(&d->b_qrot, R * qrot * 4, "row buffer");
+        alloc(&d->b_kfull, kfull * 4, "expanded keys");
+        alloc(&d->b_vfull, vfull * 4, "expanded values");
+        alloc(&d->b_qlat, qlat * 4, "row buffer");
+    }
     alloc(&d->d_h, (size_t)c.hidden * 4, "decoder buffer");
     alloc(&d->b_h2, (size_t)c.hidden * 4, "decoder buffer");
-    alloc(&d->d_delta, (size_t)c.hidden * 4, "decoder buffer");
+    alloc(&d->d_delta, (size_t)d->xn_ld * 4, "decoder buffer");
     alloc(&d->d_xn, (size_t)d->xn_ld * es, "decoder buffer");
     alloc(&d->d_logits, (size_t)c.vocab * 4, "decoder buffer");
     alloc(&d->d_final_norm, (size_t)c.hidden * 4, "final norm");
-    alloc(&d->d_state, (4 + 2 * kArgmaxBlocks) * 4, "decoder state");
+    alloc(&d->d_state, (kStateWords + 2 * kArgmaxBlocks) * 4, "decoder state");
     alloc(&d->d_tokens, (size_t)c.max_seq * 4, "token log");
     alloc(&d->d_part, part * 4, "attention partials");
     alloc(&d->d_arrived, counters * 4, "attention arrival counters");
     alloc(&d->pf_h, R * c.hidden * 4, "row buffer");
-    alloc(&d->pf_delta, R * c.hidden * 4, "row buffer");
+    alloc(&d->pf_delta, R * d->xn_ld * 4, "row buffer");   // (the experts' rows are as wide as the products' input)
     alloc(&d->pf_xn, R * d->xn_ld * es, "row buffer");
-    alloc(&d->pf_tokens, R * 4, "row buffer");
+    alloc(&d->pf_tokens, (R + 1) * 4, "row buffer");   // the token in front of a block of rows, then the block's
     alloc(&d->pf_want, R * 4, "row buffer");
     alloc(&d->b_proj, R * proj * 4, "row buffer");
     alloc(&d->b_act, R * act * es, "row buffer");
@@ -966,10 +1072,21 @@ nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_block_weig
     if (!d->blocks || layer < 0 || layer >= c.n_layers) return fail(ctx, NNQ_ERR_INVALID_ARG, "no block %d", layer);
     nnq_decoder::Block &B = d->blocks[layer];
     const nnq_block_config &b = B.cfg;
-    if (!shape_is(w->in, B.lay.in_cols, B.lay.in_k) || !shape_is(w->out, c.hidden, B.lay.out_k))
+    if (b.experts) {
+        if (!w->moe || w->moe->hidden != B.lay.in_k || w->moe->n_experts != b.experts || w->moe->fmt != NNQ_BF16_DENSE)
+            return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "block %d takes %d bf16 experts of width %d", layer, b.experts, B.lay.in_k);
+    } else if (!shape_is(w->in, B.lay.in_cols, B.lay.in_k) || !shape_is(w->out, c.hidden, B.lay.out_k))
         return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "products of block %d must be [%d, %d] and [%d, %d]", layer, B.lay.in_cols, B.lay.in_k, c.hidden, B.lay.out_k);
     if (!w->norm || (B.conv && !w->conv) || (B.a2t && (!w->decay_w || !w->decay_b)) || (B.decay && !w->decay))
         return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d lacks a tensor", layer);
+    if (b.post_norm && !w->norm_bias) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d lacks a tensor", layer);
+    if (b.mixer == NNQ_MIXER_LATENT) {
+        if (!w->q_norm || (B.kv_norm && !w->kv_norm)) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d lacks a tensor", layer);
+        if (!shape_is(w->uq, (int64_t)b.heads * (b.dim + b.rot_dims), B.lay.q_ld) || !shape_is(w->ukv, (int64_t)b.heads * (B.lay.dim_ld + B.lay.vdim_ld), B.lay.kv_ld) ||
+            w->ukv->fmt != NNQ_BF16_DENSE)
+            return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "latent products of block %d must be [%d, %d] and (bf16) [%d, %d]", layer, b.heads * (b.dim + b.rot_dims), B.lay.q_ld,
+                        b.heads * (B.lay.dim_ld + B.lay.vdim_ld), B.lay.kv_ld);
+    }
     nnq_status s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
     auto copy = [&](float *dst, const float *src, size_t n, const char *what) {
         if (s == NNQ_OK) s = check_cuda(ctx, cudaMemcpy(dst, src, n * 4, cudaMemcpyDefault), what);
@@ -980,6 +1097,10 @@ nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_block_weig
         copy(*dst, src, n, what);
     };
     copy(B.norm, w->norm, c.hidden, "norm weight");
+    if (b.post_norm) copy(B.norm_bias, w->norm_bias, c.hidden, "norm bias");
+    if (B.q_norm) copy(B.q_norm, w->q_norm, b.q_rank, "norm weight");
+    if (B.kv_norm) copy(B.kv_norm, w->kv_norm, b.kv_rank, "norm weight");
+    if (b.experts && s == NNQ_OK) s = moe_reserve(ctx, w->moe, d->pf_rows);
     optional(&B.bias_in, w->bias_in, B.lay.in_cols, "bias");
     optional(&B.bias_out, w->bias_out, c.hidden, "bias");
     optional(&B.head_norm, b.mixer == NNQ_MIXER_RECURRENT ? w->head_norm : nullptr, b.vdim, "head norm weight");
@@ -1002,6 +1123,9 @@ nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_block_weig
     if (s == NNQ_OK) {
         B.in = w->in;
         B.out = w->out;
+        B.uq = w->uq;
+        B.ukv = w->ukv;
+        B.moe = w->moe;
     }
     return s;
 }
@@ -1020,6 +1144,25 @@ nnq_status nnq_decoder_set_head_weights(nnq_decoder *d, const nnq_weight *embed,
     d->lm_head = lm_head;
     d->ready = 1;
     return NNQ_OK;
+}
+
+nnq_status nnq_decoder_set_head_options(nnq_decoder *d, const nnq_head_options *o) {
+    if (!d || !o) return NNQ_ERR_INVALID_ARG;
+    nnq_ctx *ctx = d->ctx;
+    if (!d->blocks) return fail(ctx, NNQ_ERR_INVALID_ARG, "not a block decoder");
+    if (!(o->logit_cap >= 0.0f)) return fail(ctx, NNQ_ERR_INVALID_ARG, "bad logit cap");
+    if (o->pair_table && (o->pair_buckets < 1 || o->pair_buckets >= (1ll << 31) || o->pair_mul_prev < 0 || o->pair_mul_cur < 0 || o->pair_mul_prev >= (1ll << 31) ||
+                          o->pair_mul_cur >= (1ll << 31) || !shape_is(o->pair_table, o->pair_buckets + 1, d->embed_ld) || o->pair_table->fmt != NNQ_BF16_DENSE))
+        return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "the pair table must be bf16 [buckets + 1, %d]", d->embed_ld);
+    nnq_status s = check_cuda(ctx, cudaSetDevice(ctx->device), "cudaSetDevice");
+    if (s == NNQ_OK && o->final_norm_bias) {
+        if (!d->final_bias) s = dev_alloc(ctx, (void **)&d->final_bias, (size_t)d->cfg.hidden * 4, "final norm bias");
+        if (s == NNQ_OK) s = check_cuda(ctx, cudaMemcpy(d->final_bias, o->final_norm_bias, (size_t)d->cfg.hidden * 4, cudaMemcpyDefault), "final norm bias");
+    }
+    d->logit_cap = o->logit_cap;
+    d->pairs = PairTable{};
+    if (o->pair_table) d->pairs = {(const __nv_bfloat16 *)o->pair_table->d_raw, o->pair_mul_prev, o->pair_mul_cur, o->pair_buckets};
+    return s;
 }
 
 nnq_status nnq_decoder_set_comm(nnq_decoder *d, nnq_comm *comm) {
@@ -1057,9 +1200,9 @@ nnq_status nnq_decoder_buffers(nnq_decoder *d, float **k_cache, float **v_cache,
 }
 
 // A product of the decoder: blocks with f32 activations keep f32 operands throughout.
-static nnq_status product(nnq_decoder *d, const nnq_weight *w, const void *x, int64_t m, const float *bias, float *y, cudaStream_t st) {
-    if (!d->blocks || d->act_dt != NNQ_F32) return nnq_linear(d->ctx, w, x, (nnq_dtype)d->act_dt, m, bias, y, NNQ_F32, st);
-    LinearArgs a = {w->d_raw, w->d_scales, x, bias, y, m, w->n, w->k, w->fmt, NNQ_F32, NNQ_F32};
+static nnq_status product(nnq_decoder *d, const nnq_weight *w, const void *x, int64_t m, const float *bias, void *y, cudaStream_t st, int y_dt = NNQ_F32) {
+    if (!d->blocks || d->act_dt != NNQ_F32) return nnq_linear(d->ctx, w, x, (nnq_dtype)d->act_dt, m, bias, y, (nnq_dtype)y_dt, st);
+    LinearArgs a = {w->d_raw, w->d_scales, x, bias, y, m, w->n, w->k, w->fmt, NNQ_F32, y_dt};
     return launch_linear_f32(d->ctx, a, st);
 }
 
@@ -1068,10 +1211,10 @@ static nnq_status product(nnq_decoder *d, const nnq_weight *w, const void *x, in
 static nnq_status launch_argmax(nnq_decoder *d, bool vocab_parallel, const CommView &cv, cudaStream_t st) {
     nnq_ctx *ctx = d->ctx;
     const nnq_decoder_config &c = d->cfg;
-    const float *logits = d->d_logits + d->head_row0;
-    float *bv = reinterpret_cast<float *>(d->d_state + 4);
-    int *bi = d->d_state + 4 + kArgmaxBlocks;
-    launch_pdl(dec_argmax_stage1_kernel, dim3(kArgmaxBlocks), dim3(256), st, logits, d->head_rows, bv, bi);
+    float *logits = d->d_logits + d->head_row0;
+    float *bv = reinterpret_cast<float *>(d->d_state + kStateWords);
+    int *bi = d->d_state + kStateWords + kArgmaxBlocks;
+    launch_pdl(dec_argmax_stage1_kernel, dim3(kArgmaxBlocks), dim3(256), st, logits, d->head_rows, d->logit_cap, bv, bi);
     if (vocab_parallel)
         launch_pdl(dec_argmax_exchange_kernel, dim3(1), dim3(32), st, bv, bi, kArgmaxBlocks, d->head_row0, cv.peer_table, cv.rank, cv.world,
                    cv.slot_bytes, d->d_state, d->d_tokens, c.max_seq, ctx->d_status);
@@ -1119,20 +1262,102 @@ static nnq_status ready_to_run(const nnq_decoder *d) {
     if (!d->ready) return fail(ctx, NNQ_ERR_INVALID_ARG, "decoder head has not been set");
     if (c.tp_world > 1 && !d->comm) return fail(ctx, NNQ_ERR_INVALID_ARG, "communicator has not been set");
     for (int l = 0; l < c.n_layers; l++)
-        if (d->blocks ? !d->blocks[l].in : !d->layers[l].q) return fail(ctx, NNQ_ERR_INVALID_ARG, "layer %d has not been set", l);
+        if (d->blocks ? !d->blocks[l].in && !d->blocks[l].moe : !d->layers[l].q) return fail(ctx, NNQ_ERR_INVALID_ARG, "layer %d has not been set", l);
     return NNQ_OK;
 }
 
+// What the row buffers hold in front of block l (l = n_layers: in front of the head): the last block's sum has not been
+// formed yet. h: residual rows, delta: that block's output rows.
+static NormRows pending_rows(const nnq_decoder *d, int l, float *h, const float *delta) {
+    const nnq_decoder_config &c = d->cfg;
+    NormRows r = {};
+    r.h = h;
+    r.delta = delta;
+    r.alpha = 1.0f;
+    r.delta_ld = c.hidden;
+    if (l == 0) {
+        r.embed = (const __nv_bfloat16 *)d->d_embed;
+        r.pairs = d->pairs;
+    } else if (d->blocks) {
+        const nnq_decoder::Block &P = d->blocks[l - 1];
+        if (P.moe) r.delta_ld = d->xn_ld;
+        if (P.cfg.post_norm) {
+            r.alpha = P.cfg.alpha;
+            r.post_w = P.norm;
+            r.post_b = P.norm_bias;
+        }
+    }
+    if (l == c.n_layers) r.in = {d->final_bias ? kNormLayer : kNormRms, d->d_final_norm, d->final_bias};
+    else if (d->blocks && !d->blocks[l].cfg.post_norm) r.in = {kNormRms, d->blocks[l].norm, nullptr};
+    r.eps = c.rms_eps;
+    r.act_dt = d->act_dt;
+    r.hidden = c.hidden;
+    r.embed_ld = d->embed_ld;
+    r.xn_ld = d->xn_ld;
+    return r;
+}
+
+static bool fused_steps(const nnq_decoder *d) { return d->act_dt == NNQ_BF16 && d->ctx->path == NNQ_PATH_AUTO; }
+
 // The mixer, the feed-forward activation and the output product of block l for n rows: b_proj -> delta. `state`
-// given: a decode step (n = 1, position in state[1]), else rows from position pos0.
-static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *state, float *delta, cudaStream_t st) {
+// given: a decode step (n = 1, position in state[1]), else rows from position pos0. activated: b_act holds the
+// feed-forward activation already.
+static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *state, bool activated, float *delta, cudaStream_t st) {
     nnq_ctx *ctx = d->ctx;
     const nnq_decoder::Block &B = d->blocks[l];
     const nnq_block_config &k = B.cfg;
     nnq_status s;
     const RowSpan span = {n, pos0, state};
     const FfnPart ffn = {d->b_proj, B.lay.in_cols, B.lay.gate, B.lay.up, k.ffn, d->b_act, d->act_dt, B.lay.out_k, k.heads * k.vdim, B.lay.ffn_col};
-    if (k.mixer == NNQ_MIXER_ATTENTION) {
+    if (k.mixer == NNQ_MIXER_NONE) {
+        if (!activated && (s = launch_pair_act(ctx, d->b_proj, B.lay.in_cols, n, k.ffn, k.ffn_act, d->b_act, d->act_dt, B.lay.out_k, st)) != NNQ_OK) return s;
+    } else if (k.mixer == NNQ_MIXER_LATENT) {
+        LatentAttn a = {};
+        a.span = span;
+        a.heads = k.heads; a.dim = k.dim; a.rot = k.rot_dims; a.vdim = k.vdim; a.dim_ld = B.lay.dim_ld; a.vdim_ld = B.lay.vdim_ld;
+        a.q_rank = k.q_rank; a.q_ld = B.lay.q_ld; a.kv_rank = k.kv_rank; a.kv_ld = B.lay.kv_ld; a.rot_ld = round_up(k.rot_dims, 64);
+        a.proj = d->b_proj; a.in_cols = B.lay.in_cols; a.c_q = B.lay.q; a.c_kv = B.lay.k;
+        a.eps = d->cfg.rms_eps; a.q_norm = B.q_norm; a.kv_norm = B.kv_norm;
+        a.cosv = B.cosv; a.sinv = B.sinv;
+        a.act_dt = d->act_dt;
+        a.cq = d->b_cq; a.ring_c = B.ring_c; a.ring_r = B.ring_r; a.cap = B.cap;
+        a.q = d->b_q2;
+        a.scale = k.scale; a.window = k.window > 0 ? k.window : (1 << 30);
+        a.out = d->b_act; a.out_ld = B.lay.out_k;
+        a.ukv = (const __nv_bfloat16 *)B.ukv->d_raw;
+        if (state) {
+            a.qlat = d->b_qlat; a.ranges = B.ranges; a.part = d->d_part;
+            a.keys_max = k.window > 0 && k.window < d->cfg.max_seq ? k.window : d->cfg.max_seq;
+            if (fused_steps(d) && dense_gemv_norm_supported(B.uq, k.q_rank)) {
+                // the query latent's norm in the prologue of the product that reads it
+                const TcArgs t = {B.uq->d_raw, B.uq->d_scales, nullptr, nullptr, d->b_q2, 1, B.uq->n, B.uq->k, B.uq->fmt, NNQ_BF16, NNQ_F32};
+                GemvNorm g = {};
+                g.h_in = d->b_proj + B.lay.q;
+                g.alpha = 1.0f;
+                g.in = {kNormRms, B.q_norm, nullptr};
+                g.eps = d->cfg.rms_eps;
+                g.hidden = k.q_rank;
+                s = launch_dense_gemv_norm(ctx, t, g, 0, 0, st);
+            } else {
+                s = launch_latent_prep(ctx, a, kLatentQueries, st);
+                if (s == NNQ_OK) s = product(d, B.uq, d->b_cq, 1, nullptr, d->b_q2, st);
+            }
+            if (s != NNQ_OK || (s = launch_latent_step(ctx, a, st)) != NNQ_OK) return s;
+        } else {
+            const size_t es = d->act_dt == NNQ_F32 ? 4 : 2;
+            a.first = k.window > 0 && pos0 - k.window + 1 > 0 ? pos0 - k.window + 1 : 0;
+            a.keys = pos0 + n - a.first;
+            a.linear = a.cap < d->cfg.max_seq;   // a ring that can wrap
+            a.lin_c = a.linear ? d->b_lin_c : (char *)a.ring_c + (size_t)a.first * a.kv_ld * es;
+            a.lin_r = a.linear ? d->b_lin_r : (char *)a.ring_r + (size_t)a.first * a.rot_ld * es;
+            a.kv = d->b_kv;
+            a.qrot = d->b_qrot; a.kfull = d->b_kfull; a.vfull = d->b_vfull;
+            s = launch_latent_prep(ctx, a, kLatentQueries | kLatentKeys, st);
+            if (s == NNQ_OK) s = product(d, B.uq, d->b_cq, n, nullptr, d->b_q2, st);
+            if (s == NNQ_OK) s = product(d, B.ukv, a.lin_c, a.keys, nullptr, d->b_kv, st, d->act_dt);
+            if (s != NNQ_OK || (s = launch_latent_rows(ctx, a, st)) != NNQ_OK) return s;
+        }
+    } else if (k.mixer == NNQ_MIXER_ATTENTION) {
         WindowAttn a = {};
         a.span = span;
         a.ffn = ffn;
@@ -1169,21 +1394,29 @@ static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *s
     return product(d, B.out, d->b_act, n, B.bias_out, delta, st);
 }
 
-// y = RMSNorm(residual) * norm times w^T for the step's row. The residual row is h + delta (the first block: the
-// embedding row); where the norm is part of the product kernel the sum goes to the other of two buffers.
-static nnq_status step_norm_product(nnq_decoder *d, const float *norm, bool embed, const nnq_weight *w, const float *bias, float *y, cudaStream_t st) {
+// y = what block l (l = n_layers: the head) reads times w^T for the step's row; where the residual update and the norm
+// are part of the product kernel the new residual row goes to the other of two buffers. pair_act: as in
+// launch_dense_gemv_norm; *activated tells whether y holds the activation.
+static nnq_status step_norm_product(nnq_decoder *d, int l, const nnq_weight *w, const float *bias, float *y, int pair_act, int y_ld, void *act, bool *activated,
+                                    cudaStream_t st) {
     const nnq_decoder_config &c = d->cfg;
-    const __nv_bfloat16 *table = embed ? (const __nv_bfloat16 *)d->d_embed : nullptr;
-    if (d->act_dt == NNQ_BF16 && d->ctx->path == NNQ_PATH_AUTO && dense_gemv_norm_supported(w, c.hidden)) {
-        const TcArgs a = {w->d_raw, w->d_scales, nullptr, bias, y, 1, w->n, w->k, w->fmt, NNQ_BF16, NNQ_F32};
-        const GemvNorm g = {d->d_h, d->d_delta, d->b_h2, table, d->embed_ld, d->d_state, norm, c.rms_eps, c.hidden, 0};
-        nnq_status s = launch_dense_gemv_norm(d->ctx, a, g, st);
+    NormRows r = pending_rows(d, l, d->d_h, d->d_delta);
+    *activated = false;
+    if (fused_steps(d) && dense_gemv_norm_supported(w, c.hidden)) {
+        const TcArgs a = {w->d_raw, w->d_scales, nullptr, bias, pair_act ? act : y, 1, w->n, w->k, w->fmt, NNQ_BF16, NNQ_F32};
+        GemvNorm g = {};
+        g.h_in = r.h; g.delta = r.delta; g.h_out = d->b_h2; g.alpha = r.alpha;
+        g.embed = r.embed; g.pairs = r.pairs; g.embed_ld = r.embed_ld; g.state = d->d_state;
+        g.post_w = r.post_w; g.post_b = r.post_b; g.in = r.in; g.eps = r.eps; g.hidden = r.hidden;
+        nnq_status s = launch_dense_gemv_norm(d->ctx, a, g, pair_act, y_ld, st);
         float *t = d->d_h;
         d->d_h = d->b_h2;
         d->b_h2 = t;
+        *activated = pair_act > 0;
         return s;
     }
-    const nnq_status s = launch_norm_step(d->ctx, {d->d_h, d->d_delta, table, norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld}, d->d_state, st);
+    r.xn = d->d_xn;
+    const nnq_status s = launch_norm_step(d->ctx, r, d->d_state, st);
     return s == NNQ_OK ? product(d, w, d->d_xn, 1, bias, y, st) : s;
 }
 
@@ -1191,8 +1424,17 @@ static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
     nnq_status s = NNQ_OK;
     for (int l = 0; l < d->cfg.n_layers; l++) {
         const nnq_decoder::Block &B = d->blocks[l];
-        if ((s = step_norm_product(d, B.norm, l == 0, B.in, B.bias_in, d->b_proj, st)) != NNQ_OK) return s;
-        if ((s = run_block(d, l, 1, 0, d->d_state, d->d_delta, st)) != NNQ_OK) return s;
+        if (B.moe) {
+            NormRows r = pending_rows(d, l, d->d_h, d->d_delta);
+            r.xn = d->d_xn;
+            if ((s = launch_norm_step(d->ctx, r, d->d_state, st)) != NNQ_OK) return s;
+            if ((s = moe_rows(d->ctx, B.moe, d->d_xn, (nnq_dtype)d->act_dt, 1, d->act_dt == NNQ_F32, d->d_delta, st)) != NNQ_OK) return s;
+            continue;
+        }
+        bool activated = false;
+        const int pair = B.cfg.mixer == NNQ_MIXER_NONE ? 1 + B.cfg.ffn_act : 0;
+        if ((s = step_norm_product(d, l, B.in, B.bias_in, d->b_proj, pair, B.lay.out_k, d->b_act, &activated, st)) != NNQ_OK) return s;
+        if ((s = run_block(d, l, 1, 0, d->d_state, activated, d->d_delta, st)) != NNQ_OK) return s;
     }
     return NNQ_OK;
 }
@@ -1200,10 +1442,16 @@ static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
 static nnq_status rows_blocks(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
     const nnq_decoder_config &c = d->cfg;
     for (int l = 0; l < c.n_layers; l++) {
-        nnq_status s = launch_norm_rows(d->ctx, {d->pf_h, d->pf_delta, l == 0 ? (const __nv_bfloat16 *)d->d_embed : nullptr, d->blocks[l].norm, c.rms_eps,
-                                                 d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld}, n, d->pf_tokens, nullptr, st);
-        if (s == NNQ_OK) s = product(d, d->blocks[l].in, d->pf_xn, n, d->blocks[l].bias_in, d->b_proj, st);
-        if (s == NNQ_OK) s = run_block(d, l, n, pos0, nullptr, d->pf_delta, st);
+        const nnq_decoder::Block &B = d->blocks[l];
+        NormRows r = pending_rows(d, l, d->pf_h, d->pf_delta);
+        r.xn = d->pf_xn;
+        nnq_status s = launch_norm_rows(d->ctx, r, n, d->pf_tokens + 1, pos0, nullptr, st);
+        if (s == NNQ_OK && B.moe) {
+            s = moe_rows(d->ctx, B.moe, d->pf_xn, (nnq_dtype)d->act_dt, n, d->act_dt == NNQ_F32, d->pf_delta, st);
+        } else {
+            if (s == NNQ_OK) s = product(d, B.in, d->pf_xn, n, B.bias_in, d->b_proj, st);
+            if (s == NNQ_OK) s = run_block(d, l, n, pos0, nullptr, false, d->pf_delta, st);
+        }
         if (s != NNQ_OK) return s;
     }
     return NNQ_OK;
@@ -1268,7 +1516,7 @@ static nnq_status rows_qwen3(nnq_decoder *d, int n, int pos0, cudaStream_t st) {
     for (int l = 0; l < c.n_layers; l++) {
         const nnq_decoder::Layer &L = d->layers[l];
         float *kc = d->d_kcache + l * layer_cache, *vc = d->d_vcache + l * layer_cache;
-        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? embed : nullptr, d->pf_tokens, L.in_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden);
+        dec_norm_rows_kernel<<<n, 256, 0, st>>>(d->pf_h, l == 0 ? nullptr : d->pf_delta, l == 0 ? embed : nullptr, d->pf_tokens + 1, L.in_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden);
         const nnq_weight *w3[3] = {L.q, L.k, L.v};
         const void *x3[3] = {d->pf_xn, d->pf_xn, d->pf_xn};
         void *y3[3] = {d->pf_q, d->pf_k, d->pf_v};
@@ -1321,7 +1569,8 @@ nnq_status nnq_decoder_step(nnq_decoder *d, void *stream) {
     cudaStream_t st = (cudaStream_t)stream;
     if (d->blocks) {
         if ((s = step_blocks(d, st)) != NNQ_OK) return s;
-        if ((s = step_norm_product(d, d->d_final_norm, false, d->lm_head, nullptr, d->d_logits, st)) != NNQ_OK) return s;
+        bool activated = false;
+        if ((s = step_norm_product(d, c.n_layers, d->lm_head, nullptr, d->d_logits, 0, 0, nullptr, &activated, st)) != NNQ_OK) return s;
         return launch_argmax(d, vocab_parallel, cv, st);
     }
     if ((s = step_qwen3(d, st)) != NNQ_OK) return s;
@@ -1376,7 +1625,7 @@ static nnq_status row_buffers(nnq_decoder *d, int *rows_max) {
         if (s == NNQ_OK) s = dev_alloc(ctx, &d->pf_xn, R * c.hidden * es, "prompt buffer");
         if (s == NNQ_OK) s = dev_alloc(ctx, &d->pf_attn, R * qdim * es, "prompt buffer");
         if (s == NNQ_OK) s = dev_alloc(ctx, &d->pf_mid, R * lffn * es, "prompt buffer");
-        if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->pf_tokens, R * 4, "prompt buffer");
+        if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->pf_tokens, (R + 1) * 4, "prompt buffer");
         if (s == NNQ_OK) s = dev_alloc(ctx, (void **)&d->pf_want, R * 4, "prompt buffer");
         if (s != NNQ_OK) return s;
     }
@@ -1385,8 +1634,13 @@ static nnq_status row_buffers(nnq_decoder *d, int *rows_max) {
 
 // n <= rows_max tokens through the layers: afterwards pf_h + pf_delta are the rows' final residuals.
 static nnq_status run_rows(nnq_decoder *d, const int32_t *tokens_host, int n, int pos0, cudaStream_t st) {
-    nnq_status s = check_cuda(d->ctx, cudaMemcpyAsync(d->pf_tokens, tokens_host, (size_t)n * 4, cudaMemcpyHostToDevice, st), "prompt tokens");
+    nnq_status s = check_cuda(d->ctx, cudaMemcpyAsync(d->pf_tokens + 1, tokens_host, (size_t)n * 4, cudaMemcpyHostToDevice, st), "prompt tokens");
     if (s != NNQ_OK) return s;
+    if (d->blocks) {   // the token in front of the block, and what a later block or step finds as its previous token
+        s = check_cuda(d->ctx, cudaMemcpyAsync(d->pf_tokens, d->d_state + 4, 4, cudaMemcpyDeviceToDevice, st), "prompt tokens");
+        if (s == NNQ_OK) s = check_cuda(d->ctx, cudaMemcpyAsync(d->d_state + 4, d->pf_tokens + n, 4, cudaMemcpyDeviceToDevice, st), "prompt tokens");
+        if (s != NNQ_OK) return s;
+    }
     return d->blocks ? rows_blocks(d, n, pos0, st) : rows_qwen3(d, n, pos0, st);
 }
 
@@ -1410,11 +1664,12 @@ nnq_status nnq_decoder_prefill(nnq_decoder *d, const int32_t *tokens_host, int c
         if ((s = run_rows(d, tokens_host + c0, n, start_pos + c0, st)) != NNQ_OK) return s;
     }
     // the last prompt token's state: final norm, vocabulary projection, greedy successor
-    const size_t last = (size_t)(n - 1) * c.hidden;
     const int st4[4] = {tokens_host[count - 1], start_pos + count - 1, 0, 0};
     if ((s = check_cuda(ctx, cudaMemcpyAsync(d->d_state, st4, sizeof(st4), cudaMemcpyHostToDevice, st), "decoder state")) != NNQ_OK) return s;
-    s = launch_norm_step(ctx, {d->pf_h + last, d->pf_delta + last, nullptr, d->d_final_norm, c.rms_eps, d->d_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld},
-                         d->d_state, st);
+    NormRows r = pending_rows(d, c.n_layers, d->pf_h + (size_t)(n - 1) * c.hidden, d->pf_delta);
+    r.delta += (size_t)(n - 1) * r.delta_ld;
+    r.xn = d->d_xn;
+    s = launch_norm_step(ctx, r, d->d_state, st);
     if (s != NNQ_OK || (s = launch_head(d, vocab_parallel, cv, st)) != NNQ_OK) return s;
     s = check_cuda(ctx, cudaStreamSynchronize(st), "prompt pass");   // tokens_host and st4 are the caller's / the stack's
     if (s == NNQ_OK) d->host_pos = (long long)start_pos + count;
@@ -1457,9 +1712,12 @@ nnq_status nnq_decoder_extend(nnq_decoder *d, const int32_t *tokens_host, int co
                 m++;
             }
             if ((s = check_cuda(ctx, cudaMemcpyAsync(d->pf_want, rows, (size_t)m * 4, cudaMemcpyHostToDevice, st), "wanted rows")) != NNQ_OK) return s;
-            s = launch_norm_rows(ctx, {d->pf_h, d->pf_delta, nullptr, d->d_final_norm, c.rms_eps, d->pf_xn, d->act_dt, c.hidden, d->embed_ld, d->xn_ld}, m,
-                                 d->pf_tokens, d->pf_want, st);
-            if (s == NNQ_OK && (s = product(d, d->lm_head, d->pf_xn, m, nullptr, d->d_want_logits, st)) != NNQ_OK) return s;
+            NormRows r = pending_rows(d, c.n_layers, d->pf_h, d->pf_delta);
+            r.xn = d->pf_xn;
+            s = launch_norm_rows(ctx, r, m, nullptr, 0, d->pf_want, st);
+            if (s == NNQ_OK) s = product(d, d->lm_head, d->pf_xn, m, nullptr, d->d_want_logits, st);
+            if (s == NNQ_OK && d->logit_cap > 0.0f) s = launch_logit_cap(ctx, d->d_want_logits, d->logit_cap, (long long)m * c.vocab, st);
+            if (s != NNQ_OK) return s;
             s = check_cuda(ctx, cudaMemcpyAsync(logits_host + (size_t)w0 * c.vocab, d->d_want_logits, (size_t)m * c.vocab * 4, cudaMemcpyDeviceToHost, st), "logits");
             if (s == NNQ_OK) s = check_cuda(ctx, cudaStreamSynchronize(st), "logits");   // rows[] is on the stack
             if (s != NNQ_OK) return s;
@@ -1503,7 +1761,10 @@ void nnq_decoder_destroy(nnq_decoder *d) {
             nnq_decoder::Block &B = d->blocks[l];
             cudaFree(B.norm); cudaFree(B.bias_in); cudaFree(B.bias_out); cudaFree(B.conv); cudaFree(B.head_norm);
             cudaFree(B.a2t); cudaFree(B.a2b); cudaFree(B.decay); cudaFree(B.kcache); cudaFree(B.vcache);
-            cudaFree(B.conv_ring); cudaFree(B.rec_state);
+            cudaFree(B.conv_ring); cudaFree(B.rec_state); cudaFree(B.norm_bias); cudaFree(B.q_norm); cudaFree(B.kv_norm);
+            if (B.cfg.mixer == NNQ_MIXER_LATENT && B.cfg.kv_from < 0) {
+                cudaFree(B.ring_c); cudaFree(B.ring_r);
+            }
             if (B.owns_tables) {
                 cudaFree(B.cosv); cudaFree(B.sinv);
             }
@@ -1511,6 +1772,8 @@ void nnq_decoder_destroy(nnq_decoder *d) {
         delete[] d->blocks;
     }
     cudaFree(d->b_h2); cudaFree(d->b_proj); cudaFree(d->b_q); cudaFree(d->b_k); cudaFree(d->b_a); cudaFree(d->b_o); cudaFree(d->b_vfirst); cudaFree(d->b_act);
+    cudaFree(d->b_cq); cudaFree(d->b_lin_c); cudaFree(d->b_lin_r); cudaFree(d->b_kv); cudaFree(d->b_q2); cudaFree(d->b_qrot);
+    cudaFree(d->b_kfull); cudaFree(d->b_vfull); cudaFree(d->b_qlat); cudaFree(d->final_bias);
     cudaFree(d->pf_want); cudaFree(d->d_want_logits);
     cudaFree(d->d_final_norm); cudaFree(d->d_cos); cudaFree(d->d_sin); cudaFree(d->d_kcache); cudaFree(d->d_vcache);
     cudaFree(d->d_h); cudaFree(d->d_delta); cudaFree(d->d_q); cudaFree(d->d_k); cudaFree(d->d_v); cudaFree(d->d_qrot);

@@ -38,5 +38,11 @@ __device__ __forceinline__ void store_act(void *dst, int dt, size_t i, float v) 
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)); }
+// the tanh form of gelu
+__device__ __forceinline__ float gelu_tanh_f32(float x) {
+    return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * x * x, x, x)));
+}
+// kind: nnq_gate_act
+__device__ __forceinline__ float gate_act(int kind, float x) { return kind == NNQ_ACT_GELU_TANH ? gelu_tanh_f32(x) : silu_f32(x); }
 
 }  // namespace nnq

@@ -9,11 +9,12 @@
 // weights stream while they run. Products bf16 x bf16 in f32, f32 sums. Every wait is bounded.
 //
 // With NORM the kernel also does what stands in front of a decoder's product: every CTA adds the last block's output
-// to the residual row (or reads the embedding row), takes its root mean square and keeps the normed row as bf16 in
-// shared memory; CTA 0 writes the new residual to another buffer (the others may still be reading the old one).
+// to the residual row (or reads the embedding row), norms it and keeps the normed row as bf16 in shared memory; CTA 0
+// writes the new residual to another buffer (the others may still be reading the old one). Behind a gate / up product
+// with interleaved rows the epilogue forms the gated activation.
 #include <cuda_bf16.h>
 
-#include "decoder_common.cuh"
+#include "block_norm.cuh"
 #include "gemm_tc.h"
 #include "sync.cuh"
 
@@ -32,13 +33,14 @@ constexpr int kGvNormMax = 8192;   // width of the normed row: 16 values per thr
 template <int M, bool NORM>
 __global__ void __launch_bounds__(gv_warps(M) * 32, 1)
 dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__restrict__ x, const float *__restrict__ bias, void *__restrict__ y,
-                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm) {
+                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm, int pair_act, int y_ld) {
     constexpr int kGvWarps = gv_warps(M), kGvStages = kGvTiles / kGvWarps;
     extern __shared__ __align__(128) uint8_t gv_smem[];
     __shared__ __align__(8) uint64_t bars[kGvWarps * kGvStages];
     float *part = reinterpret_cast<float *>(gv_smem + kGvRing);   // [rows of this CTA][ks][M]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int r0 = (int)((long long)N * blockIdx.x / gridDim.x), r1 = (int)((long long)N * (blockIdx.x + 1) / gridDim.x);
+    const int unit = NORM && pair_act ? 2 : 1;   // rows that stay together
+    const int r0 = (int)((long long)(N / unit) * blockIdx.x / gridDim.x) * unit, r1 = (int)((long long)(N / unit) * (blockIdx.x + 1) / gridDim.x) * unit;
     const int groups = kGvWarps / ks, group = warp / ks, kw = warp % ks;
     const int rows = r1 - r0 > group ? (r1 - r0 - group + groups - 1) / groups : 0;   // rows r0 + group, + groups, ...
     const uint32_t bar0 = smem_u32(bars + warp * kGvStages);
@@ -67,33 +69,32 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
     if constexpr (NORM) {
         __shared__ float red[32];
         __nv_bfloat16 *xn = reinterpret_cast<__nv_bfloat16 *>(gv_smem + kGvRing + nrm.xn_at);
-        const __nv_bfloat16 *er = nrm.embed ? nrm.embed + (size_t)nrm.state[0] * nrm.embed_ld : nullptr;
-        float4 h[4];
-        float ss = 0.0f;
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-            const int d = 4 * (threadIdx.x + kGvWarps * 32 * i);
-            h[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (d < nrm.hidden) {
-                if (er) {
-                    const uint2 u = *reinterpret_cast<const uint2 *>(er + d);
-                    h[i] = make_float4(bf_lo(u.x), bf_hi(u.x), bf_lo(u.y), bf_hi(u.y));
-                } else {
-                    const float4 a = *reinterpret_cast<const float4 *>(nrm.h_in + d), b = *reinterpret_cast<const float4 *>(nrm.delta + d);
-                    h[i] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
-                }
-                if (blockIdx.x == 0 && nrm.h_out) *reinterpret_cast<float4 *>(nrm.h_out + d) = h[i];
-            }
-            ss = fmaf(h[i].x, h[i].x, fmaf(h[i].y, h[i].y, fmaf(h[i].z, h[i].z, fmaf(h[i].w, h[i].w, ss))));
+        NormRow row;
+        row.h_in = nrm.h_in;
+        row.delta = nrm.delta;
+        row.h_out = blockIdx.x == 0 ? nrm.h_out : nullptr;
+        row.e0 = row.e1 = nullptr;
+        if (nrm.embed) {
+            const int tok = nrm.state[0];
+            row.e0 = nrm.embed + (size_t)tok * nrm.embed_ld;
+            if (nrm.pairs.table) row.e1 = nrm.pairs.table + pair_row(nrm.pairs, nrm.state[4], tok, nrm.state[1]) * nrm.embed_ld;
         }
-        const float rms = sqrtf(block_sum(ss, red) / (float)nrm.hidden + nrm.eps);
+        row.alpha = nrm.alpha;
+        row.post_w = nrm.post_w;
+        row.post_b = nrm.post_b;
+        row.in = nrm.in;
+        row.eps = nrm.eps;
+        row.hidden = nrm.hidden;
+        float4 h[4];
+        norm_units(row, h, red);
 #pragma unroll
         for (int i = 0; i < 4; i++) {
             const int d = 4 * (threadIdx.x + kGvWarps * 32 * i);
             if (d >= K) continue;   // columns from hidden on are zero
-            const float4 g = d < nrm.hidden ? *reinterpret_cast<const float4 *>(nrm.w + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            const __nv_bfloat162 a = __floats2bfloat162_rn(h[i].x / rms * g.x, h[i].y / rms * g.y), b = __floats2bfloat162_rn(h[i].z / rms * g.z, h[i].w / rms * g.w);
-            *reinterpret_cast<uint2 *>(xn + d) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+            const __nv_bfloat162 a = __floats2bfloat162_rn(h[i].x, h[i].y), b = __floats2bfloat162_rn(h[i].z, h[i].w);
+            const uint2 u = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+            *reinterpret_cast<uint2 *>(xn + d) = u;
+            if (nrm.xn_out && blockIdx.x == 0) *reinterpret_cast<uint2 *>(nrm.xn_out + d) = u;
         }
         __syncthreads();
         xrow = xn;
@@ -164,6 +165,20 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
         if (lane == 0) atomicExch(status, 1);
     }
     __syncthreads();
+    if (NORM && pair_act) {
+        __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(y);
+        for (int i = threadIdx.x; i < (r1 - r0) / 2; i += kGvWarps * 32) {
+            float g = 0.0f, u = 0.0f;
+            for (int q = 0; q < ks; q++) {
+                g += part[(size_t)(2 * i) * ks + q];
+                u += part[(size_t)(2 * i + 1) * ks + q];
+            }
+            out[r0 / 2 + i] = __float2bfloat16_rn(gate_act(pair_act - 1, g) * u);
+        }
+        if (blockIdx.x == 0)
+            for (int i = N / 2 + threadIdx.x; i < y_ld; i += kGvWarps * 32) out[i] = __float2bfloat16_rn(0.0f);
+        return;
+    }
     for (int i = threadIdx.x; i < (r1 - r0) * M; i += kGvWarps * 32) {
         const int m = i / (r1 - r0), r = i - m * (r1 - r0);
         float v = 0.0f;
@@ -180,11 +195,11 @@ bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt) {
 }
 
 template <int M, bool NORM>
-static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, const GemvNorm &nrm, cudaStream_t st) {
+static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, const GemvNorm &nrm, int pair_act, int y_ld, cudaStream_t st) {
     cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M, NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     launch_pdl_smem(dense_gemv_kernel<M, NORM>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
-                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm);
+                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm, pair_act, y_ld);
     return cudaGetLastError();
 }
 
@@ -192,7 +207,7 @@ bool dense_gemv_norm_supported(const nnq_weight *w, int hidden) {
     return dense_gemv_supported(w, 1, NNQ_BF16) && hidden % 4 == 0 && hidden <= w->k && w->k <= kGvNormMax;
 }
 
-static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, cudaStream_t stream) {
+static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, int pair_act, int y_ld, cudaStream_t stream) {
     // as few warps per row as keep a warp's columns within one chunk
     int ks = 1;
     while (ks < gv_warps((int)a.m) && a.k > (int64_t)ks * kGvChunk) ks *= 2;
@@ -201,21 +216,22 @@ static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, cudaStream_
     const int chunks = (int)((a.k + chunk - 1) / chunk), passes = (chunks + ks - 1) / ks;
     // partial sums of a CTA's rows within 32 KB: more CTAs than SMs for very tall weights
     const int64_t max_rows = (32 << 10) / (4 * ks * a.m);
-    int64_t grid = a.n < ctx->sm_count ? a.n : ctx->sm_count;
-    while ((a.n + grid - 1) / grid > max_rows) grid += ctx->sm_count;
-    size_t smem = kGvRing + ((size_t)((a.n + grid - 1) / grid) * ks * a.m * 4 + 15) / 16 * 16;
+    const int64_t units = pair_act ? a.n / 2 : a.n, per_unit = pair_act ? 2 : 1;   // runs of rows that stay together
+    int64_t grid = units < ctx->sm_count ? units : ctx->sm_count;
+    while ((units + grid - 1) / grid * per_unit > max_rows) grid += ctx->sm_count;
+    size_t smem = kGvRing + ((size_t)((units + grid - 1) / grid * per_unit) * ks * a.m * 4 + 15) / 16 * 16;
     cudaError_t e;
     const GemvNorm none = {};
     if (nrm) {
         nrm->xn_at = (int)(smem - kGvRing);
         smem += (size_t)a.k * 2;
-        e = gv_go<1, true>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, stream);
+        e = gv_go<1, true>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, pair_act, y_ld, stream);
     } else {
         switch (a.m) {
-            case 1: e = gv_go<1, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
-            case 2: e = gv_go<2, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
-            case 3: e = gv_go<3, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
-            case 4: e = gv_go<4, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, stream); break;
+            case 1: e = gv_go<1, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 2: e = gv_go<2, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 3: e = gv_go<3, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 4: e = gv_go<4, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
             default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "1 to 4 rows");
         }
     }
@@ -223,11 +239,11 @@ static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, cudaStream_
     return check_cuda(ctx, e, "bf16 row product launch");
 }
 
-nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) { return gemv(ctx, a, nullptr, stream); }
+nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) { return gemv(ctx, a, nullptr, 0, 0, stream); }
 
-nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, cudaStream_t stream) {
+nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, int pair_act, int y_ld, cudaStream_t stream) {
     GemvNorm n = norm;
-    return gemv(ctx, a, &n, stream);
+    return gemv(ctx, a, &n, pair_act, y_ld, stream);
 }
 
 }  // namespace nnq

@@ -2,6 +2,7 @@
 #pragma once
 #include <cuda_bf16.h>
 
+#include "blocks.h"
 #include "nnq_internal.h"
 
 namespace nnq {
@@ -58,21 +59,29 @@ nnq_status launch_gemm_dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs
 // dense_gemv.cu: one to four bf16 rows against an unquantized bf16 weight
 bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt);
 nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream);
-// the same for one row x = RMSNorm(h) * w with h = h_in + delta, or the embedding row of token state[0]; h_out (not
-// h_in) receives h, NULL to drop it. a.x is not read; a.k >= hidden, columns from hidden on are zero.
+// The same for one row that the kernel forms itself: h = alpha h_in + delta, or the embedding row of token state[0]
+// (plus its pair row: previous token state[4], position state[1]), post-normed where post_w is given; x = in(h). h_out
+// (not h_in) receives h, xn_out x as bf16 [k], NULL to drop them. a.x is not read; a.k >= hidden, columns from hidden on
+// are zero.
 struct GemvNorm {
-    const float *h_in, *delta;
+    const float *h_in, *delta;    // delta NULL: alpha h_in
     float *h_out;
-    const __nv_bfloat16 *embed;   // NULL: h_in + delta
+    __nv_bfloat16 *xn_out;
+    float alpha;
+    const __nv_bfloat16 *embed;   // NULL: alpha h_in + delta
+    PairTable pairs;
     int embed_ld;
     const int *state;
-    const float *w;
+    const float *post_w, *post_b;
+    InNorm in;
     float eps;
     int hidden;
     int xn_at;                    // (set by the launcher)
 };
 bool dense_gemv_norm_supported(const nnq_weight *w, int hidden);
-nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, cudaStream_t stream);
+// pair_act > 0: rows 2j and 2j + 1 of the weight are a gate and an up row, and y (bf16, n / 2 columns and zeros up to y_ld)
+// receives f(gate) * up, f = nnq_gate_act pair_act - 1
+nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, int pair_act, int y_ld, cudaStream_t stream);
 bool gemm_dense_shape_ok(const nnq_ctx *ctx, int64_t m, int64_t n, int64_t k, int x_dt);
 // the expert products of a prefill-sized MoE call: all local experts decoded at once
 bool gemm_dense_grouped_supported(const nnq_ctx *ctx, const TcGroupArgs &g);

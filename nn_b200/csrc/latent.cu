@@ -1,0 +1,542 @@
+// Attention through a latent (LatentAttn in blocks.h): preparation of the latents and the decode step. f32: norms,
+// rotation, scores, softmax, sums, the query carried into the latent space and the weighted latents.
+//
+// Decode step, three launches:
+//   absorb  a CTA per (head, 128 latent columns): q_lat = scale * W_uk,h^T q_h, the rotated query part beside it; one
+//           more CTA norms and appends the new latent. The weight rows are asked for before the wait.
+//   scores  a CTA per (range of keys, eight heads): scores, softmax and weighted latents of its range, one record each.
+//   values  a CTA per (head, 32 value dimensions): merges the records of the head and multiplies with W_uv,h.
+#include <math.h>
+
+#include "blocks.cuh"
+
+namespace nnq {
+
+template <typename T> __device__ __forceinline__ float to_f32(T v);
+template <> __device__ __forceinline__ float to_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// ---- preparation ----
+
+constexpr int kLpWarps = 4;
+
+// A warp per item: n query latents, n key latents, then the older positions in groups of four (copied).
+template <typename T>
+__global__ void __launch_bounds__(kLpWarps * 32) latent_prep_kernel(const LatentAttn a, int nq, int nk, int copy_end) {
+    pdl_prologue();
+    pdl_release();
+    const int lane = threadIdx.x & 31;
+    int item = blockIdx.x * kLpWarps + (threadIdx.x >> 5);
+    const int pos0 = span_pos(a.span);
+    if (item < nq) {
+        const float *p = a.proj + (size_t)item * a.in_cols + a.c_q;
+        float ss = 0.0f;
+        for (int i = lane; i < a.q_rank; i += 32) ss = fmaf(p[i], p[i], ss);
+        const float rms = sqrtf(warp_sum(ss) / (float)a.q_rank + a.eps);
+        T *o = reinterpret_cast<T *>(a.cq) + (size_t)item * a.q_ld;
+        for (int i = lane; i < a.q_ld; i += 32) o[i] = from_f32<T>(i < a.q_rank ? p[i] / rms * a.q_norm[i] : 0.0f);
+        return;
+    }
+    item -= nq;
+    if (item < nk) {
+        const int pos = pos0 + item, half = a.rot >> 1;
+        const float *p = a.proj + (size_t)item * a.in_cols + a.c_kv, *r = p + a.kv_rank;
+        float ss = 0.0f;
+        for (int i = lane; i < a.kv_rank; i += 32) ss = fmaf(p[i], p[i], ss);
+        const float rms = sqrtf(warp_sum(ss) / (float)a.kv_rank + a.eps);
+        T *oc = reinterpret_cast<T *>(a.ring_c) + (size_t)(pos % a.cap) * a.kv_ld, *orr = reinterpret_cast<T *>(a.ring_r) + (size_t)(pos % a.cap) * a.rot_ld;
+        T *lc = reinterpret_cast<T *>(a.lin_c) + (size_t)(pos - a.first) * a.kv_ld, *lr = reinterpret_cast<T *>(a.lin_r) + (size_t)(pos - a.first) * a.rot_ld;
+        for (int i = lane; i < a.kv_ld; i += 32) {
+            const T v = from_f32<T>(i < a.kv_rank ? p[i] / rms * a.kv_norm[i] : 0.0f);
+            oc[i] = v;
+            if (a.linear) lc[i] = v;
+        }
+        for (int i = lane; i < a.rot_ld; i += 32) {
+            const T v = from_f32<T>(i < a.rot ? rotated(r, i, a.rot, a.cosv + (size_t)pos * half, a.sinv + (size_t)pos * half) : 0.0f);
+            orr[i] = v;
+            if (a.linear) lr[i] = v;
+        }
+        return;
+    }
+    item -= nk;
+    constexpr int E = 16 / sizeof(T);
+    for (int p = a.first + 4 * item; p < min(a.first + 4 * item + 4, copy_end); p++) {
+        const uint4 *sc = reinterpret_cast<const uint4 *>(reinterpret_cast<const T *>(a.ring_c) + (size_t)(p % a.cap) * a.kv_ld);
+        const uint4 *sr = reinterpret_cast<const uint4 *>(reinterpret_cast<const T *>(a.ring_r) + (size_t)(p % a.cap) * a.rot_ld);
+        uint4 *dc = reinterpret_cast<uint4 *>(reinterpret_cast<T *>(a.lin_c) + (size_t)(p - a.first) * a.kv_ld);
+        uint4 *dr = reinterpret_cast<uint4 *>(reinterpret_cast<T *>(a.lin_r) + (size_t)(p - a.first) * a.rot_ld);
+        for (int i = lane; i < a.kv_ld / E; i += 32) dc[i] = sc[i];
+        for (int i = lane; i < a.rot_ld / E; i += 32) dr[i] = sr[i];
+    }
+}
+
+nnq_status launch_latent_prep(nnq_ctx *ctx, const LatentAttn &a, int parts, cudaStream_t st) {
+    const int n = a.span.n, nq = parts & kLatentQueries ? n : 0, nk = (parts & kLatentKeys) && a.c_kv >= 0 ? n : 0;
+    const int copy_end = (parts & kLatentKeys) && a.linear ? (a.c_kv >= 0 ? a.span.pos0 : a.span.pos0 + n) : a.first;
+    const int items = nq + nk + (copy_end - a.first + 3) / 4;
+    if (items == 0) return NNQ_OK;
+    const dim3 grid((items + kLpWarps - 1) / kLpWarps), block(kLpWarps * 32);
+    if (a.act_dt == NNQ_F32) launch_pdl(latent_prep_kernel<float>, grid, block, st, a, nq, nk, copy_end);
+    else launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, st, a, nq, nk, copy_end);
+    ctx->launches++;
+    return check_cuda(ctx, cudaGetLastError(), "latent preparation launch");
+}
+
+// ---- block of rows on the general attention kernels ----
+
+// f32 queries (rotated), keys and values with the shared key part in every head; zeros in the columns of out behind
+// the heads'. Grid: (elements of a row, rows of q / keys / out)
+template <typename T>
+__global__ void __launch_bounds__(256) latent_assemble_kernel(const LatentAttn a, int dl, int vl) {
+    pdl_prologue();
+    pdl_release();
+    const int row = blockIdx.y, n = a.span.n, i = blockIdx.x * 256 + threadIdx.x, dk = a.dim + a.rot, half = a.rot >> 1;
+    if (row < n) {
+        const int pos = a.span.pos0 + row;
+        const float *cs = a.cosv + (size_t)pos * half, *sn = a.sinv + (size_t)pos * half;
+        if (i < a.heads * dl) {
+            const int h = i / dl, d = i - h * dl;
+            const float *q = a.q + ((size_t)row * a.heads + h) * dk;
+            a.qrot[((size_t)row * a.heads + h) * dl + d] = d < a.dim ? q[d] : (d < dk ? rotated(q + a.dim, d - a.dim, a.rot, cs, sn) : 0.0f);
+        }
+        if (i < a.out_ld - a.heads * a.vdim) store_act(a.out, a.act_dt, (size_t)row * a.out_ld + a.heads * a.vdim + i, 0.0f);
+        return;
+    }
+    const int key = row - n;
+    const T *kv = reinterpret_cast<const T *>(a.kv) + (size_t)key * a.heads * (a.dim_ld + a.vdim_ld);
+    if (i < a.heads * dl) {
+        const int h = i / dl, d = i - h * dl;
+        const T *r = reinterpret_cast<const T *>(a.lin_r) + (size_t)key * a.rot_ld;
+        a.kfull[((size_t)h * a.keys + key) * dl + d] = d < a.dim ? to_f32(kv[h * a.dim_ld + d]) : (d < dk ? to_f32(r[d - a.dim]) : 0.0f);
+    }
+    if (i < a.heads * vl) {
+        const int h = i / vl, d = i - h * vl;
+        a.vfull[((size_t)h * a.keys + key) * vl + d] = d < a.vdim ? to_f32(kv[a.heads * a.dim_ld + h * a.vdim_ld + d]) : 0.0f;
+    }
+}
+
+nnq_status launch_latent_rows(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st) {
+    if (latent_tc_supported(a.act_dt, a.dim, a.rot, a.vdim)) return launch_latent_tc(ctx, a, st);
+    const int dl = round_up(a.dim + a.rot, 4), vl = round_up(a.vdim, 4);
+    int width = a.heads * (dl > vl ? dl : vl);
+    if (a.out_ld - a.heads * a.vdim > width) width = a.out_ld - a.heads * a.vdim;
+    const dim3 grid((width + 255) / 256, a.span.n + a.keys);
+    if (a.act_dt == NNQ_F32) launch_pdl(latent_assemble_kernel<float>, grid, dim3(256), st, a, dl, vl);
+    else launch_pdl(latent_assemble_kernel<__nv_bfloat16>, grid, dim3(256), st, a, dl, vl);
+    ctx->launches++;
+    nnq_status s = check_cuda(ctx, cudaGetLastError(), "latent expansion launch");
+    if (s != NNQ_OK) return s;
+    WindowAttn w = {};
+    w.span = {a.span.n, a.span.pos0 - a.first, nullptr};   // positions count from the first key
+    w.heads = w.kv_heads = a.heads;
+    w.dim = a.dim + a.rot; w.vdim = a.vdim; w.dim_ld = dl; w.vdim_ld = vl;
+    w.scale = a.scale; w.window = a.window;
+    w.qrot = a.qrot; w.kcache = a.kfull; w.vcache = a.vfull; w.cap = a.keys;
+    w.ffn.act = a.out; w.ffn.act_dt = a.act_dt; w.ffn.out_k = a.out_ld;
+    return launch_attn_rows(ctx, w, st);
+}
+
+// ---- decode step ----
+
+constexpr int kLsThreads = 256, kLsHeads = 8, kLsMaxRanges = 64;
+
+__device__ __forceinline__ float bf_at(uint32_t u, int hi) { return __uint_as_float(hi ? u & 0xFFFF0000u : u << 16); }
+
+template <typename T>
+__global__ void __launch_bounds__(kLsThreads) latent_absorb_kernel(const LatentAttn a) {
+    __shared__ float red[16][132];
+    __shared__ float qs[1024 + 32];
+    const int tid = threadIdx.x, h = blockIdx.x;
+    if (h == a.heads) {   // the new latent
+        pdl_prologue();
+        pdl_release();
+        if (blockIdx.y != 0 || a.c_kv < 0) return;
+        const int pos = a.span.state[1], half = a.rot >> 1;
+        const float *p = a.proj + a.c_kv, *r = p + a.kv_rank;
+        float ss = 0.0f;
+        for (int i = tid; i < a.kv_rank; i += kLsThreads) ss = fmaf(p[i], p[i], ss);
+        const float rms = sqrtf(block_sum(ss, qs) / (float)a.kv_rank + a.eps);
+        T *oc = reinterpret_cast<T *>(a.ring_c) + (size_t)(pos % a.cap) * a.kv_ld, *orr = reinterpret_cast<T *>(a.ring_r) + (size_t)(pos % a.cap) * a.rot_ld;
+        for (int i = tid; i < a.kv_ld; i += kLsThreads) oc[i] = from_f32<T>(i < a.kv_rank ? p[i] / rms * a.kv_norm[i] : 0.0f);
+        for (int i = tid; i < a.rot_ld; i += kLsThreads)
+            orr[i] = from_f32<T>(i < a.rot ? rotated(r, i, a.rot, a.cosv + (size_t)pos * half, a.sinv + (size_t)pos * half) : 0.0f);
+        return;
+    }
+    const int rg = tid >> 4, c0 = blockIdx.y * 128 + 8 * (tid & 15);
+    const bool in = c0 < a.kv_ld;
+    const __nv_bfloat16 *w = a.ukv + (size_t)h * a.dim_ld * a.kv_ld + c0;
+    uint4 wv[8];
+#pragma unroll
+    for (int i = 0; i < 8; i++) wv[i] = in && rg + 16 * i < a.dim ? *reinterpret_cast<const uint4 *>(w + (size_t)(rg + 16 * i) * a.kv_ld) : make_uint4(0, 0, 0, 0);
+    pdl_prologue();
+    pdl_release();
+    const float *q = a.q + (size_t)h * (a.dim + a.rot);
+    const int ld = a.kv_ld + a.rot_ld;
+    float acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; e++) acc[e] = 0.0f;
+    for (int d0 = 0; d0 < a.dim; d0 += 128) {
+        __syncthreads();
+        for (int i = tid; i < 128; i += kLsThreads) qs[i] = d0 + i < a.dim ? q[d0 + i] : 0.0f;
+        __syncthreads();
+        if (d0 > 0)
+#pragma unroll
+            for (int i = 0; i < 8; i++)
+                wv[i] = in && d0 + rg + 16 * i < a.dim ? *reinterpret_cast<const uint4 *>(w + (size_t)(d0 + rg + 16 * i) * a.kv_ld) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            const float x = qs[rg + 16 * i];
+            const uint32_t u[4] = {wv[i].x, wv[i].y, wv[i].z, wv[i].w};
+#pragma unroll
+            for (int e = 0; e < 8; e++) acc[e] = fmaf(bf_at(u[e >> 1], e & 1), x, acc[e]);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 8; e++) red[rg][8 * (tid & 15) + e] = acc[e];
+    __syncthreads();
+    if (tid < 128 && blockIdx.y * 128 + tid < a.kv_ld) {
+        float v = 0.0f;
+#pragma unroll
+        for (int g = 0; g < 16; g++) v += red[g][tid];
+        a.qlat[(size_t)h * ld + blockIdx.y * 128 + tid] = v * a.scale;
+    }
+    if (blockIdx.y == 0) {
+        const int pos = a.span.state[1], half = a.rot >> 1;
+        for (int i = tid; i < a.rot_ld; i += kLsThreads)
+            a.qlat[(size_t)h * ld + a.kv_ld + i] = i < a.rot ? rotated(q + a.dim, i, a.rot, a.cosv + (size_t)pos * half, a.sinv + (size_t)pos * half) * a.scale : 0.0f;
+    }
+}
+
+template <typename T> struct StepKeys;   // keys of a tile
+template <> struct StepKeys<__nv_bfloat16> { static constexpr int value = 64; };
+template <> struct StepKeys<float> { static constexpr int value = 32; };
+
+struct LatentSmem {   // bytes
+    int keys, q, dots, probs, total;
+    int key_ld;       // bytes of a key row
+};
+template <typename T>
+__host__ __device__ inline LatentSmem latent_smem(int kv_ld, int rot_ld) {
+    constexpr int KT = StepKeys<T>::value;
+    LatentSmem m;
+    m.key_ld = (kv_ld + rot_ld) * (int)sizeof(T) + 16;   // rows four banks apart
+    m.keys = 0;
+    m.q = m.keys + KT * m.key_ld;
+    m.dots = m.q + kLsHeads * (kv_ld + rot_ld) * 4;
+    m.probs = m.dots + 8 * kLsHeads * KT * 4;
+    m.total = m.probs + KT * kLsHeads * 4;
+    return m;
+}
+
+__device__ __forceinline__ void cp_async16_latent(void *dst, const void *src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+// NV: 512-wide pieces of the latent
+template <typename T, int NV>
+__global__ void __launch_bounds__(kLsThreads) latent_scores_kernel(const LatentAttn a, int per) {
+    constexpr int KT = StepKeys<T>::value, KL = KT / 32, P = kLsHeads, E = 16 / (int)sizeof(T);
+    extern __shared__ __align__(16) uint8_t ls_smem[];
+    __shared__ float run_m[P], run_l[P], corr_s[P];
+    const LatentSmem m = latent_smem<T>(a.kv_ld, a.rot_ld);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int range = blockIdx.x, h0 = blockIdx.y * P, nh = min(P, a.heads - h0);
+    const int ld = a.kv_ld + a.rot_ld, uc = a.kv_ld / E, units = ld / E;
+    const int pos = a.span.state[1];
+    const int first = max(0, pos - a.window + 1);
+    const int lo = first + range * per, hi = min(pos + 1, lo + per);
+    float *q_s = reinterpret_cast<float *>(ls_smem + m.q), *dots = reinterpret_cast<float *>(ls_smem + m.dots), *probs = reinterpret_cast<float *>(ls_smem + m.probs);
+    auto fetch = [&](int p0, int n) {   // positions p0 .. p0 + n - 1 into the tile, from row 0 on
+        for (int i = tid; i < n * units; i += kLsThreads) {
+            const int r = i / units, c = i - r * units, slot = (p0 + r) % a.cap;
+            const T *src = c < uc ? reinterpret_cast<const T *>(a.ring_c) + (size_t)slot * a.kv_ld + c * E
+                                  : reinterpret_cast<const T *>(a.ring_r) + (size_t)slot * a.rot_ld + (c - uc) * E;
+            cp_async16_latent(ls_smem + m.keys + r * m.key_ld + 16 * c, src);
+        }
+    };
+    // the older latents do not depend on the kernel in front; the current position's is written by it
+    if (lo < hi) fetch(lo, min(KT, min(hi, pos) - lo));
+    pdl_prologue();
+    pdl_release();
+    if (lo >= hi) return;
+    for (int i = tid; i < P * ld / 4; i += kLsThreads) {
+        const int p = i / (ld / 4);
+        reinterpret_cast<float4 *>(q_s)[i] = p < nh ? reinterpret_cast<const float4 *>(a.qlat + (size_t)h0 * ld)[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+    if (tid < P) {
+        run_m[tid] = -INFINITY;
+        run_l[tid] = 0.0f;
+    }
+    // weighted latents: a thread owns column pairs, groups of threads take every G-th key
+    int G = 1;
+    while (2 * G * (a.kv_ld / 2) <= kLsThreads && G < 8) G *= 2;
+    const int gt = kLsThreads / G, grp = tid / gt, ci = tid - grp * gt;
+    float acc[NV][2][P];
+#pragma unroll
+    for (int v = 0; v < NV; v++)
+#pragma unroll
+        for (int p = 0; p < P; p++) acc[v][0][p] = acc[v][1][p] = 0.0f;
+    for (int b0 = lo; b0 < hi; b0 += KT) {
+        const int n = min(KT, hi - b0);
+        if (b0 > lo) fetch(b0, n);
+        else if (n > min(KT, min(hi, pos) - lo)) {   // the current position is in the first tile
+            for (int c = tid; c < units; c += kLsThreads) {
+                const T *src = c < uc ? reinterpret_cast<const T *>(a.ring_c) + (size_t)(pos % a.cap) * a.kv_ld + c * E
+                                      : reinterpret_cast<const T *>(a.ring_r) + (size_t)(pos % a.cap) * a.rot_ld + (c - uc) * E;
+                cp_async16_latent(ls_smem + m.keys + (n - 1) * m.key_ld + 16 * c, src);
+            }
+        }
+        asm volatile("cp.async.wait_all;" ::: "memory");
+        __syncthreads();
+        {
+            float dot[KL][P];
+#pragma unroll
+            for (int k = 0; k < KL; k++)
+#pragma unroll
+                for (int p = 0; p < P; p++) dot[k][p] = 0.0f;
+            const uint8_t *krow = ls_smem + m.keys + lane * m.key_ld;
+            for (int c = warp; c < units; c += 8) {
+                float kx[KL][E];
+#pragma unroll
+                for (int k = 0; k < KL; k++) {
+                    const uint4 u = *reinterpret_cast<const uint4 *>(krow + k * 32 * m.key_ld + 16 * c);
+                    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+                    for (int e = 0; e < E; e++) kx[k][e] = sizeof(T) == 4 ? __uint_as_float(w[e & 3]) : bf_at(w[(e >> 1) & 3], e & 1);
+                }
+#pragma unroll
+                for (int p = 0; p < P; p++) {
+                    const float4 *q4 = reinterpret_cast<const float4 *>(q_s + p * ld + c * E);
+#pragma unroll
+                    for (int e = 0; e < E / 4; e++) {
+                        const float4 x = q4[e];
+#pragma unroll
+                        for (int k = 0; k < KL; k++)
+                            dot[k][p] = fmaf(x.x, kx[k][4 * e], fmaf(x.y, kx[k][4 * e + 1], fmaf(x.z, kx[k][4 * e + 2], fmaf(x.w, kx[k][4 * e + 3], dot[k][p]))));
+                    }
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < KL; k++)
+#pragma unroll
+                for (int p = 0; p < P; p++) dots[(warp * P + p) * KT + 32 * k + lane] = dot[k][p];
+        }
+        __syncthreads();
+        {   // softmax of head `warp` over the tile (eight warps, eight heads)
+            float sc[KL], mx = -INFINITY;
+#pragma unroll
+            for (int k = 0; k < KL; k++) {
+                float d = 0.0f;
+#pragma unroll
+                for (int w = 0; w < 8; w++) d += dots[(w * P + warp) * KT + 32 * k + lane];
+                sc[k] = 32 * k + lane < n ? d : -INFINITY;
+                mx = fmaxf(mx, sc[k]);
+            }
+            const float mo = run_m[warp], mn = fmaxf(mo, warp_max(mx));   // finite: the tile holds a key
+            float sum = 0.0f;
+#pragma unroll
+            for (int k = 0; k < KL; k++) {
+                const float e = expf(sc[k] - mn);
+                probs[(32 * k + lane) * P + warp] = e;
+                sum += e;
+            }
+            sum = warp_sum(sum);
+            if (lane == 0) {
+                const float corr = expf(mo - mn);
+                run_m[warp] = mn;
+                run_l[warp] = run_l[warp] * corr + sum;
+                corr_s[warp] = corr;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int v = 0; v < NV; v++)
+#pragma unroll
+            for (int p = 0; p < P; p++) {
+                acc[v][0][p] *= corr_s[p];
+                acc[v][1][p] *= corr_s[p];
+            }
+#pragma unroll 2
+        for (int jj = grp; jj < n; jj += G) {
+            float w[P];
+            const float4 w0 = *reinterpret_cast<const float4 *>(probs + jj * P), w1 = *reinterpret_cast<const float4 *>(probs + jj * P + 4);
+            w[0] = w0.x; w[1] = w0.y; w[2] = w0.z; w[3] = w0.w; w[4] = w1.x; w[5] = w1.y; w[6] = w1.z; w[7] = w1.w;
+#pragma unroll
+            for (int v = 0; v < NV; v++) {
+                const int c = 2 * (ci + gt * v);
+                if (c >= a.kv_ld) continue;
+                float x, y;
+                if (sizeof(T) == 4) {
+                    const float2 f = *reinterpret_cast<const float2 *>(ls_smem + m.keys + jj * m.key_ld + 4 * c);
+                    x = f.x;
+                    y = f.y;
+                } else {
+                    const uint32_t u = *reinterpret_cast<const uint32_t *>(ls_smem + m.keys + jj * m.key_ld + 2 * c);
+                    x = bf_at(u, 0);
+                    y = bf_at(u, 1);
+                }
+#pragma unroll
+                for (int p = 0; p < P; p++) {
+                    acc[v][0][p] = fmaf(w[p], x, acc[v][0][p]);
+                    acc[v][1][p] = fmaf(w[p], y, acc[v][1][p]);
+                }
+            }
+        }
+        __syncthreads();   // the tile may be overwritten
+    }
+    // groups meet in the key area ([G][P][kv_ld] floats, kv_ld * G <= 512 for G > 1)
+    float *sum = reinterpret_cast<float *>(ls_smem + m.keys);
+    if (G > 1) {
+        if (2 * ci < a.kv_ld)
+#pragma unroll
+            for (int p = 0; p < P; p++) *reinterpret_cast<float2 *>(sum + ((size_t)grp * P + p) * a.kv_ld + 2 * ci) = make_float2(acc[0][0][p], acc[0][1][p]);
+        __syncthreads();
+        for (int i = tid; i < nh * a.kv_ld; i += kLsThreads) {
+            float v = 0.0f;
+            for (int g = 0; g < G; g++) v += sum[(size_t)g * P * a.kv_ld + i];
+            const int p = i / a.kv_ld, c = i - p * a.kv_ld;
+            a.part[((size_t)range * a.heads + h0 + p) * (a.kv_ld + 4) + 4 + c] = v;
+        }
+    } else {
+#pragma unroll
+        for (int v = 0; v < NV; v++) {
+            const int c = 2 * (ci + gt * v);
+            if (c >= a.kv_ld) continue;
+#pragma unroll
+            for (int p = 0; p < P; p++)
+                if (p < nh) *reinterpret_cast<float2 *>(a.part + ((size_t)range * a.heads + h0 + p) * (a.kv_ld + 4) + 4 + c) = make_float2(acc[v][0][p], acc[v][1][p]);
+        }
+    }
+    if (tid < nh) {
+        float *o = a.part + ((size_t)range * a.heads + h0 + tid) * (a.kv_ld + 4);
+        o[0] = run_m[tid];
+        o[1] = run_l[tid];
+    }
+}
+
+constexpr int kLvRows = 4;   // value dimensions of a warp
+
+// grid (heads, ceil(vdim / 32))
+__global__ void __launch_bounds__(kLsThreads) latent_values_kernel(const LatentAttn a, int per) {
+    __shared__ __align__(16) float lat[1024];
+    __shared__ float wt[kLsMaxRanges];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
+    const int v0 = blockIdx.y * 8 * kLvRows + warp * kLvRows, nu = a.kv_ld >> 3;
+    const __nv_bfloat16 *w = a.ukv + ((size_t)a.heads * a.dim_ld + (size_t)h * a.vdim_ld + v0) * a.kv_ld;
+    uint4 wv[kLvRows][4];
+#pragma unroll
+    for (int r = 0; r < kLvRows; r++)
+#pragma unroll
+        for (int u = 0; u < 4; u++)
+            wv[r][u] = v0 + r < a.vdim && lane + 32 * u < nu ? *reinterpret_cast<const uint4 *>(w + (size_t)r * a.kv_ld + 8 * (lane + 32 * u)) : make_uint4(0, 0, 0, 0);
+    pdl_prologue();
+    pdl_release();
+    const int pos = a.span.state[1], keys = min(pos + 1, a.window), used = (keys + per - 1) / per;
+    const size_t step = (size_t)a.heads * (a.kv_ld + 4);
+    const float *rec = a.part + (size_t)h * (a.kv_ld + 4);
+    if (warp == 0) {
+        float mv[2], lv[2], mx = -INFINITY, sum = 0.0f;
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            const int s = lane + 32 * k;
+            mv[k] = s < used ? rec[s * step] : -INFINITY;
+            lv[k] = s < used ? rec[s * step + 1] : 0.0f;
+            mx = fmaxf(mx, mv[k]);
+        }
+        mx = warp_max(mx);
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            mv[k] = expf(mv[k] - mx);
+            sum = fmaf(lv[k], mv[k], sum);
+        }
+        sum = warp_sum(sum);
+        wt[lane] = mv[0] / sum;
+        wt[lane + 32] = mv[1] / sum;
+    }
+    __syncthreads();
+    for (int i = 4 * tid; i < a.kv_ld; i += 4 * kLsThreads) {
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int s0 = 0; s0 < used; s0 += 8) {
+            float4 x[8];
+#pragma unroll
+            for (int s = 0; s < 8; s++) x[s] = s0 + s < used ? *reinterpret_cast<const float4 *>(rec + (s0 + s) * step + 4 + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+            for (int s = 0; s < 8; s++) {
+                const float e = s0 + s < used ? wt[s0 + s] : 0.0f;
+                v.x = fmaf(e, x[s].x, v.x); v.y = fmaf(e, x[s].y, v.y); v.z = fmaf(e, x[s].z, v.z); v.w = fmaf(e, x[s].w, v.w);
+            }
+        }
+        *reinterpret_cast<float4 *>(lat + i) = v;
+    }
+    __syncthreads();
+    float acc[kLvRows];
+#pragma unroll
+    for (int r = 0; r < kLvRows; r++) acc[r] = 0.0f;
+#pragma unroll
+    for (int u = 0; u < 4; u++) {
+        if (lane + 32 * u >= nu) continue;
+        const float4 x0 = *reinterpret_cast<const float4 *>(lat + 8 * (lane + 32 * u)), x1 = *reinterpret_cast<const float4 *>(lat + 8 * (lane + 32 * u) + 4);
+        const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+#pragma unroll
+        for (int r = 0; r < kLvRows; r++) {
+            const uint32_t q[4] = {wv[r][u].x, wv[r][u].y, wv[r][u].z, wv[r][u].w};
+#pragma unroll
+            for (int e = 0; e < 8; e++) acc[r] = fmaf(bf_at(q[e >> 1], e & 1), x[e], acc[r]);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < kLvRows; r++) {
+        const float v = warp_sum(acc[r]);
+        if (lane == 0 && v0 + r < a.vdim) store_act(a.out, a.act_dt, h * a.vdim + v0 + r, v);
+    }
+    if (h == 0 && blockIdx.y == 0)
+        for (int i = a.heads * a.vdim + tid; i < a.out_ld; i += kLsThreads) store_act(a.out, a.act_dt, i, 0.0f);
+}
+
+// ---- host side ----
+
+static int step_tile(int act_dt) { return act_dt == NNQ_F32 ? StepKeys<float>::value : StepKeys<__nv_bfloat16>::value; }
+static int range_keys(int ranges, int keys, int tile) { return ((keys + ranges - 1) / ranges + tile - 1) / tile * tile; }
+
+int latent_step_ranges(int sm_count, int heads, int window, int max_seq, int act_dt) {
+    const int keys = window < max_seq ? window : max_seq, tiles = (heads + kLsHeads - 1) / kLsHeads, kt = step_tile(act_dt);
+    int r = sm_count / tiles;
+    r = r < 1 ? 1 : (r > kLsMaxRanges ? kLsMaxRanges : r);
+    return (keys + range_keys(r, keys, kt) - 1) / range_keys(r, keys, kt);
+}
+
+bool latent_step_supported(int act_dt, int kv_ld, int rot_ld) {
+    const int smem = act_dt == NNQ_F32 ? latent_smem<float>(kv_ld, rot_ld).total : latent_smem<__nv_bfloat16>(kv_ld, rot_ld).total;
+    return kv_ld <= 1024 && smem <= 220 * 1024;
+}
+
+template <typename T, int NV>
+static nnq_status go_scores(nnq_ctx *ctx, const LatentAttn &a, int per, cudaStream_t st) {
+    const int smem = latent_smem<T>(a.kv_ld, a.rot_ld).total;
+    nnq_status s = check_cuda(ctx, cudaFuncSetAttribute(latent_scores_kernel<T, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "latent attention shared memory");
+    if (s != NNQ_OK) return s;
+    launch_pdl_smem(latent_scores_kernel<T, NV>, dim3(a.ranges, (a.heads + kLsHeads - 1) / kLsHeads), dim3(kLsThreads), smem, st, a, per);
+    return check_cuda(ctx, cudaGetLastError(), "latent attention launch");
+}
+
+nnq_status launch_latent_step(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st) {
+    const bool f32 = a.act_dt == NNQ_F32;
+    const int per = range_keys(a.ranges, a.keys_max, step_tile(a.act_dt));
+    const dim3 ag(a.heads + 1, (a.kv_ld + 127) / 128), ab(kLsThreads);
+    if (f32) launch_pdl(latent_absorb_kernel<float>, ag, ab, st, a);
+    else launch_pdl(latent_absorb_kernel<__nv_bfloat16>, ag, ab, st, a);
+    nnq_status s = check_cuda(ctx, cudaGetLastError(), "latent query launch");
+    if (s == NNQ_OK) {
+        if (a.kv_ld <= 512) s = f32 ? go_scores<float, 1>(ctx, a, per, st) : go_scores<__nv_bfloat16, 1>(ctx, a, per, st);
+        else s = f32 ? go_scores<float, 2>(ctx, a, per, st) : go_scores<__nv_bfloat16, 2>(ctx, a, per, st);
+    }
+    if (s != NNQ_OK) return s;
+    launch_pdl(latent_values_kernel, dim3(a.heads, (a.vdim + 8 * kLvRows - 1) / (8 * kLvRows)), dim3(kLsThreads), st, a, per);
+    ctx->launches += 3;
+    return check_cuda(ctx, cudaGetLastError(), "latent value launch");
+}
+
+}  // namespace nnq

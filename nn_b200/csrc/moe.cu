@@ -39,42 +39,55 @@ __device__ __forceinline__ float ld_act<__nv_bfloat16>(const __nv_bfloat16 *p, i
     return __bfloat162float(p[i]);
 }
 
-constexpr int kMaxExperts = 64;
+constexpr int kMaxExperts = 256;
+constexpr int kLaneExperts = kMaxExperts / 32;   // logits held by a lane of the routing warp
 constexpr int kMaxTopK = 8;
 
 // Softmax over the E logits of one token (lg, shared memory) and top-k selection by one warp.
 __device__ __forceinline__ void route_token(const float *lg, int E, int top_k, int tok, int *__restrict__ idx,
                                             float *__restrict__ wt, int lane) {
-    // lane e (and e + 32) holds expert e's logit
-    float l0 = lane < E ? lg[lane] : -CUDART_INF_F;
-    float l1 = lane + 32 < E ? lg[lane + 32] : -CUDART_INF_F;
+    // lane l holds the logits of experts l, l + 32, ...
+    float p[kLaneExperts];
+    float mx = -CUDART_INF_F;
+#pragma unroll
+    for (int k = 0; k < kLaneExperts; k++) {
+        p[k] = lane + 32 * k < E ? lg[lane + 32 * k] : -CUDART_INF_F;
+        mx = fmaxf(mx, p[k]);
+    }
     // softmax over the E experts (max-subtracted, f32)
-    float mx = fmaxf(l0, l1);
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, off));
-    float p0 = lane < E ? expf(l0 - mx) : 0.0f;
-    float p1 = lane + 32 < E ? expf(l1 - mx) : 0.0f;
-    float sum = p0 + p1;
+    float sum = 0.0f;
+#pragma unroll
+    for (int k = 0; k < kLaneExperts; k++) {
+        p[k] = lane + 32 * k < E ? expf(p[k] - mx) : 0.0f;
+        sum += p[k];
+    }
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
-    p0 = p0 / sum;
-    p1 = p1 / sum;
-    if (lane >= E) p0 = -1.0f;
-    if (lane + 32 >= E) p1 = -1.0f;
+#pragma unroll
+    for (int k = 0; k < kLaneExperts; k++) p[k] = lane + 32 * k < E ? p[k] / sum : -1.0f;
     // top-k: k rounds of (largest probability, lowest index) selection
     float sel_p = 0.0f, wsum = 0.0f;
     int sel_e = 0;
     for (int s = 0; s < top_k; s++) {
-        float best = p0 >= p1 ? p0 : p1;
-        int be = p0 >= p1 ? lane : lane + 32;
+        float best = p[0];
+        int be = lane;
+#pragma unroll
+        for (int k = 1; k < kLaneExperts; k++)
+            if (p[k] > best) {
+                best = p[k];
+                be = lane + 32 * k;
+            }
 #pragma unroll
         for (int off = 16; off > 0; off >>= 1) {
             float ob = __shfl_xor_sync(0xFFFFFFFFu, best, off);
             int oe = __shfl_xor_sync(0xFFFFFFFFu, be, off);
             if (ob > best || (ob == best && oe < be)) { best = ob; be = oe; }
         }
-        if (be == lane) p0 = -1.0f;
-        if (be == lane + 32) p1 = -1.0f;
+#pragma unroll
+        for (int k = 0; k < kLaneExperts; k++)
+            if (be == lane + 32 * k) p[k] = -1.0f;
         if (lane == s) { sel_p = best; sel_e = be; }
         wsum += best;
     }
@@ -551,7 +564,8 @@ static size_t align256(size_t v) { return (v + 255) & ~(size_t)255; }
 // Prefill-sized calls on [N, K] expert weights go through the grouped tcgen05 products: from 32 routed
 // rows per local expert on average (below that the weights are streamed once per 16 rows by the
 // grouped token-column kernel, which is HBM-bound and wins; the gpt-oss block crosses over near 240 tokens).
-static bool moe_tensor_mode(const nnq_moe *m, int64_t T, int k, bool routed) {
+static bool moe_tensor_mode(const nnq_moe *m, int64_t T, int k, bool routed, bool exact) {
+    if (exact) return false;
     static const char *env = diag_env("NNQ_MOE_TENSOR");   // tuning aid: 0 keeps the token-column kernel
     if (env && atoi(env) == 0) return false;
     // nn-gptoss [E, K, N] experts take the decode-once form only (a transposing decode into the context's
@@ -568,7 +582,7 @@ static bool moe_tensor_mode(const nnq_moe *m, int64_t T, int k, bool routed) {
 
 // Carves the scratch buffer for T rows with k expert slots each; with base == NULL only the size
 // is computed.
-static MoeScratch carve(uint8_t *base, int64_t T, const nnq_moe *m, int k, bool routed = false) {
+static MoeScratch carve(uint8_t *base, int64_t T, const nnq_moe *m, int k, bool routed = false, bool exact = false) {
     MoeScratch s;
     const int64_t R = T * k;
     size_t off = 0;
@@ -583,7 +597,7 @@ static MoeScratch carve(uint8_t *base, int64_t T, const nnq_moe *m, int k, bool 
     s.gu = (float *)take((size_t)R * 2 * m->inter * 4 * slices);
     s.h = (float *)take((size_t)R * m->inter * 4);
     s.o = (float *)take((size_t)R * m->hidden * 4 * slices);
-    const bool tensor = moe_tensor_mode(m, T, k, routed);
+    const bool tensor = moe_tensor_mode(m, T, k, routed, exact);
     s.xg = tensor ? (__nv_bfloat16 *)take((size_t)R * m->hidden * 2) : nullptr;
     s.hb = tensor ? (__nv_bfloat16 *)take((size_t)R * m->inter * 2) : nullptr;
     s.slices = slices;
@@ -593,8 +607,8 @@ static MoeScratch carve(uint8_t *base, int64_t T, const nnq_moe *m, int k, bool 
     return s;
 }
 
-static nnq_status ensure_scratch(nnq_ctx *ctx, const nnq_moe *m, int64_t T, int k, bool routed, MoeScratch *out) {
-    MoeScratch need = carve(nullptr, T, m, k, routed);
+static nnq_status ensure_scratch(nnq_ctx *ctx, const nnq_moe *m, int64_t T, int k, bool routed, MoeScratch *out, bool exact = false) {
+    MoeScratch need = carve(nullptr, T, m, k, routed, exact);
     if (need.bytes > ctx->moe_bytes) {
         cudaFree(ctx->d_moe);
         ctx->d_moe = nullptr;
@@ -603,7 +617,7 @@ static nnq_status ensure_scratch(nnq_ctx *ctx, const nnq_moe *m, int64_t T, int 
         if (s != NNQ_OK) return s;
         ctx->moe_bytes = need.bytes;
     }
-    *out = carve(ctx->d_moe, T, m, k, routed);
+    *out = carve(ctx->d_moe, T, m, k, routed, exact);
     return NNQ_OK;
 }
 
@@ -793,6 +807,20 @@ static nnq_status forward_typed(nnq_ctx *ctx, const nnq_moe *m, const XT *x, int
     if (idx_out) cudaMemcpyAsync(idx_out, s.idx, total * 4, cudaMemcpyDeviceToDevice, st);
     if (wt_out) cudaMemcpyAsync(wt_out, s.wt, total * 4, cudaMemcpyDeviceToDevice, st);
     return check_cuda(ctx, cudaGetLastError(), "MoE routing copy");
+}
+
+nnq_status moe_reserve(nnq_ctx *ctx, const nnq_moe *m, int64_t rows) {
+    MoeScratch s;
+    if (m->ctx != ctx) return fail(ctx, NNQ_ERR_INVALID_ARG, "MoE block belongs to another context");
+    return ensure_scratch(ctx, m, rows, m->top_k, false, &s);
+}
+
+nnq_status moe_rows(nnq_ctx *ctx, const nnq_moe *m, const void *x, nnq_dtype x_dt, int64_t rows, bool exact, float *y, cudaStream_t st) {
+    MoeScratch s;
+    nnq_status rc = ensure_scratch(ctx, m, rows, m->top_k, false, &s, exact);
+    if (rc != NNQ_OK) return rc;
+    if (x_dt == NNQ_F32) return run_with_scratch<float>(ctx, m, (const float *)x, rows, m->top_k, nullptr, nullptr, y, s, false, st);
+    return run_with_scratch<__nv_bfloat16>(ctx, m, (const __nv_bfloat16 *)x, rows, m->top_k, nullptr, nullptr, y, s, false, st);
 }
 
 // Gathers rows of a [rows, H] matrix by index: out[i, :] = x[index[i], :] (the token permute of

@@ -18,3 +18,12 @@ struct nnq_moe {
     uint8_t *d_gu_tiled, *d_dn_tiled;
     size_t gu_tile_stride, dn_tile_stride;   // bytes per expert
 };
+
+namespace nnq {
+
+// moe.cu, for a decoder's blocks: scratch for calls of up to `rows` tokens, and the block over `rows` tokens (y: [rows,
+// hidden]). exact: every product in f32 (f32 activations only).
+nnq_status moe_reserve(nnq_ctx *ctx, const nnq_moe *m, int64_t rows);
+nnq_status moe_rows(nnq_ctx *ctx, const nnq_moe *m, const void *x, nnq_dtype x_dt, int64_t rows, bool exact, float *y, cudaStream_t st);
+
+}  // namespace nnq

@@ -8,13 +8,13 @@ quantized products: Qwen3DecoderLayer / Qwen3Attention / Qwen3MLP forward
 ``step`` can be captured in a CUDA graph once and replayed per token (``generate`` does that).
 
 ``BlockDecoder`` is the same decoder object made of blocks that each name their own mixer (sliding-window
-attention, linear-attention recurrences) and read one normed row per block.
+attention, linear-attention recurrences, attention through a latent, none) and form one residual sum each.
 """
 from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import Callable, List, Optional
 
 import numpy as np
 
@@ -184,7 +184,8 @@ class Decoder:
 # decoders made of blocks
 # --------------------------------------------------------------------------- #
 
-MIXER_ATTENTION, MIXER_RECURRENT = 0, 1
+MIXER_ATTENTION, MIXER_RECURRENT, MIXER_LATENT, MIXER_NONE = 0, 1, 2, 3
+ACT_SILU, ACT_GELU_TANH = 0, 1
 
 
 class _BlockConfig(ctypes.Structure):
@@ -192,22 +193,32 @@ class _BlockConfig(ctypes.Structure):
                 ("vdim", ctypes.c_int32), ("ffn", ctypes.c_int32), ("rot_dims", ctypes.c_int32), ("rot_base", ctypes.c_double),
                 ("scale", ctypes.c_float), ("window", ctypes.c_int32), ("conv_taps", ctypes.c_int32), ("value_mix", ctypes.c_int32),
                 ("out_gate", ctypes.c_int32), ("q_scale", ctypes.c_float), ("k_scale", ctypes.c_float),
-                ("decay_rank", ctypes.c_int32), ("decay_tau", ctypes.c_float)]
+                ("decay_rank", ctypes.c_int32), ("decay_tau", ctypes.c_float), ("post_norm", ctypes.c_int32), ("alpha", ctypes.c_float),
+                ("ffn_act", ctypes.c_int32), ("experts", ctypes.c_int32), ("q_rank", ctypes.c_int32), ("kv_rank", ctypes.c_int32),
+                ("kv_from", ctypes.c_int32)]
 
 
 class _BlockLayout(ctypes.Structure):
-    _fields_ = [(n, ctypes.c_int32) for n in ("in_cols", "in_k", "out_k", "ffn_col", "q", "k", "v", "g", "a1", "gate", "up")]
+    _fields_ = [(n, ctypes.c_int32) for n in ("in_cols", "in_k", "out_k", "ffn_col", "q", "k", "v", "g", "a1", "gate", "up", "ffn_step",
+                                                 "q_ld", "kv_ld", "dim_ld", "vdim_ld")]
 
 
 class _BlockWeights(ctypes.Structure):
     _fields_ = [("w_in", ctypes.c_void_p), ("w_out", ctypes.c_void_p)] + \
         [(n, ctypes.c_void_p) for n in ("norm", "bias_in", "bias_out", "conv", "head_norm", "decay_w", "decay_b", "decay")] + \
-        [("value_lambda", ctypes.c_float)]
+        [("value_lambda", ctypes.c_float)] + \
+        [(n, ctypes.c_void_p) for n in ("norm_bias", "uq", "ukv", "q_norm", "kv_norm", "moe")]
+
+
+class _HeadOptions(ctypes.Structure):
+    _fields_ = [("final_norm_bias", ctypes.c_void_p), ("logit_cap", ctypes.c_float), ("pair_table", ctypes.c_void_p),
+                ("pair_mul_prev", ctypes.c_int64), ("pair_mul_cur", ctypes.c_int64), ("pair_buckets", ctypes.c_int64)]
 
 
 @dataclass
 class BlockConfig:
-    """nnq_block_config of the C ABI; window 0 = every earlier position, decay_rank 0 = a fixed decay per head."""
+    """nnq_block_config of the C ABI; window 0 = every earlier position, decay_rank 0 = a fixed decay per head,
+    kv_from < 0 = latents of its own. top and expert_ffn describe a mixture of `experts`."""
     mixer: int = MIXER_ATTENTION
     heads: int = 1
     kv_heads: int = 1
@@ -225,21 +236,31 @@ class BlockConfig:
     k_scale: float = 1.0
     decay_rank: int = 0
     decay_tau: float = 1.0
+    post_norm: bool = False
+    alpha: float = 1.0
+    ffn_act: int = ACT_SILU
+    experts: int = 0
+    q_rank: int = 0
+    kv_rank: int = 0
+    kv_from: int = -1
+    top: int = 0
+    expert_ffn: int = 0
 
     def _c(self) -> _BlockConfig:
         return _BlockConfig(self.mixer, self.heads, self.kv_heads, self.dim, self.vdim, self.ffn, self.rot_dims, self.rot_base,
                             self.scale, self.window, self.conv_taps, int(self.value_mix), int(self.out_gate), self.q_scale,
-                            self.k_scale, self.decay_rank, self.decay_tau)
+                            self.k_scale, self.decay_rank, self.decay_tau, int(self.post_norm), self.alpha, self.ffn_act, self.experts,
+                            self.q_rank, self.kv_rank, self.kv_from)
 
 
 @dataclass
 class BlockTensors:
     """Tensors of one block: matrices [out, in] as bf16 bit patterns (uint16), everything else f32."""
     norm: np.ndarray
-    q: np.ndarray
-    k: np.ndarray
-    v: np.ndarray
-    o: np.ndarray
+    q: Optional[np.ndarray] = None
+    k: Optional[np.ndarray] = None
+    v: Optional[np.ndarray] = None
+    o: Optional[np.ndarray] = None
     g: Optional[np.ndarray] = None
     q_bias: Optional[np.ndarray] = None
     k_bias: Optional[np.ndarray] = None
@@ -255,10 +276,22 @@ class BlockTensors:
     gate: Optional[np.ndarray] = None
     up: Optional[np.ndarray] = None
     down: Optional[np.ndarray] = None
+    norm_bias: Optional[np.ndarray] = None
+    dq: Optional[np.ndarray] = None          # latent attention: [q_rank, hidden]
+    q_norm: Optional[np.ndarray] = None
+    uq: Optional[np.ndarray] = None          # [heads * (dim + rot_dims), q_rank]
+    dkv: Optional[np.ndarray] = None         # [kv_rank + rot_dims, hidden]
+    kv_norm: Optional[np.ndarray] = None
+    uk: Optional[np.ndarray] = None          # [heads * dim, kv_rank]
+    uv: Optional[np.ndarray] = None          # [heads * vdim, kv_rank]
+    router: Optional[np.ndarray] = None      # mixture of experts: f32 [experts, hidden]
+    router_bias: Optional[np.ndarray] = None
+    expert: Optional[Callable[[int], tuple]] = None   # expert -> (gate, up, down)
 
 
 class BlockDecoder(Decoder):
-    """Decoder whose layers are blocks x <- x + mixer(h) + ff(h), h = RMSNorm(x) * w."""
+    """Decoder whose layers are blocks x <- x + mixer(h) + ff(h), h = RMSNorm(x) * w, or (post_norm) x <- LN(alpha x +
+    mixer(x) + ff(x))."""
 
     def __init__(self, backend: api.Backend, *, hidden: int, vocab: int, blocks: List[BlockConfig], max_seq: int,
                  rms_eps: float = 1e-6, act_dtype: int = api.BF16, block_rows: int = 0):
@@ -289,8 +322,77 @@ class BlockDecoder(Decoder):
         self._keep.append(t)
         return t
 
+    def _heads(self, rows: int, cols: int, parts) -> api.DeviceWeight:
+        """A weight made of head-by-head matrices: (first row, rows per head, rows a head is given, matrix) parts."""
+        out = []
+        for r, per, ld, m in parts:
+            out += [(r + h * ld, 0, m[h * per:(h + 1) * per]) for h in range(m.shape[0] // per)]
+        return self._weight(rows, cols, out)
+
+    def _experts(self, b: BlockConfig, y: _BlockLayout, t: BlockTensors):
+        """The block's experts as a MoeBlock of bf16 weights, widths rounded up to whole k steps with zeros."""
+        from .moe import LAYOUT_NK, MoeBlock
+        hidden, ld, inter = self.cfg.hidden, y.in_k, -(-b.expert_ffn // 64) * 64
+        gu, dn = np.zeros((b.experts, 2, inter, ld), np.uint16), np.zeros((b.experts, ld, inter), np.uint16)
+        for e in range(b.experts):
+            gate, up, down = t.expert(e)
+            if gate.shape != (b.expert_ffn, hidden) or up.shape != gate.shape or down.shape != gate.shape[::-1]:
+                raise api.ShapeMismatch(f"expert {e}: matrices of shape {gate.shape}, {up.shape}, {down.shape}")
+            gu[e, 0, :b.expert_ffn, :hidden], gu[e, 1, :b.expert_ffn, :hidden], dn[e, :hidden, :b.expert_ffn] = gate, up, down
+        router = np.zeros((b.experts, ld), np.float32)
+        router[:, :hidden] = t.router
+        bias = np.zeros(b.experts, np.float32) if t.router_bias is None else t.router_bias
+        m = MoeBlock(b.experts, ld, inter, b.top, float("inf"), router, bias, LAYOUT_NK, QuantFormat.BF16_DENSE, gu.reshape(-1).view(np.uint8), None,
+                     np.zeros((b.experts, 2 * inter), np.float32), dn.reshape(-1).view(np.uint8), None, np.zeros((b.experts, ld), np.float32), self.backend)
+        self._keep.append(m)
+        return m
+
+    def _set_post(self, layer: int, b: BlockConfig, y: _BlockLayout, t: BlockTensors):
+        """Blocks of attention through a latent, of a feed-forward alone or of a mixture of experts."""
+        hidden, w = self.cfg.hidden, _BlockWeights()
+        want = {"norm": (hidden,), "norm_bias": (hidden,)}
+        if b.mixer == MIXER_LATENT:
+            want.update(dq=(b.q_rank, hidden), q_norm=(b.q_rank,), uq=(b.heads * (b.dim + b.rot_dims), b.q_rank), uk=(b.heads * b.dim, b.kv_rank),
+                        uv=(b.heads * b.vdim, b.kv_rank), o=(hidden, b.heads * b.vdim))
+            if b.kv_from < 0:
+                want.update(dkv=(b.kv_rank + b.rot_dims, hidden), kv_norm=(b.kv_rank,))
+        elif b.experts:
+            want.update(router=(b.experts, hidden))
+        else:
+            want.update(gate=(b.ffn, hidden), up=(b.ffn, hidden), down=(hidden, b.ffn))
+        self._check(layer, t, want, {"router_bias": (b.experts,)})
+        if b.mixer == MIXER_LATENT:
+            w.w_in = self._weight(y.in_cols, y.in_k, [(y.q, 0, t.dq), (y.k, 0, t.dkv if b.kv_from < 0 else None)]).handle()
+            w.w_out = self._weight(hidden, y.out_k, [(0, 0, t.o)]).handle()
+            w.uq = self._weight(b.heads * (b.dim + b.rot_dims), y.q_ld, [(0, 0, t.uq)]).handle()
+            w.ukv = self._heads(b.heads * (y.dim_ld + y.vdim_ld), y.kv_ld,
+                                [(0, b.dim, y.dim_ld, t.uk), (b.heads * y.dim_ld, b.vdim, y.vdim_ld, t.uv)]).handle()
+        elif b.experts:
+            w.moe = self._experts(b, y, t)._handle
+        else:
+            pairs = np.zeros((y.in_cols, hidden), np.uint16)
+            end = y.ffn_step * b.ffn
+            pairs[y.gate:end:y.ffn_step], pairs[y.up:end:y.ffn_step] = t.gate, t.up
+            w.w_in = self._weight(y.in_cols, y.in_k, [(0, 0, pairs)]).handle()
+            w.w_out = self._weight(hidden, y.out_k, [(0, 0, t.down)]).handle()
+        f32 = {n: np.ascontiguousarray(getattr(t, n), np.float32) for n in ("norm", "norm_bias", "q_norm", "kv_norm") if getattr(t, n) is not None}
+        for n, a in f32.items():
+            setattr(w, n, a.ctypes.data)
+        self.backend.check(self.backend._lib.nnq_decoder_set_block(self._handle, layer, ctypes.byref(w)))
+
+    @staticmethod
+    def _check(layer: int, t: BlockTensors, want: dict, optional: dict):
+        for name, shape in list(want.items()) + list(optional.items()):
+            a = getattr(t, name)
+            if a is None and name in optional:
+                continue
+            if a is None or tuple(a.shape) != shape:
+                raise api.ShapeMismatch(f"block {layer}: {name} must be {shape}, got {None if a is None else tuple(a.shape)}")
+
     def set_block(self, layer: int, t: BlockTensors):
         y, b, hidden = self.layout(layer), self.blocks[layer], self.cfg.hidden
+        if b.mixer in (MIXER_LATENT, MIXER_NONE):
+            return self._set_post(layer, b, y, t)
         kvh = b.kv_heads if b.mixer == MIXER_ATTENTION else b.heads
         qn, kn, vn, mix = b.heads * b.dim, kvh * b.dim, kvh * b.vdim, b.heads * b.vdim
         want = {"q": (qn, hidden), "k": (kn, hidden), "v": (vn, hidden), "o": (hidden, mix), "norm": (hidden,)}
@@ -306,12 +408,9 @@ class BlockDecoder(Decoder):
             else:
                 want["decay"] = (b.heads,)
         optional = {"q_bias": (qn,), "k_bias": (kn,), "v_bias": (vn,), "o_bias": (hidden,), "head_norm": (b.vdim,)}
-        for name, shape in list(want.items()) + list(optional.items()):
-            a = getattr(t, name)
-            if a is None and name in optional:
-                continue
-            if a is None or tuple(a.shape) != shape:
-                raise api.ShapeMismatch(f"block {layer}: {name} must be {shape}, got {None if a is None else tuple(a.shape)}")
+        if b.post_norm:
+            want["norm_bias"] = (hidden,)
+        self._check(layer, t, want, optional)
         w_in = self._weight(y.in_cols, y.in_k, [(y.q, 0, t.q), (y.k, 0, t.k), (y.v, 0, t.v), (y.g, 0, t.g), (y.a1, 0, t.a1),
                                                 (y.gate, 0, t.gate), (y.up, 0, t.up)])
         w_out = self._weight(hidden, y.out_k, [(0, 0, t.o), (0, y.ffn_col, t.down)])
@@ -324,10 +423,15 @@ class BlockDecoder(Decoder):
         f32 = [None if a is None else np.ascontiguousarray(a, np.float32)
                for a in (t.norm, bias, t.o_bias, t.conv, t.head_norm, t.decay_w, t.decay_b, t.decay)]
         w = _BlockWeights(w_in.handle(), w_out.handle(), *[None if a is None else a.ctypes.data for a in f32], float(t.value_lambda))
+        post = np.ascontiguousarray(t.norm_bias, np.float32) if b.post_norm else None
+        if b.post_norm:
+            w.norm_bias = post.ctypes.data
         self.backend.check(self.backend._lib.nnq_decoder_set_block(self._handle, layer, ctypes.byref(w)))
 
-    def set_head(self, embed, final_norm, lm_head):
-        """embed, lm_head: [vocab, hidden] as bf16 bit patterns (uint16); final_norm f32 [hidden]."""
+    def set_head(self, embed, final_norm, lm_head, *, final_norm_bias=None, logit_cap: float = 0.0, pair_table=None, pair_mul=(0, 0)):
+        """embed, lm_head: [vocab, hidden] as bf16 bit patterns (uint16); final_norm f32 [hidden], with final_norm_bias a layer
+        norm. logit_cap > 0: logits <- cap tanh(logits / cap). pair_table [buckets + 1, hidden] with the factors pair_mul of the
+        previous and the current token: the hashed embedding of token pairs."""
         c = self.cfg
         ld = self.layout(0).in_k
         for a in (embed, lm_head):
@@ -337,6 +441,17 @@ class BlockDecoder(Decoder):
         h = e if lm_head is embed else self._weight(c.vocab, ld, [(0, 0, lm_head)])
         fn = np.ascontiguousarray(final_norm, np.float32)
         self.backend.check(self.backend._lib.nnq_decoder_set_head_weights(self._handle, e.handle(), fn.ctypes.data, h.handle()))
+        o = _HeadOptions(logit_cap=float(logit_cap))
+        if final_norm_bias is not None:
+            fb = np.ascontiguousarray(final_norm_bias, np.float32)
+            o.final_norm_bias = fb.ctypes.data
+        if pair_table is not None:
+            if pair_table.shape[1] != c.hidden or pair_table.shape[0] < 2:
+                raise api.ShapeMismatch(f"pair table of shape {pair_table.shape}")
+            o.pair_table = self._weight(pair_table.shape[0], ld, [(0, 0, pair_table)]).handle()
+            o.pair_buckets = pair_table.shape[0] - 1
+            o.pair_mul_prev, o.pair_mul_cur = (int(m) % o.pair_buckets for m in pair_mul)   # (the row depends on the remainders only)
+        self.backend.check(self.backend._lib.nnq_decoder_set_head_options(self._handle, ctypes.byref(o)))
 
     def set_layer(self, *a, **k):
         raise api.Unsupported("a block decoder takes set_block")

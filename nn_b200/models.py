@@ -62,6 +62,12 @@ def _sikivik(config, folder, backend, max_seq, act_dtype, **options):
     return sikivik.load(config, os.path.join(folder, "model.safetensors"), backend, max_seq=max_seq, act_dtype=act_dtype, **options)
 
 
+@register_folder_model("Rugesun")
+def _rugesun(config, folder, backend, max_seq, act_dtype, **options):
+    from . import rugesun
+    return rugesun.load(config, os.path.join(folder, "model.safetensors"), backend, max_seq=max_seq, act_dtype=act_dtype, **options)
+
+
 @register_gguf_model("qwen3")
 def _qwen3(f, backend, max_seq, act_dtype, **options):
     from . import gguf
