@@ -1238,7 +1238,13 @@ def decode_tokens_per_s(torch, backend, layers, gen, dev, peak_hbm, prompt=2048,
     return out
 
 
-def run_sikivik(args, local_rank):
+BLOCK_MODELS = {
+    "sikivik": dict(beside=("qwen3",), config="sikivik blocks (attention, gla, gla, retention) x 2, width 4096"),
+    "rugesun": dict(beside=("sikivik", "qwen3"), config="rugesun layers (latent attention + dense, experts, dense, experts on shared latents) x 2, width 4096"),
+}
+
+
+def run_block_model(args, local_rank):
     """Prompt passes of 4096 tokens and greedy decoding behind them, random weights; `value` is the decode rate of
     the larger size, everything else is under `sizes`."""
     import torch
@@ -1247,14 +1253,14 @@ def run_sikivik(args, local_rank):
     torch.cuda.set_device(local_rank)
     prompt, new = 4096, 128
     with ClockSampler(local_rank) as clk:
-        sizes = blockbench.run(prompt, new, reps=max(3, args.steps // 4))
+        sizes = blockbench.run(prompt, new, reps=max(3, args.steps // 4), model=args.model, beside=BLOCK_MODELS[args.model]["beside"])
     peak, which = _peaks()
-    big = sizes["width 4096"]["sikivik"]
+    big = sizes["width 4096"][args.model]
     print(json.dumps({
         "metric": "decode_tokens_per_s", "value": big["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
         "dtype": "bf16", "data": "synthetic", "clocks": clk.summary(), "sizes": sizes,
         "roofline": {"bound": "hbm", "achieved_gbs": big["decode_weight_gbs"], "peak_gbs": peak, "peak": which, "frac": big["decode_weight_gbs"] / peak},
-        "config": {"model": "sikivik blocks (attention, gla, gla, retention) x 2, width 4096", "prompt": prompt, "new_tokens": new,
+        "config": {"model": BLOCK_MODELS[args.model]["config"], "prompt": prompt, "new_tokens": new,
                    "baseline": "8 Qwen3 layers of equal width, heads and feed-forward, bf16 weights", "l2": "weights larger than L2"}}))
 
 
@@ -1270,9 +1276,9 @@ def main():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--no-others", action="store_true")
-    ap.add_argument("--model", default="projections", choices=["projections", "sikivik"],
-                    help="sikivik: prefill and decode throughput of the block decoder at real layer sizes beside a "
-                         "Qwen3-shaped decoder with bf16 weights (one GPU; a JSON line of its own)")
+    ap.add_argument("--model", default="projections", choices=["projections", *BLOCK_MODELS],
+                    help="sikivik, rugesun: prefill and decode throughput of that block decoder at real layer sizes beside the "
+                         "other decoders at equal size with bf16 weights (one GPU; a JSON line of its own)")
     ap.add_argument("--no-fused", action="store_true", help="N > 1: separate all-reduce kernel after the row-parallel products")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
@@ -1281,8 +1287,8 @@ def main():
     if args.impl == "reference":
         run_reference(args, rank)
         return
-    if args.model == "sikivik":
-        run_sikivik(args, local_rank)
+    if args.model in BLOCK_MODELS:
+        run_block_model(args, local_rank)
         return
     if world != args.gpus:
         if args.gpus > 1:

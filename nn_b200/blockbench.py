@@ -1,6 +1,6 @@
-"""Prefill and decode throughput of the Sikivik design at sizes of real layers (random weights), beside a
+"""Prefill and decode throughput of the Sikivik and Rugesun designs at sizes of real layers (random weights), beside a
 Qwen3-shaped decoder of equal width, heads and feed-forward with unquantized bf16 weights. Used by
-`bench.py --model sikivik`; `python -m nn_b200.blockbench --once SIZE` issues one prompt pass and a few
+`bench.py --model sikivik | rugesun`; `python -m nn_b200.blockbench --once SIZE` issues one prompt pass and a few
 decode steps of one model (a launch list under a profiler)."""
 from __future__ import annotations
 
@@ -11,7 +11,8 @@ import time
 import numpy as np
 
 from . import api
-from .decoder import BlockConfig, BlockDecoder, BlockTensors, Decoder, DecoderConfig, MIXER_ATTENTION, MIXER_RECURRENT
+from .decoder import (ACT_GELU_TANH, BlockConfig, BlockDecoder, BlockTensors, Decoder, DecoderConfig, MIXER_ATTENTION, MIXER_LATENT, MIXER_NONE,
+                      MIXER_RECURRENT)
 from .formats import QuantFormat
 
 # layers: two periods of (attention, gla, gla, retention); Qwen3: as many layers of its own
@@ -20,6 +21,12 @@ SIZES = {
     "width 4096": dict(hidden=4096, ff=12288, heads=32, kv=8, rec_heads=16, rec_dim=128, rec_vdim=256, window=1024, rank=16, vocab=32768),
 }
 PERIODS = 2
+# Rugesun: two periods of (dense, experts, dense, experts on the latents of the layer in front); every layer's attention
+# has the heads and the window of the size above
+LATENT = {
+    "width 2048": dict(dim=128, rot=64, vdim=128, q_rank=768, kv_rank=512, experts=32, top=4, expert_ff=768),
+    "width 4096": dict(dim=128, rot=64, vdim=128, q_rank=1536, kv_rank=512, experts=32, top=4, expert_ff=1536),
+}
 
 
 def _bits(rng, *shape):
@@ -55,6 +62,44 @@ def block_model(backend, z, max_seq, act_dtype=api.BF16, seed=0):
     return dec
 
 
+def rugesun_blocks(z, y):
+    mix = dict(mixer=MIXER_LATENT, heads=z["heads"], dim=y["dim"], vdim=y["vdim"], rot_dims=y["rot"], rot_base=1e6, scale=(y["dim"] + y["rot"]) ** -0.5,
+               window=z["window"], post_norm=True, alpha=1.5, q_rank=y["q_rank"], kv_rank=y["kv_rank"])
+    dense = dict(mixer=MIXER_NONE, post_norm=True, alpha=1.5, ffn=z["ff"], ffn_act=ACT_GELU_TANH)
+    moe = dict(mixer=MIXER_NONE, post_norm=True, alpha=1.5, experts=y["experts"], top=y["top"], expert_ffn=y["expert_ff"])
+    out = []
+    for _ in range(PERIODS):
+        at = len(out)
+        for k, f in enumerate((dense, moe, dense, moe)):
+            out += [BlockConfig(**mix, kv_from=at + 4 if k == 3 else -1), BlockConfig(**f)]
+    return out
+
+
+def rugesun_model(backend, z, max_seq, act_dtype=api.BF16, seed=0):
+    D, y = z["hidden"], z["latent"]
+    blocks = rugesun_blocks(z, y)
+    dec = BlockDecoder(backend, hidden=D, vocab=z["vocab"], blocks=blocks, max_seq=max_seq, rms_eps=1e-5, act_dtype=act_dtype)
+    rng = np.random.default_rng(seed)
+    one, zero = np.ones(D, np.float32), np.zeros(D, np.float32)
+    experts = [(_bits(rng, y["expert_ff"], D), _bits(rng, y["expert_ff"], D), _bits(rng, D, y["expert_ff"])) for _ in range(y["experts"])]
+    for i, b in enumerate(blocks):
+        t = BlockTensors(norm=one, norm_bias=zero)
+        if b.mixer == MIXER_LATENT:
+            H = b.heads
+            t.dq, t.uq, t.q_norm = _bits(rng, b.q_rank, D), _bits(rng, H * (b.dim + b.rot_dims), b.q_rank), np.ones(b.q_rank, np.float32)
+            t.uk, t.uv, t.o = _bits(rng, H * b.dim, b.kv_rank), _bits(rng, H * b.vdim, b.kv_rank), _bits(rng, D, H * b.vdim)
+            if b.kv_from < 0:
+                t.dkv, t.kv_norm = _bits(rng, b.kv_rank + b.rot_dims, D), np.ones(b.kv_rank, np.float32)
+        elif b.experts:
+            t.router, t.expert = rng.standard_normal((b.experts, D)).astype(np.float32) * 0.02, experts.__getitem__
+        else:
+            t.gate, t.up, t.down = _bits(rng, b.ffn, D), _bits(rng, b.ffn, D), _bits(rng, D, b.ffn)
+        dec.set_block(i, t)
+    e = _bits(rng, z["vocab"], D)
+    dec.set_head(e, one, e, final_norm_bias=zero, logit_cap=30.0, pair_table=_bits(rng, 4097, D), pair_mul=(31, 7))
+    return dec
+
+
 def qwen3_model(backend, z, max_seq, act_dtype=api.BF16, seed=0):
     import torch
     D, F, H, G, n = z["hidden"], z["ff"], z["heads"], z["kv"], 4 * PERIODS
@@ -78,6 +123,15 @@ def qwen3_model(backend, z, max_seq, act_dtype=api.BF16, seed=0):
 def weight_bytes(name, z):
     """Bytes of the weights one decoded token streams (bf16, the vocabulary projection included)."""
     D, F = z["hidden"], z["ff"]
+    if name == "rugesun":
+        y, H, total = z["latent"], z["heads"], 0
+        for b in rugesun_blocks(z, y):
+            if b.mixer == MIXER_LATENT:
+                total += D * b.q_rank + H * (b.dim + b.rot_dims) * b.q_rank + H * (b.dim + b.vdim) * b.kv_rank + D * H * b.vdim
+                total += D * (b.kv_rank + b.rot_dims) if b.kv_from < 0 else 0
+            else:
+                total += 3 * D * (b.ffn or b.top * b.expert_ffn) + 2 * D * b.experts   # (the router is f32)
+        return 2 * total + 2 * D * z["vocab"]
     if name == "qwen3":
         per = 2 * D * (2 * z["heads"] * 128 + 2 * z["kv"] * 128 + 3 * F) * 4
     else:
@@ -88,14 +142,14 @@ def weight_bytes(name, z):
 
 
 def product_flops(name, z):
-    """Multiply-adds of the layers' products per prompt token, times two."""
+    """Multiply-adds of the layers' products per prompt token, times two (chosen experts only)."""
     return weight_bytes(name, z) - 2 * z["hidden"] * z["vocab"]
 
 
 def measure(backend, name, z, prompt, new_tokens, reps=5):
     import torch
     dev = torch.device("cuda", backend.device)
-    dec = (qwen3_model if name == "qwen3" else block_model)(backend, z, prompt + new_tokens + 16)
+    dec = MODELS[name](backend, z, prompt + new_tokens + 16)
     ids = np.random.default_rng(7).integers(0, z["vocab"], prompt).tolist()
     st = torch.cuda.Stream(device=dev)
     for _ in range(3):
@@ -134,20 +188,24 @@ def measure(backend, name, z, prompt, new_tokens, reps=5):
             "decode_launches": int(launches)}
 
 
-def run(prompt=4096, new_tokens=128, reps=5):
+MODELS = {"sikivik": block_model, "rugesun": rugesun_model, "qwen3": qwen3_model}
+
+
+def run(prompt=4096, new_tokens=128, reps=5, model="sikivik", beside=("qwen3",)):
     backend = api.gpu_backend()
     out = {}
-    for size, z in SIZES.items():
-        out[size] = {n: measure(backend, n, z, prompt, new_tokens, reps) for n in ("sikivik", "qwen3")}
-        r = out[size]
-        out[size]["sikivik_over_qwen3"] = {k: r["sikivik"][k] / r["qwen3"][k] for k in ("prefill_tokens_per_s", "decode_tokens_per_s")}
+    for size in SIZES:
+        z = dict(SIZES[size], latent=LATENT[size])
+        r = out[size] = {n: measure(backend, n, z, prompt, new_tokens, reps) for n in (model, *beside)}
+        for n in beside:
+            r[f"{model}_over_{n}"] = {k: r[model][k] / r[n][k] for k in ("prefill_tokens_per_s", "decode_tokens_per_s")}
     return out
 
 
 def main():
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--once", choices=sorted(SIZES))
-    ap.add_argument("--which", default="sikivik", choices=["sikivik", "qwen3"])
+    ap.add_argument("--which", default="sikivik", choices=sorted(MODELS))
     ap.add_argument("--prompt", type=int, default=1024)
     ap.add_argument("--new", type=int, default=2)
     a = ap.parse_args()
@@ -155,7 +213,7 @@ def main():
         print(json.dumps(run()))
         return
     b = api.gpu_backend()
-    dec = (qwen3_model if a.which == "qwen3" else block_model)(b, SIZES[a.once], a.prompt + a.new + 8)
+    dec = MODELS[a.which](b, dict(SIZES[a.once], latent=LATENT[a.once]), a.prompt + a.new + 8)
     t0 = time.perf_counter()
     dec.prefill(np.random.default_rng(7).integers(0, SIZES[a.once]["vocab"], a.prompt).tolist(), 0, 0)
     for _ in range(a.new):

@@ -795,7 +795,7 @@ static nnq_status check_block(nnq_ctx *ctx, int l, const nnq_block_config &b) {
     }
     if (b.experts || b.ffn_act != NNQ_ACT_SILU) return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: experts and other activations than silu stand in blocks without a mixer", l);
     if (b.mixer == NNQ_MIXER_LATENT) {
-        if (b.heads < 1 || b.dim < 1 || b.vdim < 1 || b.ffn || b.q_rank < 1 || b.kv_rank < 1 || b.window < 0) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad sizes", l);
+        if (b.heads < 1 || b.dim < 1 || b.vdim < 1 || b.ffn || b.q_rank < 1 || b.kv_rank < 1 || b.window < 0 || !(b.scale > 0.0f)) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad sizes", l);
         if (b.rot_dims < 0 || b.rot_dims % 2 || (b.rot_dims && !(b.rot_base > 0.0))) return fail(ctx, NNQ_ERR_INVALID_ARG, "block %d: bad rotation", l);
         if (b.vdim > kAttnMaxDim || b.dim + b.rot_dims > 2 * kAttnMaxDim) return fail(ctx, NNQ_ERR_UNSUPPORTED, "block %d: attention heads of %d + %d / %d are above %d / %d", l, b.dim, b.rot_dims, b.vdim, 2 * kAttnMaxDim, kAttnMaxDim);
         return NNQ_OK;
