@@ -411,8 +411,11 @@ NNQ_API void nnq_plan_destroy(nnq_plan *p);
  *   NNQ_MXFP4_GPTOSS.
  * NNQ_MOE_NK: gate_up is [E, 2*inter, hidden] and down is [E, hidden, inter], each expert an
  *   [N, K] weight in any nnq_format with blocks along K (the [N,K/2]+[N,K/32] MXFP4 contract of
- *   crates/nn-metal/src/mxfp4_gemm_msl.rs:47-61 when fmt = NNQ_MXFP4_SPLIT). */
-typedef enum nnq_moe_layout { NNQ_MOE_KN_GPTOSS = 0, NNQ_MOE_NK = 1 } nnq_moe_layout;
+ *   crates/nn-metal/src/mxfp4_gemm_msl.rs:47-61 when fmt = NNQ_MXFP4_SPLIT).
+ * NNQ_MOE_NK_PAIRS: as NNQ_MOE_NK with the gate and up rows of an expert alternating (row 2j: gate j, row 2j + 1:
+ *   up j), bf16 (NNQ_BF16_DENSE), hidden and inter multiples of 64, whole blocks only; the expert biases may be NULL
+ *   (the gate_up bias alternates like the rows). The experts are multiplied in place. */
+typedef enum nnq_moe_layout { NNQ_MOE_KN_GPTOSS = 0, NNQ_MOE_NK = 1, NNQ_MOE_NK_PAIRS = 2 } nnq_moe_layout;
 
 /* Build the MoE block of one decoder layer. All tensors may be host or device memory and are
  * copied. router_w [E, hidden] and router_b [E] are f32; gate_up_bias [E, 2*inter] and down_bias
@@ -687,7 +690,7 @@ typedef struct nnq_block_weights {
     const nnq_weight *uq, *ukv;   /* latent; stay owned by the caller */
     const float *q_norm;      /* [q_rank] */
     const float *kv_norm;     /* [kv_rank], NULL with kv_from */
-    const nnq_moe *moe;       /* mixture of experts: hidden = in_k, [E, N, K] bf16 experts; stays owned by the caller */
+    const nnq_moe *moe;       /* mixture of experts: NNQ_MOE_NK_PAIRS of hidden = in_k; stays owned by the caller */
 } nnq_block_weights;
 /* `blocks` holds cfg->n_layers entries. block_rows: prompt rows that go through the blocks together (0 =
  * 1024). An attention block keeps a ring of min(max_seq, window - 1 + block_rows) keys and values. */

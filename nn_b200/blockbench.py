@@ -14,6 +14,7 @@ from . import api
 from .decoder import (ACT_GELU_TANH, BlockConfig, BlockDecoder, BlockTensors, Decoder, DecoderConfig, MIXER_ATTENTION, MIXER_LATENT, MIXER_NONE,
                       MIXER_RECURRENT)
 from .formats import QuantFormat
+from .safetensors import bf16_to_f32
 
 # layers: two periods of (attention, gla, gla, retention); Qwen3: as many layers of its own
 SIZES = {
@@ -91,7 +92,7 @@ def rugesun_model(backend, z, max_seq, act_dtype=api.BF16, seed=0):
             if b.kv_from < 0:
                 t.dkv, t.kv_norm = _bits(rng, b.kv_rank + b.rot_dims, D), np.ones(b.kv_rank, np.float32)
         elif b.experts:
-            t.router, t.expert = rng.standard_normal((b.experts, D)).astype(np.float32) * 0.02, experts.__getitem__
+            t.router, t.expert = bf16_to_f32(_bits(rng, b.experts, D)), experts.__getitem__
         else:
             t.gate, t.up, t.down = _bits(rng, b.ffn, D), _bits(rng, b.ffn, D), _bits(rng, D, b.ffn)
         dec.set_block(i, t)

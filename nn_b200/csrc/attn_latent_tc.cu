@@ -5,13 +5,13 @@
 // enter the second product as two bf16 terms (p = hi + lo, remainder below 2^-16 of p), accumulation is f32.
 //
 // One CTA: 128 query rows of one head, key tiles of 64 over the union of the rows' windows.
-//   warps 0-3: softmax. Thread r owns row r: scores of tile t from tensor memory, maximum, sum, weights as two
-//              swizzled tiles; then the weighted values of tile t - 1 from tensor memory into its f32 accumulators.
-//   warp 4:    one thread issues the TMA loads: key tiles (64-wide pieces of the head's part, then the shared part) and
+//   warps 0-7: softmax. Two threads share a row, one per half of a tile's keys (they exchange their maxima) and of the
+//              value dimensions: scores of tile t from tensor memory, maximum, sum, weights as two swizzled tiles; then
+//              the weighted values of tile t - 1 from tensor memory into f32 accumulators.
+//   warp 8:    one thread issues the TMA loads: key tiles (64-wide pieces of the head's part, then the shared part) and
 //              value tiles, two stages each.
-//   warp 5:    one thread issues the MMAs: S(t + 2) = Q K^T right behind O(t) = P V. Values are the MN-major operand,
+//   warp 9:    one thread issues the MMAs: S(t + 2) = Q K^T right behind O(t) = P V. Values are the MN-major operand,
 //              so their tiles stay as they lie in memory.
-//   warps 6-7: only help to stage the queries.
 // Scores, weights and weighted values have two buffers each, so the tensor cores work on tile t while the softmax
 // warps are at t + 1. The barrier of S(t) also frees the key stage, that of O(t) the value stage. Every wait is bounded.
 #include <cuda.h>
@@ -24,11 +24,12 @@
 
 namespace nnq {
 
-constexpr int kLtKeys = 64, kLtRows = 128, kLtThreads = 256;
+constexpr int kLtKeys = 64, kLtRows = 128, kLtSoft = 256, kLtThreads = kLtSoft + 64;
 constexpr int kLtQAtom = kLtRows * 128, kLtKAtom = kLtKeys * 128;   // bytes of a tile of 64 columns (one swizzle row)
 constexpr int kLtMaxAtoms = 4;                                      // 64-wide pieces of a key
 
-static int lt_smem_bytes(int atoms, int nv) { return 1024 + atoms * kLtQAtom + 2 * (atoms + nv) * kLtKAtom + 4 * kLtQAtom; }
+// (the largest case, four pieces and two value pieces, takes all there is beside the static part)
+static int lt_smem_bytes(int atoms, int nv) { return atoms * kLtQAtom + 2 * (atoms + nv) * kLtKAtom + 4 * kLtQAtom; }
 
 __device__ __forceinline__ void lt_tma_2d(uint32_t dst, const CUtensorMap *map, int x, int y, uint32_t bar) {
     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
@@ -76,9 +77,14 @@ template <int NV>
 __global__ void __launch_bounds__(kLtThreads, 1)
 attn_latent_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap r_map, const LatentAttn a, int *status) {
     extern __shared__ __align__(1024) uint8_t lt_smem_raw[];
-    uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(lt_smem_raw) + 1023) & ~(uintptr_t)1023);
+    uint8_t *smem = lt_smem_raw;
+    if (smem_u32(smem) & 1023u) {   // the swizzled tiles start at multiples of 1024 bytes
+        if (threadIdx.x == 0) atomicExch(status, 1);
+        return;
+    }
     __shared__ __align__(8) uint64_t bars[11];   // k_full[2], v_full[2], s_full[2], o_full[2], p_full[2], drain
     __shared__ uint32_t tmem_s;
+    __shared__ float half_max[2][2][kLtRows], half_sum[kLtRows];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t kf = smem_u32(bars), vf = kf + 16, sf = kf + 32, of = kf + 48, pf = kf + 64, drain = kf + 80;
     const int h = blockIdx.x, row0 = blockIdx.y * kLtRows, rows = min(kLtRows, a.span.n - row0);
@@ -90,29 +96,39 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_c
 
     if (tid == 0) {
         for (int i = 0; i < 8; i++) mbar_init(kf + 8 * i, 1);
-        for (int i = 0; i < 2; i++) mbar_init(pf + 8 * i, 128);
+        for (int i = 0; i < 2; i++) mbar_init(pf + 8 * i, kLtSoft);
         mbar_init(drain, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    if (warp == 5) {
+    if (warp == 9) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_s)), "r"(512u) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    // the queries; a piece ends where the unrotated part ends, so the rotated part starts a piece of its own
-    for (int u = tid; u < kLtRows * 16 * atoms; u += kLtThreads) {
-        const int r = u / (16 * atoms), c = u - r * 16 * atoms, at = c >> 4, e = 4 * (c & 15);
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (r < rows) {
+    // the queries; a piece ends where the unrotated part ends, so the rotated part starts a piece of its own. A batch of
+    // loads is under way before the first is used.
+    constexpr int QB = 6;
+    for (int u0 = tid; u0 < kLtRows * 16 * atoms; u0 += QB * kLtThreads) {
+        float4 v[QB];
+#pragma unroll
+        for (int i = 0; i < QB; i++) {
+            const int u = u0 + i * kLtThreads, r = u / (16 * atoms), c = u - r * 16 * atoms, at = c >> 4, e = 4 * (c & 15);
+            v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (r >= rows) continue;
             const int d = at < da ? 64 * at + e : a.dim + 64 * (at - da) + e;
             const float *q = a.q + ((size_t)(row0 + r) * a.heads + h) * (a.dim + a.rot);
             if (at >= da) {
-                v = lt_query4(a, q, d, pos_first + r);
+                v[i] = lt_query4(a, q, d, pos_first + r);
             } else if (d < a.dim) {
-                if (d + 4 <= a.dim && ((a.dim | a.rot) & 3) == 0) v = *reinterpret_cast<const float4 *>(q + d);
-                else v = make_float4(q[d], d + 1 < a.dim ? q[d + 1] : 0.0f, d + 2 < a.dim ? q[d + 2] : 0.0f, d + 3 < a.dim ? q[d + 3] : 0.0f);
+                if (d + 4 <= a.dim && ((a.dim | a.rot) & 3) == 0) v[i] = *reinterpret_cast<const float4 *>(q + d);
+                else v[i] = make_float4(q[d], d + 1 < a.dim ? q[d + 1] : 0.0f, d + 2 < a.dim ? q[d + 2] : 0.0f, d + 3 < a.dim ? q[d + 3] : 0.0f);
             }
         }
-        *reinterpret_cast<uint2 *>(q_s + at * kLtQAtom + swz(r, e >> 3) + 2 * (e & 7)) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+#pragma unroll
+        for (int i = 0; i < QB; i++) {
+            const int u = u0 + i * kLtThreads, r = u / (16 * atoms), c = u - r * 16 * atoms, at = c >> 4, e = 4 * (c & 15);
+            if (r < kLtRows)
+                *reinterpret_cast<uint2 *>(q_s + at * kLtQAtom + swz(r, e >> 3) + 2 * (e & 7)) = make_uint2(pack_bf16(v[i].x, v[i].y), pack_bf16(v[i].z, v[i].w));
+        }
     }
     fence_async_smem();
     tc_fence_before();
@@ -121,101 +137,110 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_c
     const uint32_t tmem = tmem_s, o_tmem = tmem + 128;   // scores: two of 64 columns, weighted values: two of 64 NV
     bool ok = true;
 
-    if (warp < 4) {
+    if (warp < 8) {
         // ---------------- softmax ----------------
-        const int my_hi = pos_first + tid, my_lo = my_hi - a.window + 1;   // keys this row sees (rows past the end are not stored)
+        const int row = tid & 127, half = tid >> 7;                        // half: keys 32 half .. + 31 of a tile, value dimensions 32 NV half ..
+        const int my_hi = pos_first + row, my_lo = my_hi - a.window + 1;   // keys this row sees (rows past the end are not stored)
         const float c = a.scale * 1.4426950408889634f;
-        const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
-        float acc[NV * 64];
+        const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
+        float acc[NV * 32];
 #pragma unroll
-        for (int i = 0; i < NV * 64; i++) acc[i] = 0.0f;
+        for (int i = 0; i < NV * 32; i++) acc[i] = 0.0f;
         float m = -INFINITY, l = 0.0f, corr = 1.0f;
         auto add_values = [&](int t) {   // weighted values of tile t, weights relative to the maximum after tile t
-            if (!__all_sync(0xFFFFFFFFu, mbar_wait_fast(of + 8 * (t & 1), (t >> 1) & 1))) return false;   // (a warp agrees)
+            ok = ok && __all_sync(0xFFFFFFFFu, mbar_wait_fast(of + 8 * (t & 1), (t >> 1) & 1));   // (a warp agrees)
+            if (!ok) return;
             tc_fence_after();
 #pragma unroll
-            for (int b = 0; b < NV * 2; b++) {
+            for (int b = 0; b < NV; b++) {
                 uint32_t v[32];
-                tmem_ld32(o_tmem + (t & 1) * NV * 64 + lane_base + b * 32, v);
+                tmem_ld32(o_tmem + (t & 1) * NV * 64 + half * NV * 32 + lane_base + b * 32, v);
 #pragma unroll
                 for (int i = 0; i < 32; i++) acc[b * 32 + i] = fmaf(acc[b * 32 + i], corr, __uint_as_float(v[i]));
             }
-            return true;
         };
+        // every warp comes to the barrier of every tile, also after a wait that ran out (then without waiting again)
         for (int t = 0; t < tiles; t++) {
-            if (!__all_sync(0xFFFFFFFFu, mbar_wait_fast(sf + 8 * (t & 1), (t >> 1) & 1))) {
-                ok = false;
-                break;
-            }
-            tc_fence_after();
-            const int k0 = first + t * kLtKeys;
-            const int lo = my_lo - k0, hi = my_hi - k0;   // visible keys of the tile
-            uint32_t s[2][32];
-            tmem_ld32(tmem + (t & 1) * 64 + lane_base, s[0]);
-            tmem_ld32(tmem + (t & 1) * 64 + lane_base + 32, s[1]);
+            ok = ok && __all_sync(0xFFFFFFFFu, mbar_wait_fast(sf + 8 * (t & 1), (t >> 1) & 1));
+            uint32_t s[32];
             float mt = -INFINITY;
-            if (__all_sync(0xFFFFFFFFu, lo <= 0 && hi >= kLtKeys - 1)) {
+            if (ok) {
+                tc_fence_after();
+                const int k0 = first + t * kLtKeys + 32 * half;
+                const int lo = my_lo - k0, hi = my_hi - k0;   // visible keys of this half
+                tmem_ld32(tmem + (t & 1) * 64 + 32 * half + lane_base, s);
+                if (__all_sync(0xFFFFFFFFu, lo <= 0 && hi >= 31)) {
 #pragma unroll
-                for (int i = 0; i < 64; i++) mt = fmaxf(mt, __uint_as_float(s[i >> 5][i & 31]));
-            } else {
+                    for (int i = 0; i < 32; i++) mt = fmaxf(mt, __uint_as_float(s[i]));
+                } else {
 #pragma unroll
-                for (int i = 0; i < 64; i++) {
-                    const float x = i >= lo && i <= hi ? __uint_as_float(s[i >> 5][i & 31]) : -INFINITY;
-                    s[i >> 5][i & 31] = __float_as_uint(x);
-                    mt = fmaxf(mt, x);
+                    for (int i = 0; i < 32; i++) {
+                        const float x = i >= lo && i <= hi ? __uint_as_float(s[i]) : -INFINITY;
+                        s[i] = __float_as_uint(x);
+                        mt = fmaxf(mt, x);
+                    }
                 }
             }
-            mt = mt == -INFINITY ? mt : mt * c;          // (c > 0)
+            half_max[t & 1][half][row] = mt;
+            asm volatile("bar.sync 1, %0;" ::"n"(kLtSoft) : "memory");
+            if (!ok) continue;
+            mt = fmaxf(mt, half_max[t & 1][half ^ 1][row]);
+            mt = mt == -INFINITY ? mt : mt * c;                // (c > 0)
             const float mn = fmaxf(m, mt);
             const float next = m == mn ? 1.0f : ex2(m - mn);   // no key of this row yet: both -inf
             const float base = mn == -INFINITY ? 0.0f : mn;
             float sum = 0.0f;
             uint8_t *p_t = p_s + (t & 1) * 2 * kLtQAtom;
 #pragma unroll
-            for (int ch = 0; ch < 8; ch++) {
+            for (int ch = 0; ch < 4; ch++) {
                 uint4 hv, lv;
                 uint32_t *hp = &hv.x, *lp = &lv.x;
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int i = ch * 8 + 2 * e;
-                    const float p0 = ex2(fmaf(__uint_as_float(s[i >> 5][i & 31]), c, -base)), p1 = ex2(fmaf(__uint_as_float(s[i >> 5][(i & 31) + 1]), c, -base));
+                    const float p0 = ex2(fmaf(__uint_as_float(s[i]), c, -base)), p1 = ex2(fmaf(__uint_as_float(s[i + 1]), c, -base));
                     sum += p0 + p1;
                     hp[e] = pack_bf16(p0, p1);
                     lp[e] = pack_bf16(p0 - __uint_as_float(hp[e] << 16), p1 - __uint_as_float(hp[e] & 0xFFFF0000u));
                 }
-                *reinterpret_cast<uint4 *>(p_t + swz(tid, ch)) = hv;
-                *reinterpret_cast<uint4 *>(p_t + kLtQAtom + swz(tid, ch)) = lv;
+                *reinterpret_cast<uint4 *>(p_t + swz(row, 4 * half + ch)) = hv;
+                *reinterpret_cast<uint4 *>(p_t + kLtQAtom + swz(row, 4 * half + ch)) = lv;
             }
             fence_async_smem();
             tc_fence_before();
             mbar_arrive(pf + 8 * (t & 1));
-            if (t > 0 && !add_values(t - 1)) {
-                ok = false;
-                break;
-            }
+            if (t > 0) add_values(t - 1);
             l = l * next + sum;
             m = mn;
             corr = next;   // tile t's weighted values join sums that are still relative to the maximum before it
         }
-        ok = ok && add_values(tiles - 1);
-        if (ok && tid < rows) {
-            const float inv = 1.0f / l;
-            __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(a.out) + (size_t)(row0 + tid) * a.out_ld + h * a.vdim;
+        add_values(tiles - 1);
+        if (half) half_sum[row] = l;
+        asm volatile("bar.sync 1, %0;" ::"n"(kLtSoft) : "memory");
+        if (!half) {
+            l += half_sum[row];
+            half_max[0][0][row] = l;
+        }
+        asm volatile("bar.sync 1, %0;" ::"n"(kLtSoft) : "memory");
+        if (ok && row < rows) {
+            const float inv = 1.0f / half_max[0][0][row];
+            const int v0 = half * NV * 32;
+            __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(a.out) + (size_t)(row0 + row) * a.out_ld + h * a.vdim;
             if ((a.vdim & 7) == 0) {
 #pragma unroll
-                for (int d = 0; d < NV * 64; d += 8)
-                    if (d < a.vdim)
-                        *reinterpret_cast<uint4 *>(o + d) = make_uint4(pack_bf16(acc[d] * inv, acc[d + 1] * inv), pack_bf16(acc[d + 2] * inv, acc[d + 3] * inv),
-                                                                       pack_bf16(acc[d + 4] * inv, acc[d + 5] * inv), pack_bf16(acc[d + 6] * inv, acc[d + 7] * inv));
+                for (int d = 0; d < NV * 32; d += 8)
+                    if (v0 + d < a.vdim)
+                        *reinterpret_cast<uint4 *>(o + v0 + d) = make_uint4(pack_bf16(acc[d] * inv, acc[d + 1] * inv), pack_bf16(acc[d + 2] * inv, acc[d + 3] * inv),
+                                                                            pack_bf16(acc[d + 4] * inv, acc[d + 5] * inv), pack_bf16(acc[d + 6] * inv, acc[d + 7] * inv));
             } else {
 #pragma unroll
-                for (int d = 0; d < NV * 64; d++)
-                    if (d < a.vdim) o[d] = __float2bfloat16_rn(acc[d] * inv);
+                for (int d = 0; d < NV * 32; d++)
+                    if (v0 + d < a.vdim) o[v0 + d] = __float2bfloat16_rn(acc[d] * inv);
             }
-            if (h == a.heads - 1)
+            if (half && h == a.heads - 1)
                 for (int d = a.vdim; d < a.out_ld - h * a.vdim; d++) o[d] = __float2bfloat16_rn(0.0f);
         }
-    } else if (warp == 4 && lane == 0) {
+    } else if (warp == 8 && lane == 0) {
         // ---------------- TMA loads ----------------
         const int vcol = a.heads * a.dim_ld + h * a.vdim_ld;
         int t = 0;
@@ -241,7 +266,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_c
                 ok = mbar_wait(kf + 8 * (k & 1), (k >> 1) & 1) && ok;
                 ok = mbar_wait(vf + 8 * (k & 1), (k >> 1) & 1) && ok;
             }
-    } else if (warp == 5 && lane == 0) {
+    } else if (warp == 9 && lane == 0) {
         // ---------------- MMA issuer ----------------
         const uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kLtKeys >> 3) << 17) | ((128u >> 4) << 24);
         const uint32_t id_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(NV * 64 >> 3) << 17) | ((128u >> 4) << 24);   // B is MN-major
@@ -285,7 +310,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_c
     if (!ok) atomicExch(status, 1);
     tc_fence_before();
     __syncthreads();
-    if (warp == 5) {
+    if (warp == 9) {
         tc_fence_after();
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
     }

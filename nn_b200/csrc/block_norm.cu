@@ -6,11 +6,12 @@
 
 namespace nnq {
 
-__device__ __forceinline__ void store_units(const NormRow &r, void *xn, int act_dt, int xn_ld, float *red) {
-    float4 v[8];
+template <int K>
+__device__ __forceinline__ void store_units(const NormRow &r, void *xn, int act_dt, float *red) {
+    float4 v[K];
     norm_units(r, v, red);
 #pragma unroll
-    for (int k = 0; k < 8; k++) {
+    for (int k = 0; k < K; k++) {
         const int u = threadIdx.x + blockDim.x * k;
         if (4 * u >= r.hidden) continue;
         if (act_dt == NNQ_F32) {
@@ -23,7 +24,9 @@ __device__ __forceinline__ void store_units(const NormRow &r, void *xn, int act_
 }
 
 // One CTA of 256 per row (the row of a step: `state` given, token state[0], position state[1], the token before it
-// state[4]). With `rows` given CTA i norms row rows[i] into row i of xn and leaves h as it is.
+// state[4]). With `rows` given CTA i norms row rows[i] into row i of xn and leaves h as it is. K: units of four elements
+// per thread, 0: any width, element by element.
+template <int K>
 __global__ void __launch_bounds__(256) norm_rows_kernel(const NormRows a, const int *__restrict__ tokens, int pos0, const int *__restrict__ rows,
                                                         const int *__restrict__ state) {
     pdl_prologue();
@@ -50,19 +53,27 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const NormRows a, const 
     n.eps = a.eps;
     n.hidden = a.hidden;
     char *xr = reinterpret_cast<char *>(a.xn) + (size_t)blockIdx.x * a.xn_ld * (a.act_dt == NNQ_F32 ? 4 : 2);
-    if (a.hidden % 4 == 0 && a.hidden <= 256 * 4 * 8) store_units(n, xr, a.act_dt, a.xn_ld, red);
+    if constexpr (K > 0) store_units<K>(n, xr, a.act_dt, red);
     else norm_elements(n, red, [&](int i, float v) { store_act(xr, a.act_dt, i, v); });
     for (int i = a.hidden + threadIdx.x; i < a.xn_ld; i += blockDim.x) store_act(xr, a.act_dt, i, 0.0f);
 }
 
+static void go_norm(const NormRows &a, int n, const int *tokens, int pos0, const int *rows, const int *state, cudaStream_t st) {
+    const dim3 grid(n), block(256);
+    if (a.hidden % 4 || a.hidden > 8192) launch_pdl(norm_rows_kernel<0>, grid, block, st, a, tokens, pos0, rows, state);
+    else if (a.hidden <= 2048) launch_pdl(norm_rows_kernel<2>, grid, block, st, a, tokens, pos0, rows, state);
+    else if (a.hidden <= 4096) launch_pdl(norm_rows_kernel<4>, grid, block, st, a, tokens, pos0, rows, state);
+    else launch_pdl(norm_rows_kernel<8>, grid, block, st, a, tokens, pos0, rows, state);
+}
+
 nnq_status launch_norm_step(nnq_ctx *ctx, const NormRows &a, const int *state, cudaStream_t st) {
-    launch_pdl(norm_rows_kernel, dim3(1), dim3(256), st, a, nullptr, 0, nullptr, state);
+    go_norm(a, 1, nullptr, 0, nullptr, state, st);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "norm launch");
 }
 
 nnq_status launch_norm_rows(nnq_ctx *ctx, const NormRows &a, int n, const int *tokens, int pos0, const int *rows, cudaStream_t st) {
-    launch_pdl(norm_rows_kernel, dim3(n), dim3(256), st, a, tokens, pos0, rows, nullptr);
+    go_norm(a, n, tokens, pos0, rows, nullptr, st);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "norm launch");
 }

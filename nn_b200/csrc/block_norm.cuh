@@ -67,14 +67,14 @@ __device__ __forceinline__ void norm_units(const NormRow &r, float4 (&v)[K], flo
 #pragma unroll
         for (int k = 0; k < K; k++) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
         const float mean = block_sum(s, red) / n;
-        const float sd = sqrtf(squares(mean) / n + r.eps);
+        const float inv = 1.0f / sqrtf(squares(mean) / n + r.eps);
 #pragma unroll
         for (int k = 0; k < K; k++) {
             const int i = 4 * (threadIdx.x + blockDim.x * k);
             if (i >= r.hidden) continue;
             const float4 g = *reinterpret_cast<const float4 *>(w + i), o = *reinterpret_cast<const float4 *>(b + i);
-            v[k] = make_float4(fmaf((v[k].x - mean) / sd, g.x, o.x), fmaf((v[k].y - mean) / sd, g.y, o.y), fmaf((v[k].z - mean) / sd, g.z, o.z),
-                               fmaf((v[k].w - mean) / sd, g.w, o.w));
+            v[k] = make_float4(fmaf((v[k].x - mean) * inv, g.x, o.x), fmaf((v[k].y - mean) * inv, g.y, o.y), fmaf((v[k].z - mean) * inv, g.z, o.z),
+                               fmaf((v[k].w - mean) * inv, g.w, o.w));
         }
     };
     if (r.post_w) layer_norm(r.post_w, r.post_b);

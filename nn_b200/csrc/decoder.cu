@@ -837,8 +837,8 @@ static nnq_block_layout layout_of(const nnq_block_config &b, int hidden) {
         y.gate = 0;
         y.up = 1;
         y.ffn_step = 2;
-        y.in_cols = round_up(2 * b.ffn, 8);
         y.out_k = round_up(b.ffn, 64);
+        y.in_cols = 2 * y.out_k;
         return y;
     }
     const bool attn = b.mixer == NNQ_MIXER_ATTENTION;
@@ -1073,7 +1073,7 @@ nnq_status nnq_decoder_set_block(nnq_decoder *d, int layer, const nnq_block_weig
     nnq_decoder::Block &B = d->blocks[layer];
     const nnq_block_config &b = B.cfg;
     if (b.experts) {
-        if (!w->moe || w->moe->hidden != B.lay.in_k || w->moe->n_experts != b.experts || w->moe->fmt != NNQ_BF16_DENSE)
+        if (!w->moe || w->moe->hidden != B.lay.in_k || w->moe->n_experts != b.experts || w->moe->layout != NNQ_MOE_NK_PAIRS)
             return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "block %d takes %d bf16 experts of width %d", layer, b.experts, B.lay.in_k);
     } else if (!shape_is(w->in, B.lay.in_cols, B.lay.in_k) || !shape_is(w->out, c.hidden, B.lay.out_k))
         return fail(ctx, NNQ_ERR_SHAPE_MISMATCH, "products of block %d must be [%d, %d] and [%d, %d]", layer, B.lay.in_cols, B.lay.in_k, c.hidden, B.lay.out_k);
@@ -1394,6 +1394,19 @@ static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *s
     return product(d, B.out, d->b_act, n, B.bias_out, delta, st);
 }
 
+// The residual update and norm of r for a product kernel that has them in its prologue. The new residual row goes to the
+// other of two buffers.
+static GemvNorm step_norm(nnq_decoder *d, const NormRows &r) {
+    GemvNorm g = {};
+    g.h_in = r.h; g.delta = r.delta; g.h_out = d->b_h2; g.alpha = r.alpha;
+    g.embed = r.embed; g.pairs = r.pairs; g.embed_ld = r.embed_ld; g.state = d->d_state;
+    g.post_w = r.post_w; g.post_b = r.post_b; g.in = r.in; g.eps = r.eps; g.hidden = r.hidden;
+    float *t = d->d_h;
+    d->d_h = d->b_h2;
+    d->b_h2 = t;
+    return g;
+}
+
 // y = what block l (l = n_layers: the head) reads times w^T for the step's row; where the residual update and the norm
 // are part of the product kernel the new residual row goes to the other of two buffers. pair_act: as in
 // launch_dense_gemv_norm; *activated tells whether y holds the activation.
@@ -1404,14 +1417,7 @@ static nnq_status step_norm_product(nnq_decoder *d, int l, const nnq_weight *w, 
     *activated = false;
     if (fused_steps(d) && dense_gemv_norm_supported(w, c.hidden)) {
         const TcArgs a = {w->d_raw, w->d_scales, nullptr, bias, pair_act ? act : y, 1, w->n, w->k, w->fmt, NNQ_BF16, NNQ_F32};
-        GemvNorm g = {};
-        g.h_in = r.h; g.delta = r.delta; g.h_out = d->b_h2; g.alpha = r.alpha;
-        g.embed = r.embed; g.pairs = r.pairs; g.embed_ld = r.embed_ld; g.state = d->d_state;
-        g.post_w = r.post_w; g.post_b = r.post_b; g.in = r.in; g.eps = r.eps; g.hidden = r.hidden;
-        nnq_status s = launch_dense_gemv_norm(d->ctx, a, g, pair_act, y_ld, st);
-        float *t = d->d_h;
-        d->d_h = d->b_h2;
-        d->b_h2 = t;
+        nnq_status s = launch_dense_gemv_norm(d->ctx, a, step_norm(d, r), pair_act, y_ld, st);
         *activated = pair_act > 0;
         return s;
     }
@@ -1426,6 +1432,10 @@ static nnq_status step_blocks(nnq_decoder *d, cudaStream_t st) {
         const nnq_decoder::Block &B = d->blocks[l];
         if (B.moe) {
             NormRows r = pending_rows(d, l, d->d_h, d->d_delta);
+            if (fused_steps(d) && moe_step_supported(B.moe, d->cfg.hidden)) {
+                if ((s = moe_step(d->ctx, B.moe, step_norm(d, r), d->d_delta, st)) != NNQ_OK) return s;
+                continue;
+            }
             r.xn = d->d_xn;
             if ((s = launch_norm_step(d->ctx, r, d->d_state, st)) != NNQ_OK) return s;
             if ((s = moe_rows(d->ctx, B.moe, d->d_xn, (nnq_dtype)d->act_dt, 1, d->act_dt == NNQ_F32, d->d_delta, st)) != NNQ_OK) return s;
@@ -1449,8 +1459,15 @@ static nnq_status rows_blocks(nnq_decoder *d, int n, int pos0, cudaStream_t st) 
         if (s == NNQ_OK && B.moe) {
             s = moe_rows(d->ctx, B.moe, d->pf_xn, (nnq_dtype)d->act_dt, n, d->act_dt == NNQ_F32, d->pf_delta, st);
         } else {
-            if (s == NNQ_OK) s = product(d, B.in, d->pf_xn, n, B.bias_in, d->b_proj, st);
-            if (s == NNQ_OK) s = run_block(d, l, n, pos0, nullptr, false, d->pf_delta, st);
+            // hundreds of rows: the activation in the product's epilogue
+            const bool fused = fused_steps(d) && B.cfg.mixer == NNQ_MIXER_NONE && gemm_dense_supported(d->ctx, B.in, n, d->act_dt);
+            if (s == NNQ_OK && fused) {
+                const TcArgs a = {B.in->d_raw, B.in->d_scales, d->pf_xn, nullptr, nullptr, n, B.in->n, B.in->k, B.in->fmt, NNQ_BF16, NNQ_BF16};
+                s = launch_gemm_dense_pairs(d->ctx, a, (__nv_bfloat16 *)d->b_act, B.cfg.ffn_act, st);
+            } else if (s == NNQ_OK) {
+                s = product(d, B.in, d->pf_xn, n, B.bias_in, d->b_proj, st);
+            }
+            if (s == NNQ_OK) s = run_block(d, l, n, pos0, nullptr, fused, d->pf_delta, st);
         }
         if (s != NNQ_OK) return s;
     }

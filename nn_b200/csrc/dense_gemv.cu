@@ -11,11 +11,14 @@
 // With NORM the kernel also does what stands in front of a decoder's product: every CTA adds the last block's output
 // to the residual row (or reads the embedding row), norms it and keeps the normed row as bf16 in shared memory; CTA 0
 // writes the new residual to another buffer (the others may still be reading the old one). Behind a gate / up product
-// with interleaved rows the epilogue forms the gated activation.
+// with interleaved rows the epilogue forms the gated activation. For a mixture of experts the rows (gate / up) or the
+// segments of the columns (down) belong to the experts the row is routed to: their addresses are known only behind the
+// wait, everything else is the same.
 #include <cuda_bf16.h>
 
 #include "block_norm.cuh"
 #include "gemm_tc.h"
+#include "route.cuh"
 #include "sync.cuh"
 
 namespace nnq {
@@ -30,16 +33,19 @@ __device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 
 // grid: rows dealt to CTAs in contiguous runs. ks: warps per row (power of two), passes: chunks of a warp.
 constexpr int kGvNormMax = 8192;   // width of the normed row: 16 values per thread
 
-template <int M, bool NORM>
+enum { kGvPlain = 0, kGvNorm = 1, kGvUp = 2, kGvDown = 3 };
+
+template <int M, int MODE>
 __global__ void __launch_bounds__(gv_warps(M) * 32, 1)
 dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__restrict__ x, const float *__restrict__ bias, void *__restrict__ y,
-                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm, int pair_act, int y_ld) {
+                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm, int pair_act, int y_ld, const GemvExperts ex) {
+    constexpr bool NORM = MODE == kGvNorm, PAIRS = MODE == kGvNorm || MODE == kGvUp;
     constexpr int kGvWarps = gv_warps(M), kGvStages = kGvTiles / kGvWarps;
     extern __shared__ __align__(128) uint8_t gv_smem[];
     __shared__ __align__(8) uint64_t bars[kGvWarps * kGvStages];
     float *part = reinterpret_cast<float *>(gv_smem + kGvRing);   // [rows of this CTA][ks][M]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int unit = NORM && pair_act ? 2 : 1;   // rows that stay together
+    const int unit = PAIRS && pair_act ? 2 : 1;   // rows that stay together
     const int r0 = (int)((long long)(N / unit) * blockIdx.x / gridDim.x) * unit, r1 = (int)((long long)(N / unit) * (blockIdx.x + 1) / gridDim.x) * unit;
     const int groups = kGvWarps / ks, group = warp / ks, kw = warp % ks;
     const int rows = r1 - r0 > group ? (r1 - r0 - group + groups - 1) / groups : 0;   // rows r0 + group, + groups, ...
@@ -51,21 +57,46 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncwarp();
+    // the columns are `segs` segments of K (one expert each, or a single one), a segment is seg_chunks chunks.
     // tile i of this warp: pass i / rows, row r0 + group + groups * (i % rows); a chunk past the end has no tiles
-    const int my_passes = max(0, min(passes, ((K + chunk - 1) / chunk - kw + ks - 1) / ks));
+    __shared__ int slot_e[kMaxTopK];
+    __shared__ float slot_w[kMaxTopK];
+    const int segs = MODE == kGvDown ? ex.top : 1, seg_chunks = (K + chunk - 1) / chunk;
+    const int my_passes = max(0, min(passes, (segs * seg_chunks - kw + ks - 1) / ks));
     const int tiles = rows * my_passes;
     auto issue = [&](int i) {   // lane 0
         const int pass = i / rows, row = r0 + group + groups * (i - pass * rows);
-        const int k0 = (pass * ks + kw) * chunk, kc = min(chunk, K - k0);
+        const int q = pass * ks + kw, seg = MODE == kGvDown ? q / seg_chunks : 0;
+        const int k0 = (q - seg * seg_chunks) * chunk, kc = min(chunk, K - k0);
+        size_t wrow = row;
+        if constexpr (MODE == kGvDown) wrow += (size_t)slot_e[seg] * N;
+        if constexpr (MODE == kGvUp) {
+            const int per = N / ex.top, s = row / per;   // rows of an expert, slot
+            wrow += ((size_t)slot_e[s] - s) * per;
+        }
         const uint32_t bar = bar0 + 8 * (i % kGvStages);
         mbar_expect_tx(bar, kc * 2);
-        bulk_g2s(ring + (i % kGvStages) * kGvTileBytes, w + (size_t)row * K + k0, kc * 2, bar);
+        bulk_g2s(ring + (i % kGvStages) * kGvTileBytes, w + wrow * K + k0, kc * 2, bar);
     };
-    if (lane == 0)
+    if (MODE <= kGvNorm && lane == 0)
         for (int i = 0; i < kGvStages && i < tiles; i++) issue(i);
     pdl_prologue();
     pdl_release();   // (the whole grid is resident; the mixer behind it asks for its caches while this kernel streams)
     const __nv_bfloat16 *xrow = x;
+    if constexpr (MODE >= kGvUp) {
+        if (MODE == kGvUp) {
+            if (warp == 0) {
+                route_token(ex.logits, ex.experts, ex.top, 0, slot_e, slot_w, lane);
+                __syncwarp();
+                if (blockIdx.x == 0 && lane < ex.top) ex.idx[lane] = slot_e[lane];
+            }
+        } else if (threadIdx.x < ex.top) {
+            slot_e[threadIdx.x] = ex.idx[threadIdx.x];
+        }
+        __syncthreads();
+        if (lane == 0)
+            for (int i = 0; i < kGvStages && i < tiles; i++) issue(i);
+    }
     if constexpr (NORM) {
         __shared__ float red[32];
         __nv_bfloat16 *xn = reinterpret_cast<__nv_bfloat16 *>(gv_smem + kGvRing + nrm.xn_at);
@@ -103,13 +134,14 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
     int stage = 0, issued = min(tiles, kGvStages);
     uint32_t phase = 0;
     for (int pass = 0, i = 0; pass < my_passes && ok; pass++) {
-        const int k0 = (pass * ks + kw) * chunk, kc = min(chunk, K - k0);
+        const int q = pass * ks + kw, seg = MODE == kGvDown ? q / seg_chunks : 0;
+        const int k0 = (q - seg * seg_chunks) * chunk, kc = min(chunk, K - k0), x0 = seg * K + k0;
         uint4 xv[M][4];
 #pragma unroll
         for (int m = 0; m < M; m++)
 #pragma unroll
             for (int j = 0; j < 4; j++)
-                xv[m][j] = 8 * (lane + 32 * j) < kc ? *reinterpret_cast<const uint4 *>(xrow + (size_t)m * K + k0 + 8 * (lane + 32 * j)) : make_uint4(0, 0, 0, 0);
+                xv[m][j] = 8 * (lane + 32 * j) < kc ? *reinterpret_cast<const uint4 *>(xrow + (size_t)m * K + x0 + 8 * (lane + 32 * j)) : make_uint4(0, 0, 0, 0);
         for (int r = 0; r < rows; r++, i++) {
             if (!mbar_wait_fast(bar0 + 8 * stage, phase)) {
                 ok = false;
@@ -165,7 +197,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
         if (lane == 0) atomicExch(status, 1);
     }
     __syncthreads();
-    if (NORM && pair_act) {
+    if (PAIRS && pair_act) {
         __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(y);
         for (int i = threadIdx.x; i < (r1 - r0) / 2; i += kGvWarps * 32) {
             float g = 0.0f, u = 0.0f;
@@ -173,9 +205,11 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
                 g += part[(size_t)(2 * i) * ks + q];
                 u += part[(size_t)(2 * i + 1) * ks + q];
             }
-            out[r0 / 2 + i] = __float2bfloat16_rn(gate_act(pair_act - 1, g) * u);
+            float v = gate_act(pair_act - 1, g) * u;
+            if constexpr (MODE == kGvUp) v *= slot_w[(r0 + 2 * i) / (N / ex.top)];
+            out[r0 / 2 + i] = __float2bfloat16_rn(v);
         }
-        if (blockIdx.x == 0)
+        if (MODE == kGvNorm && blockIdx.x == 0)
             for (int i = N / 2 + threadIdx.x; i < y_ld; i += kGvWarps * 32) out[i] = __float2bfloat16_rn(0.0f);
         return;
     }
@@ -194,12 +228,13 @@ bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt) {
            w->n < (1ll << 31) && w->k < (1ll << 31) && !((uintptr_t)w->d_raw & 15u);
 }
 
-template <int M, bool NORM>
-static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, const GemvNorm &nrm, int pair_act, int y_ld, cudaStream_t st) {
-    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M, NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+template <int M, int MODE>
+static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, const GemvNorm &nrm, int pair_act, int y_ld, cudaStream_t st,
+                         const GemvExperts &ex = {}) {
+    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
-    launch_pdl_smem(dense_gemv_kernel<M, NORM>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
-                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm, pair_act, y_ld);
+    launch_pdl_smem(dense_gemv_kernel<M, MODE>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
+                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm, pair_act, y_ld, ex);
     return cudaGetLastError();
 }
 
@@ -225,18 +260,38 @@ static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, int pair_ac
     if (nrm) {
         nrm->xn_at = (int)(smem - kGvRing);
         smem += (size_t)a.k * 2;
-        e = gv_go<1, true>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, pair_act, y_ld, stream);
+        e = gv_go<1, kGvNorm>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, pair_act, y_ld, stream);
     } else {
         switch (a.m) {
-            case 1: e = gv_go<1, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
-            case 2: e = gv_go<2, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
-            case 3: e = gv_go<3, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
-            case 4: e = gv_go<4, false>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 1: e = gv_go<1, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 2: e = gv_go<2, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 3: e = gv_go<3, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 4: e = gv_go<4, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
             default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "1 to 4 rows");
         }
     }
     ctx->launches++;
     return check_cuda(ctx, e, "bf16 row product launch");
+}
+
+nnq_status launch_dense_gemv_experts(nnq_ctx *ctx, const GemvExperts &g, bool up, cudaStream_t stream) {
+    const int64_t n = up ? 2ll * g.inter * g.top : g.hidden, k = up ? g.hidden : g.inter;
+    if (g.top < 1 || g.top > kMaxTopK || g.experts < g.top || g.experts > kMaxExperts || k % 8 || k < 8) return fail(ctx, NNQ_ERR_UNSUPPORTED, "bad expert product");
+    // chunks of a segment alike, as few warps per row as there are chunks
+    const int segs = up ? 1 : g.top, seg_chunks = (int)((k + kGvChunk - 1) / kGvChunk), chunk = (int)((k + seg_chunks - 1) / seg_chunks + 7) / 8 * 8;
+    int ks = 1;
+    while (ks < gv_warps(1) && ks < segs * seg_chunks) ks *= 2;
+    const int passes = (segs * seg_chunks + ks - 1) / ks, per_unit = up ? 2 : 1;
+    const int64_t units = n / per_unit, max_rows = (32 << 10) / (4 * ks);
+    int64_t grid = units < ctx->sm_count ? units : ctx->sm_count;
+    while ((units + grid - 1) / grid * per_unit > max_rows) grid += ctx->sm_count;
+    const size_t smem = kGvRing + ((size_t)((units + grid - 1) / grid * per_unit) * ks * 4 + 15) / 16 * 16;
+    const TcArgs a = {(const uint8_t *)g.w, nullptr, g.x, nullptr, g.y, 1, n, k, NNQ_BF16_DENSE, NNQ_BF16, up ? NNQ_BF16 : NNQ_F32};
+    const GemvNorm none = {};
+    const cudaError_t e = up ? gv_go<1, kGvUp>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 1 + NNQ_ACT_SILU, 0, stream, g)
+                             : gv_go<1, kGvDown>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, g);
+    ctx->launches++;
+    return check_cuda(ctx, e, "expert row product launch");
 }
 
 nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) { return gemv(ctx, a, nullptr, 0, 0, stream); }

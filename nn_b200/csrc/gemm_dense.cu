@@ -215,13 +215,13 @@ __device__ __forceinline__ void dg_tma_2d(uint32_t dst, const CUtensorMap *map, 
 // on the device), expert e multiplies its rows with rows [e * N, (e + 1) * N) of the decoded
 // weights and adds bias + e * N. Row tiles are numbered expert by expert; rows of the next expert
 // inside a tile are computed but not stored. offsets == NULL: a plain product.
-constexpr int kDgMaxGroups = 64;
+constexpr int kDgMaxGroups = 256;
 
 template <int BN>
 __global__ void __launch_bounds__(kDgThreads, 1)
 gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap,
                   const float *__restrict__ bias, void *__restrict__ y, int M, int N, int K, int y_dt, int *status,
-                  const int *__restrict__ offsets, int groups, __nv_bfloat16 *__restrict__ h_out, float swiglu_limit) {
+                  const int *__restrict__ offsets, int groups, __nv_bfloat16 *__restrict__ h_out, float swiglu_limit, int gate_kind) {
     constexpr int kDgBN = BN, kDgStageBytes = dg_stage_bytes(BN);
     extern __shared__ __align__(1024) uint8_t smem_raw[];
     uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -371,7 +371,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
                 tmem_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * kDgBN + cc * 32), v);
                 const int col0 = n0 + cc * 32;
                 if (h_out) {
-                    // interleaved gate / up columns (2j, 2j + 1): h[row, j] = clamp(silu(g), +-limit) * u in bf16,
+                    // interleaved gate / up columns (2j, 2j + 1): h[row, j] = clamp(f(g), +-limit) * u in bf16, f silu or gelu,
                     // the input of the second expert product; the bias of column c is the gate bias of c / 2 for
                     // even c and the up bias (second half of the expert's bias row) for odd c
                     if (row < m_end && col0 < N) {
@@ -390,7 +390,9 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constan
                                 }
                                 // fast exponential and division (2^-22 relative): far below the bf16 rounding of h,
                                 // and cheap enough for the epilogue to stay hidden behind the next tile's MMAs
-                                float sv = __fdividef(gv, 1.0f + __expf(-gv));
+                                // (the tanh form of gelu is x sigmoid(2 sqrt(2 / pi) (x + 0.044715 x^3)))
+                                const float sx = gate_kind == NNQ_ACT_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * gv * gv, gv, gv) : gv;
+                                float sv = __fdividef(gv, 1.0f + __expf(-sx));
                                 sv = fminf(fmaxf(sv, -swiglu_limit), swiglu_limit);
                                 hv[q2] = sv * uv;
                             }
@@ -552,8 +554,8 @@ static nnq_status dg_configure(nnq_ctx *ctx, int bn) {
     return NNQ_OK;
 }
 
-// The GEMM alone: w_bf16 is a bf16 [n, k] weight in device memory (16-byte aligned).
-nnq_status launch_gemm_dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs &a, cudaStream_t stream) {
+// The GEMM alone: w_bf16 is a bf16 [n, k] weight in device memory (16-byte aligned). h_out: see launch_gemm_dense_pairs.
+static nnq_status dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs &a, __nv_bfloat16 *h_out, int gate_kind, cudaStream_t stream) {
     CUtensorMap xmap, wmap;
     memset(&xmap, 0, sizeof(xmap));
     memset(&wmap, 0, sizeof(wmap));
@@ -567,11 +569,17 @@ nnq_status launch_gemm_dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs
     const int64_t tiles = m_tiles * ((a.n + bn - 1) / bn);
     const int grid = (int)(tiles < ctx->sm_count ? tiles : ctx->sm_count);
     if (bn == 256)
-        gemm_dense_kernel<256><<<grid, kDgThreads, smem_bytes, stream>>>(xmap, wmap, a.bias, a.y, (int)a.m, (int)a.n, (int)a.k, a.y_dt, ctx->d_status, nullptr, 0, nullptr, 0.0f);
+        gemm_dense_kernel<256><<<grid, kDgThreads, smem_bytes, stream>>>(xmap, wmap, a.bias, a.y, (int)a.m, (int)a.n, (int)a.k, a.y_dt, ctx->d_status, nullptr, 0, h_out, INFINITY, gate_kind);
     else
-        gemm_dense_kernel<128><<<grid, kDgThreads, smem_bytes, stream>>>(xmap, wmap, a.bias, a.y, (int)a.m, (int)a.n, (int)a.k, a.y_dt, ctx->d_status, nullptr, 0, nullptr, 0.0f);
+        gemm_dense_kernel<128><<<grid, kDgThreads, smem_bytes, stream>>>(xmap, wmap, a.bias, a.y, (int)a.m, (int)a.n, (int)a.k, a.y_dt, ctx->d_status, nullptr, 0, h_out, INFINITY, gate_kind);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "bf16 GEMM launch");
+}
+
+nnq_status launch_gemm_dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs &a, cudaStream_t stream) { return dense_bf16(ctx, w_bf16, a, nullptr, 0, stream); }
+
+nnq_status launch_gemm_dense_pairs(nnq_ctx *ctx, const TcArgs &a, __nv_bfloat16 *h_out, int gate_kind, cudaStream_t stream) {
+    return dense_bf16(ctx, a.w, a, h_out, gate_kind, stream);
 }
 
 nnq_status launch_gemm_dense(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream) {
@@ -597,13 +605,13 @@ nnq_status launch_gemm_dense(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream)
 
 bool gemm_dense_grouped_supported(const nnq_ctx *ctx, const TcGroupArgs &g) {
     if (g.kn && (g.fmt != NNQ_MXFP4_GPTOSS || g.n % kKnTile || g.k % kKnTile || ((uintptr_t)g.w & 15u))) return false;
-    return ctx->d_dense && g.k >= kDgBK && g.k % kDgBK == 0 && g.experts >= 1 && g.experts <= kDgMaxGroups && g.rows_upper >= 1 &&
-           (size_t)g.experts * (size_t)g.n * (size_t)g.k * 2 <= ctx->dense_bytes && g.rows_upper < (1ll << 30) &&
+    const bool room = g.pairs || (ctx->d_dense && (size_t)g.experts * (size_t)g.n * (size_t)g.k * 2 <= ctx->dense_bytes);
+    return room && g.k >= kDgBK && g.k % kDgBK == 0 && g.experts >= 1 && g.experts <= kDgMaxGroups && g.rows_upper >= 1 && g.rows_upper < (1ll << 30) &&
            (int64_t)g.experts * g.n < (1ll << 31) && encode_fn() != nullptr;
 }
 
 bool gemm_dense_grouped_fuses_swiglu(const TcGroupArgs &g) {
-    return g.h_out != nullptr && (g.fmt == NNQ_MXFP4_SPLIT || g.fmt == NNQ_MXFP4_GPTOSS) && g.n % 2 == 0 &&
+    return g.h_out != nullptr && (g.pairs || g.fmt == NNQ_MXFP4_SPLIT || g.fmt == NNQ_MXFP4_GPTOSS) && g.n % 2 == 0 &&
            (int64_t)g.experts * g.n * (g.k / 32) < (1ll << 31);
 }
 
@@ -611,12 +619,15 @@ nnq_status launch_gemm_dense_grouped(nnq_ctx *ctx, const TcGroupArgs &g, cudaStr
     // the experts' raw blocks are one contiguous [experts, N, K] tensor: one decode launch
     Geometry geo = geometry(g.fmt);
     const int64_t nchunks = (int64_t)g.experts * g.n * (g.k / geo.elems) * (geo.elems / 32);
-    cudaError_t e;
+    cudaError_t e = cudaSuccess;
     // SwiGLU in the GEMM's epilogue (g.h_out given): needs the gate / up rows interleaved in the decoded copy,
     // which the direct MXFP4 decode can write at no cost
     const bool fuse = gemm_dense_grouped_fuses_swiglu(g);
     const int cpr = (int)(g.k / 32), half = fuse ? (int)(g.n / 2) : 0;
-    if (g.kn) {
+    const void *w_bf16 = g.pairs ? (const void *)g.w : ctx->d_dense;
+    if (g.pairs) {
+        // bf16 experts are multiplied where they are
+    } else if (g.kn) {
         dequant_kn_bf16_kernel<<<dim3((unsigned)(g.n / kKnTile), (unsigned)(g.k / kKnTile), (unsigned)g.experts), 128, 0, stream>>>(
             g.w, g.scales, static_cast<__nv_bfloat16 *>(ctx->d_dense), (int)g.k, (int)g.n, half);
         e = cudaGetLastError();
@@ -630,7 +641,7 @@ nnq_status launch_gemm_dense_grouped(nnq_ctx *ctx, const TcGroupArgs &g, cudaStr
 #undef NNQ_DB
         default: return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown format %d", g.fmt);
     }
-    ctx->launches++;
+    if (!g.pairs) ctx->launches++;
     nnq_status s = check_cuda(ctx, e, "bf16 decode launch");
     if (s != NNQ_OK) return s;
     CUtensorMap xmap, wmap;
@@ -638,17 +649,17 @@ nnq_status launch_gemm_dense_grouped(nnq_ctx *ctx, const TcGroupArgs &g, cudaStr
     memset(&wmap, 0, sizeof(wmap));
     // row tiles of all experts: at most rows / 128 + one ragged tile per expert
     const int bn = dg_pick_bn(ctx, g.rows_upper / kDgBM + g.experts, g.n);
-    if (!make_map(g.x_bf16, g.rows_upper, g.k, kDgBM, &xmap) || !make_map(ctx->d_dense, (int64_t)g.experts * g.n, g.k, bn, &wmap))
+    if (!make_map(g.x_bf16, g.rows_upper, g.k, kDgBM, &xmap) || !make_map(w_bf16, (int64_t)g.experts * g.n, g.k, bn, &wmap))
         return fail(ctx, NNQ_ERR_DISPATCH_FAILED, "tensor map creation failed");
     s = dg_configure(ctx, bn);
     if (s != NNQ_OK) return s;
     const int smem_bytes = kDgStages * dg_stage_bytes(bn) + 1024;
     if (bn == 256)
         gemm_dense_kernel<256><<<ctx->sm_count, kDgThreads, smem_bytes, stream>>>(xmap, wmap, g.bias, g.y, (int)g.rows_upper, (int)g.n, (int)g.k, NNQ_F32,
-                                                                                  ctx->d_status, g.offsets, g.experts, fuse ? g.h_out : nullptr, g.swiglu_limit);
+                                                                                  ctx->d_status, g.offsets, g.experts, fuse ? g.h_out : nullptr, g.swiglu_limit, NNQ_ACT_SILU);
     else
         gemm_dense_kernel<128><<<ctx->sm_count, kDgThreads, smem_bytes, stream>>>(xmap, wmap, g.bias, g.y, (int)g.rows_upper, (int)g.n, (int)g.k, NNQ_F32,
-                                                                                  ctx->d_status, g.offsets, g.experts, fuse ? g.h_out : nullptr, g.swiglu_limit);
+                                                                                  ctx->d_status, g.offsets, g.experts, fuse ? g.h_out : nullptr, g.swiglu_limit, NNQ_ACT_SILU);
     ctx->launches++;
     return check_cuda(ctx, cudaGetLastError(), "grouped bf16 GEMM launch");
 }

@@ -41,6 +41,9 @@ struct TcGroupArgs {
     // decode-once path only: the experts are nn-gptoss [experts, K, N] MXFP4 tensors (codes [E, K, N / 2],
     // scale bytes [E, K, N / 32], blocks along N); the decode transposes them into the [N, K] copy
     bool kn = false;
+    // bf16 experts whose gate and up rows alternate (row 2j: gate j): multiplied in place, with h_out given the epilogue
+    // forms the activation as above
+    bool pairs = false;
 };
 bool gemm_dense_grouped_fuses_swiglu(const TcGroupArgs &g);
 nnq_status launch_gemm_tc_grouped(nnq_ctx *ctx, const TcGroupArgs &a, cudaStream_t stream);
@@ -56,6 +59,9 @@ nnq_status dense_scratch_reserve(nnq_ctx *ctx, int64_t n, int64_t k);
 nnq_status launch_gemm_dense(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream);
 // the GEMM alone over an already decoded bf16 [n, k] weight (a.w / a.fmt are not read)
 nnq_status launch_gemm_dense_bf16(nnq_ctx *ctx, const void *w_bf16, const TcArgs &a, cudaStream_t stream);
+// gate / up product of a bf16 weight with alternating gate and up rows (n = 2 * width): h_out[m, width] = f(gate) * up in
+// bf16, f = gate_kind (nnq_gate_act); gemm_dense_supported tells whether it runs, a.y is not written
+nnq_status launch_gemm_dense_pairs(nnq_ctx *ctx, const TcArgs &a, __nv_bfloat16 *h_out, int gate_kind, cudaStream_t stream);
 // dense_gemv.cu: one to four bf16 rows against an unquantized bf16 weight
 bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt);
 nnq_status launch_dense_gemv(nnq_ctx *ctx, const TcArgs &a, cudaStream_t stream);
@@ -82,6 +88,19 @@ bool dense_gemv_norm_supported(const nnq_weight *w, int hidden);
 // pair_act > 0: rows 2j and 2j + 1 of the weight are a gate and an up row, and y (bf16, n / 2 columns and zeros up to y_ld)
 // receives f(gate) * up, f = nnq_gate_act pair_act - 1
 nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, int pair_act, int y_ld, cudaStream_t stream);
+// Products of one row with the experts it is routed to, bf16 [experts, N, K] weights.
+//   up    every CTA routes the row (logits f32 [experts]); slot s, row pair j of its expert: y[s * inter + j] = weight_s *
+//         silu(gate) * up in bf16; idx receives the chosen experts
+//   down  y[n] (f32) = sum over the slots of W[idx[s]][n, :] . x[s * inter ..]
+struct GemvExperts {
+    const void *w;
+    int experts, top, inter, hidden;
+    const float *logits;
+    int *idx;
+    const __nv_bfloat16 *x;
+    void *y;
+};
+nnq_status launch_dense_gemv_experts(nnq_ctx *ctx, const GemvExperts &g, bool up, cudaStream_t stream);
 bool gemm_dense_shape_ok(const nnq_ctx *ctx, int64_t m, int64_t n, int64_t k, int x_dt);
 // the expert products of a prefill-sized MoE call: all local experts decoded at once
 bool gemm_dense_grouped_supported(const nnq_ctx *ctx, const TcGroupArgs &g);

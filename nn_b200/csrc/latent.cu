@@ -21,7 +21,47 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
 
 // ---- preparation ----
 
+template <typename T> struct Four;   // four values at once
+template <> struct Four<float> { using type = float4; };
+template <> struct Four<__nv_bfloat16> { using type = uint2; };
+
 constexpr int kLpWarps = 4;
+
+// v / rms(v) * w of `n` values to o (zeros up to ld) by one warp. Up to 2048 values in whole groups of four stay in registers.
+template <typename T>
+__device__ __forceinline__ void warp_rms_row(const float *p, const float *w, int n, int ld, float eps, T *o, T *o2) {
+    const int lane = threadIdx.x & 31;
+    if ((n & 3) == 0 && n <= 2048) {
+        float4 v[16];
+        float ss = 0.0f;
+#pragma unroll
+        for (int k = 0; k < 16; k++) v[k] = 4 * (lane + 32 * k) < n ? *reinterpret_cast<const float4 *>(p + 4 * (lane + 32 * k)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+        for (int k = 0; k < 16; k++) ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
+#pragma unroll
+        for (int k = 0; k < 16; k++) {
+            const int i = 4 * (lane + 32 * k);
+            if (i >= ld) continue;
+            const float4 g = i < n ? *reinterpret_cast<const float4 *>(w + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            const float y[4] = {v[k].x * inv * g.x, v[k].y * inv * g.y, v[k].z * inv * g.z, v[k].w * inv * g.w};
+            alignas(16) T t[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) t[e] = from_f32<T>(y[e]);
+            using V = typename Four<T>::type;
+            *reinterpret_cast<V *>(o + i) = *reinterpret_cast<const V *>(t);
+            if (o2) *reinterpret_cast<V *>(o2 + i) = *reinterpret_cast<const V *>(t);
+        }
+        return;
+    }
+    float ss = 0.0f;
+    for (int i = lane; i < n; i += 32) ss = fmaf(p[i], p[i], ss);
+    const float rms = sqrtf(warp_sum(ss) / (float)n + eps);
+    for (int i = lane; i < ld; i += 32) {
+        o[i] = from_f32<T>(i < n ? p[i] / rms * w[i] : 0.0f);
+        if (o2) o2[i] = o[i];
+    }
+}
 
 // A warp per item: n query latents, n key latents, then the older positions in groups of four (copied).
 template <typename T>
@@ -32,28 +72,16 @@ __global__ void __launch_bounds__(kLpWarps * 32) latent_prep_kernel(const Latent
     int item = blockIdx.x * kLpWarps + (threadIdx.x >> 5);
     const int pos0 = span_pos(a.span);
     if (item < nq) {
-        const float *p = a.proj + (size_t)item * a.in_cols + a.c_q;
-        float ss = 0.0f;
-        for (int i = lane; i < a.q_rank; i += 32) ss = fmaf(p[i], p[i], ss);
-        const float rms = sqrtf(warp_sum(ss) / (float)a.q_rank + a.eps);
-        T *o = reinterpret_cast<T *>(a.cq) + (size_t)item * a.q_ld;
-        for (int i = lane; i < a.q_ld; i += 32) o[i] = from_f32<T>(i < a.q_rank ? p[i] / rms * a.q_norm[i] : 0.0f);
+        warp_rms_row<T>(a.proj + (size_t)item * a.in_cols + a.c_q, a.q_norm, a.q_rank, a.q_ld, a.eps, reinterpret_cast<T *>(a.cq) + (size_t)item * a.q_ld, nullptr);
         return;
     }
     item -= nq;
     if (item < nk) {
         const int pos = pos0 + item, half = a.rot >> 1;
         const float *p = a.proj + (size_t)item * a.in_cols + a.c_kv, *r = p + a.kv_rank;
-        float ss = 0.0f;
-        for (int i = lane; i < a.kv_rank; i += 32) ss = fmaf(p[i], p[i], ss);
-        const float rms = sqrtf(warp_sum(ss) / (float)a.kv_rank + a.eps);
         T *oc = reinterpret_cast<T *>(a.ring_c) + (size_t)(pos % a.cap) * a.kv_ld, *orr = reinterpret_cast<T *>(a.ring_r) + (size_t)(pos % a.cap) * a.rot_ld;
         T *lc = reinterpret_cast<T *>(a.lin_c) + (size_t)(pos - a.first) * a.kv_ld, *lr = reinterpret_cast<T *>(a.lin_r) + (size_t)(pos - a.first) * a.rot_ld;
-        for (int i = lane; i < a.kv_ld; i += 32) {
-            const T v = from_f32<T>(i < a.kv_rank ? p[i] / rms * a.kv_norm[i] : 0.0f);
-            oc[i] = v;
-            if (a.linear) lc[i] = v;
-        }
+        warp_rms_row<T>(p, a.kv_norm, a.kv_rank, a.kv_ld, a.eps, oc, a.linear ? lc : nullptr);
         for (int i = lane; i < a.rot_ld; i += 32) {
             const T v = from_f32<T>(i < a.rot ? rotated(r, i, a.rot, a.cosv + (size_t)pos * half, a.sinv + (size_t)pos * half) : 0.0f);
             orr[i] = v;

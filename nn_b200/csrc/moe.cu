@@ -22,6 +22,7 @@
 #include "gemm_tc.h"
 #include "moe.h"
 #include "pdl.cuh"
+#include "route.cuh"
 #include "skinny.h"
 
 namespace nnq {
@@ -37,64 +38,6 @@ __device__ __forceinline__ float ld_act<float>(const float *p, int64_t i) { retu
 template <>
 __device__ __forceinline__ float ld_act<__nv_bfloat16>(const __nv_bfloat16 *p, int64_t i) {
     return __bfloat162float(p[i]);
-}
-
-constexpr int kMaxExperts = 256;
-constexpr int kLaneExperts = kMaxExperts / 32;   // logits held by a lane of the routing warp
-constexpr int kMaxTopK = 8;
-
-// Softmax over the E logits of one token (lg, shared memory) and top-k selection by one warp.
-__device__ __forceinline__ void route_token(const float *lg, int E, int top_k, int tok, int *__restrict__ idx,
-                                            float *__restrict__ wt, int lane) {
-    // lane l holds the logits of experts l, l + 32, ...
-    float p[kLaneExperts];
-    float mx = -CUDART_INF_F;
-#pragma unroll
-    for (int k = 0; k < kLaneExperts; k++) {
-        p[k] = lane + 32 * k < E ? lg[lane + 32 * k] : -CUDART_INF_F;
-        mx = fmaxf(mx, p[k]);
-    }
-    // softmax over the E experts (max-subtracted, f32)
-#pragma unroll
-    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, off));
-    float sum = 0.0f;
-#pragma unroll
-    for (int k = 0; k < kLaneExperts; k++) {
-        p[k] = lane + 32 * k < E ? expf(p[k] - mx) : 0.0f;
-        sum += p[k];
-    }
-#pragma unroll
-    for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
-#pragma unroll
-    for (int k = 0; k < kLaneExperts; k++) p[k] = lane + 32 * k < E ? p[k] / sum : -1.0f;
-    // top-k: k rounds of (largest probability, lowest index) selection
-    float sel_p = 0.0f, wsum = 0.0f;
-    int sel_e = 0;
-    for (int s = 0; s < top_k; s++) {
-        float best = p[0];
-        int be = lane;
-#pragma unroll
-        for (int k = 1; k < kLaneExperts; k++)
-            if (p[k] > best) {
-                best = p[k];
-                be = lane + 32 * k;
-            }
-#pragma unroll
-        for (int off = 16; off > 0; off >>= 1) {
-            float ob = __shfl_xor_sync(0xFFFFFFFFu, best, off);
-            int oe = __shfl_xor_sync(0xFFFFFFFFu, be, off);
-            if (ob > best || (ob == best && oe < be)) { best = ob; be = oe; }
-        }
-#pragma unroll
-        for (int k = 0; k < kLaneExperts; k++)
-            if (be == lane + 32 * k) p[k] = -1.0f;
-        if (lane == s) { sel_p = best; sel_e = be; }
-        wsum += best;
-    }
-    if (lane < top_k) {
-        idx[(int64_t)tok * top_k + lane] = sel_e;
-        wt[(int64_t)tok * top_k + lane] = sel_p / wsum;
-    }
 }
 
 // A CTA serves TOK consecutive tokens: their activations sit in shared memory as f32, the 8 warps
@@ -391,6 +334,7 @@ moe_kn_gptoss_kernel(const uint8_t *__restrict__ data, const uint8_t *__restrict
 
 // Weights stored per expert as [N, K] in any block format (blocks along K):
 // one warp per output column, the lanes share the 32-weight chunks of the row.
+// (bias NULL: none)
 template <int FMT, typename XT>
 __global__ void __launch_bounds__(128)
 moe_nk_kernel(const uint8_t *__restrict__ data, const uint8_t *__restrict__ scales, size_t expert_bytes,
@@ -427,7 +371,7 @@ moe_nk_kernel(const uint8_t *__restrict__ data, const uint8_t *__restrict__ scal
             float v = acc[t];
 #pragma unroll
             for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, off);
-            if (lane == 0 && t < mt) out[(size_t)(r0 + t) * N + n] = v + __ldg(bias + (size_t)e * N + n);
+            if (lane == 0 && t < mt) out[(size_t)(r0 + t) * N + n] = v + (bias ? __ldg(bias + (size_t)e * N + n) : 0.0f);
         }
     }
 }
@@ -442,7 +386,7 @@ __device__ __forceinline__ float swiglu_one(float g, float u, float limit) {
 }
 __global__ void __launch_bounds__(256)
 moe_swiglu_kernel(const float *__restrict__ gu, float *__restrict__ h, const int *__restrict__ offset,
-                  int E, int inter, float limit, int slices, size_t slice_stride, __nv_bfloat16 *__restrict__ h_bf16) {
+                  int E, int inter, float limit, int slices, size_t slice_stride, __nv_bfloat16 *__restrict__ h_bf16, bool pairs) {
     pdl_prologue();
     const int64_t r = blockIdx.x;
     if (r >= offset[E]) return;
@@ -450,6 +394,11 @@ moe_swiglu_kernel(const float *__restrict__ gu, float *__restrict__ h, const int
     if (j0 >= inter) return;
     const float *grow = gu + r * 2 * inter;
     float out[4];
+    if (pairs) {   // gate and up columns alternate; inter is a multiple of 64
+        const float4 a = *reinterpret_cast<const float4 *>(grow + 2 * j0), b = *reinterpret_cast<const float4 *>(grow + 2 * j0 + 4);
+        *reinterpret_cast<float4 *>(h + r * inter + j0) = make_float4(swiglu_one(a.x, a.y, limit), swiglu_one(a.z, a.w, limit), swiglu_one(b.x, b.y, limit), swiglu_one(b.z, b.w, limit));
+        return;
+    }
     if (slices == 1 && (inter & 3) == 0) {
         const float4 g = *reinterpret_cast<const float4 *>(grow + j0);
         const float4 u = *reinterpret_cast<const float4 *>(grow + inter + j0);
@@ -566,6 +515,7 @@ static size_t align256(size_t v) { return (v + 255) & ~(size_t)255; }
 // grouped token-column kernel, which is HBM-bound and wins; the gpt-oss block crosses over near 240 tokens).
 static bool moe_tensor_mode(const nnq_moe *m, int64_t T, int k, bool routed, bool exact) {
     if (exact) return false;
+    if (m->layout == NNQ_MOE_NK_PAIRS) return true;   // (row tiles of few rows still read every weight once)
     static const char *env = diag_env("NNQ_MOE_TENSOR");   // tuning aid: 0 keeps the token-column kernel
     if (env && atoi(env) == 0) return false;
     // nn-gptoss [E, K, N] experts take the decode-once form only (a transposing decode into the context's
@@ -643,6 +593,8 @@ static nnq_status launch_product(nnq_ctx *ctx, const nnq_moe *m, bool first, con
         const size_t eb = (size_t)N * (K / g.elems) * g.bytes, es = (size_t)N * (K / g.elems) * g.scale_bytes;
         TcGroupArgs a = {d, sc, eb, es, first ? (const void *)s.xg : (const void *)s.hb, b, out, s.offset, E, rows, N, K, m->fmt};
         a.kn = m->layout == NNQ_MOE_KN_GPTOSS;
+        a.pairs = m->layout == NNQ_MOE_NK_PAIRS;
+        if (a.pairs && !gemm_dense_grouped_supported(ctx, a)) return fail(ctx, NNQ_ERR_UNSUPPORTED, "no tensor maps for the expert products");
         // all local experts decoded to bf16 once, then the plain grouped GEMM -- or the grouped product with
         // the decode fused in. Measured (32 experts of about 3000 x 3000, top-4; ms per block fused / decoded
         // once at 64, 128 and 256 rows per expert): MXFP4 1.24 / 0.87 at 64 rows, decoded once at every size
@@ -658,7 +610,7 @@ static nnq_status launch_product(nnq_ctx *ctx, const nnq_moe *m, bool first, con
         if (const char *e = getenv("NNQ_MOE_DENSE_ROWS")) dense_rows = atoi(e);
 #endif
         if (a.kn && !gemm_dense_grouped_supported(ctx, a)) return fail(ctx, NNQ_ERR_UNSUPPORTED, "[E, K, N] experts: no bf16 scratch for the prefill-sized product");
-        if ((a.kn || rows >= dense_rows * (int64_t)E) && gemm_dense_grouped_supported(ctx, a)) {
+        if ((a.kn || a.pairs || rows >= dense_rows * (int64_t)E) && gemm_dense_grouped_supported(ctx, a)) {
             if (first && swiglu_done && s.slices == 1) {
                 // gate / up product: SwiGLU in the GEMM's epilogue where the decode can interleave the rows
                 a.h_out = s.hb;
@@ -786,7 +738,7 @@ static nnq_status run_with_scratch(nnq_ctx *ctx, const nnq_moe *m, const XT *x, 
     nnq_status prc = launch_product<XT>(ctx, m, true, x, s.rowtok, k, s, s.gu, total, st, &swiglu_done);
     if (prc != NNQ_OK) return prc;
     if (!swiglu_done)
-        launch_pdl(moe_swiglu_kernel, dim3((unsigned)total, (unsigned)((m->inter + 1023) / 1024)), dim3(256), st, s.gu, s.h, s.offset, m->e_local, m->inter, m->limit, s.slices, s.gu_stride, s.hb);
+        launch_pdl(moe_swiglu_kernel, dim3((unsigned)total, (unsigned)((m->inter + 1023) / 1024)), dim3(256), st, s.gu, s.h, s.offset, m->e_local, m->inter, m->limit, s.slices, s.gu_stride, s.hb, m->layout == NNQ_MOE_NK_PAIRS);
     prc = launch_product<float>(ctx, m, false, s.h, nullptr, k, s, s.o, total, st);
     if (prc != NNQ_OK) return prc;
     launch_pdl(moe_combine_kernel, dim3((unsigned)T, T < 1024 ? 4 : 1), dim3(256), st, s.o, idx, wt, s.pos, (int)T, m->hidden, k, y, s.slices, s.o_stride);
@@ -807,6 +759,25 @@ static nnq_status forward_typed(nnq_ctx *ctx, const nnq_moe *m, const XT *x, int
     if (idx_out) cudaMemcpyAsync(idx_out, s.idx, total * 4, cudaMemcpyDeviceToDevice, st);
     if (wt_out) cudaMemcpyAsync(wt_out, s.wt, total * 4, cudaMemcpyDeviceToDevice, st);
     return check_cuda(ctx, cudaGetLastError(), "MoE routing copy");
+}
+
+bool moe_step_supported(const nnq_moe *m, int hidden) { return m->router && m->limit == INFINITY && dense_gemv_norm_supported(m->router, hidden); }
+
+nnq_status moe_step(nnq_ctx *ctx, const nnq_moe *m, const GemvNorm &norm, float *y, cudaStream_t st) {
+    MoeScratch s;
+    nnq_status rc = ensure_scratch(ctx, m, 1, m->top_k, false, &s);
+    if (rc != NNQ_OK) return rc;
+    // logits in the place of the gate / up rows, the normed row in that of the outputs, the activation in its own
+    GemvNorm g = norm;
+    g.xn_out = reinterpret_cast<__nv_bfloat16 *>(s.o);
+    const TcArgs a = {m->router->d_raw, nullptr, nullptr, m->d_router_b, s.gu, 1, m->n_experts, m->hidden, NNQ_BF16_DENSE, NNQ_BF16, NNQ_F32};
+    if ((rc = launch_dense_gemv_norm(ctx, a, g, 0, 0, st)) != NNQ_OK) return rc;
+    GemvExperts e = {m->d_gu, m->n_experts, m->top_k, m->inter, m->hidden, s.gu, s.idx, g.xn_out, s.h};
+    if ((rc = launch_dense_gemv_experts(ctx, e, true, st)) != NNQ_OK) return rc;
+    e.w = m->d_dn;
+    e.x = reinterpret_cast<const __nv_bfloat16 *>(s.h);
+    e.y = y;
+    return launch_dense_gemv_experts(ctx, e, false, st);
 }
 
 nnq_status moe_reserve(nnq_ctx *ctx, const nnq_moe *m, int64_t rows) {
@@ -847,6 +818,24 @@ static nnq_status upload(nnq_ctx *ctx, void **dst, const void *src, size_t bytes
     return check_cuda(ctx, cudaMemcpy(*dst, src, bytes, cudaMemcpyDefault), what);
 }
 
+// the router as a bf16 weight, if no value of it is rounded by that
+static nnq_status bf16_router(nnq_moe *m) {
+    const size_t n = (size_t)m->n_experts * m->hidden;
+    uint32_t *w = new (std::nothrow) uint32_t[n];
+    uint16_t *b = new (std::nothrow) uint16_t[n];
+    nnq_status s = w && b ? check_cuda(m->ctx, cudaMemcpy(w, m->d_router_w, n * 4, cudaMemcpyDeviceToHost), "router weight")
+                          : fail(m->ctx, NNQ_ERR_OUT_OF_MEMORY, "host allocation failed");
+    bool exact = s == NNQ_OK;
+    for (size_t i = 0; i < n && exact; i++) {
+        exact = (w[i] & 0xFFFFu) == 0;
+        b[i] = (uint16_t)(w[i] >> 16);
+    }
+    if (exact) s = nnq_weight_create(m->ctx, NNQ_BF16_DENSE, b, n * 2, nullptr, 0, m->n_experts, m->hidden, &m->router);
+    delete[] b;
+    delete[] w;
+    return s;
+}
+
 nnq_status nnq_moe_create_shard(nnq_ctx *ctx, int n_experts, int expert_begin, int expert_count, int hidden,
                                 int inter, int top_k, float swiglu_limit, const float *router_w,
                                 const float *router_b, nnq_moe_layout layout, nnq_format fmt, const void *gate_up,
@@ -861,11 +850,14 @@ nnq_status nnq_moe_create_shard(nnq_ctx *ctx, int n_experts, int expert_begin, i
         return fail(ctx, NNQ_ERR_INVALID_ARG, "bad MoE dimensions (experts %d, top_k %d, hidden %d, inter %d)", n_experts, top_k, hidden, inter);
     if (expert_begin < 0 || expert_count < 1 || expert_begin + expert_count > n_experts)
         return fail(ctx, NNQ_ERR_INVALID_ARG, "bad expert range [%d, %d) of %d", expert_begin, expert_begin + expert_count, n_experts);
-    if (!router_w || !router_b || !gate_up || !down || !gate_up_bias || !down_bias) return fail(ctx, NNQ_ERR_INVALID_ARG, "NULL MoE tensor");
+    const bool pairs = layout == NNQ_MOE_NK_PAIRS;
+    if (!router_w || !router_b || !gate_up || !down || (!pairs && (!gate_up_bias || !down_bias))) return fail(ctx, NNQ_ERR_INVALID_ARG, "NULL MoE tensor");
     if ((int)fmt < 0 || fmt >= NNQ_FORMAT_COUNT) return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown format %d", (int)fmt);
     if (layout == NNQ_MOE_KN_GPTOSS && fmt != NNQ_MXFP4_GPTOSS)
         return fail(ctx, NNQ_ERR_WRONG_QUANT_TYPE, "the [E,K,N] layout holds nn-gptoss MXFP4 tensors only");
-    if (layout != NNQ_MOE_KN_GPTOSS && layout != NNQ_MOE_NK) return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown MoE layout %d", (int)layout);
+    if (pairs && (fmt != NNQ_BF16_DENSE || hidden % 64 || inter % 64 || expert_count != n_experts || (gate_up_bias && swiglu_limit != INFINITY)))
+        return fail(ctx, NNQ_ERR_UNSUPPORTED, "the alternating layout holds whole bf16 blocks with widths of multiples of 64");
+    if (layout != NNQ_MOE_KN_GPTOSS && layout != NNQ_MOE_NK && !pairs) return fail(ctx, NNQ_ERR_INVALID_ARG, "unknown MoE layout %d", (int)layout);
     Geometry g = geometry(fmt);
     // blocks must not cross rows of the axis they run along
     const int64_t gu_inner = layout == NNQ_MOE_KN_GPTOSS ? 2 * (int64_t)inter : hidden;
@@ -892,10 +884,11 @@ nnq_status nnq_moe_create_shard(nnq_ctx *ctx, int n_experts, int expert_begin, i
     if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_router_b, router_b, (size_t)n_experts * 4, "router bias");
     if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_gu, gate_up, gate_up_bytes, "gate_up");
     if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_gu_scales, gate_up_scales, gate_up_scales_bytes, "gate_up scales");
-    if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_gu_bias, gate_up_bias, (size_t)expert_count * 2 * inter * 4, "gate_up bias");
+    if (s == NNQ_OK && gate_up_bias) s = upload(ctx, (void **)&m->d_gu_bias, gate_up_bias, (size_t)expert_count * 2 * inter * 4, "gate_up bias");
     if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_dn, down, down_bytes, "down");
     if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_dn_scales, down_scales, down_scales_bytes, "down scales");
-    if (s == NNQ_OK) s = upload(ctx, (void **)&m->d_dn_bias, down_bias, (size_t)expert_count * hidden * 4, "down bias");
+    if (s == NNQ_OK && down_bias) s = upload(ctx, (void **)&m->d_dn_bias, down_bias, (size_t)expert_count * hidden * 4, "down bias");
+    if (s == NNQ_OK && pairs && !gate_up_bias && !down_bias) s = bf16_router(m);
     // tiled copies for the grouped kernel
     static const char *env_tiled = diag_env("NNQ_MOE_TILED");   // tuning aid: 0 keeps the row kernels
     if (s == NNQ_OK && layout == NNQ_MOE_KN_GPTOSS && !(env_tiled && atoi(env_tiled) == 0)) {
@@ -966,6 +959,7 @@ void nnq_moe_destroy(nnq_moe *m) {
     cudaFree(m->d_router_w); cudaFree(m->d_router_b); cudaFree(m->d_gu); cudaFree(m->d_gu_scales);
     cudaFree(m->d_gu_bias); cudaFree(m->d_dn); cudaFree(m->d_dn_scales); cudaFree(m->d_dn_bias);
     cudaFree(m->d_gu_tiled); cudaFree(m->d_dn_tiled);
+    if (m->router) nnq_weight_destroy(m->router);
     cudaGetLastError();
     delete m;
 }

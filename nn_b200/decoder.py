@@ -331,19 +331,19 @@ class BlockDecoder(Decoder):
 
     def _experts(self, b: BlockConfig, y: _BlockLayout, t: BlockTensors):
         """The block's experts as a MoeBlock of bf16 weights, widths rounded up to whole k steps with zeros."""
-        from .moe import LAYOUT_NK, MoeBlock
+        from .moe import LAYOUT_NK_PAIRS, MoeBlock
         hidden, ld, inter = self.cfg.hidden, y.in_k, -(-b.expert_ffn // 64) * 64
-        gu, dn = np.zeros((b.experts, 2, inter, ld), np.uint16), np.zeros((b.experts, ld, inter), np.uint16)
+        gu, dn = np.zeros((b.experts, inter, 2, ld), np.uint16), np.zeros((b.experts, ld, inter), np.uint16)
         for e in range(b.experts):
             gate, up, down = t.expert(e)
             if gate.shape != (b.expert_ffn, hidden) or up.shape != gate.shape or down.shape != gate.shape[::-1]:
                 raise api.ShapeMismatch(f"expert {e}: matrices of shape {gate.shape}, {up.shape}, {down.shape}")
-            gu[e, 0, :b.expert_ffn, :hidden], gu[e, 1, :b.expert_ffn, :hidden], dn[e, :hidden, :b.expert_ffn] = gate, up, down
+            gu[e, :b.expert_ffn, 0, :hidden], gu[e, :b.expert_ffn, 1, :hidden], dn[e, :hidden, :b.expert_ffn] = gate, up, down
         router = np.zeros((b.experts, ld), np.float32)
         router[:, :hidden] = t.router
         bias = np.zeros(b.experts, np.float32) if t.router_bias is None else t.router_bias
-        m = MoeBlock(b.experts, ld, inter, b.top, float("inf"), router, bias, LAYOUT_NK, QuantFormat.BF16_DENSE, gu.reshape(-1).view(np.uint8), None,
-                     np.zeros((b.experts, 2 * inter), np.float32), dn.reshape(-1).view(np.uint8), None, np.zeros((b.experts, ld), np.float32), self.backend)
+        m = MoeBlock(b.experts, ld, inter, b.top, float("inf"), router, bias, LAYOUT_NK_PAIRS, QuantFormat.BF16_DENSE,
+                     gu.reshape(-1).view(np.uint8), None, None, dn.reshape(-1).view(np.uint8), None, None, self.backend)
         self._keep.append(m)
         return m
 

@@ -12,7 +12,7 @@ import numpy as np
 from . import api
 from .formats import QuantFormat
 
-LAYOUT_KN_GPTOSS, LAYOUT_NK = 0, 1
+LAYOUT_KN_GPTOSS, LAYOUT_NK, LAYOUT_NK_PAIRS = 0, 1, 2
 
 
 def _u8(a):
@@ -29,6 +29,7 @@ class MoeBlock:
     router_w [E, H], router_b [E]; expert tensors as raw quantized bytes:
       layout KN_GPTOSS: gate_up logical [E, H, 2I], down [E, I, H] (nn-gptoss Mxfp4Tensor, blocks along N)
       layout NK:        gate_up logical [E, 2I, H], down [E, H, I] (any format, blocks along K)
+      layout NK_PAIRS:  as NK with alternating gate and up rows (bf16; biases may be None)
     gate_up_bias [E, 2I], down_bias [E, H].
     """
 
@@ -39,12 +40,12 @@ class MoeBlock:
         self.n_experts, self.hidden, self.inter, self.top_k = n_experts, hidden, inter, top_k
         b = self.backend
         rw, rb = _f32(router_w), _f32(router_b)
-        gu, gus, gub = _u8(gate_up), _u8(gate_up_scales), _f32(gate_up_bias)
-        dn, dns, dnb = _u8(down), _u8(down_scales), _f32(down_bias)
+        gu, gus, gub = _u8(gate_up), _u8(gate_up_scales), None if gate_up_bias is None else _f32(gate_up_bias)
+        dn, dns, dnb = _u8(down), _u8(down_scales), None if down_bias is None else _f32(down_bias)
         if rw.shape != (n_experts, hidden) or rb.shape != (n_experts,):
             raise api.InvalidShape("router weight must be [E, hidden] and router bias [E]")
         e0, ec = expert_range if expert_range is not None else (0, n_experts)
-        if gub.shape != (ec, 2 * inter) or dnb.shape != (ec, hidden):
+        if (gub is not None and gub.shape != (ec, 2 * inter)) or (dnb is not None and dnb.shape != (ec, hidden)):
             raise api.BiasMismatch("expert biases must be [E, 2*inter] and [E, hidden]")
         h = ctypes.c_void_p()
         p = lambda a: None if a is None else a.ctypes.data

@@ -269,7 +269,7 @@ def test_far_key_over_several_decode_ranges(tmp_path):
         dec.release()
 
 
-@pytest.mark.parametrize("heads,dim,rot,vdim,kv_rank,window", [(4, 24, 8, 20, 40, 9), (2, 128, 64, 128, 512, 100), (3, 64, 32, 64, 128, 300), (5, 100, 20, 72, 200, 64),
+@pytest.mark.parametrize("heads,dim,rot,vdim,kv_rank,window", [(4, 24, 8, 20, 40, 9), (2, 180, 64, 120, 256, 90), (2, 128, 64, 128, 512, 100), (3, 64, 32, 64, 128, 300), (5, 100, 20, 72, 200, 64),
                                                                 (8, 64, 64, 128, 64, 1), (2, 32, 128, 96, 96, 2000), (10, 64, 16, 40, 320, 65)])
 def test_expanded_and_absorbed_attention_agree(tmp_path, heads, dim, rot, vdim, kv_rank, window):
     """A bf16 decoder's prompt pass (expanded keys and values) against its own decode steps (latents as they are). Queries
