@@ -30,6 +30,19 @@ __device__ __forceinline__ float4 bf4(const __nv_bfloat16 *p) {
     return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
 }
 
+// Asks L2 for the weights and biases of the norms (constants: also before the kernel in front has ended).
+template <int K>
+__device__ __forceinline__ void norm_prefetch(const NormRow &r) {
+    const float *p[4] = {r.post_w, r.post_b, r.in.kind == kNormNone ? nullptr : r.in.w, r.in.kind == kNormLayer ? r.in.b : nullptr};
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+#pragma unroll
+        for (int k = 0; k < K; k++) {
+            const int i = 4 * (threadIdx.x + blockDim.x * k);
+            if (p[j] && i < r.hidden && (threadIdx.x & 7) == 0) asm volatile("prefetch.global.L2 [%0];" ::"l"(p[j] + i));
+        }
+}
+
 // The row as units of four elements, unit threadIdx.x + blockDim.x * k in v[k] (hidden a multiple of 4 and at most
 // 4 * K * blockDim.x; units past the end are zero). Every thread of the block calls it; red: 32 floats.
 template <int K>
@@ -63,6 +76,15 @@ __device__ __forceinline__ void norm_units(const NormRow &r, float4 (&v)[K], flo
         return block_sum(ss, red);
     };
     auto layer_norm = [&](const float *w, const float *b) {
+        float4 g[K], o[K];   // (asked for before the sums are formed)
+#pragma unroll
+        for (int k = 0; k < K; k++) {
+            const int i = 4 * (threadIdx.x + blockDim.x * k);
+            g[k] = o[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (i >= r.hidden) continue;
+            g[k] = *reinterpret_cast<const float4 *>(w + i);
+            o[k] = *reinterpret_cast<const float4 *>(b + i);
+        }
         float s = 0.0f;
 #pragma unroll
         for (int k = 0; k < K; k++) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
@@ -72,9 +94,8 @@ __device__ __forceinline__ void norm_units(const NormRow &r, float4 (&v)[K], flo
         for (int k = 0; k < K; k++) {
             const int i = 4 * (threadIdx.x + blockDim.x * k);
             if (i >= r.hidden) continue;
-            const float4 g = *reinterpret_cast<const float4 *>(w + i), o = *reinterpret_cast<const float4 *>(b + i);
-            v[k] = make_float4(fmaf((v[k].x - mean) * inv, g.x, o.x), fmaf((v[k].y - mean) * inv, g.y, o.y), fmaf((v[k].z - mean) * inv, g.z, o.z),
-                               fmaf((v[k].w - mean) * inv, g.w, o.w));
+            v[k] = make_float4(fmaf((v[k].x - mean) * inv, g[k].x, o[k].x), fmaf((v[k].y - mean) * inv, g[k].y, o[k].y), fmaf((v[k].z - mean) * inv, g[k].z, o[k].z),
+                               fmaf((v[k].w - mean) * inv, g[k].w, o[k].w));
         }
     };
     if (r.post_w) layer_norm(r.post_w, r.post_b);
@@ -86,13 +107,17 @@ __device__ __forceinline__ void norm_units(const NormRow &r, float4 (&v)[K], flo
         }
     }
     if (r.in.kind == kNormRms) {
-        const float rms = sqrtf(squares(0.0f) / n + r.eps);
+        float4 g[K];
 #pragma unroll
         for (int k = 0; k < K; k++) {
             const int i = 4 * (threadIdx.x + blockDim.x * k);
-            if (i >= r.hidden) continue;
-            const float4 g = *reinterpret_cast<const float4 *>(r.in.w + i);
-            v[k] = make_float4(v[k].x / rms * g.x, v[k].y / rms * g.y, v[k].z / rms * g.z, v[k].w / rms * g.w);
+            g[k] = i < r.hidden ? *reinterpret_cast<const float4 *>(r.in.w + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+        const float rms = sqrtf(squares(0.0f) / n + r.eps);
+#pragma unroll
+        for (int k = 0; k < K; k++) {
+            if (4 * (threadIdx.x + blockDim.x * k) >= r.hidden) continue;
+            v[k] = make_float4(v[k].x / rms * g[k].x, v[k].y / rms * g[k].y, v[k].z / rms * g[k].z, v[k].w / rms * g[k].w);
         }
     } else if (r.in.kind == kNormLayer) {
         layer_norm(r.in.w, r.in.b);

@@ -164,7 +164,7 @@ struct LatentAttn {
     float *qrot, *kfull, *vfull;    // rows on the general attention kernels: f32 copies with the shared part per head
     // decode step
     const __nv_bfloat16 *ukv;
-    float *qlat;                    // [heads, kv_ld + rot_ld]
+    float *qlat;                    // queries in the latent space (latent_step_query_floats)
     int ranges, keys_max;
     float *part;                    // [ranges, heads, kv_ld + 4]: maximum, sum, -, -, weighted latents
 };
@@ -176,6 +176,7 @@ nnq_status launch_latent_rows(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st
 bool latent_tc_supported(int act_dt, int dim, int rot, int vdim);                    // attn_latent_tc.cu: on the tensor cores
 nnq_status launch_latent_tc(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st);
 nnq_status launch_latent_step(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st);   // one row, appends its latent
+size_t latent_step_query_floats(int heads, int kv_ld, int rot_ld);
 bool latent_step_supported(int act_dt, int kv_ld, int rot_ld);
 int latent_step_ranges(int sm_count, int heads, int window, int max_seq, int act_dt);
 

@@ -971,7 +971,7 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
                 most(kfull, keys * b.heads * dl);
                 most(vfull, keys * b.heads * vl);
             }
-            most(qlat, (size_t)b.heads * (y.kv_ld + rot_ld));
+            most(qlat, latent_step_query_floats(b.heads, y.kv_ld, rot_ld));
             most(part, (size_t)B.ranges * b.heads * (y.kv_ld + 4));
         } else if (b.mixer == NNQ_MIXER_RECURRENT) {
             B.dim_ld = b.dim <= 64 ? 64 : round_up(b.dim, 128);
@@ -1337,6 +1337,7 @@ static nnq_status run_block(nnq_decoder *d, int l, int n, int pos0, const int *s
                 g.in = {kNormRms, B.q_norm, nullptr};
                 g.eps = d->cfg.rms_eps;
                 g.hidden = k.q_rank;
+                g.half = true;
                 s = launch_dense_gemv_norm(ctx, t, g, 0, 0, st);
             } else {
                 s = launch_latent_prep(ctx, a, kLatentQueries, st);
@@ -1417,7 +1418,9 @@ static nnq_status step_norm_product(nnq_decoder *d, int l, const nnq_weight *w, 
     *activated = false;
     if (fused_steps(d) && dense_gemv_norm_supported(w, c.hidden)) {
         const TcArgs a = {w->d_raw, w->d_scales, nullptr, bias, pair_act ? act : y, 1, w->n, w->k, w->fmt, NNQ_BF16, NNQ_F32};
-        nnq_status s = launch_dense_gemv_norm(d->ctx, a, step_norm(d, r), pair_act, y_ld, st);
+        GemvNorm g = step_norm(d, r);
+        g.half = l < c.n_layers && d->blocks[l].cfg.mixer == NNQ_MIXER_LATENT;   // a small product in front of another
+        nnq_status s = launch_dense_gemv_norm(d->ctx, a, g, pair_act, y_ld, st);
         *activated = pair_act > 0;
         return s;
     }

@@ -6,7 +6,8 @@
 // registers (a lane's 32 of them as bf16 pairs) and a tile is one row's chunk, 2 KB. KS warps share a row; their
 // partial sums meet in shared memory once, at the end. The ring is filled before the kernel waits for its
 // predecessor (programmatic dependent launch): the small kernels in front of a product release it early, so the
-// weights stream while they run. Products bf16 x bf16 in f32, f32 sums. Every wait is bounded.
+// weights stream while they run. With GemvNorm.half it takes half of the warps and of the ring, so that two of them, or one
+// and a small kernel, fit on an SM. Products bf16 x bf16 in f32, f32 sums. Every wait is bounded.
 //
 // With NORM the kernel also does what stands in front of a decoder's product: every CTA adds the last block's output
 // to the residual row (or reads the embedding row), norms it and keeps the normed row as bf16 in shared memory; CTA 0
@@ -35,25 +36,26 @@ constexpr int kGvNormMax = 8192;   // width of the normed row: 16 values per thr
 
 enum { kGvPlain = 0, kGvNorm = 1, kGvUp = 2, kGvDown = 3 };
 
-template <int M, int MODE>
-__global__ void __launch_bounds__(gv_warps(M) * 32, 1)
+template <int M, int MODE, int W>
+__global__ void __launch_bounds__(W * 32, 1)
 dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__restrict__ x, const float *__restrict__ bias, void *__restrict__ y,
-                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm, int pair_act, int y_ld, const GemvExperts ex) {
+                  int N, int K, int ks, int chunk, int passes, int y_dt, int *status, const GemvNorm nrm, int pair_act, int y_ld, const GemvExperts ex, int stages) {
     constexpr bool NORM = MODE == kGvNorm, PAIRS = MODE == kGvNorm || MODE == kGvUp;
-    constexpr int kGvWarps = gv_warps(M), kGvStages = kGvTiles / kGvWarps;
+    constexpr int kGvWarps = W, kGvMaxStages = kGvTiles / kGvWarps;
     extern __shared__ __align__(128) uint8_t gv_smem[];
-    __shared__ __align__(8) uint64_t bars[kGvWarps * kGvStages];
-    float *part = reinterpret_cast<float *>(gv_smem + kGvRing);   // [rows of this CTA][ks][M]
+    __shared__ __align__(8) uint64_t bars[kGvWarps * kGvMaxStages];
+    const int ring_bytes = kGvWarps * stages * kGvTileBytes;
+    float *part = reinterpret_cast<float *>(gv_smem + ring_bytes);   // [rows of this CTA][ks][M]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int unit = PAIRS && pair_act ? 2 : 1;   // rows that stay together
     const int r0 = (int)((long long)(N / unit) * blockIdx.x / gridDim.x) * unit, r1 = (int)((long long)(N / unit) * (blockIdx.x + 1) / gridDim.x) * unit;
     const int groups = kGvWarps / ks, group = warp / ks, kw = warp % ks;
     const int rows = r1 - r0 > group ? (r1 - r0 - group + groups - 1) / groups : 0;   // rows r0 + group, + groups, ...
-    const uint32_t bar0 = smem_u32(bars + warp * kGvStages);
-    const uint32_t ring = smem_u32(gv_smem) + warp * kGvStages * kGvTileBytes;
-    const uint8_t *ring_p = gv_smem + warp * kGvStages * kGvTileBytes;
+    const uint32_t bar0 = smem_u32(bars + warp * kGvMaxStages);
+    const uint32_t ring = smem_u32(gv_smem) + warp * stages * kGvTileBytes;
+    const uint8_t *ring_p = gv_smem + warp * stages * kGvTileBytes;
     if (lane == 0) {
-        for (int s = 0; s < kGvStages; s++) mbar_init(bar0 + 8 * s, 1);
+        for (int s = 0; s < stages; s++) mbar_init(bar0 + 8 * s, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncwarp();
@@ -64,7 +66,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
     const int segs = MODE == kGvDown ? ex.top : 1, seg_chunks = (K + chunk - 1) / chunk;
     const int my_passes = max(0, min(passes, (segs * seg_chunks - kw + ks - 1) / ks));
     const int tiles = rows * my_passes;
-    auto issue = [&](int i) {   // lane 0
+    auto issue = [&](int i, int st) {   // lane 0; st = i % stages
         const int pass = i / rows, row = r0 + group + groups * (i - pass * rows);
         const int q = pass * ks + kw, seg = MODE == kGvDown ? q / seg_chunks : 0;
         const int k0 = (q - seg * seg_chunks) * chunk, kc = min(chunk, K - k0);
@@ -74,33 +76,38 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
             const int per = N / ex.top, s = row / per;   // rows of an expert, slot
             wrow += ((size_t)slot_e[s] - s) * per;
         }
-        const uint32_t bar = bar0 + 8 * (i % kGvStages);
+        const uint32_t bar = bar0 + 8 * st;
         mbar_expect_tx(bar, kc * 2);
-        bulk_g2s(ring + (i % kGvStages) * kGvTileBytes, w + wrow * K + k0, kc * 2, bar);
+        bulk_g2s(ring + st * kGvTileBytes, w + wrow * K + k0, kc * 2, bar);
     };
-    if (MODE <= kGvNorm && lane == 0)
-        for (int i = 0; i < kGvStages && i < tiles; i++) issue(i);
+    auto route = [&]() {   // every CTA for itself
+        if (warp == 0) {
+            route_token(ex.logits, ex.experts, ex.top, 0, slot_e, slot_w, lane);
+        }
+        __syncthreads();
+    };
+    if constexpr (MODE == kGvDown) route();   // the logits are older than the kernel in front
+    if (MODE != kGvUp && lane == 0)
+        for (int i = 0; i < stages && i < tiles; i++) issue(i, i);
+    NormRow row;
+    if constexpr (NORM) {
+        row.post_w = nrm.post_w;
+        row.post_b = nrm.post_b;
+        row.in = nrm.in;
+        row.hidden = nrm.hidden;
+        norm_prefetch<4>(row);
+    }
     pdl_prologue();
     pdl_release();   // (the whole grid is resident; the mixer behind it asks for its caches while this kernel streams)
     const __nv_bfloat16 *xrow = x;
-    if constexpr (MODE >= kGvUp) {
-        if (MODE == kGvUp) {
-            if (warp == 0) {
-                route_token(ex.logits, ex.experts, ex.top, 0, slot_e, slot_w, lane);
-                __syncwarp();
-                if (blockIdx.x == 0 && lane < ex.top) ex.idx[lane] = slot_e[lane];
-            }
-        } else if (threadIdx.x < ex.top) {
-            slot_e[threadIdx.x] = ex.idx[threadIdx.x];
-        }
-        __syncthreads();
+    if constexpr (MODE == kGvUp) {
+        route();
         if (lane == 0)
-            for (int i = 0; i < kGvStages && i < tiles; i++) issue(i);
+            for (int i = 0; i < stages && i < tiles; i++) issue(i, i);
     }
     if constexpr (NORM) {
         __shared__ float red[32];
-        __nv_bfloat16 *xn = reinterpret_cast<__nv_bfloat16 *>(gv_smem + kGvRing + nrm.xn_at);
-        NormRow row;
+        __nv_bfloat16 *xn = reinterpret_cast<__nv_bfloat16 *>(gv_smem + ring_bytes + nrm.xn_at);
         row.h_in = nrm.h_in;
         row.delta = nrm.delta;
         row.h_out = blockIdx.x == 0 ? nrm.h_out : nullptr;
@@ -111,11 +118,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
             if (nrm.pairs.table) row.e1 = nrm.pairs.table + pair_row(nrm.pairs, nrm.state[4], tok, nrm.state[1]) * nrm.embed_ld;
         }
         row.alpha = nrm.alpha;
-        row.post_w = nrm.post_w;
-        row.post_b = nrm.post_b;
-        row.in = nrm.in;
         row.eps = nrm.eps;
-        row.hidden = nrm.hidden;
         float4 h[4];
         norm_units(row, h, red);
 #pragma unroll
@@ -131,7 +134,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
         xrow = xn;
     }
     bool ok = true;
-    int stage = 0, issued = min(tiles, kGvStages);
+    int stage = 0, issued = min(tiles, stages);
     uint32_t phase = 0;
     for (int pass = 0, i = 0; pass < my_passes && ok; pass++) {
         const int q = pass * ks + kw, seg = MODE == kGvDown ? q / seg_chunks : 0;
@@ -155,7 +158,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
 #pragma unroll
             for (int j = 0; j < 4; j++) wv[j] = 8 * (lane + 32 * j) < kc ? tile[lane + 32 * j] : make_uint4(0, 0, 0, 0);
             __syncwarp();
-            if (lane == 0 && issued < tiles) issue(issued);   // the tile's values are in registers
+            if (lane == 0 && issued < tiles) issue(issued, stage);   // the tile's values are in registers
             issued++;
 #pragma unroll
             for (int j = 0; j < 4; j++) {
@@ -181,7 +184,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
                     *p = pass == 0 ? v : *p + v;
                 }
             }
-            if (++stage == kGvStages) {
+            if (++stage == stages) {
                 stage = 0;
                 phase ^= 1u;
             }
@@ -193,7 +196,7 @@ dense_gemv_kernel(const __nv_bfloat16 *__restrict__ w, const __nv_bfloat16 *__re
             for (int m = 0; m < M; m++) part[((size_t)(group + groups * r) * ks + kw) * M + m] = 0.0f;
     if (!ok) {
         // give the copies in flight a bounded chance to land before the shared memory goes
-        for (int s = 0; s < kGvStages; s++) mbar_wait(bar0 + 8 * s, phase);
+        for (int s = 0; s < stages; s++) mbar_wait(bar0 + 8 * s, phase);
         if (lane == 0) atomicExch(status, 1);
     }
     __syncthreads();
@@ -228,13 +231,13 @@ bool dense_gemv_supported(const nnq_weight *w, int64_t m, int x_dt) {
            w->n < (1ll << 31) && w->k < (1ll << 31) && !((uintptr_t)w->d_raw & 15u);
 }
 
-template <int M, int MODE>
+template <int M, int MODE, int W>
 static cudaError_t gv_go(const TcArgs &a, int grid, int ks, int chunk, int passes, size_t smem, int *status, const GemvNorm &nrm, int pair_act, int y_ld, cudaStream_t st,
-                         const GemvExperts &ex = {}) {
-    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+                         int stages, const GemvExperts &ex = {}) {
+    cudaError_t e = cudaFuncSetAttribute(dense_gemv_kernel<M, MODE, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
-    launch_pdl_smem(dense_gemv_kernel<M, MODE>, dim3(grid), dim3(gv_warps(M) * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
-                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm, pair_act, y_ld, ex);
+    launch_pdl_smem(dense_gemv_kernel<M, MODE, W>, dim3(grid), dim3(W * 32), smem, st, reinterpret_cast<const __nv_bfloat16 *>(a.w),
+                    reinterpret_cast<const __nv_bfloat16 *>(a.x), a.bias, a.y, (int)a.n, (int)a.k, ks, chunk, passes, a.y_dt, status, nrm, pair_act, y_ld, ex, stages);
     return cudaGetLastError();
 }
 
@@ -244,8 +247,10 @@ bool dense_gemv_norm_supported(const nnq_weight *w, int hidden) {
 
 static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, int pair_act, int y_ld, cudaStream_t stream) {
     // as few warps per row as keep a warp's columns within one chunk
+    const bool half = nrm && nrm->half && a.k <= kGvNormMax / 2;
+    const int warps = half ? 8 : gv_warps((int)a.m);
     int ks = 1;
-    while (ks < gv_warps((int)a.m) && a.k > (int64_t)ks * kGvChunk) ks *= 2;
+    while (ks < warps && a.k > (int64_t)ks * kGvChunk) ks *= 2;
     int chunk = (int)(((a.k + ks - 1) / ks + 7) / 8 * 8);
     if (chunk > kGvChunk) chunk = kGvChunk;
     const int chunks = (int)((a.k + chunk - 1) / chunk), passes = (chunks + ks - 1) / ks;
@@ -254,19 +259,22 @@ static nnq_status gemv(nnq_ctx *ctx, const TcArgs &a, GemvNorm *nrm, int pair_ac
     const int64_t units = pair_act ? a.n / 2 : a.n, per_unit = pair_act ? 2 : 1;   // runs of rows that stay together
     int64_t grid = units < ctx->sm_count ? units : ctx->sm_count;
     while ((units + grid - 1) / grid * per_unit > max_rows) grid += ctx->sm_count;
-    size_t smem = kGvRing + ((size_t)((units + grid - 1) / grid * per_unit) * ks * a.m * 4 + 15) / 16 * 16;
+    const int stages = half ? kGvTiles / 16 : kGvTiles / warps;
+    const size_t ring = (size_t)warps * stages * kGvTileBytes;
+    size_t smem = ring + ((size_t)((units + grid - 1) / grid * per_unit) * ks * a.m * 4 + 15) / 16 * 16;
     cudaError_t e;
     const GemvNorm none = {};
     if (nrm) {
-        nrm->xn_at = (int)(smem - kGvRing);
+        nrm->xn_at = (int)(smem - ring);
         smem += (size_t)a.k * 2;
-        e = gv_go<1, kGvNorm>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, pair_act, y_ld, stream);
+        e = half ? gv_go<1, kGvNorm, 8>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, pair_act, y_ld, stream, stages)
+                 : gv_go<1, kGvNorm, 16>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, *nrm, pair_act, y_ld, stream, stages);
     } else {
         switch (a.m) {
-            case 1: e = gv_go<1, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
-            case 2: e = gv_go<2, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
-            case 3: e = gv_go<3, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
-            case 4: e = gv_go<4, kGvPlain>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream); break;
+            case 1: e = gv_go<1, kGvPlain, 16>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, stages); break;
+            case 2: e = gv_go<2, kGvPlain, 16>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, stages); break;
+            case 3: e = gv_go<3, kGvPlain, 8>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, stages); break;
+            case 4: e = gv_go<4, kGvPlain, 8>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, stages); break;
             default: return fail(ctx, NNQ_ERR_UNSUPPORTED, "1 to 4 rows");
         }
     }
@@ -285,11 +293,12 @@ nnq_status launch_dense_gemv_experts(nnq_ctx *ctx, const GemvExperts &g, bool up
     const int64_t units = n / per_unit, max_rows = (32 << 10) / (4 * ks);
     int64_t grid = units < ctx->sm_count ? units : ctx->sm_count;
     while ((units + grid - 1) / grid * per_unit > max_rows) grid += ctx->sm_count;
+    const int stages = kGvTiles / gv_warps(1);
     const size_t smem = kGvRing + ((size_t)((units + grid - 1) / grid * per_unit) * ks * 4 + 15) / 16 * 16;
     const TcArgs a = {(const uint8_t *)g.w, nullptr, g.x, nullptr, g.y, 1, n, k, NNQ_BF16_DENSE, NNQ_BF16, up ? NNQ_BF16 : NNQ_F32};
     const GemvNorm none = {};
-    const cudaError_t e = up ? gv_go<1, kGvUp>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 1 + NNQ_ACT_SILU, 0, stream, g)
-                             : gv_go<1, kGvDown>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, g);
+    const cudaError_t e = up ? gv_go<1, kGvUp, 16>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 1 + NNQ_ACT_SILU, 0, stream, stages, g)
+                             : gv_go<1, kGvDown, 16>(a, (int)grid, ks, chunk, passes, smem, ctx->d_status, none, 0, 0, stream, stages, g);
     ctx->launches++;
     return check_cuda(ctx, e, "expert row product launch");
 }

@@ -82,6 +82,7 @@ struct GemvNorm {
     InNorm in;
     float eps;
     int hidden;
+    bool half;                    // half of the warps and of the ring: products whose weight is a few hundred kilobytes per SM
     int xn_at;                    // (set by the launcher)
 };
 bool dense_gemv_norm_supported(const nnq_weight *w, int hidden);
@@ -89,14 +90,14 @@ bool dense_gemv_norm_supported(const nnq_weight *w, int hidden);
 // receives f(gate) * up, f = nnq_gate_act pair_act - 1
 nnq_status launch_dense_gemv_norm(nnq_ctx *ctx, const TcArgs &a, const GemvNorm &norm, int pair_act, int y_ld, cudaStream_t stream);
 // Products of one row with the experts it is routed to, bf16 [experts, N, K] weights.
-//   up    every CTA routes the row (logits f32 [experts]); slot s, row pair j of its expert: y[s * inter + j] = weight_s *
-//         silu(gate) * up in bf16; idx receives the chosen experts
-//   down  y[n] (f32) = sum over the slots of W[idx[s]][n, :] . x[s * inter ..]
+// Every CTA routes the row (logits f32 [experts]).
+//   up    slot s, row pair j of its expert: y[s * inter + j] = weight_s * silu(gate) * up in bf16
+//   down  y[n] (f32) = sum over the slots of W[expert of s][n, :] . x[s * inter ..]; routes before it waits for the kernel in
+//         front, so that kernel must not be the one that forms the logits
 struct GemvExperts {
     const void *w;
     int experts, top, inter, hidden;
     const float *logits;
-    int *idx;
     const __nv_bfloat16 *x;
     void *y;
 };

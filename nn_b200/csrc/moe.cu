@@ -772,7 +772,7 @@ nnq_status moe_step(nnq_ctx *ctx, const nnq_moe *m, const GemvNorm &norm, float 
     g.xn_out = reinterpret_cast<__nv_bfloat16 *>(s.o);
     const TcArgs a = {m->router->d_raw, nullptr, nullptr, m->d_router_b, s.gu, 1, m->n_experts, m->hidden, NNQ_BF16_DENSE, NNQ_BF16, NNQ_F32};
     if ((rc = launch_dense_gemv_norm(ctx, a, g, 0, 0, st)) != NNQ_OK) return rc;
-    GemvExperts e = {m->d_gu, m->n_experts, m->top_k, m->inter, m->hidden, s.gu, s.idx, g.xn_out, s.h};
+    GemvExperts e = {m->d_gu, m->n_experts, m->top_k, m->inter, m->hidden, s.gu, g.xn_out, s.h};
     if ((rc = launch_dense_gemv_experts(ctx, e, true, st)) != NNQ_OK) return rc;
     e.w = m->d_dn;
     e.x = reinterpret_cast<const __nv_bfloat16 *>(s.h);

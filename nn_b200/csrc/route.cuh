@@ -17,6 +17,8 @@ __device__ __forceinline__ void route_token(const float *lg, int E, int top_k, i
     float mx = -CUDART_INF_F;
 #pragma unroll
     for (int k = 0; k < kLaneExperts; k++) {
+        p[k] = -1.0f;
+        if (32 * k >= E) continue;   // (the same in every lane: few experts cost few steps)
         p[k] = lane + 32 * k < E ? lg[lane + 32 * k] : -CUDART_INF_F;
         mx = fmaxf(mx, p[k]);
     }
@@ -26,13 +28,15 @@ __device__ __forceinline__ void route_token(const float *lg, int E, int top_k, i
     float sum = 0.0f;
 #pragma unroll
     for (int k = 0; k < kLaneExperts; k++) {
+        if (32 * k >= E) continue;
         p[k] = lane + 32 * k < E ? expf(p[k] - mx) : 0.0f;
         sum += p[k];
     }
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xFFFFFFFFu, sum, off);
 #pragma unroll
-    for (int k = 0; k < kLaneExperts; k++) p[k] = lane + 32 * k < E ? p[k] / sum : -1.0f;
+    for (int k = 0; k < kLaneExperts; k++)
+        if (32 * k < E) p[k] = lane + 32 * k < E ? p[k] / sum : -1.0f;
     // top-k: k rounds of (largest probability, lowest index) selection
     float sel_p = 0.0f, wsum = 0.0f;
     int sel_e = 0;
@@ -41,7 +45,7 @@ __device__ __forceinline__ void route_token(const float *lg, int E, int top_k, i
         int be = lane;
 #pragma unroll
         for (int k = 1; k < kLaneExperts; k++)
-            if (p[k] > best) {
+            if (32 * k < E && p[k] > best) {
                 best = p[k];
                 be = lane + 32 * k;
             }
