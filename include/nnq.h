@@ -693,7 +693,7 @@ typedef struct nnq_block_weights {
     const nnq_moe *moe;       /* mixture of experts: NNQ_MOE_NK_PAIRS of hidden = in_k; stays owned by the caller */
 } nnq_block_weights;
 /* `blocks` holds cfg->n_layers entries. block_rows: prompt rows that go through the blocks together (0 =
- * 1024). An attention block keeps a ring of min(max_seq, window - 1 + block_rows) keys and values. */
+ * 1024, 4096 with experts among the blocks). An attention block keeps a ring of min(max_seq, window - 1 + block_rows) keys and values. */
 NNQ_API nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg, const nnq_block_config *blocks,
                                              int block_rows, nnq_decoder **out);
 NNQ_API nnq_status nnq_decoder_block_layout(const nnq_decoder *d, int layer, nnq_block_layout *out);

@@ -100,6 +100,8 @@ constexpr int kAttnWarps = 4;
 // decode-once tensor path with several row tiles per weight tile (about 210 KB of buffers per row at
 // the Qwen3-8B shape).
 constexpr int kPrefillRows = 1024;
+// with experts among the blocks: their weights are read once per block of rows, whatever part of the rows each expert gets
+constexpr int kPrefillRowsExperts = 4096;
 constexpr int kArgmaxBlocks = 128;
 constexpr int kStateWords = 8;    // token, position, steps, context full, previous token
 constexpr int kWantRows = 64;     // rows of logits formed together
@@ -901,7 +903,9 @@ nnq_status nnq_decoder_create_blocks(nnq_ctx *ctx, const nnq_decoder_config *cfg
         delete d;
         return fail(ctx, NNQ_ERR_OUT_OF_MEMORY, "host allocation failed");
     }
-    const int want_rows = block_rows ? block_rows : kPrefillRows;
+    bool experts = false;
+    for (int l = 0; l < c.n_layers; l++) experts = experts || blocks[l].experts > 0;
+    const int want_rows = block_rows ? block_rows : (experts ? kPrefillRowsExperts : kPrefillRows);
     const int rows = d->pf_rows = want_rows < c.max_seq ? want_rows : c.max_seq;
     const size_t R = rows, es = c.act_dtype == NNQ_F32 ? 4 : 2;
     size_t proj = 0, act = 0, q = 0, k = 0, o = 0, vf = 0, part = 0, counters = 1;

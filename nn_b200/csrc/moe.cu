@@ -96,6 +96,13 @@ moe_router_kernel(const XT *__restrict__ x, const float *__restrict__ rw, const 
     for (int t = warp; t < ntok; t += 8) route_token(logits + t * E, E, top_k, tok0 + t, idx, wt, lane);
 }
 
+// routing of tokens whose logits are formed already, a warp per token
+__global__ void __launch_bounds__(256) moe_route_kernel(const float *__restrict__ logits, int T, int E, int top_k, int *__restrict__ idx, float *__restrict__ wt) {
+    pdl_prologue();
+    const int tok = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (tok < T) route_token(logits + (size_t)tok * E, E, top_k, tok, idx, wt, threadIdx.x & 31);
+}
+
 // Fewer tokens than fill the machine one CTA each: a cluster of four CTAs serves a token, every CTA
 // forms a quarter of the logits (a warp per expert, the same lane-strided sums as above: identical
 // bits) and sends them into the first CTA's shared memory, which then routes the token.
@@ -715,6 +722,13 @@ static nnq_status run_with_scratch(nnq_ctx *ctx, const nnq_moe *m, const XT *x, 
     if (given_idx) {
         idx = given_idx;
         wt = given_wt;
+    } else if (m->router && s.xg && sizeof(XT) == 2 && gemm_dense_supported(ctx, m->router, T, NNQ_BF16) && (size_t)T * E <= s.gu_stride) {
+        // hundreds of bf16 rows and an exact bf16 router: the logits on the tensor cores (in the place of the gate / up rows)
+        const TcArgs a = {m->router->d_raw, nullptr, x, m->d_router_b, s.gu, T, E, m->hidden, NNQ_BF16_DENSE, NNQ_BF16, NNQ_F32};
+        nnq_status rc = launch_gemm_dense(ctx, a, st);
+        if (rc != NNQ_OK) return rc;
+        launch_pdl(moe_route_kernel, dim3((unsigned)((T + 7) / 8)), dim3(256), st, s.gu, (int)T, E, k, s.idx, s.wt);
+        ctx->launches++;
     } else {
         launch_router<XT>(m, x, T, s.idx, s.wt, st);
         ctx->launches++;
