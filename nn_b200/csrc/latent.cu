@@ -611,18 +611,20 @@ __global__ void __launch_bounds__(kLsThreads) latent_scores_mma_kernel(const Lat
 
 constexpr int kLvRows = 4, kLvGroups = 8;   // value dimensions of a warp; most groups of threads that share the records
 
-// grid (heads, ceil(vdim / 32))
-__global__ void __launch_bounds__(kLsThreads) latent_values_kernel(const LatentAttn a, int per) {
+// grid (heads, ceil(vdim / 32)). NU: 256-wide pieces of the latent
+// (NU = 2: few enough registers for the product behind it to become resident)
+template <int NU>
+__global__ void __launch_bounds__(kLsThreads, NU <= 2 ? 3 : 1) latent_values_kernel(const LatentAttn a, int per) {
     __shared__ __align__(16) float parts[1024];   // G rows of kv_ld
     __shared__ float wt[8][kLsMaxRanges];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x;
     const int v0 = blockIdx.y * 8 * kLvRows + warp * kLvRows, nu = a.kv_ld >> 3;
     const __nv_bfloat16 *w = a.ukv + ((size_t)a.heads * a.dim_ld + (size_t)h * a.vdim_ld + v0) * a.kv_ld;
-    uint4 wv[kLvRows][4];
+    uint4 wv[kLvRows][NU];
 #pragma unroll
     for (int r = 0; r < kLvRows; r++)
 #pragma unroll
-        for (int u = 0; u < 4; u++)
+        for (int u = 0; u < NU; u++)
             wv[r][u] = v0 + r < a.vdim && lane + 32 * u < nu ? *reinterpret_cast<const uint4 *>(w + (size_t)r * a.kv_ld + 8 * (lane + 32 * u)) : make_uint4(0, 0, 0, 0);
     pdl_prologue();
     pdl_release();
@@ -687,7 +689,7 @@ __global__ void __launch_bounds__(kLsThreads) latent_values_kernel(const LatentA
 #pragma unroll
     for (int r = 0; r < kLvRows; r++) acc[r] = 0.0f;
 #pragma unroll
-    for (int u = 0; u < 4; u++) {
+    for (int u = 0; u < NU; u++) {
         if (lane + 32 * u >= nu) continue;
         const float4 x0 = *reinterpret_cast<const float4 *>(lat + 8 * (lane + 32 * u)), x1 = *reinterpret_cast<const float4 *>(lat + 8 * (lane + 32 * u) + 4);
         const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
@@ -751,7 +753,9 @@ nnq_status launch_latent_step(nnq_ctx *ctx, const LatentAttn &a, cudaStream_t st
         s = a.kv_ld <= 512 ? go_scores(ctx, latent_scores_mma_kernel<4>, a, per, smem, st) : go_scores(ctx, latent_scores_mma_kernel<8>, a, per, smem, st);
     }
     if (s != NNQ_OK) return s;
-    launch_pdl(latent_values_kernel, dim3(a.heads, (a.vdim + 8 * kLvRows - 1) / (8 * kLvRows)), dim3(kLsThreads), st, a, per);
+    const dim3 vg(a.heads, (a.vdim + 8 * kLvRows - 1) / (8 * kLvRows));
+    if (a.kv_ld <= 512) launch_pdl(latent_values_kernel<2>, vg, ab, st, a, per);
+    else launch_pdl(latent_values_kernel<4>, vg, ab, st, a, per);
     ctx->launches += 3;
     return check_cuda(ctx, cudaGetLastError(), "latent value launch");
 }
