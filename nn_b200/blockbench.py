@@ -97,7 +97,7 @@ def rugesun_model(backend, z, max_seq, act_dtype=api.BF16, seed=0):
             t.gate, t.up, t.down = _bits(rng, b.ffn, D), _bits(rng, b.ffn, D), _bits(rng, D, b.ffn)
         dec.set_block(i, t)
     e = _bits(rng, z["vocab"], D)
-    dec.set_head(e, one, e, final_norm_bias=zero, logit_cap=30.0, pair_table=_bits(rng, 4097, D), pair_mul=(31, 7))
+    dec.set_head(e, one, e, final_norm_bias=zero, logit_cap=30.0, pair_table=_bits(rng, 4097, D), pair_mul=(29, 13))
     return dec
 
 

@@ -163,7 +163,7 @@ def test_portions_on_the_tensor_core_products(tmp_path):
 
 def test_first_token_and_the_pair_of_every_portion(tmp_path):
     """The pair table stands out: the row of a sequence's first token, and the previous token over cuts and restarts."""
-    cfg = M.config([M.layer(mlp=None)], pairs=(97, 31, 7))
+    cfg = M.config([M.layer(mlp=None)], pairs=(97, 29, 13))
     t = M.tensors(cfg, 4)
     t["bigram"] *= 4.0
     ids = tokens(30, cfg["vocab"], 8)

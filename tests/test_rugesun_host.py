@@ -66,7 +66,7 @@ def test_registry():
 # ---- closed forms for the restatement ----
 
 def test_restated_pairs():
-    assert ref.pair_rows([3, 5, 0, 5], 31, 7, 10) == [10, (93 + 35) % 10, 155 % 10, 35 % 10]
+    assert ref.pair_rows([3, 5, 0, 5], 13, 4, 10) == [10, (39 + 20) % 10, 65 % 10, 20 % 10]
 
 
 def test_restated_norm_and_activation():
